@@ -147,3 +147,7 @@ register_architecture(_rukedra.NAME, _rukedra.RukedraConfig.from_dict, _rukedra.
 from . import piratar as _piratar  # noqa: E402
 
 register_architecture(_piratar.NAME, _piratar.PiratarConfig.from_dict, _piratar.piratar_spec)
+
+from . import memilorn as _memilorn  # noqa: E402
+
+register_architecture(_memilorn.NAME, _memilorn.MemilornConfig.from_dict, _memilorn.memilorn_spec)

@@ -18,6 +18,7 @@
 // (token, head) that multiplies the head's output.
 #include "common.cuh"
 #include "kernel_args.h"
+#include "attention_reduce.cuh"
 
 LLG_API const char* llg_last_error() { return g_llg_error; }
 
@@ -299,35 +300,6 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(DecodeArgs a) {
   }
 }
 
-template <typename T>
-__global__ void attn_decode_reduce_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
-                                          T* __restrict__ out, int nh, int hd, int n_splits, int has_sink,
-                                          float sink_score, const float* __restrict__ gate,
-                                          const float* __restrict__ sinks) {
-  // (hd: elements of a value head)
-  const int h = blockIdx.x, b = blockIdx.y;
-  if (sinks) sink_score = sinks[h];
-  const long long base = ((long long)b * nh + h) * n_splits;
-  float M = -INFINITY;
-  for (int s = 0; s < n_splits; ++s) M = fmaxf(M, part_ml[(base + s) * 2]);
-  if (has_sink) M = fmaxf(M, sink_score);
-  float L = has_sink ? expf(sink_score - M) : 0.f;
-  for (int s = 0; s < n_splits; ++s) {
-    const float ms = part_ml[(base + s) * 2];
-    if (ms != -INFINITY) L += expf(ms - M) * part_ml[(base + s) * 2 + 1];
-  }
-  float inv = L > 0.f ? 1.0f / L : 0.f;
-  if (gate) inv *= gate[(long long)b * nh + h];
-  for (int d = threadIdx.x; d < hd; d += blockDim.x) {
-    float o = 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-      const float ms = part_ml[(base + s) * 2];
-      if (ms != -INFINITY) o += expf(ms - M) * part_o[(base + s) * hd + d];
-    }
-    out[((long long)b * nh + h) * hd + d] = from_f32<T>(o * inv);
-  }
-}
-
 }  // namespace
 
 LLG_API int llg_attn_prefill_simt(const PrefillArgs* args, int dtype, cudaStream_t stream) {
@@ -466,5 +438,7 @@ int llg_attn_decode_noalloc(const void* q, const void* k_pages, const void* v_pa
   a.gate = nullptr;
   a.sinks = nullptr;
   a.chunked = 0;
+  a.softcap = 0.f;
+  a.head_mix = nullptr;
   return llg_attn_decode_simt(&a, out, dtype, stream);
 }

@@ -30,7 +30,8 @@ SOURCES: Dict[str, List[str]] = {
     "elementwise": ["elementwise.cu", "common.cuh", "kernel_args.h"],
     "gemm_simt": ["gemm_simt.cu", "common.cuh"],
     "gemm_tc": ["gemm_tc.cu", "common.cuh", "kernel_args.h"],
-    "attention_simt": ["attention_simt.cu", "common.cuh", "kernel_args.h", "attention_noalloc.h"],
+    "attention_simt": ["attention_simt.cu", "common.cuh", "kernel_args.h", "attention_noalloc.h", "attention_reduce.cuh"],
+    "attention_mix": ["attention_mix.cu", "common.cuh", "kernel_args.h", "attention_reduce.cuh"],
     "attention_mma": ["attention_mma.cu", "common.cuh", "kernel_args.h"],
     "attention_tc": ["attention_tc.cu", "common.cuh", "kernel_args.h"],
     "attention_decode_tma": ["attention_decode_tma.cu", "common.cuh", "kernel_args.h"],
@@ -41,6 +42,7 @@ SOURCES: Dict[str, List[str]] = {
     "latent": ["latent.cu", "common.cuh", "kernel_args.h"],
     "groupnorm": ["groupnorm.cu", "common.cuh", "kernel_args.h"],
     "recurrent": ["recurrent.cu", "common.cuh", "kernel_args.h"],
+    "matrix_memory": ["matrix_memory.cu", "common.cuh", "kernel_args.h"],
     "addnorm": ["addnorm.cu", "common.cuh", "kernel_args.h"],
     "moe": ["moe.cu", "common.cuh", "kernel_args.h"],
 }

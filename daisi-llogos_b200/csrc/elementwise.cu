@@ -317,16 +317,27 @@ __global__ void qk_prep_kernel(QkPrepArgs a) {
   extern __shared__ float sm[];
   const int warps = blockDim.x >> 5;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int heads = a.nh + 2 * a.nkv;
+  const int heads = a.nh + 2 * a.nkv, units = heads + (a.gate_out ? 1 : 0);     // the gates of a token's heads are one unit more
   const long long item = (long long)blockIdx.x * warps + warp;
-  if (item >= (long long)a.n_tokens * heads) return;
-  const int n = (int)(item / heads);
-  const int h = (int)(item % heads);
+  if (item >= (long long)a.n_tokens * units) return;
+  const int n = (int)(item / units);
+  const int h = (int)(item % units);
   const int kind = h < a.nh ? 0 : (h < a.nh + a.nkv ? 1 : 2);  // 0 query, 1 key, 2 value
   const int vd = a.vd > 0 ? a.vd : a.hd;
   const int hd = kind == 2 ? vd : a.hd;                        // elements of this head
   float* x = sm + warp * max(a.hd, vd);
-  const long long row_w = (long long)(a.nh + a.nkv) * a.hd + (long long)a.nkv * vd;
+  const long long qkv_w = (long long)(a.nh + a.nkv) * a.hd + (long long)a.nkv * vd;
+  const long long row_w = qkv_w + (a.gate_out ? a.nh : 0);
+  if (h == heads) {
+    const IT* z = (const IT*)a.qkv + (long long)n * row_w + qkv_w;
+    const float zs = row_scale_of(a.row_scale, n);
+    for (int i = lane; i < a.nh; i += 32) {
+      float v = 0.f;
+      for (int s = 0; s < a.n_partials; ++s) v += to_f32(z[s * a.partial_stride + i]);
+      a.gate_out[(long long)n * a.nh + i] = 1.0f / (1.0f + expf(-v * zs));
+    }
+    return;
+  }
   const long long col = kind == 2 ? (long long)(a.nh + a.nkv) * a.hd + (long long)(h - a.nh - a.nkv) * vd : (long long)h * a.hd;
   const long long off = (long long)n * row_w + col;
   const IT* src = (const IT*)a.qkv + off;
@@ -549,12 +560,12 @@ LLG_API int llg_qk_prep(const QkPrepArgs* args, int out_dtype, cudaStream_t stre
   const bool plain_values = (a.vd == 0 || a.vd == a.hd) && !a.v_first_in && !a.v_first_out;
   LLG_REQUIRE(a.vd >= 0 && a.vd <= 1024, "qk_prep: value head size %d is larger than 1024", a.vd);
   LLG_REQUIRE(!a.v_first_in || a.v_mix, "qk_prep: blending values needs the blend's weight");
-  const bool lane_ok = plain_values && (a.hd == 64 || a.hd == 128 || a.hd == 256) &&
+  const bool lane_ok = plain_values && !a.gate_out && (a.hd == 64 || a.hd == 128 || a.hd == 256) &&
                        (!a.cos_table || (a.pairing == 0 && a.rotary_dim == a.hd)) && a.partial_stride % 4 == 0 &&
                        aligned(a.qkv) && aligned(a.q_norm_w) && aligned(a.k_norm_w) && aligned(a.bias) &&
                        aligned(a.cos_table) && aligned(a.sin_table) && aligned(a.q_out) && aligned(a.k_new) &&
                        aligned(a.v_new) && aligned(a.k_pages) && aligned(a.v_pages);
-  const long long items = (long long)a.n_tokens * (a.nh + 2 * a.nkv);
+  const long long items = (long long)a.n_tokens * (a.nh + 2 * a.nkv + (a.gate_out ? 1 : 0));
   // a step of few tokens spreads its heads over many small blocks: nothing but memory latency bounds it
   const bool few = lane_ok && items * (a.hd / 8) <= (long long)2 * 64 * llg_sm_count();
   const int warps = lane_ok ? (few ? 2 : 8) : 4;
@@ -653,10 +664,10 @@ LLG_API int llg_kv_write(const void* k_new, const void* v_new, void* k_pages, vo
 // to a multiple P of 128, then the up rows in the same way (the layout the tensor-core product's
 // gated epilogue wants).  A product's output row therefore holds, for feature i, g at i and u at P + i:
 // out[n][i] = silu(g) * u, silu(g) = g / (1 + exp(-g))  (Daisi.Llogos.Cpu/Silu.cs:9-16).
-// `act`: what the gate passes: 2 silu, 1 the tanh form of gelu (the kinds of llg_act in common.cuh).
+// `act`: what the gate passes: 2 silu, 1 the tanh form of gelu (the kinds of llg_act in common.cuh), -1: what `form` says.
 template <typename IT, typename OT>
 __global__ void silu_mul_kernel(const IT* __restrict__ gu, int n_partials, long long partial_stride,
-                                OT* __restrict__ out, long long total, int inter, int width, int act) {
+                                OT* __restrict__ out, long long total, int inter, int width, int act, GateForm form) {
   pdl_launch_dependents();
   pdl_wait();
   for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total;
@@ -669,27 +680,34 @@ __global__ void silu_mul_kernel(const IT* __restrict__ gu, int n_partials, long 
       g += to_f32(p[s * partial_stride]);
       u += to_f32(p[s * partial_stride + width / 2]);
     }
-    out[idx] = from_f32<OT>((act == 2 ? g / (1.0f + expf(-g)) : llg_act(act, g)) * u);
+    out[idx] = from_f32<OT>(act < 0 ? gate_form_of(form, g, u) : (act == 2 ? g / (1.0f + expf(-g)) : llg_act(act, g)) * u);
   }
 }
 
 static int gate_mul(const void* gu, int in_dtype, int n_partials, long long partial_stride, void* out,
-                    int out_dtype, int n_tokens, int inter, int act, cudaStream_t stream);
+                    int out_dtype, int n_tokens, int inter, int act, const GateForm& form, cudaStream_t stream);
+static const GateForm SILU_FORM = {1.0f, 0.0f, INFINITY, 0.0f};
 
 LLG_API int llg_silu_mul(const void* gu, int in_dtype, int n_partials, long long partial_stride, void* out,
                          int out_dtype, int n_tokens, int inter, cudaStream_t stream) {
-  return gate_mul(gu, in_dtype, n_partials, partial_stride, out, out_dtype, n_tokens, inter, 2, stream);
+  return gate_mul(gu, in_dtype, n_partials, partial_stride, out, out_dtype, n_tokens, inter, 2, SILU_FORM, stream);
 }
 
 // out[n][i] = act(g) * u with the gate's activation given by its kind (llg_act in common.cuh).
 LLG_API int llg_gate_mul(const void* gu, int in_dtype, int n_partials, long long partial_stride, void* out,
                          int out_dtype, int n_tokens, int inter, int act, cudaStream_t stream) {
   LLG_REQUIRE(act >= 0 && act < LLG_ACT_KINDS, "gate_mul: activation kind %d is not known", act);
-  return gate_mul(gu, in_dtype, n_partials, partial_stride, out, out_dtype, n_tokens, inter, act, stream);
+  return gate_mul(gu, in_dtype, n_partials, partial_stride, out, out_dtype, n_tokens, inter, act, SILU_FORM, stream);
+}
+
+// out[n][i] by a form of gating (GateForm in kernel_args.h).
+LLG_API int llg_gate_form_mul(const void* gu, int in_dtype, int n_partials, long long partial_stride, void* out, int out_dtype,
+                              int n_tokens, int inter, const GateForm* form, cudaStream_t stream) {
+  return gate_mul(gu, in_dtype, n_partials, partial_stride, out, out_dtype, n_tokens, inter, -1, *form, stream);
 }
 
 static int gate_mul(const void* gu, int in_dtype, int n_partials, long long partial_stride, void* out,
-                    int out_dtype, int n_tokens, int inter, int act, cudaStream_t stream) {
+                    int out_dtype, int n_tokens, int inter, int act, const GateForm& form, cudaStream_t stream) {
   LLG_REQUIRE(n_tokens >= 0 && inter > 0 && n_partials >= 1, "silu_mul: bad sizes");
   const long long total = (long long)n_tokens * inter;
   if (total == 0) return 0;
@@ -699,7 +717,7 @@ static int gate_mul(const void* gu, int in_dtype, int n_partials, long long part
   if (blocks > (long long)llg_sm_count() * 16) blocks = (long long)llg_sm_count() * 16;
 #define LAUNCH(IT, OT)                                                                                          \
   silu_mul_kernel<IT, OT><<<(unsigned)blocks, threads, 0, stream>>>((const IT*)gu, n_partials, partial_stride, \
-                                                                     (OT*)out, total, inter, width, act)
+                                                                     (OT*)out, total, inter, width, act, form)
   if (in_dtype == LLG_F32 && out_dtype == LLG_F32) LAUNCH(float, float);
   else if (in_dtype == LLG_F32 && out_dtype == LLG_BF16) LAUNCH(float, __nv_bfloat16);
   else if (in_dtype == LLG_BF16 && out_dtype == LLG_BF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);

@@ -125,13 +125,16 @@ __device__ __forceinline__ void tmem_ld16(uint32_t taddr, uint32_t (&r)[16]) {
       : "r"(taddr));
 }
 
-// What the gate of a gated epilogue passes: g sigmoid(g (a + b g^2)).  (a, b) = (1, 0) is silu; the tanh form of gelu,
+// What a gated epilogue makes of gate and up values (GateForm in kernel_args.h): g sigmoid(g (a + b g^2)) times the up value,
+// both clamped first and the up value shifted.  (a, b) = (1, 0) is silu; the tanh form of gelu,
 // 0.5 g (1 + tanh(c (g + 0.044715 g^3))), is the same as g sigmoid(2 c (g + 0.044715 g^3)), so (a, b) = (2 c, 2 c 0.044715)
 // with c = sqrt(2 / pi).  One form without a branch: the epilogue of every gated product costs what silu's did.
 #define LLG_GELU_GATE_A 1.5957691216057308f
 #define LLG_GELU_GATE_B 0.07135481627260025f
-__device__ __forceinline__ float gate_act(float a, float b, float g) {
-  return __fdividef(g, 1.0f + __expf(-g * fmaf(b * g, g, a)));
+__device__ __forceinline__ float gate_act(const GateForm& f, float g, float u) {
+  g = fminf(g, f.limit);
+  u = fmaxf(fminf(u, f.limit), -f.limit) + f.up_offset;
+  return __fdividef(g, 1.0f + __expf(-g * fmaf(f.b * g, g, f.a))) * u;
 }
 
 struct GemmParams {
@@ -145,12 +148,13 @@ struct GemmParams {
   RowScale scale;   // of the token rows of x: the result's rows are multiplied by it (EPI 2 / 3 take prep.row_scale)
   int act;          // EPI -1 (the plain epilogue with an activation; one split): kind + 1, every element goes through
                     // llg_act(kind, .) before it is stored.  A variant of its own, so that the plain products carry none of it.
-                    // EPI 1 (the gated epilogue): 0 = the gate passes silu, else the tanh form of gelu.
   // Grouped products (SWAP 1, one token tile per block): token tile t multiplies with the matrix of group tile_group[t],
   // whose rows start at row tile_group[t] * group_rows of w; a tile whose group is negative is left out by every role.
   // The list is written by a kernel earlier in the step, so nothing of w is requested ahead of the dependency wait.
   const int* tile_group;
   int group_rows;
+  GateForm gate;            // EPI 1 (the gated epilogue)
+  const float* row_weight;  // EPI 1, SWAP 1: null, or one number per token row that both products are multiplied by
 };
 
 // The activation of an epilogue on sixteen values.  The square of relu is two instructions a value and stays in line; the
@@ -418,7 +422,7 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
   } else {
     // ---- epilogue: warps 0-3, each its quarter of the lanes: tensor memory -> registers -> out ----------------------
     pdl_wait();                 // before anything of the previous kernel is read or overwritten
-    const float gate_a = EPI == 1 && p.act ? LLG_GELU_GATE_A : 1.0f, gate_b = EPI == 1 && p.act ? LLG_GELU_GATE_B : 0.0f;
+    const GateForm gate = p.gate;
     int round = 0;
     for (int tile = blockIdx.x; tile < total_tiles; tile += gridDim.x, ++round) {
       if (grouped && group_of(tile) < 0) { --round; continue; }
@@ -535,7 +539,7 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
           for (int mt = 0; mt < MT; ++mt) {
             if (o0 + mt * BM >= p.o) break;
             const int tok = o0 + mt * BM + warp * 32 + lane;
-            const float rs = tok < p.o ? row_scale_of(p.scale, tok) : 1.0f;
+            const float rs = tok >= p.o ? 1.0f : (EPI == 1 && p.row_weight) ? p.row_weight[tok] : row_scale_of(p.scale, tok);
             OT* row = out + (long long)tok * width;
             constexpr int COLS = EPI == 1 ? TN / 2 : TN;
   #pragma unroll
@@ -552,7 +556,7 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
   #pragma unroll
                 for (int c = 0; c < 16; ++c) {
                   const float g = __uint_as_float(r[c]) * rs;
-                  v[c] = gate_act(gate_a, gate_b, g) * (__uint_as_float(ru[c]) * rs);
+                  v[c] = gate_act(gate, g, __uint_as_float(ru[c]) * rs);
                 }
               } else {
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -651,7 +655,7 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
                 for (int c = 0; c < 16; ++c) {
                   const float rs = p.scale.ss ? col_scale[c0 + 16 * q + c] : 1.0f;
                   const float g = __uint_as_float(rg[q][c]) * rs, u = __uint_as_float(ru[q][c]) * rs;
-                  v[c] = gate_act(gate_a, gate_b, g) * u;
+                  v[c] = gate_act(gate, g, u);
                 }
                 OT* dst = out + (long long)(n0 + c0 + 16 * q) * inter + f;
   #pragma unroll
@@ -774,11 +778,12 @@ LLG_API int llg_gemm_tc_splits(int k, int splits) {
 // `scale` (may be null): what a norm left for the rows of x; the rows of the result are multiplied by it (with several
 // splits every partial is).
 static int gemm_tc_run(const void* x, const void* w, void* out, int out_dtype, int n, int o, int k, int splits,
-                       int tile_n, int gated_features, const RowScale* scale, int act, cudaStream_t stream);
+                       int tile_n, int gated_features, const RowScale* scale, int act, const GateForm& gate, cudaStream_t stream);
+static const GateForm SILU_FORM = {1.0f, 0.0f, INFINITY, 0.0f};
 
 LLG_API int llg_gemm_tc(const void* x, const void* w, void* out, int out_dtype, int n, int o, int k, int splits,
                         int tile_n, int gated_features, const RowScale* scale, cudaStream_t stream) {
-  return gemm_tc_run(x, w, out, out_dtype, n, o, k, splits, tile_n, gated_features, scale, 0, stream);
+  return gemm_tc_run(x, w, out, out_dtype, n, o, k, splits, tile_n, gated_features, scale, 0, SILU_FORM, stream);
 }
 
 // The gated product (llg_gemm_tc with gated_features > 0) with another activation of the gate than silu: out[n][F] =
@@ -787,7 +792,15 @@ LLG_API int llg_gemm_tc_gated(const void* x, const void* w, void* out, int out_d
                               int gated_features, int kind, const RowScale* scale, cudaStream_t stream) {
   LLG_REQUIRE((kind == 1 || kind == 2) && gated_features > 0, "gemm_tc_gated: activation kind %d (1 gelu, 2 silu), %d features",
               kind, gated_features);
-  return gemm_tc_run(x, w, out, out_dtype, n, o, k, 1, tile_n, gated_features, scale, kind == 2 ? 0 : kind + 1, stream);
+  const GateForm gelu = {LLG_GELU_GATE_A, LLG_GELU_GATE_B, INFINITY, 0.0f};
+  return gemm_tc_run(x, w, out, out_dtype, n, o, k, 1, tile_n, gated_features, scale, 0, kind == 2 ? SILU_FORM : gelu, stream);
+}
+
+// The gated product with any form of gating.
+LLG_API int llg_gemm_tc_gate_form(const void* x, const void* w, void* out, int out_dtype, int n, int o, int k, int tile_n,
+                                  int gated_features, const GateForm* form, const RowScale* scale, cudaStream_t stream) {
+  LLG_REQUIRE(gated_features > 0, "gemm_tc_gate_form: %d features", gated_features);
+  return gemm_tc_run(x, w, out, out_dtype, n, o, k, 1, tile_n, gated_features, scale, 0, *form, stream);
 }
 
 // out[n][o] = act(x w^T) in one split, the activation (kind as in llg_act, common.cuh) applied to the float32 sums
@@ -795,18 +808,18 @@ LLG_API int llg_gemm_tc_gated(const void* x, const void* w, void* out, int out_d
 LLG_API int llg_gemm_tc_act(const void* x, const void* w, void* out, int out_dtype, int n, int o, int k, int kind,
                             const RowScale* scale, cudaStream_t stream) {
   LLG_REQUIRE(kind >= 0 && kind < LLG_ACT_KINDS, "gemm_tc_act: activation kind %d is not known", kind);
-  return gemm_tc_run(x, w, out, out_dtype, n, o, k, 1, 0, 0, scale, kind + 1, stream);
+  return gemm_tc_run(x, w, out, out_dtype, n, o, k, 1, 0, 0, scale, kind + 1, SILU_FORM, stream);
 }
 
 static int gemm_tc_run(const void* x, const void* w, void* out, int out_dtype, int n, int o, int k, int splits,
-                       int tile_n, int gated_features, const RowScale* scale, int act, cudaStream_t stream) {
+                       int tile_n, int gated_features, const RowScale* scale, int act, const GateForm& gate, cudaStream_t stream) {
   const RowScale rs = scale ? *scale : RowScale{nullptr, 0, 0.f, 0.f};
   LLG_REQUIRE(llg_gemm_tc_supported(x, w, n, o, k), "gemm_tc: needs k %% 8 == 0 and 16-byte aligned operands (n=%d o=%d k=%d)",
               n, o, k);
   splits = llg_gemm_tc_splits(k, splits);
   LLG_REQUIRE(out_dtype == LLG_F32 || (out_dtype == LLG_BF16 && splits == 1), "gemm_tc: bfloat16 output needs one split");
   const bool gated = gated_features > 0;
-  LLG_REQUIRE(act == 0 || gated || (splits == 1 && out_dtype == LLG_BF16),
+  LLG_REQUIRE(act == 0 || (splits == 1 && out_dtype == LLG_BF16),
               "gemm_tc: an activation needs one split and bfloat16 output");
   LLG_REQUIRE(!gated || (splits == 1 && o == ((gated_features + BM - 1) / BM) * 2 * BM),
               "gemm_tc: the gated epilogue needs one split and ceil(features / 128) * 256 rows of w (features=%d rows=%d splits=%d)",
@@ -816,7 +829,7 @@ static int gemm_tc_run(const void* x, const void* w, void* out, int out_dtype, i
   if (n >= 256 && tile_n <= 0) {
     // ---- prompt steps: activations are the first operand (128 tokens per tile), up to 256 features per tile ----
     // in this orientation the kernel's first-operand rows (field o) are the tokens, the second's (field n) the features
-    GemmParams ps{out, /*n=*/o, /*o=*/n, k, (nkb + splits - 1) / splits, gated_features, o / 2, BM, QkPrepArgs{}, rs, act};
+    GemmParams ps{out, /*n=*/o, /*o=*/n, k, (nkb + splits - 1) / splits, gated_features, o / 2, BM, QkPrepArgs{}, rs, act, nullptr, 0, gate, nullptr};
     // Tile shape: blocks run in rounds of one per SM (148 on a B200); a round costs its tile's width, and a narrower tile can save a
     // round (4096 features: 16 tiles of 256 in two token rows of 8 are 128 blocks, 18 of 240 are 144).  Two token
     // tiles per block halve the weight traffic per flop (worth about 15 %) but double the tile.
@@ -883,7 +896,7 @@ static int gemm_tc_run(const void* x, const void* w, void* out, int out_dtype, i
     if (gate_rows < 16) gate_rows = 16;
     if (gate_rows > BM) gate_rows = BM;
   }
-  GemmParams p{out, n, o, k, (nkb + splits - 1) / splits, gated_features, o / 2, gate_rows, QkPrepArgs{}, rs, act};
+  GemmParams p{out, n, o, k, (nkb + splits - 1) / splits, gated_features, o / 2, gate_rows, QkPrepArgs{}, rs, act, nullptr, 0, gate, nullptr};
   LLG_REQUIRE(splits <= 65535, "gemm_tc: grid too large");
   LLG_REQUIRE(tensor_map(w, o, k, gated ? gate_rows : BM, &map_w) && tensor_map(x, n, k, tile_n, &map_x),
               "gemm_tc: cuTensorMapEncodeTiled failed or is not available");
@@ -924,19 +937,22 @@ static int gemm_tc_run(const void* x, const void* w, void* out, int out_dtype, i
 // tiles of 128 rows each belong to one group (tile_group[t], negative: the tile is left out and its rows of out are not
 // written).  w holds the groups' matrices one after another, group_rows rows each: plain rows (o of them, out float32 or
 // bfloat16) or, with gated_features, the gated layout (gate rows filled up to a multiple of 128, then the up rows; out is
-// [rows][gated_features] = silu(gate) * up).  Tokens are the tensor cores' rows, as in a prompt step's products.
+// [rows][gated_features], what `form` makes of gate and up (null: silu(gate) * up), both multiplied by row_weight[r] first
+// where given).  Tokens are the tensor cores' rows, as in a prompt step's products.
 LLG_API int llg_gemm_tc_grouped(const void* x, const void* w, void* out, int out_dtype, int rows, int o, int k, int gated_features,
-                                const int* tile_group, int n_groups, int group_rows, cudaStream_t stream) {
+                                const int* tile_group, int n_groups, int group_rows, const GateForm* form,
+                                const float* row_weight, cudaStream_t stream) {
   LLG_REQUIRE(rows > 0 && rows % BM == 0, "gemm_tc_grouped: %d rows are no multiple of %d", rows, BM);
   LLG_REQUIRE(tile_group != nullptr && n_groups > 0 && group_rows >= o, "gemm_tc_grouped: needs the tiles' groups and their rows of w");
   LLG_REQUIRE(llg_gemm_tc_supported(x, w, rows, o, k), "gemm_tc_grouped: needs k %% 8 == 0 and 16-byte aligned operands (k=%d)", k);
   const bool gated = gated_features > 0;
   LLG_REQUIRE(!gated || (o == ((gated_features + BM - 1) / BM) * 2 * BM && out_dtype == LLG_BF16),
               "gemm_tc_grouped: the gated epilogue needs ceil(features / 128) * 256 rows of w per group and bfloat16 output");
+  LLG_REQUIRE(gated || (!form && !row_weight), "gemm_tc_grouped: a form of gating and row weights go with the gated layout");
   LLG_REQUIRE((long long)n_groups * group_rows < 2147483647LL, "gemm_tc_grouped: too many rows of w");
   const int nkb = (k + BK - 1) / BK;
   const RowScale rs{nullptr, 0, 0.f, 0.f};
-  GemmParams ps{out, /*n=*/o, /*o=*/rows, k, nkb, gated_features, o / 2, BM, QkPrepArgs{}, rs, 0, tile_group, group_rows};
+  GemmParams ps{out, /*n=*/o, /*o=*/rows, k, nkb, gated_features, o / 2, BM, QkPrepArgs{}, rs, 0, tile_group, group_rows, form ? *form : SILU_FORM, row_weight};
   CUtensorMap map_w, map_x;
   LLG_REQUIRE(tensor_map(x, rows, k, BM, &map_x) && tensor_map(w, n_groups * group_rows, k, gated ? 128 : 256, &map_w),
               "gemm_tc_grouped: cuTensorMapEncodeTiled failed or is not available");

@@ -38,6 +38,23 @@ __device__ __forceinline__ float row_scale_of(const RowScale& s, long long row) 
 }
 #endif
 
+// What a gated feed-forward makes of a gate value g and an up value u:
+//   g' = min(g, limit), u' = clamp(u, -limit, limit);   g' sigmoid(g' (a + b g'^2)) (u' + up_offset)
+// silu is (1, 0), the tanh form of gelu (2 c, 2 c 0.044715) with c = sqrt(2 / pi); both with an infinite limit and
+// up_offset 0.  A gate that passes g sigmoid(alpha g) is (alpha, 0).
+struct GateForm {
+  float a, b, limit, up_offset;
+};
+
+#ifdef __CUDACC__
+// (expf and an ordinary division: for kernels whose time the epilogue does not decide)
+__device__ __forceinline__ float gate_form_of(const GateForm& f, float g, float u) {
+  g = fminf(g, f.limit);
+  u = fmaxf(fminf(u, f.limit), -f.limit) + f.up_offset;
+  return g / (1.0f + expf(-g * fmaf(f.b * g, g, f.a))) * u;
+}
+#endif
+
 struct QkPrepArgs {
   const void* qkv;            // [n_partials][n_tokens][(nh + 2 nkv) * hd], float32 or bfloat16
   int qkv_dtype;
@@ -74,6 +91,7 @@ struct QkPrepArgs {
   const float* v_mix;         // one number lam, or null: with v_first_in the values become (1 - lam) v + lam v_first_in
   const float* v_first_in;    // [n_tokens][nkv][vd] float32 or null
   float* v_first_out;         // [n_tokens][nkv][vd] float32 or null: receives the values as projected (before any blend)
+  float* gate_out;            // [n_tokens][nh] or null: a row of qkv then ends with nh more numbers z, and gate_out = sigmoid(z)
 };
 
 // Attention for a step with several tokens per sequence (attention_simt.cu, attention_mma.cu, attention_tc.cu).
@@ -104,6 +122,9 @@ struct PrefillArgs {
   const float* sinks;       // [nh] or null: with has_sink, query head h's sink has the score sinks[h] instead of sink_score
   int chunked;              // 1: `window` is a chunk size: a query at position p sees the keys from (p / window) * window
                             // on (its own chunk, counted from position 0) instead of the last `window` keys
+  // Only the kernels of attention_mix.cu read these:
+  float softcap;            // > 0: a score s becomes softcap * tanh(s / softcap)
+  const float* head_mix;    // [nh][nh] or null: then head h's score is sum_g head_mix[h][g] * (head g's score)
 };
 
 // Attention of one new token per sequence, split kernels (attention_simt.cu, attention_mma.cu).
@@ -127,6 +148,8 @@ struct DecodeArgs {
   const float* gate;        // [B][nh] or null
   const float* sinks;       // as in PrefillArgs
   int chunked;
+  float softcap;            // as in PrefillArgs (attention_mix.cu only)
+  const float* head_mix;
 };
 
 // Attention of one new token per sequence, TMA kernel (attention_decode_tma.cu).
@@ -206,18 +229,20 @@ struct QkvRowPrepArgs {
 };
 
 // Layer norm fused with the residual add (layernorm.cu).  For output row j (token r = rows ? rows[j] : j):
-//   v = residual[r] + scale * (sum over all given sets of partials)      (written back when there are any)
+//   v = residual[r] + scale * (sum over all given sets of gain_i * partials)      (written back when there are any)
 //   out[j] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight + bias
+// A set's gain is a vector that its sum is multiplied by element by element (null: 1).
 // Up to LLG_LN_BRANCHES sets of partials (sublayers that ran side by side on the same norm's output).
 #define LLG_LN_BRANCHES 4
 struct LayerNormArgs {
   float* residual;            // [n_tokens][hidden]
   const float* branch[LLG_LN_BRANCHES];   // each [n_partials[i]][n_tokens][hidden] or null
   int n_partials[LLG_LN_BRANCHES];
+  const float* gain[LLG_LN_BRANCHES];     // each [hidden] or null
   long long partial_stride;   // elements between partials (n_tokens * hidden)
   float scale;
   const void* weight;         // [hidden]
-  const void* bias;           // [hidden]
+  const void* bias;           // [hidden] or null
   int w_dtype;
   float eps;
   void* out;                  // [n_out][hidden]
@@ -285,10 +310,12 @@ struct MinGruArgs {
 //            score is the sum of its group_top largest s, and only experts of the keep_groups best groups are eligible;
 //            the `top` eligible experts of largest s, weights = s / (sum of the chosen s + sum_eps) * scale.
 //   score 2: s = softmax over all experts' logits; the `top` experts of largest s, weights as for score 1.
+// raw = 1 (scores 1 and 2): weights = s * scale, not divided by the chosen scores' sum.
 struct RouterRule {
   int score;
   int groups, keep_groups, group_top;
   float scale, sum_eps;
+  int raw;
 };
 
 // Preparation for latent attention (latent.cu: latent_prep).  A row of the input product holds, per token, up to three
@@ -324,6 +351,8 @@ struct LatentPrepArgs {
   const int* seq_of_token;
   const int* slots;
   int n_tokens, nh, dim, rdim, rank;
+  int gate_col;               // with gate_out: the column of nh numbers z, one per head
+  float* gate_out;            // [n_tokens][nh] or null: sigmoid(z)
 };
 
 // y[n][h][o] = sum_k w[h][o][k] x[n][h][k] (latent.cu: head_linear).  x and y may be parts of wider rows: their
@@ -346,7 +375,8 @@ struct HeadLinearArgs {
 #define LLG_MOE_MAX_TOP 32
 
 // y[r][o] = sum_k w[e][o][k] x[src(r)][k] for every row r of every tile with an expert e; GATED: two matrices per expert
-// and y = silu(w . x) * (w2 . x).
+// and y = gate(w . x, w2 . x) as GateForm says.  With row_weight both products of row r are multiplied by row_weight[r]
+// first (the products are linear: it is the row's input that is weighed).
 struct GroupedLinearArgs {
   const void* x;              // [.][n_in]; row src(r) = token_of_row ? token_of_row[r] : r
   const int* token_of_row;    // [rows] or null
@@ -362,6 +392,8 @@ struct GroupedLinearArgs {
   long long x_group_stride, y_group_stride;   // elements by which group e's rows are shifted in x and y
   int n_rows;                                 // without token_of_row: rows from n_rows on are neither read nor written (0: all are)
   long long w_group_stride;                   // elements between the groups' matrices in w and w2 (0: n_out * n_in)
+  const float* row_weight;                    // [rows] or null
+  GateForm gate;                              // GATED
 };
 
 // Residual add of several terms, each optionally RMS-normed first, fused with the norm of the sum (addnorm.cu).  For
@@ -510,4 +542,41 @@ struct RetentionArgs {
   float* carry;               // [n_seqs][pieces][nh][dim][vdim] or null
   int pieces;
   int n_seqs, n_tokens, nh, dim, vdim;
+};
+
+// A matrix memory per head with exponential gates and a running maximum (matrix_memory.cu).  A row of the input product
+// holds q and k (nh * dim each), v and the output gate's arguments g (nh * vdim each) and the two gates' arguments (nh
+// each) at their columns.  Per head, with q times q_scale:
+//   i = cap tanh((zi + i_bias) / cap),  f = logsigmoid(cap tanh((zf + f_bias) / cap))
+//   m' = max(f + m, i);  S' = e^{f + m - m'} S + e^{i - m'} k v^T;  n' = e^{f + m - m'} n + e^{i - m'} k
+//   o = S'^T q / (max(|n' . q|, e^{-m'}) + denom_eps)
+//   out = o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(g)
+// state_s [slots][nh][dim][vdim], state_n [slots][nh][dim] and state_m [slots][nh] hold S, n and m before the step's first
+// token and receive them after its last.  A block owns `cols` columns of a head's S.  A head cut into several runs of
+// columns leaves its o in raw, and n and m in next, and a second kernel finishes (norm, gate, n and m into the state).
+// With carry, pieces of LLG_MEMORY_PIECE tokens run side by side from zero, are joined, and run again; a piece's entry in
+// carry is S [dim][vdim], n [dim] and three numbers: the sum of its f, its own maximum, the maximum it starts from.
+#define LLG_MEMORY_PIECE 128
+#define LLG_MEMORY_CARRY_EXTRA 3
+struct MatrixMemoryArgs {
+  const float* rows;          // [n_partials][n_tokens][row_width]
+  int n_partials;
+  long long partial_stride;
+  int row_width, q_col, k_col, v_col, g_col, i_col, f_col;
+  const float* i_bias;        // [nh] or null
+  const float* f_bias;        // [nh] or null
+  float gate_cap, q_scale, denom_eps, eps;
+  const float* norm_w;        // [nh * vdim]
+  float* state_s;
+  float* state_n;
+  float* state_m;
+  const int* slots;           // [n_seqs]
+  const int* cu_tokens;       // [n_seqs + 1]
+  void* out;                  // [n_tokens][nh * vdim]
+  int out_dtype;
+  float* carry;               // [n_seqs][pieces][nh][dim * vdim + dim + LLG_MEMORY_CARRY_EXTRA] or null
+  int pieces;
+  float* raw;                 // [n_tokens][nh * vdim], where cols < vdim
+  float* next;                // [n_seqs][nh][dim + 1], where cols < vdim and there is no carry
+  int n_seqs, n_tokens, nh, dim, vdim, cols;
 };

@@ -92,7 +92,7 @@ __device__ __forceinline__ void query_latent_norm(const LatentPrepArgs& a, int n
 }
 
 // One warp per unit of a token.  The units a launch has, in this order: the nh query heads (q_col >= 0), the latent with
-// the shared key part (kv_col >= 0).  The blocks behind the units' (unit_blocks of them) take the queries' latent
+// the shared key part (kv_col >= 0), the heads' gates (gate_out).  The blocks behind the units' (unit_blocks of them) take the queries' latent
 // (cq_col >= 0), one block a token.
 template <typename OT, typename WT>
 __global__ void latent_prep_kernel(LatentPrepArgs a, int unit_blocks, int cq_vec) {
@@ -104,7 +104,7 @@ __global__ void latent_prep_kernel(LatentPrepArgs a, int unit_blocks, int cq_vec
   }
   const int warps = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int q_units = a.q_col >= 0 ? a.nh : 0, kv_units = a.kv_col >= 0 ? 1 : 0;
-  const int units = q_units + kv_units;
+  const int units = q_units + kv_units + (a.gate_out ? 1 : 0);
   const long long item = (long long)blockIdx.x * warps + warp;
   if (item >= (long long)a.n_tokens * units) return;
   const int n = (int)(item / units), u = (int)(item % units);
@@ -132,6 +132,10 @@ __global__ void latent_prep_kernel(LatentPrepArgs a, int unit_blocks, int cq_vec
       qo[e0] = from_f32<OT>(x0 * cs[i] - x1 * sn[i]);
       qo[e1] = from_f32<OT>(x1 * cs[i] + x0 * sn[i]);
     }
+    return;
+  }
+  if (u == q_units + kv_units) {
+    for (int h = lane; h < a.nh; h += 32) a.gate_out[(long long)n * a.nh + h] = 1.0f / (1.0f + expf(-summed(a.gate_col + h)));
     return;
   }
   const WT* w = (const WT*)a.c_norm_w;
@@ -282,10 +286,11 @@ LLG_API int llg_latent_prep(const LatentPrepArgs* args, int out_dtype, cudaStrea
   LLG_REQUIRE(a.rdim == 0 || (a.cos_table && a.sin_table && a.table_positions > 0), "latent_prep: rotated elements need the tables");
   LLG_REQUIRE(!a.k_pages || (a.page_table && a.slots && a.seq_of_token && a.ring_pages > 0),
               "latent_prep: a cache write needs page_table, slots and seq_of_token");
+  LLG_REQUIRE(!a.gate_out || (a.gate_col >= 0 && a.gate_col + a.nh <= a.row_width), "latent_prep: the gates' columns must lie inside the row");
   LLG_REQUIRE((!a.v_new || a.k_new) && (!a.v_pages || a.k_pages), "latent_prep: values are written beside keys only");
   if (a.n_tokens == 0) return 0;
   const int warps = 4;
-  const long long items = (long long)a.n_tokens * ((a.q_col >= 0 ? a.nh : 0) + (a.kv_col >= 0 ? 1 : 0));
+  const long long items = (long long)a.n_tokens * ((a.q_col >= 0 ? a.nh : 0) + (a.kv_col >= 0 ? 1 : 0) + (a.gate_out ? 1 : 0));
   const int unit_blocks = (int)((items + warps - 1) / warps);
   const int cq_vec = a.cq_col >= 0 && a.cq_col % 4 == 0 && a.cq_rank % 4 == 0 && a.row_width % 4 == 0 && a.partial_stride % 4 == 0 &&
              (size_t)a.rows % 16 == 0 && (size_t)a.cq_norm_w % 16 == 0 && (size_t)a.cq_out % 16 == 0;

@@ -1,4 +1,4 @@
-// Layer norm (mean and variance, weight and bias) fused with the residual add; see LayerNormArgs in kernel_args.h.
+// Layer norm (mean and variance, weight and, where given, bias) fused with the residual add; see LayerNormArgs in kernel_args.h.
 // One block per output row; the row is kept in shared memory between the passes (sum, squared deviations, output),
 // so the variance is the mean of the squared deviations from the mean and not a difference of two large sums.  The
 // residual, every sum and both statistics are float32.
@@ -30,6 +30,16 @@ __global__ void add_layernorm_kernel(LayerNormArgs a) {
         for (int b = 0; b < LLG_LN_BRANCHES; ++b) {
           if (!a.branch[b]) break;
           const float* p = a.branch[b] + (long long)r * hidden + i;
+          if (a.gain[b]) {
+            float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int s = 0; s < a.n_partials[b]; ++s) {
+              const float4 u = *reinterpret_cast<const float4*>(p + s * a.partial_stride);
+              g.x += u.x; g.y += u.y; g.z += u.z; g.w += u.w;
+            }
+            const float4 k = *reinterpret_cast<const float4*>(a.gain[b] + i);
+            t.x = fmaf(k.x, g.x, t.x); t.y = fmaf(k.y, g.y, t.y); t.z = fmaf(k.z, g.z, t.z); t.w = fmaf(k.w, g.w, t.w);
+            continue;
+          }
           for (int s = 0; s < a.n_partials[b]; ++s) {
             const float4 u = *reinterpret_cast<const float4*>(p + s * a.partial_stride);
             t.x += u.x; t.y += u.y; t.z += u.z; t.w += u.w;
@@ -51,6 +61,12 @@ __global__ void add_layernorm_kernel(LayerNormArgs a) {
         for (int b = 0; b < LLG_LN_BRANCHES; ++b) {
           if (!a.branch[b]) break;
           const float* p = a.branch[b] + (long long)r * hidden + i;
+          float g = 0.f;
+          if (a.gain[b]) {
+            for (int s = 0; s < a.n_partials[b]; ++s) g += p[s * a.partial_stride];
+            t = fmaf(a.gain[b][i], g, t);
+            continue;
+          }
           for (int s = 0; s < a.n_partials[b]; ++s) t += p[s * a.partial_stride];
         }
         v = fmaf(a.scale, t, v);
@@ -71,7 +87,7 @@ __global__ void add_layernorm_kernel(LayerNormArgs a) {
   const WT* bs = (const WT*)a.bias;
   OT* o = (OT*)a.out + (long long)j * hidden;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x)
-    o[i] = from_f32<OT>((row[i] - mean) * inv * to_f32(w[i]) + to_f32(bs[i]));
+    o[i] = from_f32<OT>((row[i] - mean) * inv * to_f32(w[i]) + (bs ? to_f32(bs[i]) : 0.f));
 }
 
 }  // namespace
@@ -83,10 +99,11 @@ LLG_API int llg_add_layernorm(const LayerNormArgs* args, cudaStream_t stream) {
   for (int b = 0; b < LLG_LN_BRANCHES; ++b) {
     LLG_REQUIRE(!a.branch[b] || a.n_partials[b] >= 1, "add_layernorm: a set of partials needs at least one");
     LLG_REQUIRE(!a.branch[b] || b == 0 || a.branch[b - 1], "add_layernorm: sets of partials must be given in order");
+    LLG_REQUIRE(!a.gain[b] || a.branch[b], "add_layernorm: a gain without its set of partials");
   }
   if (a.n_out == 0) return 0;
   bool vec = a.hidden % 4 == 0 && a.partial_stride % 4 == 0 && ((uintptr_t)a.residual % 16) == 0;
-  for (int b = 0; b < LLG_LN_BRANCHES; ++b) vec = vec && ((uintptr_t)a.branch[b] % 16) == 0;
+  for (int b = 0; b < LLG_LN_BRANCHES; ++b) vec = vec && ((uintptr_t)a.branch[b] % 16) == 0 && ((uintptr_t)a.gain[b] % 16) == 0;
   const int threads = a.hidden >= 4096 ? 512 : (a.hidden >= 1024 ? 256 : 128);
   const size_t smem = (size_t)a.hidden * sizeof(float);
   LLG_REQUIRE(smem <= 200 * 1024, "add_layernorm: rows of %d elements do not fit shared memory", a.hidden);

@@ -10,7 +10,8 @@
 //                 alone, and a token's rows are added in the order of its choices).
 //   grouped products: a block takes one tile of rows (one expert) and a run of outputs: bfloat16 with rows that start on
 //                 16-byte boundaries on the tensor cores (mma.sync), everything else on the CUDA cores.
-//   moe_combine : out[n] = sum_k weight[n][k] y[row of (n, k)] + the shared expert's partial sums.
+//   moe_combine : out[n] = sum_k weight[n][k] y[row of (n, k)] + the shared expert's partial sums (a design whose weights
+//                 are on the experts' inputs has them in the first product's epilogue, and adds its rows as they are).
 #include "common.cuh"
 #include "kernel_args.h"
 
@@ -111,6 +112,10 @@ __device__ __forceinline__ void choose_and_weigh(float* z, float* gsc, float* ch
     __syncwarp();
   }
   if (rule.score != 0) {
+    if (rule.raw) {                                 // the chosen scores as they are
+      if (lane < top) weight[lane] = chosen[lane] * rule.scale;
+      return;
+    }
     // the chosen scores divided by their sum
     const float sv = lane < top ? chosen[lane] : 0.f;
     const float total = warp_sum(sv);
@@ -183,13 +188,17 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
 
 __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ choice, int n_pairs, int top, int n_exp,
                                                         int* __restrict__ row_of_pair, int* __restrict__ token_of_row,
-                                                        int* __restrict__ tile_expert, int cap, int tile_rows) {
+                                                        int* __restrict__ tile_expert, int cap, int tile_rows,
+                                                        const float* __restrict__ weight, float* __restrict__ weight_of_row) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ int counts[LLG_MOE_MAX_EXPERTS], starts[LLG_MOE_MAX_EXPERTS], cursor[LLG_MOE_MAX_EXPERTS];
   const int tid = threadIdx.x, nt = blockDim.x;
   for (int e = tid; e < n_exp; e += nt) counts[e] = cursor[e] = 0;
-  for (int r = tid; r < cap; r += nt) token_of_row[r] = -1;
+  for (int r = tid; r < cap; r += nt) {
+    token_of_row[r] = -1;
+    if (weight_of_row) weight_of_row[r] = 0.f;
+  }
   for (int t = tid; t < cap / tile_rows; t += nt) tile_expert[t] = -1;
   __syncthreads();
   for (int p = tid; p < n_pairs; p += nt) {
@@ -215,6 +224,7 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
     if (e >= 0 && e < n_exp) {
       row = starts[e] + atomicAdd(&cursor[e], 1);
       token_of_row[row] = p / top;
+      if (weight_of_row) weight_of_row[row] = weight[p];
     }
     row_of_pair[p] = row;
   }
@@ -278,7 +288,10 @@ __global__ void __launch_bounds__(256) grouped_linear_kernel(GroupedLinearArgs a
   for (int i = 0; i < RPT; ++i) {
     const int r = r0 + ty + 8 * i;
     float v = acc[i];
-    if (GATED) v = v / (1.0f + expf(-v)) * acc2[i];
+    if (GATED) {
+      const float rw = a.row_weight ? a.row_weight[r] : 1.0f;
+      v = gate_form_of(a.gate, v * rw, acc2[i] * rw);
+    }
     y[(long long)r * a.n_out + o] = from_f32<YT>(v);         // filling rows hold zeros
   }
 }
@@ -288,7 +301,7 @@ __global__ void __launch_bounds__(256) grouped_linear_kernel(GroupedLinearArgs a
 // A block of four warps takes one tile of LLG_MOE_TILE rows (one expert) and MM_O outputs; the activations' rows (gathered
 // through token_of_row) and the expert's matrix rows arrive in shared memory by 16-byte asynchronous copies, two stages
 // deep, in k-blocks of MM_K; every warp owns MM_O / 4 outputs of all rows and multiplies with mma.sync m16n8k16 (bfloat16
-// in, float32 sums).  GATED: a second matrix's tile beside the first, and silu(first) * second is what is stored.
+// in, float32 sums).  GATED: a second matrix's tile beside the first, and what the gate's form makes of the two is stored.
 constexpr int MM_O = 128, MM_K = 64, MM_PAD = 8;            // MM_PAD halves between rows: fragment loads meet no bank twice
 constexpr int MM_LD = MM_K + MM_PAD;
 
@@ -409,7 +422,10 @@ __global__ void __launch_bounds__(128) grouped_linear_mma_kernel(GroupedLinearAr
         const int o = o0 + warp * (MM_O / 4) + j * 8 + 2 * t + (c & 1);
         if (o >= a.n_out || (a.n_rows && r >= a.n_rows)) continue;
         float v = acc[i][j][c];
-        if (GATED) v = v / (1.0f + expf(-v)) * acc2[i][j][c];
+        if (GATED) {
+          const float rw = a.row_weight ? a.row_weight[r] : 1.0f;
+          v = gate_form_of(a.gate, v * rw, acc2[i][j][c] * rw);
+        }
         y[(long long)r * y_ld + o] = from_f32<YT>(v);
       }
 }
@@ -438,7 +454,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     float v = 0.f;
     for (int k = 0; k < top; ++k) {
       const int row = row_of_pair[(long long)n * top + k];
-      v = fmaf(weight[(long long)n * top + k], y[(long long)row * hidden + d], v);
+      v = fmaf(weight ? weight[(long long)n * top + k] : 1.0f, y[(long long)row * hidden + d], v);
     }
     float sh = 0.f;
     for (int s = 0; s < n_shared; ++s) sh += shared[s * shared_stride + (long long)n * hidden + d];
@@ -460,7 +476,7 @@ __global__ void moe_combine_vec4_kernel(const float* __restrict__ y, const int* 
   float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int k = 0; k < top; ++k) {
     const int row = row_of_pair[(long long)n * top + k];
-    const float wk = weight[(long long)n * top + k];
+    const float wk = weight ? weight[(long long)n * top + k] : 1.0f;
     const float4 u = *reinterpret_cast<const float4*>(y + (long long)row * hidden + d);
     v.x = fmaf(wk, u.x, v.x); v.y = fmaf(wk, u.y, v.y); v.z = fmaf(wk, u.z, v.z); v.w = fmaf(wk, u.w, v.w);
   }
@@ -478,6 +494,7 @@ __global__ void moe_combine_vec4_kernel(const float* __restrict__ y, const int* 
 
 static int check_rule(const char* what, const RouterRule& r, int n_exp, int top) {
   LLG_REQUIRE(r.score >= 0 && r.score <= 2, "%s: score kind %d is not known", what, r.score);
+  LLG_REQUIRE(!r.raw || r.score != 0, "%s: undivided scores go with sigmoid or softmax-over-all scores", what);
   LLG_REQUIRE(r.groups >= 0 && (r.groups == 0 || r.score == 1), "%s: groups of experts go with sigmoid scores", what);
   if (r.groups > 0) {
     LLG_REQUIRE(n_exp % r.groups == 0 && r.keep_groups > 0 && r.keep_groups <= r.groups && r.group_top > 0,
@@ -495,7 +512,7 @@ LLG_API int llg_moe_route(const void* x, int x_dtype, const float* w, const floa
   LLG_REQUIRE(n_exp > 0 && n_exp <= LLG_MOE_MAX_EXPERTS, "moe_route: %d experts are outside [1, %d]", n_exp, LLG_MOE_MAX_EXPERTS);
   LLG_REQUIRE(top > 0 && top <= n_exp && top <= LLG_MOE_MAX_TOP, "moe_route: top %d of %d experts (at most %d)", top, n_exp,
               LLG_MOE_MAX_TOP);
-  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f};
+  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f, 0};
   if (check_rule("moe_route", r, n_exp, top)) return 1;
   if (n_tokens == 0) return 0;
   const size_t smem = (size_t)(hidden + 2 * n_exp + 1) * sizeof(float);
@@ -522,7 +539,7 @@ LLG_API int llg_moe_topk(const float* logits, int n_partials, long long partial_
   LLG_REQUIRE(n_exp > 0 && n_exp <= LLG_MOE_MAX_EXPERTS, "moe_topk: %d experts are outside [1, %d]", n_exp, LLG_MOE_MAX_EXPERTS);
   LLG_REQUIRE(top > 0 && top <= n_exp && top <= LLG_MOE_MAX_TOP, "moe_topk: top %d of %d experts (at most %d)", top, n_exp,
               LLG_MOE_MAX_TOP);
-  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f};
+  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f, 0};
   if (check_rule("moe_topk", r, n_exp, top)) return 1;
   if (n_tokens == 0) return 0;
   llg_launch(moe_topk_kernel, dim3((n_tokens + 3) / 4), dim3(128), (size_t)4 * (2 * n_exp + 1) * sizeof(float), stream, logits,
@@ -530,8 +547,10 @@ LLG_API int llg_moe_topk(const float* logits, int n_partials, long long partial_
   return llg_check_launch("moe_topk");
 }
 
+// weight, weight_of_row: null, or the pairs' weights and [cap] for every row's weight (0 for filling rows).
 LLG_API int llg_moe_plan(const int* choice, int n_pairs, int top, int n_exp, int* row_of_pair, int* token_of_row,
-                         int* tile_expert, int cap, int tile_rows, cudaStream_t stream) {
+                         int* tile_expert, int cap, int tile_rows, const float* weight, float* weight_of_row, cudaStream_t stream) {
+  LLG_REQUIRE((weight == nullptr) == (weight_of_row == nullptr), "moe_plan: weights and their rows come together");
   LLG_REQUIRE(tile_rows > 0, "moe_plan: tiles of %d rows", tile_rows);
   LLG_REQUIRE(n_exp > 0 && n_exp <= LLG_MOE_MAX_EXPERTS, "moe_plan: %d experts are outside [1, %d]", n_exp, LLG_MOE_MAX_EXPERTS);
   LLG_REQUIRE(top > 0 && n_pairs >= 0 && n_pairs % top == 0, "moe_plan: %d pairs, top %d", n_pairs, top);
@@ -539,7 +558,7 @@ LLG_API int llg_moe_plan(const int* choice, int n_pairs, int top, int n_exp, int
   LLG_REQUIRE(cap % tile_rows == 0 && cap >= need, "moe_plan: %d rows, %lld needed (whole tiles)", cap, need);
   if (n_pairs == 0) return 0;
   llg_launch(moe_plan_kernel, dim3(1), dim3(1024), 0, stream, choice, n_pairs, top, n_exp, row_of_pair, token_of_row, tile_expert, cap,
-             tile_rows);
+             tile_rows, weight, weight_of_row);
   return llg_check_launch("moe_plan");
 }
 
@@ -640,7 +659,7 @@ LLG_API int llg_moe_gather_rows(const void* x, const int* token_of_row, void* ou
   return llg_check_launch("moe_gather_rows");
 }
 
-// shared_scale: null, or [n_tokens]: the sum of the shared expert's partials is multiplied by it.
+// weight: null = every pair counts once.  shared_scale: null, or [n_tokens]: the sum of the shared expert's partials is multiplied by it.
 LLG_API int llg_moe_combine(const float* y, const int* row_of_pair, const float* weight, const float* shared, int n_shared,
                             long long shared_stride, const float* shared_scale, float* out, int n_tokens, int hidden, int top,
                             cudaStream_t stream) {

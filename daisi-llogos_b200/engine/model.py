@@ -11,7 +11,7 @@ from typing import Dict, List, Optional, Tuple
 
 import torch
 
-from ..parts.base import Branch, BuildEnv, Part, TensorDecl, part_class, part_families
+from ..parts.base import Branch, BuildEnv, Part, TensorDecl, Term, part_class, part_families
 from ..parts.spec import ModelSpec
 
 # importing the modules registers the stock parts
@@ -22,6 +22,7 @@ from ..parts import feedforward as _feedforward  # noqa: F401
 from ..parts import gated_attention as _gated_attention  # noqa: F401
 from ..parts import hyper as _hyper  # noqa: F401
 from ..parts import latent_attention as _latent_attention  # noqa: F401
+from ..parts import matrix_memory as _matrix_memory  # noqa: F401
 from ..parts import moe as _moe  # noqa: F401
 from ..parts import norm as _norm  # noqa: F401
 from ..parts import position as _position  # noqa: F401
@@ -75,6 +76,7 @@ class DecoderModel:
                         raise ValueError(f"schedule[{e_i}].cache_of = {e.cache_of}: {err}") from None
         self.final_norm = part_class("norm", spec.final_norm.kind)(spec.final_norm.params, spec.final_norm.prefix, self.env)
         self.head = part_class("head", spec.head.kind)(spec.head.params, spec.head.prefix, self.env)
+        self._adds_embedding = any(e.add_embedding for e in spec.schedule)
         self._bound = False
 
     # ---- tensors -------------------------------------------------------------------------
@@ -140,6 +142,13 @@ class DecoderModel:
             residual = self.embedding.forward(ctx)
         for enc in self.encodings.values():
             enc.on_embeddings(residual, ctx)
+        start = None
+        if self._adds_embedding:
+            # the residual is updated in place: later entries that add the embedding's output need a copy of it
+            if residual.dim() != 2:
+                raise ValueError("add_embedding: the residual must be one stream [tokens, hidden]")
+            start = ctx.buffer("embedding.output", residual.shape, torch.float32)
+            start.copy_(residual)
         pending: Optional[Branch] = None
         if runner is not None:
             pending = runner.run(ctx, residual)
@@ -149,6 +158,8 @@ class DecoderModel:
             unit = e.cache_of if e.cache_of is not None else e_i
             view = cache.view(unit, owner=e.cache_of is None, keep_step_kv=e_i in borrowed,
                               shared=shared.setdefault(unit, {}))
+            if e.add_embedding:
+                pending = Branch.of_terms((pending.as_terms() if pending is not None else ()) + (Term(start.unsqueeze(0)),))
             pending = self.blocks[e.layer].forward(residual, pending, ctx, view)
             # what an owner put off until its cache's last reader has run (a ring's writes would
             # overwrite keys that a reader of the same step still needs)

@@ -151,7 +151,7 @@ class BlockRunner:
         if os.environ.get("LLOGOS_RUNNER", "1") == "0" or model.device.type != "cuda" or model.env.ops is not ops:
             return None
         spec = model.spec
-        if not spec.schedule or any(e.cache_of is not None for e in spec.schedule):
+        if not spec.schedule or any(e.cache_of is not None or e.add_embedding for e in spec.schedule):
             return None
         layers, keep, geom, fusable = [], [], None, 1
         for e_i, e in enumerate(spec.schedule):

@@ -118,9 +118,9 @@ def gated_layout(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:
 
 
 def gated_linear(ctx, x: torch.Tensor, w_gated: torch.Tensor, out: torch.Tensor, row_scale=None,
-                 activation: str = "silu") -> None:
+                 activation: str = "silu", form=None) -> None:
     """out[n, i] = act(x . gate_i) * (x . up_i) for a gate/up matrix in ``gated_layout``; ``activation`` is "silu" or
-    "gelu_tanh" (one of ``ops.GATE_ACTIVATIONS``).
+    "gelu_tanh" (one of ``ops.GATE_ACTIVATIONS``).  With ``form`` (an ``ops.GateForm``) out is what that makes of the two products.
 
     On the tensor cores the gating is the epilogue of the product; otherwise the product writes
     gate and up values and the gating kernel follows.  ``row_scale`` as in ``linear``: both products' rows are
@@ -130,6 +130,8 @@ def gated_linear(ctx, x: torch.Tensor, w_gated: torch.Tensor, out: torch.Tensor,
     rows = w_gated.shape[0]
     tc = getattr(ops, "gemm_tc_supported", None)
     kw = {} if activation == "silu" else {"gate_activation": activation}      # the stock form's calls stay as they were
+    if form is not None:
+        kw = {"gate_form": form}
     if tc is not None and tc(x, w_gated) and out.dtype == torch.bfloat16:
         if row_scale is not None:
             ops.gemm_tc(x, w_gated, out.unsqueeze(0), gated_features=out.shape[1], row_scale=row_scale, **kw)
@@ -143,4 +145,4 @@ def gated_linear(ctx, x: torch.Tensor, w_gated: torch.Tensor, out: torch.Tensor,
             ops.gemm_simt(x[r0:r1], w_gated, gu[0], row_scale=row_scale.slice(r0, r1))
         else:
             ops.gemm_simt(x[r0:r1], w_gated, gu[0])
-        ops.silu_mul(gu, out[r0:r1], **({} if activation == "silu" else {"activation": activation}))
+        ops.silu_mul(gu, out[r0:r1], **({"form": form} if form is not None else {} if activation == "silu" else {"activation": activation}))

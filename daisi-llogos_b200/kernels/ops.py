@@ -111,6 +111,25 @@ def _scale_ref(row_scale: Optional[RowScale], rows: int):
     return byref(row_scale.c())
 
 
+class _GateForm(Structure):
+    _fields_ = [("a", c_float), ("b", c_float), ("limit", c_float), ("up_offset", c_float)]
+
+
+class GateForm:
+    """What a gated feed-forward makes of a gate value g and an up value u: with ``g' = min(g, limit)`` and ``u' = clamp(u,
+    -limit, limit)`` it is ``g' sigmoid(alpha g') (u' + up_offset)`` (``limit`` None: no clamping; alpha 1, no limit and offset 0
+    is silu)."""
+
+    def __init__(self, alpha: float = 1.0, limit: Optional[float] = None, up_offset: float = 0.0):
+        if limit is not None and not limit > 0:
+            raise KernelError(f"gate form: the limit must be positive, got {limit}")
+        self.alpha, self.limit, self.up_offset = float(alpha), (None if limit is None else float(limit)), float(up_offset)
+        self.c = _GateForm(self.alpha, 0.0, float("inf") if limit is None else self.limit, self.up_offset)
+
+
+SILU_FORM = GateForm()
+
+
 class _QkPrepArgs(Structure):
     _fields_ = [
         ("qkv", c_void_p), ("qkv_dtype", c_int), ("n_partials", c_int), ("partial_stride", c_longlong),
@@ -124,7 +143,7 @@ class _QkPrepArgs(Structure):
         ("seq_of_token", c_void_p), ("slots", c_void_p),
         ("n_tokens", c_int), ("nh", c_int), ("nkv", c_int), ("hd", c_int),
         ("row_scale", _RowScale),
-        ("vd", c_int), ("v_mix", c_void_p), ("v_first_in", c_void_p), ("v_first_out", c_void_p),
+        ("vd", c_int), ("v_mix", c_void_p), ("v_first_in", c_void_p), ("v_first_out", c_void_p), ("gate_out", c_void_p),
     ]
 
 
@@ -137,7 +156,7 @@ class _PrefillArgs(Structure):
         ("n_tiles", c_int), ("nh", c_int), ("nkv", c_int), ("hd", c_int),
         ("scale", c_float), ("window", c_int), ("n_tokens", c_int), ("n_pages", c_int),
         ("vd", c_int), ("has_sink", c_int), ("sink_score", c_float), ("gate", c_void_p),
-        ("sinks", c_void_p), ("chunked", c_int),
+        ("sinks", c_void_p), ("chunked", c_int), ("softcap", c_float), ("head_mix", c_void_p),
     ]
 
 
@@ -149,7 +168,7 @@ class _DecodeArgs(Structure):
         ("n_seqs", c_int), ("nh", c_int), ("nkv", c_int), ("hd", c_int), ("n_splits", c_int),
         ("scale", c_float), ("window", c_int),
         ("vd", c_int), ("has_sink", c_int), ("sink_score", c_float), ("gate", c_void_p),
-        ("sinks", c_void_p), ("chunked", c_int),
+        ("sinks", c_void_p), ("chunked", c_int), ("softcap", c_float), ("head_mix", c_void_p),
     ]
 
 
@@ -190,6 +209,7 @@ _LN_BRANCHES = 4
 class _LayerNormArgs(Structure):
     _fields_ = [
         ("residual", c_void_p), ("branch", c_void_p * _LN_BRANCHES), ("n_partials", c_int * _LN_BRANCHES),
+        ("gain", c_void_p * _LN_BRANCHES),
         ("partial_stride", c_longlong), ("scale", c_float), ("weight", c_void_p), ("bias", c_void_p), ("w_dtype", c_int),
         ("eps", c_float), ("out", c_void_p), ("out_dtype", c_int), ("rows", c_void_p), ("n_out", c_int), ("hidden", c_int),
     ]
@@ -284,7 +304,7 @@ class _RetentionArgs(Structure):
 
 class _RouterRule(Structure):
     _fields_ = [("score", c_int), ("groups", c_int), ("keep_groups", c_int), ("group_top", c_int), ("scale", c_float),
-                ("sum_eps", c_float)]
+                ("sum_eps", c_float), ("raw", c_int)]
 
 
 class _LatentPrepArgs(Structure):
@@ -298,6 +318,7 @@ class _LatentPrepArgs(Structure):
         ("k_pages", c_void_p), ("v_pages", c_void_p), ("page_table", c_void_p), ("table_width", c_int),
         ("ring_pages", c_int), ("seq_of_token", c_void_p), ("slots", c_void_p),
         ("n_tokens", c_int), ("nh", c_int), ("dim", c_int), ("rdim", c_int), ("rank", c_int),
+        ("gate_col", c_int), ("gate_out", c_void_p),
     ]
 
 
@@ -315,6 +336,19 @@ class _GroupedLinearArgs(Structure):
         ("y", c_void_p), ("rows", c_int), ("n_in", c_int), ("n_out", c_int),
         ("x_row_stride", c_longlong), ("y_row_stride", c_longlong), ("x_group_stride", c_longlong),
         ("y_group_stride", c_longlong), ("n_rows", c_int), ("w_group_stride", c_longlong),
+        ("row_weight", c_void_p), ("gate", _GateForm),
+    ]
+
+
+class _MatrixMemoryArgs(Structure):
+    _fields_ = [
+        ("rows", c_void_p), ("n_partials", c_int), ("partial_stride", c_longlong),
+        ("row_width", c_int), ("q_col", c_int), ("k_col", c_int), ("v_col", c_int), ("g_col", c_int), ("i_col", c_int),
+        ("f_col", c_int), ("i_bias", c_void_p), ("f_bias", c_void_p),
+        ("gate_cap", c_float), ("q_scale", c_float), ("denom_eps", c_float), ("eps", c_float), ("norm_w", c_void_p),
+        ("state_s", c_void_p), ("state_n", c_void_p), ("state_m", c_void_p), ("slots", c_void_p), ("cu_tokens", c_void_p),
+        ("out", c_void_p), ("out_dtype", c_int), ("carry", c_void_p), ("pieces", c_int), ("raw", c_void_p), ("next", c_void_p),
+        ("n_seqs", c_int), ("n_tokens", c_int), ("nh", c_int), ("dim", c_int), ("vdim", c_int), ("cols", c_int),
     ]
 
 
@@ -365,6 +399,7 @@ def _load_lib(name: str):
         lib.llg_kv_write.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
                                      c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.llg_silu_mul.argtypes = [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_void_p]
+        lib.llg_gate_form_mul.argtypes = [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_int, POINTER(_GateForm), c_void_p]
         lib.llg_gate_mul.argtypes = [c_void_p, c_int, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.llg_tanh_cap.argtypes = [c_void_p, c_longlong, c_float, c_void_p]
         lib.llg_scatter_i32.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_void_p]
@@ -384,8 +419,10 @@ def _load_lib(name: str):
         lib.llg_gemm_tc_gated.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                           POINTER(_RowScale), c_void_p]
         lib.llg_gemm_tc_qkv.argtypes = [c_void_p, c_void_p, c_int, c_int, POINTER(_QkPrepArgs), c_void_p]
+        lib.llg_gemm_tc_gate_form.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int,
+                                              POINTER(_GateForm), POINTER(_RowScale), c_void_p]
         lib.llg_gemm_tc_grouped.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int,
-                                            c_int, c_void_p]
+                                            c_int, POINTER(_GateForm), c_void_p, c_void_p]
         lib.llg_gemm_tc_act.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                         POINTER(_RowScale), c_void_p]
     elif name == "attention_simt":
@@ -393,6 +430,16 @@ def _load_lib(name: str):
         lib.llg_attn_decode_simt.argtypes = [POINTER(_DecodeArgs), c_void_p, c_int, c_void_p]
         lib.llg_attn_decode_scratch_floats.argtypes = [c_int, c_int, c_int, c_int]
         lib.llg_attn_decode_scratch_floats.restype = c_longlong
+    elif name == "attention_mix":
+        lib.llg_attn_mix_simt_supported.argtypes = [c_int, c_int, c_int]
+        lib.llg_attn_mix_prefill_simt.argtypes = [POINTER(_PrefillArgs), c_int, c_int, c_void_p]
+        lib.llg_attn_mix_decode_simt.argtypes = [POINTER(_DecodeArgs), c_void_p, c_int, c_void_p]
+    elif name == "matrix_memory":
+        lib.llg_matrix_memory_fits.argtypes = [c_int, c_int]
+        lib.llg_matrix_memory.argtypes = [POINTER(_MatrixMemoryArgs), c_int, c_void_p]
+        if lib.llg_matrix_memory_piece() != MEMORY_PIECE:
+            raise KernelError(f"the matrix memory kernel works on pieces of {lib.llg_matrix_memory_piece()} tokens, Python "
+                              f"expects {MEMORY_PIECE}")
     elif name == "attention_mma":
         lib.llg_attn_mma_supported.argtypes = [c_int]
         lib.llg_attn_prefill_mma.argtypes = [POINTER(_PrefillArgs), c_void_p]
@@ -443,7 +490,7 @@ def _load_lib(name: str):
                                             c_int, c_int, c_int, c_int, c_int, c_void_p]
         lib.llg_moe_topk.argtypes = [c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
                                      POINTER(_RouterRule), c_void_p, c_void_p]
-        lib.llg_moe_plan.argtypes = [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
+        lib.llg_moe_plan.argtypes = [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p]
         lib.llg_moe_gather_rows.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
         lib.llg_grouped_linear.argtypes = [POINTER(_GroupedLinearArgs), c_int, c_int, c_void_p]
         lib.llg_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int,
@@ -581,12 +628,13 @@ GATE_ACTIVATIONS = ("silu", "gelu_tanh")     # what the gate of a gated feed-for
 
 
 def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, tile_n: int = 0, gated_features: int = 0,
-            row_scale: Optional[RowScale] = None, gate_activation: str = "silu") -> None:
+            row_scale: Optional[RowScale] = None, gate_activation: str = "silu", gate_form: Optional[GateForm] = None) -> None:
     """out[s, n, o] = split-K partials of x[n, k] w[o, k] on the tensor cores (tcgen05, TMA).
 
     ``out`` is ``[S, N, O]`` float32 with S = ``gemm_tc_splits(k, wish)``, or ``[1, N, O]`` bfloat16.
     With ``gated_features = F`` the matrix ``w`` is in the gated layout (``gated_rows(F)`` rows) and
-    ``out`` is ``[1, N, F]`` holding ``act(gate) * up`` with ``act`` = ``gate_activation`` (one of ``GATE_ACTIVATIONS``).  ``row_scale``: what a norm left for the rows of ``x``;
+    ``out`` is ``[1, N, F]`` holding ``act(gate) * up`` with ``act`` = ``gate_activation`` (one of ``GATE_ACTIVATIONS``), or what
+    ``gate_form`` (a ``GateForm``) makes of the two.  ``row_scale``: what a norm left for the rows of ``x``;
     the rows of the product are multiplied by it (before the gating).
     """
     lib = _lib("gemm_tc")
@@ -596,6 +644,12 @@ def gemm_tc(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, tile_n: int 
     assert k == k2 and out.shape == (s, n, gated_features if gated_features else o), (x.shape, w.shape, out.shape)
     if gemm_tc_splits(k, s) != s:
         raise KernelError(f"gemm_tc: {s} splits cannot be had for k = {k}")
+    if gate_form is not None:
+        if not gated_features or s != 1:
+            raise KernelError("gemm_tc: a form of gating goes with a gated product in one split")
+        _check(lib, lib.llg_gemm_tc_gate_form(_ptr(x, torch.bfloat16), _ptr(w, torch.bfloat16), _ptr(out), _dt(out), n, o, k, tile_n,
+                                              gated_features, byref(gate_form.c), _scale_ref(row_scale, n), _stream()))
+        return
     if gate_activation != "silu":
         if gate_activation not in GATE_ACTIVATIONS or not gated_features:
             raise KernelError(f"gemm_tc: gate activation '{gate_activation}' (known: {', '.join(GATE_ACTIVATIONS)}; gated products only)")
@@ -635,7 +689,8 @@ def qk_prep(qkv: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim: int,
             page_table: Optional[torch.Tensor] = None, ring_pages: int = 0,
             seq_of_token: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
             row_scale: Optional[RowScale] = None, value_dim: int = 0, v_mix: Optional[torch.Tensor] = None,
-            v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None) -> None:
+            v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None,
+            gate_out: Optional[torch.Tensor] = None) -> None:
     """Per-head norm (optional), bias (optional), rotation, and the writes of q, k, v.
 
     ``qkv`` is ``[S, N, (nh + nkv) * hd + nkv * vd]`` (partials are summed; ``vd = value_dim or hd``).  Queries go to
@@ -643,12 +698,14 @@ def qk_prep(qkv: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim: int,
     the cache pages (for a one-token step).  ``row_scale``: what a norm left for the token rows; the summed
     partials are multiplied by it before anything else.  Values blended across layers: ``v_first_out`` (float32
     ``[N, nkv, vd]``) receives the values as projected; with ``v_first_in`` and ``v_mix`` (one float32 number lam on the
-    device) the values written are ``(1 - lam) v + lam v_first_in``.
+    device) the values written are ``(1 - lam) v + lam v_first_in``.  ``gate_out`` (float32 ``[N, nh]``): the rows of ``qkv`` end
+    with one more number z per query head, and ``gate_out`` receives ``sigmoid(z)``.
     """
     lib = _lib("elementwise")
     s, n, width = qkv.shape
     vd = value_dim or head_dim
-    assert width == (n_heads + n_kv_heads) * head_dim + n_kv_heads * vd
+    assert width == (n_heads + n_kv_heads) * head_dim + n_kv_heads * vd + (n_heads if gate_out is not None else 0)
+    assert gate_out is None or gate_out.shape == (n, n_heads)
     a = _prep_args(n, n_heads, n_kv_heads, head_dim, q_norm_w, k_norm_w, norm_eps, bias, cos, sin, rotary_dim, pairing,
                    positions, q_out, k_new, v_new, k_pages, v_pages, page_table, ring_pages, seq_of_token, slots)
     a.qkv, a.qkv_dtype, a.n_partials, a.partial_stride = _ptr(qkv), _dt(qkv), s, n * width
@@ -660,6 +717,7 @@ def qk_prep(qkv: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim: int,
         raise KernelError("qk_prep: the values to blend with and the blend's weight come together")
     a.v_mix, a.v_first_in = _ptr(v_mix, torch.float32), _ptr(v_first_in, torch.float32)
     a.v_first_out = _ptr(v_first_out, torch.float32)
+    a.gate_out = _ptr(gate_out, torch.float32)
     _set_scale(a, row_scale, n)
     _check(lib, lib.llg_qk_prep(byref(a), _dt(q_out), _stream()))
 
@@ -804,25 +862,30 @@ def qkv_row_prep(qkvg: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim:
     _check(lib, lib.llg_qkv_row_prep(byref(a), _dt(q_out), _stream()))
 
 
-def add_layernorm(residual: torch.Tensor, parts, scale: float, weight: torch.Tensor, bias: torch.Tensor, eps: float,
-                  out: torch.Tensor, rows: Optional[torch.Tensor] = None) -> None:
+def add_layernorm(residual: torch.Tensor, parts, scale: float, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
+                  out: torch.Tensor, rows: Optional[torch.Tensor] = None, gains=None) -> None:
     """residual += scale * (sum of every set of partials in ``parts``); out[j] = layer norm of residual[rows[j] or j]:
-    ``(v - mean) / sqrt(mean((v - mean)^2) + eps) * weight + bias``.  ``residual`` float32 ``[N, H]``; ``parts`` a sequence
-    of float32 ``[S_i, N, H]`` tensors (up to four; none: nothing is added)."""
+    ``(v - mean) / sqrt(mean((v - mean)^2) + eps) * weight + bias`` (``bias`` None: none).  ``residual`` float32 ``[N, H]``;
+    ``parts`` a sequence of float32 ``[S_i, N, H]`` tensors (up to four; none: nothing is added).  ``gains``: None, or one
+    entry per set: None or a float32 ``[H]`` that the set's sum is multiplied by element by element."""
     lib = _lib("layernorm")
     n, hidden = residual.shape
     m = out.shape[0]
-    assert out.shape[1] == hidden and weight.shape == (hidden,) and bias.shape == (hidden,)
+    assert out.shape[1] == hidden and weight.shape == (hidden,) and (bias is None or bias.shape == (hidden,))
+    assert gains is None or len(gains) == len(parts)
     assert rows.numel() == m if rows is not None else m == n
     if len(parts) > _LN_BRANCHES:
         raise KernelError(f"add_layernorm: {len(parts)} sets of partials, at most {_LN_BRANCHES}")
-    if weight.dtype != bias.dtype:
+    if bias is not None and weight.dtype != bias.dtype:
         raise KernelError("add_layernorm: weight and bias must share a dtype")
     a = _LayerNormArgs()
     a.residual = _ptr(residual, torch.float32)
     for i, p in enumerate(parts):
         assert p.dim() == 3 and p.shape[1:] == (n, hidden), (p.shape, residual.shape)
         a.branch[i], a.n_partials[i] = _ptr(p, torch.float32), p.shape[0]
+        if gains is not None and gains[i] is not None:
+            assert gains[i].shape == (hidden,)
+            a.gain[i] = _ptr(gains[i], torch.float32)
     a.partial_stride, a.scale = n * hidden, float(scale)
     a.weight, a.bias, a.w_dtype, a.eps = _ptr(weight), _ptr(bias), _dt(weight), float(eps)
     a.out, a.out_dtype, a.rows, a.n_out, a.hidden = _ptr(out), _dt(out), _ptr(rows, torch.int32), m, hidden
@@ -837,7 +900,8 @@ def latent_prep(rows: torch.Tensor, *, n_heads: int, head_dim: int, rot_dim: int
                 page_table: Optional[torch.Tensor] = None, ring_pages: int = 0,
                 seq_of_token: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
                 pairing: int = 0, q_col: int = 0, kv_col: Optional[int] = None, cq_col: int = -1,
-                cq_norm_w: Optional[torch.Tensor] = None, cq_out: Optional[torch.Tensor] = None) -> None:
+                cq_norm_w: Optional[torch.Tensor] = None, cq_out: Optional[torch.Tensor] = None,
+                gate_col: int = 0, gate_out: Optional[torch.Tensor] = None) -> None:
     """Preparation for latent attention from the rows of one product, float32 partials ``[P, N, width]``.  A row holds up to
     three runs of columns, each starting at a column of its own (negative: absent, its work is left out).  At ``kv_col``
     (default: behind the queries): the latent (``rank`` elements, RMS-normed with ``c_norm_w``) and the shared key part
@@ -846,7 +910,8 @@ def latent_prep(rows: torch.Tensor, *, n_heads: int, head_dim: int, rot_dim: int
     elements; every head's unrotated part goes to ``q_plain_out`` ``[N, nh, dim]`` and its rotated part, rotated, to the
     last ``rdim`` elements of ``q_out`` ``[N, nh, rank + rdim]`` (the first ``rank`` are ``head_linear``'s to fill).  At
     ``cq_col``: a latent of the queries, RMS-normed with ``cq_norm_w`` into ``cq_out`` ``[N, cq_rank]``.  ``pairing``: which
-    elements a rotation pairs, 0 (i, i + rdim / 2) or 1 (2i, 2i + 1)."""
+    elements a rotation pairs, 0 (i, i + rdim / 2) or 1 (2i, 2i + 1).  With ``gate_out`` (float32 ``[N, nh]``) the row holds one
+    number z per head at ``gate_col``, and ``gate_out`` receives ``sigmoid(z)``."""
     lib = _lib("latent")
     p_n, n, width = rows.shape
     kd = kv_rank + rot_dim
@@ -885,6 +950,9 @@ def latent_prep(rows: torch.Tensor, *, n_heads: int, head_dim: int, rot_dim: int
     a.ring_pages = ring_pages
     a.seq_of_token, a.slots = _ptr(seq_of_token, torch.int32), _ptr(slots, torch.int32)
     a.n_tokens, a.nh, a.dim, a.rdim, a.rank = n, n_heads, head_dim, rot_dim, kv_rank
+    if gate_out is not None:
+        assert gate_out.shape == (n, n_heads)
+        a.gate_col, a.gate_out = gate_col, _ptr(gate_out, torch.float32)
     _check(lib, lib.llg_latent_prep(byref(a), _dtype_code(dtype), _stream()))
 
 
@@ -1165,6 +1233,95 @@ def retention(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, g_col: 
     _check(lib, lib.llg_retention(byref(a), max_count, _stream()), kernels=3 if carry is not None else 1)
 
 
+MEMORY_PIECE = 128          # tokens per piece of ``matrix_memory``; checked against the library at first use
+MEMORY_CARRY_EXTRA = 3
+_MEMORY_COLS = (256, 128, 64, 32, 16, 8)
+
+
+def matrix_memory_pieces(max_count: int) -> int:
+    """Pieces per sequence that ``matrix_memory`` wants a carry for when the longest sequence of a step brings ``max_count``
+    tokens (1: no carry)."""
+    return max(1, -(-int(max_count) // MEMORY_PIECE))
+
+
+_memory_cols_cache = {}
+
+
+def matrix_memory_cols(dim: int, vdim: int, groups: int) -> int:
+    """Columns of a head's state per block, for a step of ``groups`` (sequence or piece, head) pairs: all of them where a
+    block can hold them and there are pairs enough for every multiprocessor, else a run of a power of two."""
+    key = (dim, vdim, groups)
+    cols = _memory_cols_cache.get(key)
+    if cols is not None:
+        return cols
+    lib = _lib("matrix_memory")
+    fits = [c for c in (vdim,) + tuple(c for c in _MEMORY_COLS if c < vdim) if lib.llg_matrix_memory_fits(dim, c)]
+    if not fits:
+        raise KernelError(f"matrix_memory: a state of {dim} x {vdim} elements a head does not fit any block")
+    want = 2 * sm_count()
+    cols = fits[0]
+    for c in fits:
+        cols = c
+        if groups * -(-vdim // c) >= want:
+            break
+    _memory_cols_cache[key] = cols
+    return cols
+
+
+def matrix_memory_supported(dim: int, vdim: int) -> bool:
+    """Whether a head's state of ``dim`` x ``vdim`` elements can be cut into runs of columns that a block holds."""
+    lib = _lib("matrix_memory")
+    return any(lib.llg_matrix_memory_fits(dim, c) for c in (vdim,) + _MEMORY_COLS if c <= vdim)
+
+
+def matrix_memory(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, g_col: int, i_col: int, f_col: int, n_heads: int,
+                  dim: int, vdim: int, i_bias: Optional[torch.Tensor], f_bias: Optional[torch.Tensor], gate_cap: float,
+                  q_scale: float, denom_eps: float, eps: float, norm_w: torch.Tensor, state_s: torch.Tensor,
+                  state_n: torch.Tensor, state_m: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor,
+                  out: torch.Tensor, cols: int, carry: Optional[torch.Tensor] = None, raw: Optional[torch.Tensor] = None,
+                  next_nm: Optional[torch.Tensor] = None) -> None:
+    """A matrix memory per head along every sequence of a step, from float32 partials ``rows`` ``[P, N, width]`` that hold q and k
+    (``n_heads * dim`` columns each), v and the output gate's arguments (``n_heads * vdim`` each) and the two gates' arguments
+    (``n_heads`` each) at their columns.  Per head, q times ``q_scale``:
+
+        i = cap tanh((zi + i_bias) / cap),  f = logsigmoid(cap tanh((zf + f_bias) / cap)),  m' = max(f + m, i)
+        S' = e^(f + m - m') S + e^(i - m') k v^T,  n' = e^(f + m - m') n + e^(i - m') k
+        o = S'^T q / (max(|n' . q|, e^-m') + denom_eps),  out = o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(g)
+
+    ``state_s`` float32 ``[slots, n_heads, dim, vdim]``, ``state_n`` ``[slots, n_heads, dim]``, ``state_m`` ``[slots, n_heads]``; ``cols``
+    from ``matrix_memory_cols``.  ``carry`` float32 ``[B, pieces, n_heads, dim * vdim + dim + 3]`` lets a long prompt run in
+    pieces side by side (``pieces = matrix_memory_pieces(longest sequence)``).  With ``cols < vdim``: ``raw`` float32 ``[N, n_heads *
+    vdim]`` and, without a carry, ``next_nm`` float32 ``[B, n_heads, dim + 1]``."""
+    lib = _lib("matrix_memory")
+    p_n, n, width = rows.shape
+    n_seqs = slots.numel()
+    assert out.shape == (n, n_heads * vdim) and norm_w.shape == (n_heads * vdim,)
+    assert state_s.shape[1:] == (n_heads, dim, vdim) and state_n.shape[1:] == (n_heads, dim) and state_m.shape[1:] == (n_heads,)
+    assert cu_tokens.numel() == n_seqs + 1
+    a = _MatrixMemoryArgs()
+    a.rows, a.n_partials, a.partial_stride = _ptr(rows, torch.float32), p_n, n * width
+    a.row_width, a.q_col, a.k_col, a.v_col, a.g_col, a.i_col, a.f_col = width, q_col, k_col, v_col, g_col, i_col, f_col
+    for b_ in (i_bias, f_bias):
+        assert b_ is None or b_.shape == (n_heads,)
+    a.i_bias, a.f_bias = _ptr(i_bias, torch.float32), _ptr(f_bias, torch.float32)
+    a.gate_cap, a.q_scale, a.denom_eps, a.eps = float(gate_cap), float(q_scale), float(denom_eps), float(eps)
+    a.norm_w = _ptr(norm_w, torch.float32)
+    a.state_s, a.state_n, a.state_m = _ptr(state_s, torch.float32), _ptr(state_n, torch.float32), _ptr(state_m, torch.float32)
+    a.slots, a.cu_tokens = _ptr(slots, torch.int32), _ptr(cu_tokens, torch.int32)
+    a.out, a.out_dtype = _ptr(out), _dt(out)
+    max_count = 0
+    if carry is not None:
+        assert carry.dim() == 4 and carry.shape[0] >= n_seqs and carry.shape[2:] == (n_heads, dim * vdim + dim + MEMORY_CARRY_EXTRA)
+        a.carry, a.pieces = _ptr(carry, torch.float32), carry.shape[1]
+        max_count = min(n, carry.shape[1] * MEMORY_PIECE)
+    if cols < vdim:
+        assert raw is not None and raw.shape == (n, n_heads * vdim)
+        assert carry is not None or (next_nm is not None and next_nm.shape == (n_seqs, n_heads, dim + 1))
+        a.raw, a.next = _ptr(raw, torch.float32), _ptr(next_nm, torch.float32)
+    a.n_seqs, a.n_tokens, a.nh, a.dim, a.vdim, a.cols = n_seqs, n, n_heads, dim, vdim, cols
+    _check(lib, lib.llg_matrix_memory(byref(a), max_count, _stream()), kernels=(3 if carry is not None else 1) + (1 if cols < vdim else 0))
+
+
 def head_linear(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor) -> None:
     """y[n, h, :] = w[h] x[n, h, :]: ``x`` ``[N, nh, a]``, ``w`` ``[nh, b, a]`` (contiguous), ``y`` ``[N, nh, b]``.  ``x`` and
     ``y`` may be views into wider rows (their last elements contiguous); float32 sums; ``x`` and ``w`` share a dtype, ``y``
@@ -1236,14 +1393,14 @@ class RouterRule:
     the sigmoid scores are.  "sigmoid": scores ``s = sigmoid(logit)``; with ``groups`` the experts form that many equal groups of
     neighbours, a group is judged by the sum of its ``group_score_top`` largest scores and only the ``keep_groups`` best
     groups' experts can be chosen; the ``top`` largest eligible scores, ``weight = s / (sum of the chosen + weight_sum_eps) *
-    weight_scale``."""
+    weight_scale``.  ``normalize`` False: ``weight = s * weight_scale`` instead."""
 
     def __init__(self, score: str = "softmax", groups: int = 0, keep_groups: int = 0, group_score_top: int = 2,
-                 weight_scale: float = 1.0, weight_sum_eps: float = 0.0):
+                 weight_scale: float = 1.0, weight_sum_eps: float = 0.0, normalize: bool = True):
         if score not in ROUTER_SCORES:
             raise KernelError(f"router rule: score '{score}' is not known ({', '.join(ROUTER_SCORES)})")
         self.c = _RouterRule(ROUTER_SCORES[score], int(groups), int(keep_groups), int(group_score_top),
-                             float(weight_scale), float(weight_sum_eps))
+                             float(weight_scale), float(weight_sum_eps), int(not normalize))
 
 
 def _rule_ref(rule: Optional["RouterRule"]):
@@ -1284,19 +1441,22 @@ def moe_topk(logits: torch.Tensor, b_router: Optional[torch.Tensor], choice: tor
 
 
 def moe_plan(choice: torch.Tensor, n_experts: int, row_of_pair: torch.Tensor, token_of_row: torch.Tensor,
-             tile_expert: torch.Tensor) -> None:
+             tile_expert: torch.Tensor, weight: Optional[torch.Tensor] = None,
+             weight_of_row: Optional[torch.Tensor] = None) -> None:
     """Lays the pairs ``(n, k)`` of ``choice`` ``[N, top]`` out as rows in the order of their experts, every expert's run
     filled up to whole tiles of ``MOE_TILE_ROWS``: ``row_of_pair[n * top + k]`` the pair's row, ``token_of_row[r]`` the
     row's token (-1: a filling row), ``tile_expert[t]`` the expert of tile t (-1: unused).  ``token_of_row`` has
     ``moe_row_capacity(N * top, n_experts, tile)`` entries and ``tile_expert`` one per tile: their sizes say which tile
-    size is meant."""
+    size is meant.  With ``weight`` ``[N, top]``, ``weight_of_row`` receives every row's pair's weight (0 for filling rows)."""
     lib = _moe_lib()
     n, top = choice.shape
     cap = token_of_row.numel()
     tile = _tile_of(cap, tile_expert)
     assert row_of_pair.numel() == n * top
+    assert (weight is None) == (weight_of_row is None) and (weight is None or (weight.shape == (n, top) and weight_of_row.numel() == cap))
     _check(lib, lib.llg_moe_plan(_ptr(choice, torch.int32), n * top, top, n_experts, _ptr(row_of_pair, torch.int32),
-                                 _ptr(token_of_row, torch.int32), _ptr(tile_expert, torch.int32), cap, tile, _stream()))
+                                 _ptr(token_of_row, torch.int32), _ptr(tile_expert, torch.int32), cap, tile,
+                                 _ptr(weight, torch.float32), _ptr(weight_of_row, torch.float32), _stream()))
 
 
 def _tile_of(rows: int, tile_expert: torch.Tensor) -> int:
@@ -1315,16 +1475,18 @@ def moe_gather_rows(x: torch.Tensor, token_of_row: torch.Tensor, out: torch.Tens
     _check(lib, lib.llg_moe_gather_rows(_ptr(x), _ptr(token_of_row, torch.int32), _ptr(out), rows, width * x.element_size(), _stream()))
 
 
-def _grouped_tc(x, tile_expert, w, out, gated_features: int) -> None:
+def _grouped_tc(x, tile_expert, w, out, gated_features: int, form: Optional[GateForm] = None,
+                row_weight: Optional[torch.Tensor] = None) -> None:
     lib = _lib("gemm_tc")
     rows, k = x.shape
     n_groups, group_rows, k2 = w.shape
     assert k == k2 and tile_expert.numel() * MOE_TC_TILE_ROWS == rows
     _check(lib, lib.llg_gemm_tc_grouped(_ptr(x, torch.bfloat16), _ptr(w, torch.bfloat16), _ptr(out), _dt(out), rows, group_rows, k,
-                                        gated_features, _ptr(tile_expert, torch.int32), n_groups, group_rows, _stream()))
+                                        gated_features, _ptr(tile_expert, torch.int32), n_groups, group_rows,
+                                        byref(form.c) if form is not None else None, _ptr(row_weight, torch.float32), _stream()))
 
 
-def _grouped(x, token_of_row, tile_expert, w, w2_offset, n_out, y) -> None:
+def _grouped(x, token_of_row, tile_expert, w, w2_offset, n_out, y, form: GateForm = SILU_FORM, row_weight=None) -> None:
     """The kernels of csrc/moe.cu: ``w`` ``[E, rows per expert, n_in]``, of which the first ``n_out`` rows of an expert are the
     (first) matrix and, with ``w2_offset``, the rows from there on the second."""
     lib = _moe_lib()
@@ -1341,25 +1503,27 @@ def _grouped(x, token_of_row, tile_expert, w, w2_offset, n_out, y) -> None:
     a.w2 = (a.w + w2_offset * n_in * w.element_size()) if w2_offset else None
     a.rows, a.n_in, a.n_out = rows, n_in, n_out
     a.w_group_stride = w.shape[1] * n_in
+    a.row_weight, a.gate = _ptr(row_weight, torch.float32), form.c
     _check(lib, lib.llg_grouped_linear(byref(a), _dt(x), _dt(y), _stream()))
 
 
 def moe_gated(x: torch.Tensor, token_of_row: Optional[torch.Tensor], tile_expert: torch.Tensor, w_gate_up: torch.Tensor,
-              act: torch.Tensor) -> None:
-    """act[r] = silu(gate_e x_r) * (up_e x_r) for every row r of the layout (e its tile's expert); filling rows of a used
+              act: torch.Tensor, form: Optional[GateForm] = None, row_weight: Optional[torch.Tensor] = None) -> None:
+    """act[r] = silu(gate_e x_r) * (up_e x_r), or what ``form`` makes of the two products, for every row r of the layout (e its tile's expert); filling rows of a used
     tile get zeros.  ``w_gate_up`` ``[E, 2 P, hidden]`` holds every expert's matrices in the gated layout (gate rows,
     filled up to P = a multiple of 128, then the up rows); ``act`` ``[rows, inner]``.  With tiles of ``MOE_TILE_ROWS``,
     ``x`` is the step's activations and ``token_of_row`` says which row reads which; with tiles of ``MOE_TC_TILE_ROWS``,
-    ``x`` is the gathered rows themselves (``moe_gather_rows``) and the product runs on tcgen05."""
+    ``x`` is the gathered rows themselves (``moe_gather_rows``) and the product runs on tcgen05.  ``row_weight`` (float32
+    ``[rows]``): both products of row r are multiplied by ``row_weight[r]`` first, as if the row's input were."""
     rows, inner = act.shape
     pad = w_gate_up.shape[1] // 2
-    assert w_gate_up.shape[1] == gated_rows(inner)
+    assert w_gate_up.shape[1] == gated_rows(inner) and (row_weight is None or row_weight.numel() == rows)
     if _tile_of(rows, tile_expert) == MOE_TC_TILE_ROWS:
         if token_of_row is not None or x.shape[0] != rows:
             raise KernelError("moe_gated: tiles of 128 rows take the gathered rows")
-        _grouped_tc(x, tile_expert, w_gate_up, act, inner)
+        _grouped_tc(x, tile_expert, w_gate_up, act, inner, form, row_weight)
         return
-    _grouped(x, token_of_row, tile_expert, w_gate_up, pad, inner, act)
+    _grouped(x, token_of_row, tile_expert, w_gate_up, pad, inner, act, form or SILU_FORM, row_weight)
 
 
 def moe_down(act: torch.Tensor, tile_expert: torch.Tensor, w_down: torch.Tensor, y: torch.Tensor) -> None:
@@ -1372,14 +1536,14 @@ def moe_down(act: torch.Tensor, tile_expert: torch.Tensor, w_down: torch.Tensor,
     _grouped(act, None, tile_expert, w_down, None, w_down.shape[1], y)
 
 
-def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, weight: torch.Tensor, shared: Optional[torch.Tensor],
+def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, weight: Optional[torch.Tensor], shared: Optional[torch.Tensor],
                 out: torch.Tensor, shared_scale: Optional[torch.Tensor] = None) -> None:
-    """out[n] = sum_k weight[n, k] y[row_of_pair[n * top + k]] + the sum of ``shared``'s partials ``[S, N, H]`` (if any),
+    """out[n] = sum_k weight[n, k] y[row_of_pair[n * top + k]] (``weight`` None: every row counts once) + the sum of ``shared``'s partials ``[S, N, H]`` (if any),
     that sum times ``shared_scale[n]`` where given (float32 ``[N]``)."""
     lib = _moe_lib()
-    n, top = weight.shape
-    hidden = y.shape[1]
-    assert out.shape == (n, hidden) and row_of_pair.numel() == n * top
+    n, hidden = out.shape
+    top = row_of_pair.numel() // max(n, 1)
+    assert y.shape[1] == hidden and row_of_pair.numel() == n * top and (weight is None or weight.shape == (n, top))
     n_shared = 0
     if shared is not None:
         assert shared.dim() == 3 and shared.shape[1:] == (n, hidden)
@@ -1427,13 +1591,16 @@ def kv_write(k_new, v_new, k_pages, v_pages, page_table, ring_pages, positions, 
                                  _ptr(len_before, torch.int32), n, nkv, hd, _dt(k_new), _stream()))
 
 
-def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out[n, i] = act(g) * u, act = ``activation`` (one of ``GATE_ACTIVATIONS``; silu by default); the summed partials ``[S, N, gated_rows(I)]`` hold g and u in the gated
+def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", form: Optional[GateForm] = None) -> None:
+    """out[n, i] = act(g) * u, act = ``activation`` (one of ``GATE_ACTIVATIONS``; silu by default), or what ``form`` makes of g and u; the summed partials ``[S, N, gated_rows(I)]`` hold g and u in the gated
     layout (g of feature i at i, u at ``gated_rows(I) / 2 + i``)."""
     lib = _lib("elementwise")
     s, n, two_i = gate_up.shape
     inter = out.shape[1]
     assert out.shape == (n, inter) and two_i == gated_rows(inter)
+    if form is not None:
+        _check(lib, lib.llg_gate_form_mul(_ptr(gate_up), _dt(gate_up), s, n * two_i, _ptr(out), _dt(out), n, inter, byref(form.c), _stream()))
+        return
     if activation != "silu":
         if activation not in GATE_ACTIVATIONS:
             raise KernelError(f"silu_mul: gate activation '{activation}' is not known ({', '.join(GATE_ACTIVATIONS)})")
@@ -1488,6 +1655,11 @@ def _use_tc_attn(dtype: torch.dtype, head_dim: int) -> bool:
     return USE_TC_PROMPT_ATTENTION and dtype == torch.bfloat16 and head_dim in (64, 128)
 
 
+def attention_mix_supported(n_heads: int, head_dim: int, value_dim: int) -> bool:
+    """Whether the kernels for capped and mixed scores take these sizes."""
+    return bool(_lib("attention_mix").llg_attn_mix_simt_supported(n_heads, head_dim, value_dim))
+
+
 class AttentionForm:
     """What an attention computes beyond the plain causal softmax over keys and values of one head size:
     ``value_dim`` (elements of a value head; 0 = the key heads' size), ``sink`` (None, or the score of a sink that
@@ -1495,18 +1667,33 @@ class AttentionForm:
     (the output of every (token, head) is multiplied by a float32 gate ``[N, nh]`` that the caller passes), ``sinks``
     (a float32 tensor ``[nh]`` on the device: a sink per query head, instead of one score for all), ``chunked`` (the
     ``window`` of the call is a chunk size: a query sees the keys of its own chunk of that many positions, chunks
-    counted from position 0, instead of the last ``window`` keys)."""
+    counted from position 0, instead of the last ``window`` keys), ``softcap`` (c > 0: a scaled score s becomes ``c tanh(s /
+    c)``), ``head_mix`` (a float32 tensor ``[nh, nh]`` on the device: behind the cap, head h's scores become ``sum_g
+    head_mix[h, g] s_g``).  The last two run on kernels of their own (csrc/attention_mix.cu): a block then works on all
+    query heads of its queries."""
 
     def __init__(self, value_dim: int = 0, sink: Optional[float] = None, gated: bool = False,
-                 sinks: Optional[torch.Tensor] = None, chunked: bool = False):
+                 sinks: Optional[torch.Tensor] = None, chunked: bool = False, softcap: float = 0.0,
+                 head_mix: Optional[torch.Tensor] = None):
         self.value_dim, self.sink, self.gated = int(value_dim), (None if sink is None else float(sink)), bool(gated)
         if sinks is not None and (sinks.dtype != torch.float32 or sinks.dim() != 1):
             raise KernelError("AttentionForm: per-head sinks are a float32 vector [query heads]")
         self.sinks, self.chunked = sinks, bool(chunked)
+        self.softcap = float(softcap or 0.0)
+        if self.softcap < 0:
+            raise KernelError(f"AttentionForm: the scores' cap must not be negative, got {softcap}")
+        if head_mix is not None and (head_mix.dtype != torch.float32 or head_mix.dim() != 2 or head_mix.shape[0] != head_mix.shape[1]):
+            raise KernelError("AttentionForm: the mix of the heads' scores is a float32 matrix [query heads, query heads]")
+        self.head_mix = head_mix
+
+    @property
+    def mixes(self) -> bool:
+        """The scores are not the plain scaled products."""
+        return self.softcap > 0 or self.head_mix is not None
 
     def plain(self, head_dim: int) -> bool:
         return (self.value_dim in (0, head_dim) and self.sink is None and self.sinks is None and not self.gated
-                and not self.chunked)
+                and not self.chunked and not self.mixes)
 
     def one_head_size(self, head_dim: int) -> bool:
         """Keys and values of one head size: what the tensor-core kernels take (sink and gate they all apply)."""
@@ -1522,19 +1709,29 @@ PLAIN_ATTENTION = AttentionForm()
 def _prefill_kernel(dtype: torch.dtype, head_dim: int, form: AttentionForm) -> str:
     """Which prompt attention kernel takes this geometry and form: the tensor-core kernels want keys and values
     of one head size."""
+    if form.mixes:
+        return "mix"
     if form.one_head_size(head_dim):
         return "tc" if _use_tc_attn(dtype, head_dim) else "mma" if _use_mma(dtype, head_dim) else "simt"
     return "simt"
 
 
+MIX_TILE_QUERIES = 16        # queries per entry of a step's tile list for the kernels of csrc/attention_mix.cu
+
+
 def prefill_tile_queries(dtype: torch.dtype, head_dim: int, form: AttentionForm = PLAIN_ATTENTION) -> int:
     """Queries per block of the prompt attention kernel that ``attn_prefill`` will run."""
-    return {"tc": 256, "mma": 64, "simt": 16}[_prefill_kernel(dtype, head_dim, form)]
+    return {"tc": 256, "mma": 64, "simt": 16, "mix": MIX_TILE_QUERIES}[_prefill_kernel(dtype, head_dim, form)]
 
 
 def _set_form(a, form: AttentionForm, head_dim: int, gate: Optional[torch.Tensor]) -> None:
     """The fields of a prompt or decode argument block that say which form of attention is wanted."""
     a.vd = 0 if form.value_dim in (0, head_dim) else form.value_dim
+    a.softcap = form.softcap
+    if form.head_mix is not None:
+        if form.head_mix.shape[0] != a.nh:
+            raise KernelError(f"attention: a mix of {form.head_mix.shape[0]} heads' scores for {a.nh} query heads")
+        a.head_mix = _ptr(form.head_mix, torch.float32)
     _set_sink(a, form)
     a.gate = _ptr(gate, torch.float32)
 
@@ -1578,7 +1775,7 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
         raise KernelError("attn_prefill: a gated form needs a gate [tokens, heads], and only a gated form takes one")
     kernel = _prefill_kernel(q.dtype, hd, form)
     tc, mma = kernel == "tc", kernel == "mma"
-    lib = _lib("attention_tc" if tc else "attention_mma" if mma else "attention_simt")
+    lib = _lib("attention_mix" if kernel == "mix" else "attention_tc" if tc else "attention_mma" if mma else "attention_simt")
     a = _PrefillArgs()
     a.q, a.k_new, a.v_new = _ptr(q), _ptr(k_new, q.dtype), _ptr(v_new, q.dtype)
     a.k_pages, a.v_pages = _ptr(k_pages, q.dtype), _ptr(v_pages, q.dtype)
@@ -1590,7 +1787,9 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
     a.scale, a.window = float(scale), int(window)
     a.n_tokens, a.n_pages = k_new.shape[0], k_pages.shape[0]
     _set_form(a, form, hd, gate)
-    if tc:
+    if kernel == "mix":
+        _check(lib, lib.llg_attn_mix_prefill_simt(byref(a), tile_queries, _dt(q), _stream()))
+    elif tc:
         _check(lib, lib.llg_attn_prefill_tc(byref(a), _stream()))
     elif mma:
         _check(lib, lib.llg_attn_prefill_mma(byref(a), _stream()))
@@ -1644,6 +1843,10 @@ def attn_decode_plan(dtype: torch.dtype, n_seqs: int, n_heads: int, n_kv_heads: 
     the device.  Other multiples of 16 up to 128: the mma.sync kernel with a split count from ``max_len`` (per
     sequence by its length for small batches).  Everything else, and values of another head size than the keys: the
     CUDA-core kernel."""
+    if form.mixes:
+        # one block works on all heads of a sequence's share of the keys
+        splits = _splits_for(n_seqs, 1, max_len, sm_count(), 1)
+        return DecodePlan("mix", splits, False, max_len, attn_decode_scratch_floats(n_seqs, n_heads, form.vd(head_dim), splits), 0)
     plain = form.one_head_size(head_dim)
     if plain and _use_tma_decode(dtype, head_dim, n_heads, n_kv_heads, n_seqs):
         lib = _lib("attention_decode_tma")
@@ -1707,7 +1910,7 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         raise KernelError("attn_decode: the scratch must be float32")
     if form.gated != (gate is not None) or (gate is not None and tuple(gate.shape) != (b, nh)):
         raise KernelError("attn_decode: a gated form needs a gate [sequences, heads], and only a gated form takes one")
-    if not form.one_head_size(hd) and plan is not None and plan.kind != "simt":
+    if not form.one_head_size(hd) and plan is not None and plan.kind not in ("simt", "mix"):
         raise KernelError(f"attn_decode: the {plan.kind} kernel takes keys and values of one head size")
     assert out.shape == (b, nh * vd) and v_pages.shape[3] == vd
     if plan is not None and plan.kind == "tma":
@@ -1730,8 +1933,8 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         return
     if plan is not None:
         n_splits, balance = plan.n_splits, plan.balance
-    mma = form.one_head_size(hd) and _use_mma(q.dtype, hd)
-    lib = _lib("attention_mma" if mma else "attention_simt")
+    mma = form.one_head_size(hd) and _use_mma(q.dtype, hd) and not form.mixes
+    lib = _lib("attention_mix" if form.mixes else "attention_mma" if mma else "attention_simt")
     need = b * nh * n_splits * (vd + 2)
     if n_splits < 1 or scratch.numel() < need:
         raise KernelError(f"attn_decode: {n_splits} splits, scratch of {scratch.numel()} floats, {need} needed")
@@ -1750,6 +1953,8 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
             raise KernelError(f"attn_decode: needs {b * nkv} zeroed int32 counters")
         _check(lib, lib.llg_attn_decode_mma(byref(a), _ptr(out, q.dtype), _ptr(counters, torch.int32),
                                             int(bool(balance) and b * nkv <= attn_decode_balance_pairs() and b <= 32), _stream()))
+    elif form.mixes:
+        _check(lib, lib.llg_attn_mix_decode_simt(byref(a), _ptr(out, q.dtype), _dt(q), _stream()), kernels=2)
     else:
         _check(lib, lib.llg_attn_decode_simt(byref(a), _ptr(out, q.dtype), _dt(q), _stream()), kernels=2)
 

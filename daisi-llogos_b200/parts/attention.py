@@ -12,7 +12,9 @@ Beyond the reference, all by parameter: value heads of another size than the key
 the keys of its own chunk of ``window`` positions, chunks counted from position 0) instead of the sliding window; a
 learned sink per query head in the softmax's denominator (``p_j = e^{s_j} / (e^{sink_h} + sum e^{s_j})``, no key, no
 value, not scaled); and values blended across layers: the first layer of a group keeps its own values and lends them
-(float32, per step) to the others, which cache ``(1 - lam) v + lam v_first`` with a learned number ``lam`` each.
+(float32, per step) to the others, which cache ``(1 - lam) v + lam v_first`` with a learned number ``lam`` each.  Ahead of
+the softmax the scaled scores may pass a cap ``c tanh(s / c)`` and then be mixed over the heads, ``s'_h = sum_g T[h, g] s_g``;
+every head's output may be multiplied by one number ``sigmoid(w_h . x)`` from the mixer's own input.
 """
 from __future__ import annotations
 
@@ -35,7 +37,9 @@ class Attention(Mixer):
     directly behind the projections: tensors ``q_proj.conv``, ``k_proj.conv``, ``v_proj.conv`` [channels, taps], the last
     column the current token's; the last ``taps - 1`` projected rows of a sequence are kept as float32 state beside the
     keys and values), out_gate (False, or True: the concatenated heads are multiplied by ``sigmoid(g_proj x)`` before
-    the output projection; a tensor ``g_proj.weight`` [num_heads * value_dim, hidden])."""
+    the output projection; a tensor ``g_proj.weight`` [num_heads * value_dim, hidden]), head_gate (bool: one gate per query
+    head instead, a tensor ``gate_proj.weight`` [num_heads, hidden]; its rows ride in the projections' product and the
+    attention kernel applies it), softcap (0: none), head_mix (bool: a tensor ``head_mix.weight`` [num_heads, num_heads])."""
 
     TAKES_ROW_SCALE = True
 
@@ -78,8 +82,21 @@ class Attention(Mixer):
         if self.conv_taps and not self.own_kv:
             raise ValueError("attention: the convolution goes with the layer that projects its keys and values (own_kv)")
         self.out_gate = bool(p.get("out_gate", False))
-        self.special = (self.vd != self.hd or self.mask != "window" or self.sink_kind is not None or bool(self.conv_taps)
-                        or self.out_gate)
+        self.head_gate = bool(p.get("head_gate", False))
+        if self.head_gate and (self.conv_taps or not self.own_kv or bool(p.get("qkv_bias", False))):
+            raise ValueError("attention: gates per head go with plain projections of queries, keys and values (own_kv, no biases, "
+                             "no convolutions)")
+        self.softcap = float(p.get("softcap") or 0.0)
+        if self.softcap < 0:
+            raise ValueError(f"attention: softcap must not be negative, got {self.softcap}")
+        self.head_mix = bool(p.get("head_mix", False))
+        mix_fits = getattr(env.ops, "attention_mix_supported", None)
+        if (self.head_mix or self.softcap) and mix_fits is not None and not mix_fits(self.nh, self.hd, self.vd):
+            raise ValueError(f"attention: {self.nh} heads of {self.hd} (keys) and {self.vd} (values) elements are more than the "
+                             f"kernels for capped and mixed scores take")
+        self.own_form = (self.vd != self.hd or self.mask != "window" or self.sink_kind is not None or self.head_gate
+                         or self.softcap > 0 or self.head_mix)
+        self.special = self.own_form or bool(self.conv_taps) or self.out_gate
         self.w_gate = self.w_conv = None
         if self.conv_taps:
             self.TAKES_ROW_SCALE = False      # the convolution mixes rows: every row arrives finished
@@ -117,11 +134,17 @@ class Attention(Mixer):
             t["v_proj.conv"] = TensorDecl((self.nkv * self.vd, self.conv_taps), "conv")
         if self.out_gate:
             t["g_proj.weight"] = TensorDecl((self.nh * self.vd, self.hidden))
+        if self.head_gate:
+            t["gate_proj.weight"] = TensorDecl((self.nh, self.hidden))
+        if self.head_mix:
+            t["head_mix.weight"] = TensorDecl((self.nh, self.nh), "stream_mix")
         return t
 
     def bind(self, tensors):
         names = ["q_proj", "k_proj", "v_proj"] if self.own_kv else ["q_proj"]
         ws = [tensors[n + ".weight"] for n in names]
+        if self.head_gate:
+            ws.append(tensors["gate_proj.weight"])
         if len({w.dtype for w in ws}) != 1:
             raise ValueError(f"{self.prefix}: q/k/v projections are stored with different types")
         self.w_qkv = torch.cat(ws, dim=0).contiguous() if len(ws) > 1 else ws[0]
@@ -148,8 +171,12 @@ class Attention(Mixer):
                 # projections' product
                 self.w_qkv = torch.cat([self.w_qkv, self.w_gate], dim=0).contiguous()
                 self.w_gate = None
-        if self.vd != self.hd or self.mask != "window" or self.sink_kind is not None:
-            self.form = self.env.ops.AttentionForm(value_dim=self.vd, sinks=self.sinks, chunked=self.mask == "chunk")
+        if self.own_form:
+            mix = {}
+            if self.softcap > 0 or self.head_mix:
+                mix = dict(softcap=self.softcap, head_mix=as_f32(tensors["head_mix.weight"], self.env) if self.head_mix else None)
+            self.form = self.env.ops.AttentionForm(value_dim=self.vd, sinks=self.sinks, chunked=self.mask == "chunk",
+                                                   gated=self.head_gate, **mix)
 
     def cache_need(self):
         if not self.own_kv:
@@ -203,7 +230,7 @@ class Attention(Mixer):
                 if tuple(lent.shape) != (n, self.nkv, self.vd):
                     raise ValueError(f"attention: layers of the value group '{self.blend_group}' differ in their values' shape")
                 extra["v_first_in"], extra["v_mix"] = lent, self.v_lambda
-        if (not ctx.decode and fused_qkv is not None and not extra and not self.conv_taps and not self.out_gate
+        if (not ctx.decode and fused_qkv is not None and not extra and not self.conv_taps and not self.out_gate and not self.head_gate
                 and fused_qkv(x, self.w_qkv, self.hd, rot.rotary_dim if rot else 0, rot.pairing if rot else 0)):
             def prep(qkv_, **kw):
                 ops.gemm_tc_qkv(x, self.w_qkv, **kw, **scale_kw)
@@ -213,6 +240,8 @@ class Attention(Mixer):
                 ops.qk_prep(qkv_, **kw, **scale_kw, **extra)
             qkv = linear(ctx, x, self.w_qkv, "attn.qkv", torch.float32)
         gate, gate_col = None, 0
+        if self.head_gate:
+            extra["gate_out"] = form_kw["gate"] = ctx.buffer("attn.head_gate", (n, self.nh), torch.float32)
         if self.out_gate:
             if self.w_gate is None:
                 gate, gate_col = qkv, self.qkv_width                 # the gate's arguments lie behind q, k, v in the same rows
@@ -242,7 +271,8 @@ class Attention(Mixer):
             else:
                 prep(qkv, **common)
             # which kernel runs and how it splits the keys is the kernels' business: the plan says what scratch it wants
-            plan = ops.attn_decode_plan(q.dtype, ctx.n_seqs, self.nh, self.nkv, self.hd, ctx.max_len_after, **form_kw)
+            plan_kw = {"form": self.form} if self.form is not None else {}
+            plan = ops.attn_decode_plan(q.dtype, ctx.n_seqs, self.nh, self.nkv, self.hd, ctx.max_len_after, **plan_kw)
             scratch = ctx.buffer("attn.scratch", (max(1, plan.scratch_floats),), torch.float32)
             counters = None
             if plan.n_counters:
@@ -269,7 +299,7 @@ class Attention(Mixer):
             else:
                 prep(qkv, **common)
                 k_new, v_new = cache.shared["k_new"], cache.shared["v_new"]
-            tq = ops.prefill_tile_queries(q.dtype, self.hd, **form_kw)
+            tq = ops.prefill_tile_queries(q.dtype, self.hd, **({"form": self.form} if self.form is not None else {}))
             ops.attn_prefill(q, k_new, v_new, cache.k_pages, cache.v_pages, cache.page_table, cache.ring_pages,
                              ctx.query_tiles(tq), ctx.cu_tokens, ctx.len_before, ctx.slots, out,
                              scale=self.scale, window=self.window, tile_queries=tq, **form_kw)

@@ -24,7 +24,7 @@ are the ``Norm.forward`` contract here.
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Any, Callable, Dict, Optional, Tuple
 
 import torch
@@ -42,13 +42,14 @@ class TensorDecl:
 @dataclass(frozen=True)
 class Term:
     """One summand of what enters the residual: float32 partials ``[S, N, H]``; with ``weight`` (float32 ``[H]``) their sum
-    is divided by its own root mean square (``eps`` inside the root) and multiplied by that weight first; ``scale`` times
-    the result is added."""
+    is divided by its own root mean square (``eps`` inside the root) and multiplied by that weight first; with ``gain``
+    (float32 ``[H]``) it is multiplied by that vector element by element; ``scale`` times the result is added."""
 
     data: torch.Tensor
     weight: Optional[torch.Tensor] = None
     eps: float = 0.0
     scale: float = 1.0
+    gain: Optional[torch.Tensor] = None
 
 
 @dataclass
@@ -74,6 +75,12 @@ class Branch:
     @property
     def n_partials(self) -> int:
         return self.data.shape[0]
+
+    def with_gain(self, gain: torch.Tensor) -> "Branch":
+        """The branch with every summand multiplied by ``gain`` (float32 ``[H]``) element by element."""
+        if any(t.gain is not None for t in self.as_terms()):
+            raise ValueError("a branch's summands have a gain already")
+        return Branch.of_terms(replace(t, gain=gain) for t in self.as_terms())
 
     @classmethod
     def of_terms(cls, terms) -> "Branch":

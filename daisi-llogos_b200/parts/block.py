@@ -9,22 +9,44 @@ from __future__ import annotations
 
 from typing import Optional
 
-from .base import Block, Branch, register_part
+from .base import Block, Branch, Part, TensorDecl, as_f32, register_part
+
+
+class LayerScale(Part):
+    """A vector that a sublayer's output is multiplied by, element by element, as it enters the residual.  params: size.
+    Tensor: ``weight`` [size].  Nothing is computed here: the branch names the vector (``Branch.with_gain``) and the norm that
+    adds the branch applies it in float32."""
+
+    def __init__(self, params, prefix, env):
+        super().__init__(params, prefix, env)
+        self.size = int(params["size"])
+        self.weight = None
+
+    def tensors(self):
+        return {"weight": TensorDecl((self.size,), "norm")}
+
+    def bind(self, tensors):
+        self.weight = as_f32(tensors["weight"], self.env)
 
 
 class PreNormBlock(Block):
-    """roles: norm1, mixer, norm2, ffn (a layer without a feed-forward leaves norm2 and ffn out)."""
+    """roles: norm1, mixer, norm2, ffn (a layer without a feed-forward leaves norm2 and ffn out), and optionally scale1,
+    scale2 (``layer_scale`` parts on the mixer's and the feed-forward's output; the norms must then take gains:
+    ``layernorm``)."""
 
-    ROLES = {"norm1": "norm", "mixer": "mixer", "norm2": "norm", "ffn": "ffn"}
+    ROLES = {"norm1": "norm", "mixer": "mixer", "scale1": "connection", "norm2": "norm", "ffn": "ffn", "scale2": "connection"}
 
     def forward(self, residual, pending: Optional[Branch], ctx, cache) -> Optional[Branch]:
         p = self.parts
         h, kw = normed_for(p["norm1"], p["mixer"], residual, pending, ctx)
         a = p["mixer"].forward(h, ctx, cache, **kw)
+        if "scale1" in p:
+            a = a.with_gain(p["scale1"].weight)
         if "ffn" not in p:
             return a
         h, kw = normed_for(p["norm2"], p["ffn"], residual, a, ctx)
-        return p["ffn"].forward(h, ctx, **kw)
+        f = p["ffn"].forward(h, ctx, **kw)
+        return f.with_gain(p["scale2"].weight) if "scale2" in p else f
 
 
 class ParallelBlock(Block):
@@ -103,6 +125,7 @@ def normed_for(norm, consumer, residual, pending, ctx, rows=None):
     return norm.forward(residual, pending, ctx, rows), {}
 
 
+register_part("connection", "layer_scale", LayerScale)
 register_part("block", "prenorm", PreNormBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "two_norm_parallel", TwoNormParallelBlock)

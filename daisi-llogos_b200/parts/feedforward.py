@@ -13,9 +13,15 @@ from ..kernels.linear import activated_linear, gated_layout, gated_linear, linea
 from .base import Branch, FeedForward, TensorDecl, register_part
 
 
+def gate_form(params, env):
+    """The ``ops.GateForm`` of a gated feed-forward with ``activation`` "clamped" (see ``SwiGLU``)."""
+    return env.ops.GateForm(float(params.get("gate_alpha", 1.0)), params.get("limit"), float(params.get("up_offset", 0.0)))
+
+
 class SwiGLU(FeedForward):
     """``down(act(gate(x)) * up(x))``.  params: hidden_size, intermediate_size, activation (of the gate: one of
-    ``ops.GATE_ACTIVATIONS``, "silu" by default, or "gelu_tanh")."""
+    ``ops.GATE_ACTIVATIONS``, "silu" by default, or "gelu_tanh"; or "clamped": with ``g = min(gate, limit)`` and ``u = clamp(up,
+    -limit, limit)`` the product is ``g sigmoid(gate_alpha g) (u + up_offset)``; params gate_alpha, up_offset, limit)."""
 
     TAKES_ROW_SCALE = True
 
@@ -25,7 +31,8 @@ class SwiGLU(FeedForward):
         self.inter = int(params["intermediate_size"])
         self.activation = str(params.get("activation", "silu"))
         known = getattr(env.ops, "GATE_ACTIVATIONS", ("silu",))
-        if self.activation not in known:
+        self.form = gate_form(params, env) if self.activation == "clamped" else None
+        if self.form is None and self.activation not in known:
             raise ValueError(f"swiglu: gate activation '{self.activation}' is not known ({', '.join(known)})")
         self.w_gate_up = None
         self.w_down = None
@@ -46,7 +53,7 @@ class SwiGLU(FeedForward):
 
     def forward(self, x, ctx, row_scale=None) -> Branch:
         act = ctx.buffer("ffn.act", (x.shape[0], self.inter))
-        gated_linear(ctx, x, self.w_gate_up, act, row_scale, self.activation)
+        gated_linear(ctx, x, self.w_gate_up, act, row_scale, self.activation, **({"form": self.form} if self.form is not None else {}))
         return Branch(linear(ctx, act, self.w_down, "ffn.out", torch.float32))
 
 

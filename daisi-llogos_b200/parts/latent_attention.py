@@ -22,7 +22,9 @@ Two further forms, by parameter.  ``q_rank``: the queries pass a bottleneck of t
 (the norm with a weight of ``q_rank`` elements); the input product then yields the queries' latent, which the same
 kernel norms, and a second product makes the queries.  ``out_gate``: the concatenated heads are multiplied element by
 element by ``sigmoid(W_g h)`` before the output product; ``W_g`` rides in the input product and ``ops.sigmoid_gate``
-applies it to the per-head products' result.  Which elements a rotation pairs (halves, or neighbours) is the position
+applies it to the per-head products' result.  ``head_gate``: every head's output is multiplied by one number ``sigmoid(w_g,h .
+h)`` instead; its rows ride in the input product too, and the attention kernel applies it (a factor per head commutes with the
+product with ``W_uv``).  Which elements a rotation pairs (halves, or neighbours) is the position
 encoding's.
 """
 from __future__ import annotations
@@ -40,7 +42,8 @@ class LatentAttention(Mixer):
     value_dim, kv_rank, norm_eps (of the latent's norm), window (0 = all keys), mask ("window" or "chunk"),
     softmax_scale, sink (None or "learned": a tensor ``sink`` [num_heads]), position (name of a rotary encoding over
     ``rot_dim`` elements), q_rank (0: queries by one matrix ``q_proj``; else ``q_down_proj`` [q_rank, hidden],
-    ``q_norm.weight`` [q_rank], ``q_up_proj``), out_gate (bool: a tensor ``gate_proj.weight`` [num_heads value_dim, hidden])."""
+    ``q_norm.weight`` [q_rank], ``q_up_proj``), out_gate (bool: a tensor ``gate_proj.weight`` [num_heads value_dim, hidden]),
+    head_gate (bool: a tensor ``gate_proj.weight`` [num_heads, hidden])."""
 
     def __init__(self, params, prefix, env):
         super().__init__(params, prefix, env)
@@ -77,6 +80,9 @@ class LatentAttention(Mixer):
             raise ValueError("latent_attention: rotated elements and a position encoding come together")
         self.q_rank = int(p.get("q_rank") or 0)
         self.out_gate = bool(p.get("out_gate", False))
+        self.head_gate = bool(p.get("head_gate", False))
+        if self.out_gate and self.head_gate:
+            raise ValueError("latent_attention: one output gate, per element or per head")
         self.w_in = self.w_o = self.w_absorb = self.w_uv = self.c_norm_w = self.sinks = self.form = None
         self.w_uq = self.q_norm_w = None
 
@@ -90,6 +96,8 @@ class LatentAttention(Mixer):
             t = {_Q: TensorDecl((qw, self.hidden))}
         if self.out_gate:
             t["gate_proj.weight"] = TensorDecl((self.nh * self.vdim, self.hidden))
+        if self.head_gate:
+            t["gate_proj.weight"] = TensorDecl((self.nh, self.hidden))
         t.update({
              _DKV: TensorDecl((self.rank + self.rdim, self.hidden)),
              "kv_norm.weight": TensorDecl((self.rank,), "norm"),
@@ -103,7 +111,7 @@ class LatentAttention(Mixer):
     def bind(self, tensors):
         # rows of the input product: [queries, or their latent | latent and rotated key part | gate arguments]
         ws = [tensors["q_down_proj.weight"] if self.q_rank else tensors[_Q], tensors[_DKV]]
-        if self.out_gate:
+        if self.out_gate or self.head_gate:
             ws.append(tensors["gate_proj.weight"])
         if len({w.dtype for w in ws}) != 1:
             raise ValueError(f"{self.prefix}: the input projections are stored with different types")
@@ -117,7 +125,8 @@ class LatentAttention(Mixer):
         self.c_norm_w = tensors["kv_norm.weight"]
         if self.sink_kind == "learned":
             self.sinks = as_f32(tensors["sink"], self.env)
-        self.form = self.env.ops.AttentionForm(sinks=self.sinks, chunked=self.mask == "chunk")
+        self.form = self.env.ops.AttentionForm(sinks=self.sinks, chunked=self.mask == "chunk",
+                                               **({"gated": True} if self.head_gate else {}))
 
     def cache_need(self):
         return KvNeed(1, self.kd, self.window, values_in_keys=True)
@@ -134,6 +143,10 @@ class LatentAttention(Mixer):
                       norm_eps=self.eps, cos=rot.cos if rot else None, sin=rot.sin if rot else None,
                       pairing=rot.pairing if rot else 0, positions=ctx.positions, kv_col=q_cols)
         queries = dict(q_plain_out=q_plain, q_out=q)
+        gate_kw = {}
+        if self.head_gate:
+            gate_kw["gate"] = ctx.buffer("lattn.head_gate", (n, self.nh), torch.float32)
+            common.update(gate_col=q_cols + self.kd, gate_out=gate_kw["gate"])
         pages = dict(k_pages=cache.k_pages, page_table=cache.page_table,
                      ring_pages=cache.ring_pages, seq_of_token=ctx.seq_of_token, slots=ctx.slots)
         write_now = ctx.decode or self.window == 0       # a ring's pages may hold keys that this step's queries still need
@@ -144,7 +157,8 @@ class LatentAttention(Mixer):
             cq = ctx.buffer("lattn.cq", (n, self.q_rank))
             ops.latent_prep(rows, **common, **kv, q_col=-1, cq_col=0, cq_norm_w=self.q_norm_w, cq_out=cq)
             q_rows = linear(ctx, cq, self.w_uq, "lattn.q_rows", torch.float32)
-            ops.latent_prep(q_rows, **dict(common, kv_col=-1), **queries, q_col=0)
+            ops.latent_prep(q_rows, **{k: v for k, v in dict(common, kv_col=-1).items() if k not in ("gate_col", "gate_out")},
+                            **queries, q_col=0)
         else:
             ops.latent_prep(rows, **common, **kv, **queries, q_col=0)
         ops.head_linear(q_plain, self.w_absorb, q[:, :, :self.rank])
@@ -157,13 +171,13 @@ class LatentAttention(Mixer):
                 counters = ctx.buffer("attn.counters", (plan.n_counters,), torch.int32, zero=True)
             ops.attn_decode(q, cache.k_pages, cache.v_pages, cache.page_table, cache.ring_pages, ctx.slots,
                             ctx.len_before, mixed.view(n, self.nh * self.kd), scratch, scale=self.scale,
-                            window=self.window, plan=plan, counters=counters, form=self.form)
+                            window=self.window, plan=plan, counters=counters, form=self.form, **gate_kw)
         else:
             tq = ops.prefill_tile_queries(q.dtype, self.kd, self.form)
             ops.attn_prefill(q, k_new, k_new, cache.k_pages, cache.v_pages, cache.page_table, cache.ring_pages,
                              ctx.query_tiles(tq), ctx.cu_tokens, ctx.len_before, ctx.slots,
                              mixed.view(n, self.nh * self.kd), scale=self.scale, window=self.window,
-                             tile_queries=tq, form=self.form)
+                             tile_queries=tq, form=self.form, **gate_kw)
             if not write_now:
                 ops.kv_write(k_new, k_new, cache.k_pages, cache.v_pages, cache.page_table, cache.ring_pages,
                              ctx.positions, ctx.seq_of_token, ctx.slots, ctx.cu_tokens, ctx.len_before)

@@ -8,7 +8,10 @@ and only the experts of the ``keep_groups`` best groups can be chosen; the ``top
 weighted by ``s / (sum of the chosen s + weight_sum_eps) * weight_scale``.  Every expert is the gated form ``W_down (silu(W_gate h) * W_up h)`` without
 biases; the token's output is the weighted sum of its experts' outputs, plus the shared expert's (which every token
 runs) where the layer has one; with ``shared_gate`` the shared expert's output is multiplied by ``sigmoid(w_sg . h)``, one
-number per token, whose row ``w_sg`` rides in the router's product.
+number per token, whose row ``w_sg`` rides in the router's product.  Further forms, by parameter: weights that are the chosen
+scores themselves (``normalize`` False); weights on the experts' INPUT, ``sum_e expert_e(w_e h)``, which the first product's
+epilogue applies (it is linear in its rows) and the sum at the end does not; experts gated in a clamped form (``activation``
+"clamped", parts/feedforward.py), the shared expert with constants of its own.
 
 On the device the step's (token, choice) pairs are put in the order of their experts, every expert's run of rows
 filled up to a whole tile (``ops.moe_plan``), so that two grouped products (gate/up with the gating as its epilogue,
@@ -23,6 +26,7 @@ import torch
 
 from ..kernels.linear import gated_layout, linear
 from .base import Branch, FeedForward, TensorDecl, as_f32, part_class, register_part
+from .feedforward import gate_form
 
 
 class MoeFeedForward(FeedForward):
@@ -30,7 +34,9 @@ class MoeFeedForward(FeedForward):
     expert), router_bias (bool), shared_prefix (where the shared expert's tensors lie under this part's prefix,
     default "shared."), shared_names (its ``tensor_names``), score ("softmax", the default, "softmax_all" or "sigmoid"), groups and
     keep_groups (0: every expert is eligible), group_score_top (default 2), weight_scale (default 1), weight_sum_eps
-    (default 0), shared_gate (bool: a tensor ``shared_gate.weight`` [1, hidden]).  Tensors: ``router.weight`` [experts, hidden],
+    (default 0), normalize (default True: scores other than "softmax" are divided by the chosen ones' sum), weight_on ("output",
+    the default, or "input"), activation ("silu", or "clamped" with gate_alpha, up_offset, limit), shared_params (further params
+    of the shared expert), shared_gate (bool: a tensor ``shared_gate.weight`` [1, hidden]).  Tensors: ``router.weight`` [experts, hidden],
     ``router.bias`` [experts], and per expert i ``experts.<i>.{gate_proj,up_proj,down_proj}.weight``."""
 
     def __init__(self, params, prefix, env):
@@ -63,13 +69,23 @@ class MoeFeedForward(FeedForward):
         self.group_score_top = int(p.get("group_score_top", 2))
         self.weight_scale = float(p.get("weight_scale", 1.0))
         self.weight_sum_eps = float(p.get("weight_sum_eps", 0.0))
+        self.normalize = bool(p.get("normalize", True))
+        if not self.normalize and self.score == "softmax":
+            raise ValueError("moe: undivided scores go with sigmoid or softmax_all")
+        self.weight_on = str(p.get("weight_on", "output"))
+        if self.weight_on not in ("output", "input"):
+            raise ValueError(f"moe: weight_on '{self.weight_on}' is not known (output, input)")
+        activation = str(p.get("activation", "silu"))
+        if activation not in ("silu", "clamped"):
+            raise ValueError(f"moe: the experts' activation '{activation}' is not known (silu, clamped)")
+        self.form = gate_form(p, env) if activation == "clamped" else None
         self.shared_gate = bool(p.get("shared_gate", False))
         if self.shared_gate and not int(p.get("shared_size") or 0):
             raise ValueError("moe: a shared gate needs a shared expert")
         self.shared = None
         shared = int(p.get("shared_size") or 0)
         if shared:
-            sp = {"hidden_size": self.hidden, "intermediate_size": shared}
+            sp = {"hidden_size": self.hidden, "intermediate_size": shared, **dict(p.get("shared_params") or {})}
             if p.get("shared_names"):
                 sp["tensor_names"] = dict(p["shared_names"])
             self.shared_rel = str(p.get("shared_prefix", "shared."))
@@ -143,7 +159,8 @@ class MoeFeedForward(FeedForward):
         plain = self.score == "softmax" and not self.shared_gate
         shared_scale = ctx.buffer("moe.shared_scale", (n,), torch.float32) if self.shared_gate else None
         rule = {} if plain else dict(rule=ops.RouterRule(self.score, self.groups, self.keep_groups, self.group_score_top,
-                                                        self.weight_scale, self.weight_sum_eps), extra_out=shared_scale)
+                                                        self.weight_scale, self.weight_sum_eps,
+                                                        **({} if self.normalize else {"normalize": False})), extra_out=shared_scale)
         if self.w_router_same is not None and x.dtype == self.w_router_same.dtype and hasattr(ops, "moe_topk"):
             ops.moe_topk(linear(ctx, x, self.w_router_same, "moe.logits", torch.float32), self.b_router, choice, weight, **rule)
         else:
@@ -155,15 +172,21 @@ class MoeFeedForward(FeedForward):
         row_of_pair = ctx.buffer("moe.row_of_pair", (pairs,), torch.int32)
         token_of_row = ctx.buffer("moe.token_of_row", (cap,), torch.int32)
         tile_expert = ctx.buffer("moe.tile_expert", (cap // tile,), torch.int32)
-        ops.moe_plan(choice, self.n_exp, row_of_pair, token_of_row, tile_expert)
+        gated_kw = {"form": self.form} if self.form is not None else {}
+        if self.weight_on == "input":
+            gated_kw["row_weight"] = ctx.buffer("moe.weight_of_row", (cap,), torch.float32)
+            ops.moe_plan(choice, self.n_exp, row_of_pair, token_of_row, tile_expert, weight, gated_kw["row_weight"])
+            weight = None
+        else:
+            ops.moe_plan(choice, self.n_exp, row_of_pair, token_of_row, tile_expert)
         act = ctx.buffer("moe.act", (cap, self.inter))
         if tile == ops.MOE_TILE_ROWS:
-            ops.moe_gated(x, token_of_row, tile_expert, self.w_gate_up, act)
+            ops.moe_gated(x, token_of_row, tile_expert, self.w_gate_up, act, **gated_kw)
         else:
             # a prompt step on the tensor cores: the layout's rows as a matrix of their own, then the grouped tcgen05 product
             rows = ctx.buffer("moe.rows", (cap, self.hidden))
             ops.moe_gather_rows(x, token_of_row, rows)
-            ops.moe_gated(rows, None, tile_expert, self.w_gate_up, act)
+            ops.moe_gated(rows, None, tile_expert, self.w_gate_up, act, **gated_kw)
         y = ctx.buffer("moe.y", (cap, self.hidden), torch.float32)
         ops.moe_down(act, tile_expert, self.w_down, y)
         shared = self.shared.forward(x, ctx).data if self.shared is not None else None

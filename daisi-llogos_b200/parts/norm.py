@@ -58,6 +58,8 @@ class RmsNorm(Norm):
             raise ValueError(f"rmsnorm: norms that share a launch write to buffers of their own (out_name), got {names}")
         outs = [ctx.buffer(o.out_name, (m, self.size)) for o in norms]
         terms = () if branch is None else branch.as_terms()
+        if any(t.gain is not None for t in terms):
+            raise ValueError("rmsnorm: a summand of the pending branch has a gain per element; this norm adds outputs as they are")
         ws = [o.weight if o.weight.dtype == torch.float32 else as_f32(o.weight, self.env) for o in norms]
         ctx.ops.multi_add_rmsnorm(residual, [(t.data, t.weight, t.eps, t.scale) for t in terms],
                                   [(out, w, o.weight_offset) for out, w, o in zip(outs, ws, norms)], self.eps, rows)
@@ -89,7 +91,8 @@ class LayerNorm(Norm):
     """Layer norm fused with the residual add: ``v = residual + scale * (sum of the pending branch's partials)``,
     ``out = (v - mean(v)) / sqrt(var(v) + eps) * weight + bias`` with the variance as the mean of the squared
     deviations.  Takes a branch of several sublayers' outputs and a scale on their sum (``Branch.more``,
-    ``Branch.scale``).  Statistics, the residual and its sum are float32.  params: size, eps."""
+    ``Branch.scale``), and terms with a vector each that they are multiplied by (``Term.gain``).  Statistics, the residual and
+    its sum are float32.  params: size, eps, bias (default True)."""
 
     def __init__(self, params, prefix, env):
         super().__init__(params, prefix, env)
@@ -97,15 +100,19 @@ class LayerNorm(Norm):
         self.eps = float(params["eps"])
         if self.eps <= 0:
             raise ValueError("layer norm eps must be positive")
+        self.biased = bool(params.get("bias", True))
         self.weight: Optional[torch.Tensor] = None
         self.bias: Optional[torch.Tensor] = None
 
     def tensors(self):
-        return {"weight": TensorDecl((self.size,), "norm"), "bias": TensorDecl((self.size,), "bias")}
+        t = {"weight": TensorDecl((self.size,), "norm")}
+        if self.biased:
+            t["bias"] = TensorDecl((self.size,), "bias")
+        return t
 
     def bind(self, tensors):
-        self.weight, self.bias = tensors["weight"], tensors["bias"]
-        if self.weight.dtype != self.bias.dtype:
+        self.weight, self.bias = tensors["weight"], tensors.get("bias")
+        if self.bias is not None and self.weight.dtype != self.bias.dtype:
             raise ValueError(f"{self.prefix}: a layer norm's weight and bias are stored with different types")
 
     def forward(self, residual, branch: Optional[Branch], ctx, rows=None):
@@ -113,9 +120,17 @@ class LayerNorm(Norm):
             raise ValueError("layernorm: the residual must be one stream [tokens, hidden]")
         m = residual.shape[0] if rows is None else rows.numel()
         out = ctx.buffer("norm.out", (m, self.size))
-        parts = () if branch is None else (branch.data,) + tuple(branch.more)
-        ctx.ops.add_layernorm(residual, parts, branch.scale if branch is not None else 1.0, self.weight, self.bias,
-                              self.eps, out, rows)
+        if branch is not None and branch.terms:
+            if any(t.weight is not None for t in branch.terms) or len({t.scale for t in branch.terms}) != 1:
+                raise ValueError("layernorm: the pending branch's terms carry norms or factors that differ; this norm takes "
+                                 "plain terms with one factor on their sum")
+            parts, scale = tuple(t.data for t in branch.terms), branch.terms[0].scale
+            gains = [t.gain for t in branch.terms]
+            kw = {"gains": gains} if any(g is not None for g in gains) else {}
+        else:
+            parts = () if branch is None else (branch.data,) + tuple(branch.more)
+            scale, kw = (branch.scale if branch is not None else 1.0), {}
+        ctx.ops.add_layernorm(residual, parts, scale, self.weight, self.bias, self.eps, out, rows, **kw)
         return out
 
 

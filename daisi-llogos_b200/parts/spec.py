@@ -42,10 +42,14 @@ class ScheduleEntry:
     ``layer`` indexes ``ModelSpec.layers``; a layer may appear in several entries
     (its weights are then shared, each entry keeps its own cache).  ``cache_of``
     names an EARLIER entry whose cache this entry reads instead of keeping one.
+    ``add_embedding``: the embedding's output (the residual as it was ahead of the
+    first entry) is added to the residual once, ahead of this entry; the entry's
+    first norm adds it together with the branch that is pending.
     """
 
     layer: int
     cache_of: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -68,6 +72,8 @@ class ModelSpec:
         for e_i, e in enumerate(self.schedule):
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"schedule[{e_i}] names layer {e.layer}, but there are {len(self.layers)}")
+            if e.add_embedding and e_i == 0:
+                raise ValueError("schedule[0].add_embedding: the residual is the embedding's output there")
             if e.cache_of is not None:
                 if not 0 <= e.cache_of < e_i:
                     raise ValueError(

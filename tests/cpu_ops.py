@@ -46,8 +46,12 @@ def _rows_of(page_table, ring_pages, slot, pos, kvh, nkv):
 
 def qk_prep(qkv, *, n_heads, n_kv_heads, head_dim, q_norm_w, k_norm_w, norm_eps, bias, cos, sin, rotary_dim,
             pairing, positions, q_out, k_new=None, v_new=None, k_pages=None, v_pages=None, page_table=None,
-            ring_pages=0, seq_of_token=None, slots=None, value_dim=0, v_mix=None, v_first_in=None, v_first_out=None):
+            ring_pages=0, seq_of_token=None, slots=None, value_dim=0, v_mix=None, v_first_in=None, v_first_out=None,
+            gate_out=None):
     x = qkv.float().sum(0)
+    if gate_out is not None:
+        gate_out.copy_(torch.sigmoid(x[:, x.shape[1] - n_heads:]))
+        x = x[:, :x.shape[1] - n_heads]
     n = x.shape[0]
     nh, nkv, hd = n_heads, n_kv_heads, head_dim
     vd = value_dim or hd
@@ -108,21 +112,24 @@ def _store_kv(k, v, positions, k_new, v_new, k_pages, v_pages, page_table, ring_
                 v_pages[pg, hh, off] = v[t, h]
 
 
-def add_layernorm(residual, parts, scale, weight, bias, eps, out, rows=None):
+def add_layernorm(residual, parts, scale, weight, bias, eps, out, rows=None, gains=None):
     idx = slice(None) if rows is None else rows.long()
     if parts:
-        total = sum(p.sum(0) for p in parts)
+        gains = gains or [None] * len(parts)
+        total = sum(p.sum(0) if g is None else p.sum(0) * g for p, g in zip(parts, gains))
         residual[idx] += float(scale) * total[idx]
     x = residual[idx]
     mu = x.mean(-1, keepdim=True)
     var = ((x - mu) ** 2).mean(-1, keepdim=True)
-    out.copy_(((x - mu) * torch.rsqrt(var + eps) * weight.float() + bias.float()).to(out.dtype))
+    out.copy_(((x - mu) * torch.rsqrt(var + eps) * weight.float() + (0.0 if bias is None else bias.float())).to(out.dtype))
 
 
 def latent_prep(rows, *, n_heads, head_dim, rot_dim, kv_rank, c_norm_w, norm_eps, cos, sin, positions, q_plain_out=None,
                 q_out=None, k_new=None, v_new=None, k_pages=None, v_pages=None, page_table=None, ring_pages=0, seq_of_token=None,
-                slots=None, pairing=0, q_col=0, kv_col=None, cq_col=-1, cq_norm_w=None, cq_out=None):
+                slots=None, pairing=0, q_col=0, kv_col=None, cq_col=-1, cq_norm_w=None, cq_out=None, gate_col=0, gate_out=None):
     x = rows.float().sum(0)
+    if gate_out is not None:
+        gate_out.copy_(torch.sigmoid(x[:, gate_col:gate_col + n_heads]))
     n = x.shape[0]
     qw = n_heads * (head_dim + rot_dim)
     if kv_col is None:
@@ -335,6 +342,47 @@ def retention(rows, *, q_col, k_col, v_col, g_col, n_heads, dim, vdim, cos, sin,
         state[int(slots[b])] = st
 
 
+MEMORY_PIECE = 4
+MEMORY_CARRY_EXTRA = 3
+
+
+def matrix_memory_pieces(max_count):
+    return -(-max_count // MEMORY_PIECE)
+
+
+def matrix_memory_cols(dim, vdim, groups):
+    return vdim if groups % 2 else max(1, vdim // 2)
+
+
+def matrix_memory(rows, *, q_col, k_col, v_col, g_col, i_col, f_col, n_heads, dim, vdim, i_bias, f_bias, gate_cap, q_scale,
+                  denom_eps, eps, norm_w, state_s, state_n, state_m, slots, cu_tokens, out, cols, carry=None, raw=None,
+                  next_nm=None):
+    x = rows.float().sum(0)
+    n, nh = x.shape[0], n_heads
+    assert carry is None or carry.shape[2:] == (nh, dim * vdim + dim + MEMORY_CARRY_EXTRA)
+    assert cols == vdim or (raw.shape == (n, nh * vdim) and (carry is not None or next_nm.shape == (slots.numel(), nh, dim + 1)))
+    q = x[:, q_col:q_col + nh * dim].view(n, nh, dim) * q_scale
+    k = x[:, k_col:k_col + nh * dim].view(n, nh, dim)
+    v = x[:, v_col:v_col + nh * vdim].view(n, nh, vdim)
+    g = torch.sigmoid(x[:, g_col:g_col + nh * vdim])
+    i = gate_cap * torch.tanh((x[:, i_col:i_col + nh] + (0 if i_bias is None else i_bias)) / gate_cap)
+    f = torch.nn.functional.logsigmoid(gate_cap * torch.tanh((x[:, f_col:f_col + nh] + (0 if f_bias is None else f_bias)) / gate_cap))
+    for b in range(slots.numel()):
+        sl = int(slots[b])
+        S, nv, m = state_s[sl].clone(), state_n[sl].clone(), state_m[sl].clone()
+        for t in range(int(cu_tokens[b]), int(cu_tokens[b + 1])):
+            m2 = torch.maximum(f[t] + m, i[t])
+            keep, take = torch.exp(f[t] + m - m2), torch.exp(i[t] - m2)
+            S = keep[:, None, None] * S + take[:, None, None] * k[t][:, :, None] * v[t][:, None, :]
+            nv = keep[:, None] * nv + take[:, None] * k[t]
+            m = m2
+            o = torch.einsum("hdv,hd->hv", S, q[t])
+            o = o / (torch.maximum((nv * q[t]).sum(-1).abs(), torch.exp(-m)) + denom_eps)[:, None]
+            o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps)
+            out[t] = (o.reshape(-1) * norm_w * g[t]).to(out.dtype)
+        state_s[sl], state_n[sl], state_m[sl] = S, nv, m
+
+
 def tanh_cap(x, cap):
     x.copy_(cap * torch.tanh(x / cap))
 
@@ -358,7 +406,9 @@ def moe_row_capacity(pairs, n_experts, tile=MOE_TILE_ROWS):
 
 
 class RouterRule:
-    def __init__(self, score="softmax", groups=0, keep_groups=0, group_score_top=2, weight_scale=1.0, weight_sum_eps=0.0):
+    def __init__(self, score="softmax", groups=0, keep_groups=0, group_score_top=2, weight_scale=1.0, weight_sum_eps=0.0,
+                 normalize=True):
+        self.normalize = normalize
         self.score, self.groups, self.keep_groups, self.group_score_top = score, groups, keep_groups, group_score_top
         self.weight_scale, self.weight_sum_eps = weight_scale, weight_sum_eps
 
@@ -387,10 +437,15 @@ def moe_route(x, w_router, b_router, choice, weight, rule=None, extra_out=None):
         masked = s.masked_fill(~ok[:, :, None].expand(-1, -1, per).reshape(n, n_exp), -1.0)
     val, idx = torch.topk(masked, top, dim=-1)
     choice.copy_(idx.to(torch.int32))
+    if not rule.normalize:
+        weight.copy_(val * rule.weight_scale)
+        return
     weight.copy_(val / (val.sum(-1, keepdim=True) + rule.weight_sum_eps) * rule.weight_scale)
 
 
-def moe_plan(choice, n_experts, row_of_pair, token_of_row, tile_expert):
+def moe_plan(choice, n_experts, row_of_pair, token_of_row, tile_expert, weight=None, weight_of_row=None):
+    if weight is not None:
+        weight_of_row.zero_()
     top = choice.shape[1]
     flat = choice.reshape(-1).tolist()
     token_of_row.fill_(-1)
@@ -401,6 +456,8 @@ def moe_plan(choice, n_experts, row_of_pair, token_of_row, tile_expert):
         for p in reversed(mine):                 # any order inside an expert's run is allowed
             row_of_pair[p] = row
             token_of_row[row] = p // top
+            if weight is not None:
+                weight_of_row[row] = weight.reshape(-1)[p]
             row += 1
         while row % MOE_TILE_ROWS:
             row += 1
@@ -412,7 +469,17 @@ def moe_plan(choice, n_experts, row_of_pair, token_of_row, tile_expert):
         # tiles of an expert without rows stay -1 (it has none)
 
 
-def moe_gated(x, token_of_row, tile_expert, w_gate_up, act):
+class GateForm:
+    def __init__(self, alpha=1.0, limit=None, up_offset=0.0):
+        self.alpha, self.limit, self.up_offset = alpha, float("inf") if limit is None else limit, up_offset
+
+    def __call__(self, g, u):
+        g, u = g.clamp(max=self.limit), u.clamp(-self.limit, self.limit)
+        return g * torch.sigmoid(self.alpha * g) * (u + self.up_offset)
+
+
+def moe_gated(x, token_of_row, tile_expert, w_gate_up, act, form=None, row_weight=None):
+    form = form or GateForm()
     act.zero_()
     inner, pad = act.shape[1], w_gate_up.shape[1] // 2
     for r in range(token_of_row.numel()):
@@ -422,7 +489,8 @@ def moe_gated(x, token_of_row, tile_expert, w_gate_up, act):
         e = int(tile_expert[r // MOE_TILE_ROWS])
         g = w_gate_up[e, :inner].float() @ x[t].float()
         u = w_gate_up[e, pad:pad + inner].float() @ x[t].float()
-        act[r] = (g / (1 + torch.exp(-g)) * u).to(act.dtype)
+        rw = 1.0 if row_weight is None else row_weight[r]
+        act[r] = form(g * rw, u * rw).to(act.dtype)
 
 
 def moe_down(act, tile_expert, w_down, y):
@@ -434,9 +502,9 @@ def moe_down(act, tile_expert, w_down, y):
 
 
 def moe_combine(y, row_of_pair, weight, shared, out, shared_scale=None):
-    n, top = weight.shape
-    rows = row_of_pair.view(n, top).long()
-    out.copy_((weight[:, :, None] * y[rows]).sum(1))
+    n = out.shape[0]
+    rows = row_of_pair.view(n, -1).long()
+    out.copy_((y[rows] if weight is None else weight[:, :, None] * y[rows]).sum(1))
     if shared is not None:
         out += shared.sum(0) if shared_scale is None else shared.sum(0) * shared_scale[:, None]
 
@@ -460,11 +528,14 @@ def kv_write(k_new, v_new, k_pages, v_pages, page_table, ring_pages, positions, 
 GATE_ACTIVATIONS = ("silu", "gelu_tanh")
 
 
-def silu_mul(gate_up, out, activation="silu"):
+def silu_mul(gate_up, out, activation="silu", form=None):
     x = gate_up.float().sum(0)
     inter = out.shape[1]
     half = x.shape[1] // 2
     g, u = x[:, :inter], x[:, half:half + inter]
+    if form is not None:
+        out.copy_(form(g, u).to(out.dtype))
+        return
     if activation == "gelu_tanh":
         a = 0.5 * g * (1 + torch.tanh(0.7978845608028654 * (g + 0.044715 * g ** 3)))
     else:
@@ -551,7 +622,8 @@ def zero_rows(base, rows):
 
 
 class AttentionForm:
-    def __init__(self, value_dim=0, sink=None, gated=False, sinks=None, chunked=False):
+    def __init__(self, value_dim=0, sink=None, gated=False, sinks=None, chunked=False, softcap=0.0, head_mix=None):
+        self.softcap, self.head_mix = softcap, head_mix
         self.value_dim, self.sink, self.gated = int(value_dim), sink, bool(gated)
         self.sinks, self.chunked = sinks, bool(chunked)
 
@@ -572,8 +644,17 @@ def _lowest(form, window, pos):
     return (pos // window) * window if form.chunked else max(0, pos - window + 1)
 
 
-def _attend(q, keys, vals, scale, form=PLAIN_ATTENTION, gate=None, head=0):
+def _score(q, keys, scale, form):
     s = (keys.float() @ q.float()) * scale
+    return form.softcap * torch.tanh(s / form.softcap) if form.softcap else s
+
+
+def _attend(q, keys, vals, scale, form=PLAIN_ATTENTION, gate=None, head=0, others=None):
+    """``others``: one (query, keys) per head, where the scores are mixed over the heads."""
+    if form.head_mix is None:
+        s = _score(q, keys, scale, form)
+    else:
+        s = sum(form.head_mix[head, g] * _score(qg, kg, scale, form) for g, (qg, kg) in enumerate(others))
     sink = form.sink if form.sinks is None else float(form.sinks[head])
     if sink is not None:
         s = torch.cat([s, torch.tensor([float(sink)])])
@@ -610,15 +691,17 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
         for t in range(t0, t1):
             pos = lb + (t - t0)
             lo = _lowest(form, window, pos)
-            for h in range(nh):
-                kvh = h // g
+            kv = []
+            for kvh in range(nkv):
                 old = [p for p in range(lo, pos + 1) if p < lb]
                 ks, vs = _gather(k_pages, v_pages, page_table, ring_pages, slot, old, kvh)
                 for p in range(max(lo, lb), pos + 1):
                     ks.append(k_new[t0 + p - lb, kvh])
                     vs.append(v_new[t0 + p - lb, kvh])
-                o[t, h] = _attend(q[t, h], torch.stack(ks), torch.stack(vs), scale, form,
-                                  None if gate is None else gate[t, h], h).to(out.dtype)
+                kv.append((torch.stack(ks), torch.stack(vs)))
+            others = [(q[t, h], kv[h // g][0]) for h in range(nh)]
+            for h in range(nh):
+                o[t, h] = _attend(q[t, h], *kv[h // g], scale, form, None if gate is None else gate[t, h], h, others).to(out.dtype)
 
 
 class _Plan:
@@ -639,10 +722,11 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         length = int(len_before[b]) + 1
         lo = _lowest(form, window, length - 1)
         slot = int(slots[b])
+        kv = [tuple(map(torch.stack, _gather(k_pages, v_pages, page_table, ring_pages, slot, range(lo, length), kvh)))
+              for kvh in range(nkv)]
+        others = [(q[b, h], kv[h // g][0]) for h in range(nh)]
         for h in range(nh):
-            ks, vs = _gather(k_pages, v_pages, page_table, ring_pages, slot, range(lo, length), h // g)
-            o[b, h] = _attend(q[b, h], torch.stack(ks), torch.stack(vs), scale, form,
-                              None if gate is None else gate[b, h], h).to(out.dtype)
+            o[b, h] = _attend(q[b, h], *kv[h // g], scale, form, None if gate is None else gate[b, h], h, others).to(out.dtype)
 
 
 def argmax(logits, out):
