@@ -173,10 +173,19 @@ def route(h, w_router, top) -> Tuple[torch.Tensor, torch.Tensor]:
     return c, s
 
 
-def mixture(h, w, p, ml, routes_out: Optional[list] = None) -> torch.Tensor:
+def route_margin(h, w_router, top) -> torch.Tensor:
+    """[T]: by how much the last chosen expert's logit beats the next one's (infinite where nothing is left out)."""
+    z = linear(h, w_router)
+    if int(top) == z.shape[-1]:
+        return torch.full((z.shape[0],), math.inf, dtype=F64)
+    v = z.topk(int(top) + 1, dim=-1).values
+    return v[:, -2] - v[:, -1]
+
+
+def mixture(h, w, p, ml, margins: Optional[list] = None) -> torch.Tensor:
     chosen, score = route(h, w[p + "router"], ml["router"]["top"])
-    if routes_out is not None:
-        routes_out.append(chosen)
+    if margins is not None:
+        margins.append(route_margin(h, w[p + "router"], ml["router"]["top"]))
     out = torch.zeros_like(h, dtype=F64)
     for e in range(int(ml["router"]["experts"])):
         t, j = (chosen == e).nonzero(as_tuple=True)
@@ -201,8 +210,9 @@ def run_order(cfg: dict) -> List[Tuple[int, bool]]:
 
 
 def forward(w: Dict[str, torch.Tensor], cfg: dict, tokens: Sequence[int], layers_out: Optional[list] = None,
-            routes_out: Optional[list] = None) -> torch.Tensor:
-    """Logits [T, vocab] of one whole sequence; ``layers_out`` receives x after every layer that runs."""
+            margins: Optional[list] = None) -> torch.Tensor:
+    """Logits [T, vocab] of one whole sequence; ``layers_out`` receives x after every layer that runs, ``margins`` every
+    router's margins (``route_margin``)."""
     eps = float(cfg["norm"]["eps"])
     e = w["embed"].to(F64)[torch.as_tensor(list(tokens), dtype=torch.long)]
     x = e.clone()
@@ -219,7 +229,7 @@ def forward(w: Dict[str, torch.Tensor], cfg: dict, tokens: Sequence[int], layers
             y = attention(h, w, p + "mix.", mx)
         x = x + y * w[p + "ls1"].to(F64)
         if lay.get("mlp"):
-            x = x + mixture(layer_norm(x, w[p + "norm2"], eps), w, p + "mlp.", lay["mlp"], routes_out) * w[p + "ls2"].to(F64)
+            x = x + mixture(layer_norm(x, w[p + "norm2"], eps), w, p + "mlp.", lay["mlp"], margins) * w[p + "ls2"].to(F64)
         if layers_out is not None:
             layers_out.append(x.clone())
     return linear(layer_norm(x, w["final.norm"], eps), w["embed"])
