@@ -27,7 +27,10 @@ stock model's feed-forward) in Karitar's place; ``--design rukedra`` puts the Ru
 and a minGRU mixer between grouped norms with gated residuals, dense and mixture feed-forwards in turn) beside Fipavik, the
 closest model the library has, at equal latent, expert and feed-forward sizes; ``--design piratar`` puts the Piratar design
 (softmax attention with short convolutions beside retention, an RG-LRU block, two norms over one residual, a per-token
-input) beside Rukedra at equal widths, experts and feed-forward sizes.
+input) beside Rukedra at equal widths, experts and feed-forward sizes; ``--design memilorn`` puts the Memilorn design (a
+matrix memory with exponential gates, attention with capped scores mixed over the heads, latent attention, a mixture weighed
+on its input) beside the two closest models the library has, Piratar (retention, attention over every key) and Rukedra
+(latent attention over every key), at equal widths, heads, states and experts.
 """
 import argparse
 import json
@@ -438,6 +441,24 @@ def piratar_config(size):
             "token_side": {"dim": 64}, "layers": layers}
 
 
+def memilorn_config(size):
+    """Memilorn at a size, four layers: a matrix memory, latent attention, attention, a matrix memory, each with a mixture.  The
+    memory has Piratar's retention heads (a quarter as many of the stock model's head size), attention the stock model's
+    heads (values of the keys' size, half of every head rotated, scores capped at 50), the latent is one head size long (a
+    cached row as long as Fipavik's and Rukedra's); the experts (sixteen, four per token, a shared expert) are Piratar's."""
+    width, heads, kv, hd, ff, window, _ = DESIGN_SIZES[size]
+    mem = {"heads": max(1, heads // 4), "dim": hd, "vdim": hd, "gate_cap": 15.0}
+    lat = {"heads": heads, "dim": hd, "vdim": hd, "kv_rank": hd, "scale": hd ** -0.5}
+    att = {"heads": heads, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "softcap": 50.0,
+           "rot": {"base": 1000000.0, "dims": hd // 2}}
+    moe = {"kind": "moe", "router": {"experts": FIPAVIK_EXPERTS, "top": FIPAVIK_TOP}, "expert": {"ff": ff // 8, "limit": 7.0},
+           "shared": {"ff": ff // 2, "limit": 7.0}}
+    layers = [{"type": t, "mixer": dict(m), "mlp": dict(moe)} for t, m in (("mlstm", mem), ("latent_attention", lat),
+                                                                          ("attention", att), ("mlstm", mem))]
+    assert len(layers) == DESIGN_LAYERS
+    return {"architecture": "Memilorn", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
+
+
 def design_configs(size, design="karitar"):
     """The configuration of ``design`` (Karitar or Fipavik) at a size and the closest stock model's (Qwen3: grouped-query
     attention with normed queries and keys and the same window, pre-norm blocks) with the same width, heads, head size
@@ -460,6 +481,8 @@ def design_configs(size, design="karitar"):
         return {"rukedra": rukedra_config(size), "fipavik": fipavik_config(size)}
     if design == "piratar":
         return {"piratar": piratar_config(size), "rukedra": rukedra_config(size)}
+    if design == "memilorn":
+        return {"memilorn": memilorn_config(size), "piratar": piratar_config(size), "rukedra": rukedra_config(size)}
     return {"karitar": karitar, "qwen3": qwen3}
 
 
@@ -467,7 +490,7 @@ _TIMED_OPS = ("embed_rows", "add_rmsnorm", "hc_add_rmsnorm", "qk_prep", "qkv_row
               "act_rows", "silu_mul", "attn_prefill", "attn_decode", "kv_write", "add_layernorm", "latent_prep", "head_linear",
               "moe_route", "moe_topk", "moe_plan", "moe_gather_rows", "moe_gated", "moe_down", "moe_combine",
               "gated_add_group_rmsnorm", "mingru_scan", "sigmoid_gate", "tanh_cap", "multi_add_rmsnorm", "hash_embed",
-              "table_gate", "causal_conv", "rglru_scan", "retention")
+              "table_gate", "causal_conv", "rglru_scan", "retention", "matrix_memory")
 
 # What the float32 multiply-adds of a B200's CUDA cores can do at most (148 multiprocessors x 128 lanes x 2 flops at
 # 1.9 GHz): the arithmetic bound of kernels whose products must stay float32 (retention's state).
@@ -480,6 +503,12 @@ def _kernel_label(name, args, kw):
         o, k = args[1].shape
         what = "gated" if kw.get("gated_features") else "act" if name == "gemm_tc_act" else "qkv+prep" if name == "gemm_tc_qkv" else ""
         return f"product {k}->{o} {what}".strip()
+    form = kw.get("form")
+    if name in ("attn_prefill", "attn_decode"):
+        if getattr(form, "mixes", False):
+            return name + " (mixed heads)"
+        if args[3 if name == "attn_prefill" else 1] is args[4 if name == "attn_prefill" else 2]:
+            return name + " (latent)"
     return name
 
 
@@ -500,7 +529,11 @@ def _kernel_cost(name, args, kw, keys_read):
         kp, vp = (args[3], args[4]) if name == "attn_prefill" else (args[1], args[2])
         nkv, vd = kp.shape[1], vp.shape[3]
         pairs, rows = keys_read
-        return rows * nkv * (hd + vd) * q.element_size() + 2 * q.nbytes, 2.0 * nh * (hd + vd) * pairs
+        mixed = 0.0
+        if getattr(kw.get("form"), "head_mix", None) is not None:
+            # the mixture of the heads' scores: float32 products, counted against the CUDA cores' peak as retention's are
+            mixed = 2.0 * nh * nh * pairs * _TENSOR_PER_FP32[0]
+        return rows * nkv * (hd + vd) * q.element_size() + 2 * q.nbytes, 2.0 * nh * (hd + vd) * pairs + mixed
     if name in ("add_rmsnorm", "hc_add_rmsnorm"):
         # the residual (one array or several streams) is read and, with a branch, written back; only the rows that
         # are normalised are touched
@@ -551,6 +584,15 @@ def _kernel_cost(name, args, kw, keys_read):
         moved = rows.nbytes * (2 if carry is not None else 1) + out.nbytes + 2 * kw["slots"].numel() * state[0].numel() * 4
         flops = 4.0 * n * nh * dim * vdim * (2 if carry is not None else 1)
         return moved, flops * _TENSOR_PER_FP32[0]
+    if name == "matrix_memory":
+        # as retention: the step's sums (with pieces q, k, v and the gates twice), the outputs, every sequence's state in and
+        # out, the float32 products of update and read-out (the normaliser's left out)
+        rows, out, state = args[0], kw["out"], kw["state_s"]
+        carry = kw.get("carry")
+        n, nh, dim, vdim = out.shape[0], kw["n_heads"], kw["dim"], kw["vdim"]
+        moved = rows.nbytes * (2 if carry is not None else 1) + out.nbytes + 2 * kw["slots"].numel() * state[0].numel() * 4
+        flops = 4.0 * n * nh * dim * vdim * (2 if carry is not None else 1)
+        return moved, flops * _TENSOR_PER_FP32[0]
     if name == "sigmoid_gate":
         x, gate = args[0], args[1]
         return 2 * x.nbytes + gate.shape[0] * x.numel() * 4, 0.0
@@ -591,7 +633,7 @@ def probe_designs(torch, L, ops, pk, sizes, batch, which="karitar"):
     report = {}
     real = {n: getattr(ops, n) for n in _TIMED_OPS}
     for size in sizes:
-        window, context = DESIGN_SIZES[size][5], DESIGN_SIZES[size][6]
+        context = DESIGN_SIZES[size][6]
         for design, cfg in design_configs(size, which).items():
             model = L.weights.random_model(cfg, seed=0, dtype=torch.bfloat16, device=dev, std=0.02)
             out = {}
@@ -662,14 +704,13 @@ def probe_designs(torch, L, ops, pk, sizes, batch, which="karitar"):
                                decode_context=context, decode_ms_per_step=round(dec_ms, 4),
                                decode_tokens_per_s=round(batch / dec_ms * 1e3, 1))
                 else:
-                    keys = min(window, context) if window else context
                     t = PREFILL_TOKENS
-                    pre_pairs = sum(min(i + 1, window) if window else i + 1 for i in range(t))
                     table = {}
                     for ph, name, a, kw, ev0, ev1 in records:
                         if ph == "warm":
                             continue
-                        kr = (pre_pairs, t) if ph == "prefill" else (batch * keys, batch * keys)
+                        seen = kw.get("window") or context                  # the keys a query sees at most
+                        kr = (sum(min(i + 1, seen) for i in range(t)), t) if ph == "prefill" else (batch * min(seen, context),) * 2
                         nbytes, flops = _kernel_cost(name, a, kw, kr)
                         row = table.setdefault((ph, _kernel_label(name, a, kw)), [0, 0.0, 0.0, 0.0])
                         row[0] += 1
@@ -710,7 +751,7 @@ def main():
     ap.add_argument("--tokens", type=int, default=0,
                     help="with --probe timeline: the time line of a prompt step of so many tokens instead of a decode step")
     ap.add_argument("--sizes", default=",".join(DESIGN_SIZES), help="with --probe designs: which of " + ", ".join(DESIGN_SIZES))
-    ap.add_argument("--design", choices=["karitar", "fipavik", "rukedra", "piratar"], default="karitar",
+    ap.add_argument("--design", choices=["karitar", "fipavik", "rukedra", "piratar", "memilorn"], default="karitar",
                     help="with --probe designs: the design that stands beside the closest stock model")
     ap.add_argument("--probe", choices=["decode-attention", "leave-one-out", "timeline", "designs"],
                     help="instead of the bench line, print a table: decode attention alone over batch shapes; what "
