@@ -434,6 +434,11 @@ def _load_lib(name: str):
         lib.llg_attn_mix_simt_supported.argtypes = [c_int, c_int, c_int]
         lib.llg_attn_mix_prefill_simt.argtypes = [POINTER(_PrefillArgs), c_int, c_int, c_void_p]
         lib.llg_attn_mix_decode_simt.argtypes = [POINTER(_DecodeArgs), c_void_p, c_int, c_void_p]
+    elif name == "attention_mix_mma":
+        lib.llg_attn_mix_prefill_mma_supported.argtypes = [c_int, c_int, c_int, c_int]
+        lib.llg_attn_mix_decode_mma_supported.argtypes = [c_int, c_int, c_int, c_int]
+        lib.llg_attn_mix_prefill_mma.argtypes = [POINTER(_PrefillArgs), c_int, c_void_p]
+        lib.llg_attn_mix_decode_mma.argtypes = [POINTER(_DecodeArgs), c_void_p, c_void_p]
     elif name == "matrix_memory":
         lib.llg_matrix_memory_fits.argtypes = [c_int, c_int]
         lib.llg_matrix_memory.argtypes = [POINTER(_MatrixMemoryArgs), c_int, c_void_p]
@@ -1660,6 +1665,22 @@ def attention_mix_supported(n_heads: int, head_dim: int, value_dim: int) -> bool
     return bool(_lib("attention_mix").llg_attn_mix_simt_supported(n_heads, head_dim, value_dim))
 
 
+_mix_mma_cache = {}
+
+
+def _use_mix_mma(step: str, dtype: torch.dtype, n_heads: int, n_kv_heads: int, head_dim: int, value_dim: int) -> bool:
+    """Whether a ``step`` ("prefill" or "decode") of attention with capped and mixed scores runs on the tensor cores
+    (csrc/attention_mix_mma.cu): bfloat16, head sizes in steps of 16 up to 128, and what a block's shared memory holds."""
+    if not USE_MIX_MMA or dtype != torch.bfloat16:
+        return False
+    key = (step, n_heads, n_kv_heads, head_dim, value_dim)
+    ok = _mix_mma_cache.get(key)
+    if ok is None:
+        fits = getattr(_lib("attention_mix_mma"), f"llg_attn_mix_{step}_mma_supported")
+        ok = _mix_mma_cache[key] = bool(fits(n_heads, n_kv_heads, head_dim, value_dim))
+    return ok
+
+
 class AttentionForm:
     """What an attention computes beyond the plain causal softmax over keys and values of one head size:
     ``value_dim`` (elements of a value head; 0 = the key heads' size), ``sink`` (None, or the score of a sink that
@@ -1669,7 +1690,8 @@ class AttentionForm:
     ``window`` of the call is a chunk size: a query sees the keys of its own chunk of that many positions, chunks
     counted from position 0, instead of the last ``window`` keys), ``softcap`` (c > 0: a scaled score s becomes ``c tanh(s /
     c)``), ``head_mix`` (a float32 tensor ``[nh, nh]`` on the device: behind the cap, head h's scores become ``sum_g
-    head_mix[h, g] s_g``).  The last two run on kernels of their own (csrc/attention_mix.cu): a block then works on all
+    head_mix[h, g] s_g``).  The last two run on kernels of their own (csrc/attention_mix_mma.cu on the tensor cores,
+    csrc/attention_mix.cu on the CUDA cores): a block then works on all
     query heads of its queries."""
 
     def __init__(self, value_dim: int = 0, sink: Optional[float] = None, gated: bool = False,
@@ -1716,7 +1738,8 @@ def _prefill_kernel(dtype: torch.dtype, head_dim: int, form: AttentionForm) -> s
     return "simt"
 
 
-MIX_TILE_QUERIES = 16        # queries per entry of a step's tile list for the kernels of csrc/attention_mix.cu
+MIX_TILE_QUERIES = 64        # queries per entry of a step's tile list for the kernels for capped and mixed scores
+USE_MIX_MMA = True           # tests switch it off to reach the CUDA-core kernels with bfloat16
 
 
 def prefill_tile_queries(dtype: torch.dtype, head_dim: int, form: AttentionForm = PLAIN_ATTENTION) -> int:
@@ -1775,7 +1798,8 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
         raise KernelError("attn_prefill: a gated form needs a gate [tokens, heads], and only a gated form takes one")
     kernel = _prefill_kernel(q.dtype, hd, form)
     tc, mma = kernel == "tc", kernel == "mma"
-    lib = _lib("attention_mix" if kernel == "mix" else "attention_tc" if tc else "attention_mma" if mma else "attention_simt")
+    mix_mma = kernel == "mix" and _use_mix_mma("prefill", q.dtype, nh, nkv, hd, vd)
+    lib = _lib("attention_mix_mma" if mix_mma else "attention_mix" if kernel == "mix" else "attention_tc" if tc else "attention_mma" if mma else "attention_simt")
     a = _PrefillArgs()
     a.q, a.k_new, a.v_new = _ptr(q), _ptr(k_new, q.dtype), _ptr(v_new, q.dtype)
     a.k_pages, a.v_pages = _ptr(k_pages, q.dtype), _ptr(v_pages, q.dtype)
@@ -1787,7 +1811,9 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
     a.scale, a.window = float(scale), int(window)
     a.n_tokens, a.n_pages = k_new.shape[0], k_pages.shape[0]
     _set_form(a, form, hd, gate)
-    if kernel == "mix":
+    if mix_mma:
+        _check(lib, lib.llg_attn_mix_prefill_mma(byref(a), tile_queries, _stream()))
+    elif kernel == "mix":
         _check(lib, lib.llg_attn_mix_prefill_simt(byref(a), tile_queries, _dt(q), _stream()))
     elif tc:
         _check(lib, lib.llg_attn_prefill_tc(byref(a), _stream()))
@@ -1934,7 +1960,8 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
     if plan is not None:
         n_splits, balance = plan.n_splits, plan.balance
     mma = form.one_head_size(hd) and _use_mma(q.dtype, hd) and not form.mixes
-    lib = _lib("attention_mix" if form.mixes else "attention_mma" if mma else "attention_simt")
+    mix_mma = form.mixes and _use_mix_mma("decode", q.dtype, nh, nkv, hd, vd)
+    lib = _lib("attention_mix_mma" if mix_mma else "attention_mix" if form.mixes else "attention_mma" if mma else "attention_simt")
     need = b * nh * n_splits * (vd + 2)
     if n_splits < 1 or scratch.numel() < need:
         raise KernelError(f"attn_decode: {n_splits} splits, scratch of {scratch.numel()} floats, {need} needed")
@@ -1953,6 +1980,8 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
             raise KernelError(f"attn_decode: needs {b * nkv} zeroed int32 counters")
         _check(lib, lib.llg_attn_decode_mma(byref(a), _ptr(out, q.dtype), _ptr(counters, torch.int32),
                                             int(bool(balance) and b * nkv <= attn_decode_balance_pairs() and b <= 32), _stream()))
+    elif mix_mma:
+        _check(lib, lib.llg_attn_mix_decode_mma(byref(a), _ptr(out, q.dtype), _stream()), kernels=2)
     elif form.mixes:
         _check(lib, lib.llg_attn_mix_decode_simt(byref(a), _ptr(out, q.dtype), _dt(q), _stream()), kernels=2)
     else:

@@ -328,16 +328,19 @@ def _mixed_attention(q, k, v, scale, cap, talk, sink, gate, first):
 
 
 MIX_SIZES = [(4, 2, 16, 24, 5.0), (6, 1, 128, 128, 50.0), (8, 2, 64, 32, 30.0), (5, 5, 32, 80, 10.0), (3, 1, 10, 6, 0.0), (1, 1, 12, 20, 2.0),
-             (16, 4, 128, 64, 20.0), (24, 8, 64, 64, 15.0), (7, 7, 48, 16, 8.0), (32, 8, 32, 32, 25.0), (12, 4, 16, 48, 3.0)]
+             (16, 4, 128, 64, 20.0), (24, 8, 64, 64, 15.0), (7, 7, 48, 16, 8.0), (32, 8, 32, 32, 25.0), (12, 4, 16, 48, 3.0),
+             (32, 8, 128, 128, 50.0), (40, 8, 128, 64, 50.0), (16, 16, 128, 128, 9.0), (48, 2, 16, 16, 5.0), (2, 1, 64, 112, 4.0)]
 
 
-@pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
+@pytest.mark.parametrize("dtype,tensor_cores", [(torch.float32, False), (torch.bfloat16, True), (torch.bfloat16, False)],
+                         ids=["f32", "bf16", "bf16-cuda-cores"])
 @pytest.mark.parametrize("window,chunked", [(0, False), (70, False), (50, True)])
 @pytest.mark.parametrize("nh,nkv,hd,vd,cap", MIX_SIZES)
-def test_attention_with_capped_and_mixed_scores(dtype, nh, nkv, hd, vd, cap, window, chunked):
+def test_attention_with_capped_and_mixed_scores(monkeypatch, dtype, tensor_cores, nh, nkv, hd, vd, cap, window, chunked):
     """A prompt step (old keys in shuffled pages, new ones packed) and a decode step of unequal sequences; sinks, gates and the
     masks beside the mixture; one key far back stands out for one query's head, so that a mixture that lost it would show."""
     ops = ops_module()
+    monkeypatch.setattr(ops, "USE_MIX_MMA", tensor_cores)
     gen = torch.Generator().manual_seed(nh * hd + window)
     talk = torch.eye(nh) + 0.5 * torch.randn(nh, nh, generator=gen)
     sinks = torch.randn(nh, generator=gen)
