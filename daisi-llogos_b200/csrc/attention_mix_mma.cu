@@ -121,17 +121,21 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
   const bf16 *kp = (const bf16*)a.k_pages, *vp = (const bf16*)a.v_pages;
 
   // rows of a key tile of the block's key/value heads; a tile's old positions lie in one page (KT divides the page)
-  auto load = [&](int tile, const bf16* fresh_base, const bf16* page_base, int d, unsigned char* dst, int rs) {
-    const int kt = k_begin + tile * KT, cpr = d / 8;
-    for (int idx = tid; idx < kvn * KT * cpr; idx += MT) {
-      const int ch = idx % cpr, r = idx / cpr, row = r % KT, kv = r / KT, pos = kt + row;
-      const bool valid = pos < k_end;
-      const bf16* src = fresh_base;
-      if (valid) {
-        if (pos >= lb) src = fresh_base + ((long long)(tok0 + pos - lb) * a.nkv + kv0 + kv) * d + ch * 8;
-        else src = page_base + kv_row(a.page_table, a.table_width, a.ring_pages, slot, pos, kv0 + kv, a.nkv) * d + ch * 8;
+  // (a thread copies 16-byte piece `ch` of rows r0, r0 + step, ...: no division in the loop)
+  const int k_cpr = hd / 8, v_cpr = vd / 8;
+  const int k_ch = tid % k_cpr, k_r0 = tid / k_cpr, k_step = MT / k_cpr, v_ch = tid % v_cpr, v_r0 = tid / v_cpr, v_step = MT / v_cpr;
+  auto load = [&](int tile, const bf16* fresh_base, const bf16* page_base, int d, unsigned char* dst, int rs, int ch, int r0, int step) {
+    const int kt = k_begin + tile * KT;
+    const bf16* fresh = fresh_base + ((long long)(tok0 + kt - lb) * a.nkv + kv0) * d + ch * 8;
+    const bf16* old = kt < lb ? page_base + kv_row(a.page_table, a.table_width, a.ring_pages, slot, kt, kv0, a.nkv) * d + ch * 8 : nullptr;
+    const uint32_t to = smem_u32(dst) + ch * 16;
+    if (r0 < step) {
+      for (int r = r0; r < kvn * KT; r += step) {
+        const int row = r % KT, kv = r / KT, pos = kt + row;
+        const bool valid = pos < k_end;
+        const bf16* src = pos >= lb ? fresh + (long long)(row * a.nkv + kv) * d : old + (kv * LLG_PAGE + row) * d;
+        cp_async16(to + r * rs, valid ? src : fresh_base, valid);
       }
-      cp_async16(smem_u32(dst + (size_t)(kv * KT + row) * rs + ch * 16), src, valid);
     }
     cp_async_commit();
   };
@@ -140,7 +144,7 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
     const bool valid = row < nq;
     cp_async16(smem_u32(Qs + (size_t)r * rsk + ch * 16), qg + ((long long)(tok0 + q_off + (valid ? row : 0)) * nh + h0 + h) * hd + ch * 8, valid);
   }
-  load(0, kn, kp, hd, Ks, rsk);                   // (one group with the queries)
+  load(0, kn, kp, hd, Ks, rsk, k_ch, k_r0, k_step);                   // (one group with the queries)
   for (int idx = tid; idx < nh * hc8; idx += MT) {
     const int j = idx % hc8, gg = idx / hc8;
     T[idx] = j >= hn ? 0.f : a.head_mix ? a.head_mix[(h0 + j) * nh + gg] : (gg == h0 + j ? 1.f : 0.f);
@@ -157,12 +161,14 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
   const float two_over_cap = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
   const int qpos0 = pos0 + sub * 16 + g;
   const uint32_t s_base = smem_u32(S);
+  // pairs of neighbouring positions in a tile (a power of two: qt is 1 or 2), and the mixture's items, at most one a thread
+  const int pairs = BQ * (KT / 2), pairs_log2 = 31 - __clz(pairs), items = pairs * (hc8 / 8);
   cluster_arrive();
   for (int tile = 0; tile < n_tiles; ++tile) {
     const int kt = k_begin + tile * KT;
     cp_async_wait<0>();
     __syncthreads();                              // keys are here; every warp is done with the last tile's values
-    load(tile, vn, vp, vd, Vs, rsv);
+    load(tile, vn, vp, vd, Vs, rsv, v_ch, v_r0, v_step);
     // this warp's scores: 16 queries x KT keys of its head
     float s[KT / 8][4];
     if (working) {
@@ -209,45 +215,34 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
     }
     cluster_arrive();
     cluster_wait();                               // all heads' scores are here; the keys may be replaced
-    if (tile + 1 < n_tiles) load(tile + 1, kn, kp, hd, Ks, rsk);
+    if (tile + 1 < n_tiles) load(tile + 1, kn, kp, hd, Ks, rsk, k_ch, k_r0, k_step);
     else cp_async_commit();
     // the mixture: an item is two neighbouring positions for eight of the block's heads
-    constexpr int ITEMS = 2;
-    const int pairs = BQ * (KT / 2), items = pairs * (hc8 / 8);
-    float mx[ITEMS][8][2];
+    float mx[8][2];
+    const bool mixing = tid < items;
+    float* sp = S + ((tid & (pairs - 1)) / (KT / 2)) * SR + 2 * (tid % (KT / 2));
+    const int j0 = (tid >> pairs_log2) * 8;
+    if (mixing) {
 #pragma unroll
-    for (int it = 0; it < ITEMS; ++it) {
-      const int item = tid + it * MT;
-      if (item < items) {
-#pragma unroll
-        for (int j = 0; j < 8; ++j) mx[it][j][0] = mx[it][j][1] = 0.f;
-        const int pr = item % pairs, hg = item / pairs;
-        const float* sp = S + (pr / (KT / 2)) * SR + 2 * (pr % (KT / 2));
-        const float* tp = T + hg * 8;
+      for (int j = 0; j < 8; ++j) mx[j][0] = mx[j][1] = 0.f;
+      const float* tp = T + j0;
 #pragma unroll 4
-        for (int gg = 0; gg < nh; ++gg) {
-          const float2 v = *reinterpret_cast<const float2*>(sp + gg * BQ * SR);
-          const float4 t0 = *reinterpret_cast<const float4*>(tp + gg * hc8), t1 = *reinterpret_cast<const float4*>(tp + gg * hc8 + 4);
-          const float tt[8] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
+      for (int gg = 0; gg < nh; ++gg) {
+        const float2 v = *reinterpret_cast<const float2*>(sp + gg * BQ * SR);
+        const float4 t0 = *reinterpret_cast<const float4*>(tp + gg * hc8), t1 = *reinterpret_cast<const float4*>(tp + gg * hc8 + 4);
+        const float tt[8] = {t0.x, t0.y, t0.z, t0.w, t1.x, t1.y, t1.z, t1.w};
 #pragma unroll
-          for (int j = 0; j < 8; ++j) {
-            mx[it][j][0] = fmaf(tt[j], v.x, mx[it][j][0]);
-            mx[it][j][1] = fmaf(tt[j], v.y, mx[it][j][1]);
-          }
+        for (int j = 0; j < 8; ++j) {
+          mx[j][0] = fmaf(tt[j], v.x, mx[j][0]);
+          mx[j][1] = fmaf(tt[j], v.y, mx[j][1]);
         }
       }
     }
     __syncthreads();                              // every thread has read all heads' scores: the mixed ones take their place
+    if (mixing) {
 #pragma unroll
-    for (int it = 0; it < ITEMS; ++it) {
-      const int item = tid + it * MT;
-      if (item < items) {
-        const int pr = item % pairs, hg = item / pairs;
-        float* sp = S + (pr / (KT / 2)) * SR + 2 * (pr % (KT / 2));
-#pragma unroll
-        for (int j = 0; j < 8; ++j)
-          if (hg * 8 + j < hn) *reinterpret_cast<float2*>(sp + (hg * 8 + j) * BQ * SR) = make_float2(mx[it][j][0], mx[it][j][1]);
-      }
+      for (int j = 0; j < 8; ++j)
+        if (j0 + j < hn) *reinterpret_cast<float2*>(sp + (j0 + j) * BQ * SR) = make_float2(mx[j][0], mx[j][1]);
     }
     cp_async_wait<1>();                           // the values are here (the next keys may still be on their way)
     __syncthreads();
@@ -338,15 +333,16 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
 
 // ---- one new token per sequence ------------------------------------------------------------------
 
-constexpr int DK = 32;                  // keys per tile
+constexpr int DK = 16;                  // keys per tile
 constexpr int DS = DK + 8;              // floats per row of scores
+constexpr int MAX_STAGES = 6;           // tiles of keys and values in shared memory at most
 constexpr int PR = DK * 2 + 16;         // bytes per row of weights
 constexpr int MAX_ACC = 8;              // 16-row x 16-column pieces of the outputs that a warp may own
-constexpr int MAX_ROWS = 8;             // heads whose softmax a warp may own
+constexpr int MAX_ROWS = 4;             // heads whose softmax half a warp may own
 
-// Shared memory: Q [nh][rsk], K [nkv][DK][rsk], V [nkv][DK][rsv], P [nh][PR] bytes, then floats: scores [nh][DS], corr [nh],
-// the mixture [nh][nh].
-__global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a) {
+// Shared memory: Q [nh][rsk], `stages` times K [nkv][DK][rsk] and V [nkv][DK][rsv], P [nh][PR] bytes, then floats: scores
+// [nh][DS], corr [nh], the mixture [nh][nh].  A tile's keys and values arrive together, stages - 1 tiles ahead.
+__global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a, int stages) {
   extern __shared__ __align__(16) unsigned char smraw[];
   pdl_launch_dependents();
   pdl_wait();
@@ -356,8 +352,8 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
   const int split = blockIdx.x, b = blockIdx.y;
   unsigned char* Qs = smraw;
   unsigned char* Ks = Qs + (size_t)nh * rsk;
-  unsigned char* Vs = Ks + (size_t)nkv * DK * rsk;
-  unsigned char* Ps = Vs + (size_t)nkv * DK * rsv;
+  const int k_bytes = nkv * DK * rsk, stage_bytes = k_bytes + nkv * DK * rsv;
+  unsigned char* Ps = Ks + (size_t)stages * stage_bytes;
   float* S = reinterpret_cast<float*>(Ps + (size_t)nh * PR);
   float* corr = S + nh * DS;
   float* T = corr + nh;
@@ -367,15 +363,33 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
   const int per = (t_end - t0 + a.n_splits - 1) / a.n_splits;
   const int my0 = min(t_end, t0 + split * per), my1 = min(t_end, my0 + per);
   const bf16 *qg = (const bf16*)a.q + (long long)b * nh * hd, *kp = (const bf16*)a.k_pages, *vp = (const bf16*)a.v_pages;
-  auto load = [&](int tile, const bf16* pages, int d, unsigned char* dst, int rs) {
+  const int k_cpr = hd / 8, v_cpr = vd / 8;
+  const int k_ch = tid % k_cpr, k_r0 = tid / k_cpr, k_step = MT / k_cpr, v_ch = tid % v_cpr, v_r0 = tid / v_cpr, v_step = MT / v_cpr;
+  const uint32_t k_to = smem_u32(Ks) + k_ch * 16, v_to = smem_u32(Ks) + k_bytes + v_ch * 16;
+  const bool k_copies = k_r0 < k_step, v_copies = v_r0 < v_step;
+  // the page of a tile is looked up one tile ahead of its copies
+  auto page_of = [&](int tile) {
+    return tile < my1 ? a.page_table[(long long)slot * a.table_width + (tile * DK / LLG_PAGE) % a.ring_pages] : 0;
+  };
+  int page = page_of(my0);
+  auto load = [&](int tile, int stage) {
     if (tile < my1) {
-      const int cpr = d / 8, pos0 = tile * DK;
-      const int page = a.page_table[(long long)slot * a.table_width + (pos0 / LLG_PAGE) % a.ring_pages];
-      const bf16* base = pages + ((long long)page * nkv * LLG_PAGE + pos0 % LLG_PAGE) * d;
-      for (int idx = tid; idx < nkv * DK * cpr; idx += MT) {
-        const int ch = idx % cpr, r = idx / cpr, row = r % DK, kv = r / DK;
-        const bool valid = pos0 + row < len;
-        cp_async16(smem_u32(dst + (size_t)r * rs + ch * 16), valid ? base + ((long long)kv * LLG_PAGE + row) * d + ch * 8 : pages, valid);
+      const int pos0 = tile * DK;
+      const long long base = (long long)page * nkv * LLG_PAGE + pos0 % LLG_PAGE;
+      page = page_of(tile + 1);
+      if (k_copies) {
+        const bf16* src = kp + base * hd + k_ch * 8;
+        for (int r = k_r0; r < nkv * DK; r += k_step) {
+          const bool valid = pos0 + r % DK < len;
+          cp_async16(k_to + stage * stage_bytes + r * rsk, valid ? src + (long long)(r / DK * LLG_PAGE + r % DK) * hd : kp, valid);
+        }
+      }
+      if (v_copies) {
+        const bf16* src = vp + base * vd + v_ch * 8;
+        for (int r = v_r0; r < nkv * DK; r += v_step) {
+          const bool valid = pos0 + r % DK < len;
+          cp_async16(v_to + stage * stage_bytes + r * rsv, valid ? src + (long long)(r / DK * LLG_PAGE + r % DK) * vd : vp, valid);
+        }
       }
     }
     cp_async_commit();
@@ -384,8 +398,7 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
     const int ch = idx % (hd / 8), h = idx / (hd / 8);
     cp_async16(smem_u32(Qs + (size_t)h * rsk + ch * 16), qg + (long long)h * hd + ch * 8, true);
   }
-  load(my0, kp, hd, Ks, rsk);
-  load(my0, vp, vd, Vs, rsv);
+  for (int st = 0; st < stages - 1; ++st) load(my0 + st, st);      // (the queries belong to the first group)
   for (int idx = tid; idx < nh * nh; idx += MT) T[idx] = a.head_mix ? a.head_mix[idx] : (idx / nh == idx % nh ? 1.f : 0.f);
   const int v16 = vd / 16, acc_items = nkv * RC * v16, qk_items = nkv * RC * (DK / 16);
   float o[MAX_ACC][2][4];
@@ -401,14 +414,32 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
   }
   const float two_over_cap = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
   const int frag_row = (lane & 7) + ((lane >> 3) & 1) * 8;
+  // this warp's pieces of the outputs: shared-memory offsets of their weights' and values' rows, first head
+  int p_off[MAX_ACC], v_off[MAX_ACC], c_off[MAX_ACC];
+#pragma unroll
+  for (int i = 0; i < MAX_ACC; ++i) {
+    const int it = min(warp + i * MW, acc_items - 1), vc = it % v16, u = it / v16, row0 = u / RC * G + u % RC * 16;
+    p_off[i] = min(row0 + frag_row, nh - 1) * PR + (lane >> 4) * 16;
+    v_off[i] = (u / RC * DK + frag_row) * rsv + (lane >> 4) * 16 + vc * 32;
+    c_off[i] = min(row0 + g, nh - 1) | min(row0 + g + 8, nh - 1) << 16;
+  }
+  const uint32_t ps_at = smem_u32(Ps);
+  int stage = 0;
   for (int tile = my0; tile < my1; ++tile) {
-    cp_async_wait<1>();
-    __syncthreads();
+    if (stages == 2) cp_async_wait<0>();
+    else if (stages == 3) cp_async_wait<1>();
+    else if (stages == 4) cp_async_wait<2>();
+    else if (stages == 5) cp_async_wait<3>();
+    else cp_async_wait<4>();
+    __syncthreads();                              // the tile is here; the tile before last is no longer read
+    load(tile + stages - 1, stage == 0 ? stages - 1 : stage - 1);
+    const uint32_t k_at = smem_u32(Ks) + stage * stage_bytes, v_at = k_at + k_bytes;
+    stage = stage + 1 == stages ? 0 : stage + 1;
     for (int it = warp; it < qk_items; it += MW) {
-      const int kh = it % (DK / 16), u = it / (DK / 16), rc = u % RC, kv = u / RC;
+      const int kh = it % (DK / 16), u = it / (DK / 16), rc = RC == 1 ? 0 : u % RC, kv = RC == 1 ? u : u / RC;
       const int row0 = kv * G + rc * 16;
       const uint32_t q_addr = smem_u32(Qs + (size_t)min(row0 + frag_row, nh - 1) * rsk) + (lane >> 4) * 16;
-      const uint32_t k_addr = smem_u32(Ks + (size_t)(kv * DK + kh * 16 + (lane & 7) + (lane >> 4) * 8) * rsk) + ((lane >> 3) & 1) * 16;
+      const uint32_t k_addr = k_at + (kv * DK + kh * 16 + (lane & 7) + (lane >> 4) * 8) * rsk + ((lane >> 3) & 1) * 16;
       float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
 #pragma unroll 4
       for (int ks = 0; ks < hd / 16; ++ks) {
@@ -427,37 +458,44 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
                 make_float2(capped(s[j][2 * r] * a.scale, a.softcap, two_over_cap), capped(s[j][2 * r + 1] * a.scale, a.softcap, two_over_cap));
     }
     __syncthreads();
-    load(tile + 1, kp, hd, Ks, rsk);
-    // mixture and softmax: a warp per head, a lane per key
-    const int pos = tile * DK + lane;
+    // mixture and softmax: half a warp per head, a lane per key
+    const int key = lane & 15, pos = tile * DK + key;
     const bool valid = pos < len && pos >= lo;
 #pragma unroll
     for (int i = 0; i < MAX_ROWS; ++i) {
-      const int h = warp + i * MW;
-      if (h >= nh) break;
-      float s = 0.f;
-      const float* tr = T + h * nh;
-#pragma unroll 8
-      for (int gg = 0; gg < nh; ++gg) s = fmaf(tr[gg], S[gg * DS + lane], s);
+      const int h = 2 * warp + (lane >> 4) + i * 2 * MW;
+      if (2 * warp + i * 2 * MW >= nh) break;
+      const bool mine = h < nh;
+      const float* tr = T + (mine ? h : 0) * nh;
+      float s4[4] = {0.f, 0.f, 0.f, 0.f};
+      int gg = 0;
+      for (; gg + 4 <= nh; gg += 4) {
+#pragma unroll
+        for (int x = 0; x < 4; ++x) s4[x] = fmaf(tr[gg + x], S[(gg + x) * DS + key], s4[x]);
+      }
+      for (; gg < nh; ++gg) s4[0] = fmaf(tr[gg], S[gg * DS + key], s4[0]);
+      float s = (s4[0] + s4[1]) + (s4[2] + s4[3]);
       if (!valid) s = -INFINITY;
-      const float m_new = fmaxf(m[i], ceilf(warp_max(s) * LOG2E));
+      float mx = s;
+#pragma unroll
+      for (int x = 8; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
+      const float m_new = fmaxf(m[i], ceilf(mx * LOG2E));
       const float c = m_new == -INFINITY ? 1.f : pow2_whole(m[i] - m_new);
       const float p = m_new == -INFINITY ? 0.f : fast_exp2(fmaf(s, LOG2E, -m_new));
       m[i] = m_new;
       l[i] = l[i] * c + p;                        // this lane's share of the sum
-      *reinterpret_cast<bf16*>(Ps + (size_t)h * PR + lane * 2) = __float2bfloat16_rn(p);
-      if (lane == 0) corr[h] = c;
+      if (mine) {
+        *reinterpret_cast<bf16*>(Ps + (size_t)h * PR + key * 2) = __float2bfloat16_rn(p);
+        if (key == 0) corr[h] = c;
+      }
     }
-    cp_async_wait<1>();
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < MAX_ACC; ++i) {
       const int it = warp + i * MW;
       if (it >= acc_items) break;
-      const int vc = it % v16, u = it / v16, rc = u % RC, kv = u / RC, row0 = kv * G + rc * 16;
-      const float c0 = corr[min(row0 + g, nh - 1)], c1 = corr[min(row0 + g + 8, nh - 1)];
-      const uint32_t p_addr = smem_u32(Ps + (size_t)min(row0 + frag_row, nh - 1) * PR) + (lane >> 4) * 16;
-      const uint32_t v_addr = smem_u32(Vs + (size_t)(kv * DK + frag_row) * rsv) + (lane >> 4) * 16 + vc * 32;
+      const float c0 = corr[c_off[i] & 0xffff], c1 = corr[c_off[i] >> 16];
+      const uint32_t p_addr = ps_at + p_off[i], v_addr = v_at + v_off[i];
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         o[i][j][0] *= c0; o[i][j][1] *= c0; o[i][j][2] *= c1; o[i][j][3] *= c1;
@@ -471,8 +509,6 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
         mma_16816(o[i][1], pa, vb[2], vb[3]);
       }
     }
-    __syncthreads();
-    load(tile + 1, vp, vd, Vs, rsv);
   }
   cp_async_wait<0>();
 #pragma unroll
@@ -494,10 +530,12 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a
   }
 #pragma unroll
   for (int i = 0; i < MAX_ROWS; ++i) {
-    const int h = warp + i * MW;
-    if (h >= nh) break;
-    const float sum = warp_sum(l[i]);
-    if (lane == 0) {
+    const int h = 2 * warp + (lane >> 4) + i * 2 * MW;
+    if (2 * warp + i * 2 * MW >= nh) break;
+    float sum = l[i];
+#pragma unroll
+    for (int x = 8; x > 0; x >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, x);
+    if ((lane & 15) == 0 && h < nh) {
       float* ml = a.part_ml + (((long long)b * nh + h) * a.n_splits + split) * 2;
       ml[0] = m[i] == -INFINITY ? -INFINITY : m[i] * 0.6931471805599453f;      // natural units
       ml[1] = sum;
@@ -520,9 +558,10 @@ bool plan_prefill(int nh, int nkv, int hd, int vd, MixCut* out) {
       MixCut p;
       p.c = c;
       p.hc = (nh + c - 1) / c;
-      p.qt = p.hc <= 4 ? 4 : p.hc <= 8 ? 2 : 1;
+      p.qt = p.hc <= 8 ? 2 : 1;                   // at most MT items of the mixture
       p.kt = kt;
-      p.kvn = min(nkv, (p.hc + G - 2) / G + 1);   // a run of hc heads touches at most that many key/value heads
+      p.kvn = 0;                                  // the most key/value heads that a block's heads reach
+      for (int h0 = 0; h0 < nh; h0 += p.hc) p.kvn = max(p.kvn, (min(h0 + p.hc, nh) - 1) / G - h0 / G + 1);
       p.smem = prefill_smem(nh, hd, vd, p);
       if (p.smem <= SMEM_MAX) {
         *out = p;
@@ -533,13 +572,13 @@ bool plan_prefill(int nh, int nkv, int hd, int vd, MixCut* out) {
   return false;
 }
 
-size_t decode_smem(int nh, int nkv, int hd, int vd) {
+size_t decode_smem(int nh, int nkv, int hd, int vd, int stages) {
   const size_t rsk = 2 * hd + 16, rsv = 2 * vd + 16;
-  return (size_t)nh * rsk + (size_t)nkv * DK * (rsk + rsv) + (size_t)nh * PR + ((size_t)nh * DS + nh + (size_t)nh * nh) * sizeof(float);
+  return (size_t)nh * rsk + (size_t)stages * nkv * DK * (rsk + rsv) + (size_t)nh * PR + ((size_t)nh * DS + nh + (size_t)nh * nh) * sizeof(float);
 }
 
 bool head_sizes_ok(int nh, int nkv, int hd, int vd) {
-  return nh > 0 && nkv > 0 && nh % nkv == 0 && nh <= MW * MAX_ROWS && hd >= 16 && hd <= 128 && hd % 16 == 0 && vd >= 16 && vd <= 128 && vd % 16 == 0;
+  return nh > 0 && nkv > 0 && nh % nkv == 0 && nh <= 2 * MW * MAX_ROWS && hd >= 16 && hd <= 128 && hd % 16 == 0 && vd >= 16 && vd <= 128 && vd % 16 == 0;
 }
 
 }  // namespace
@@ -552,7 +591,7 @@ LLG_API int llg_attn_mix_prefill_mma_supported(int nh, int nkv, int hd, int vd) 
 LLG_API int llg_attn_mix_decode_mma_supported(int nh, int nkv, int hd, int vd) {
   if (!head_sizes_ok(nh, nkv, hd, vd)) return 0;
   const int G = nh / nkv;
-  return nkv * ((G + 15) / 16) * (vd / 16) <= MW * MAX_ACC && decode_smem(nh, nkv, hd, vd) <= SMEM_MAX;
+  return nkv * ((G + 15) / 16) * (vd / 16) <= MW * MAX_ACC && decode_smem(nh, nkv, hd, vd, 2) <= SMEM_MAX;
 }
 
 // tile_queries: queries per entry of `tiles`, a multiple of 64.
@@ -608,10 +647,12 @@ LLG_API int llg_attn_mix_decode_mma(const DecodeArgs* args, void* out, cudaStrea
   LLG_REQUIRE(a.n_splits >= 1 && a.n_splits <= 65535 && a.n_seqs <= 65535, "attn_mix_decode_mma: grid too large");
   LLG_REQUIRE(a.window >= 0 && a.ring_pages > 0 && a.table_width >= a.ring_pages, "attn_mix_decode_mma: bad cache geometry");
   if (a.n_seqs <= 0) return 0;
-  const size_t smem = decode_smem(a.nh, a.nkv, a.hd, vd);
+  int stages = 2;
+  while (stages < MAX_STAGES && decode_smem(a.nh, a.nkv, a.hd, vd, stages + 1) <= SMEM_MAX) ++stages;
+  const size_t smem = decode_smem(a.nh, a.nkv, a.hd, vd, stages);
   cudaError_t e = cudaFuncSetAttribute(attn_mix_decode_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) return llg_fail("attn_mix_decode_mma: shared memory %zu: %s", smem, cudaGetErrorString(e));
-  llg_launch(attn_mix_decode_mma_kernel, dim3(a.n_splits, a.n_seqs), dim3(MT), smem, stream, a);
+  llg_launch(attn_mix_decode_mma_kernel, dim3(a.n_splits, a.n_seqs), dim3(MT), smem, stream, a, stages);
   attn_decode_reduce_kernel<bf16><<<dim3(a.nh, a.n_seqs), 64, 0, stream>>>(a.part_o, a.part_ml, (bf16*)out, a.nh, vd, a.n_splits, a.has_sink,
                                                                         a.sink_score, a.gate, a.sinks);
   return llg_check_launch("attn_mix_decode_mma");
