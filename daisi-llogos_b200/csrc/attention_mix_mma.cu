@@ -8,10 +8,10 @@
 //                          block computes its heads' scores and writes them into the shared memory of every block of the
 //                          cluster; behind a cluster barrier each block mixes all heads' scores into its own heads' and
 //                          goes on with their softmax and values by itself.
-//   attn_mix_decode_mma  : one new token per sequence; a block takes a share of a sequence's keys for all heads (the
-//                          partial results are joined by attn_decode_reduce).
+//   attn_mix_decode_mma  : one new token per sequence; scores, mixture with weights, and values by a kernel each (the partial
+//                          results of a sequence's key splits are joined by attn_decode_reduce).
 //
-// Shared-memory rows of bfloat16 are padded by 16 bytes (conflict-free ldmatrix), rows of scores by 8 floats.
+// In prompt steps shared-memory rows of bfloat16 are padded by 16 bytes (conflict-free ldmatrix), rows of scores by 8 floats.
 #include "common.cuh"
 #include "kernel_args.h"
 #include "attention_reduce.cuh"
@@ -332,214 +332,235 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
 }
 
 // ---- one new token per sequence ------------------------------------------------------------------
+//
+// Three kernels that each stream what they read once, over all the GPU's blocks: the scores of every head (keys read straight
+// into operand registers, a warp per 16 keys of one key/value head), the mixture with the softmax's weights per chunk of
+// CHUNK keys, and the weighted values (read straight into operand registers again).  Between them lie, per sequence, the
+// scores [key][nh] in float32, the weights [nh][key] in bfloat16, and per (head, chunk) the maximum and the sum.  Keys are
+// counted from the first page that the query sees.
+//
+// The order of the elements inside a product over the head's elements is free, and so is the order of an output's columns.
+// Both are chosen so that a lane's operands are 16 neighbouring bytes of a row: for the scores lane (g, t) takes elements
+// 32 c + 8 t .. + 7 of keys g and g + 8 as the operands of two products; for the values lane (g, t) takes elements
+// 64 c + 8 g .. + 7 of keys 2t, 2t + 1, 2t + 8, 2t + 9, and product j of eight uses element j of each.
 
-constexpr int DK = 16;                  // keys per tile
-constexpr int DS = DK + 8;              // floats per row of scores
-constexpr int MAX_STAGES = 6;           // tiles of keys and values in shared memory at most
-constexpr int PR = DK * 2 + 16;         // bytes per row of weights
-constexpr int MAX_ACC = 8;              // 16-row x 16-column pieces of the outputs that a warp may own
-constexpr int MAX_ROWS = 4;             // heads whose softmax half a warp may own
+constexpr int CHUNK = LLG_PAGE;         // keys per chunk of the softmax (one page)
+constexpr int SCORE_KEYS = 128;         // keys per block of the scores' kernel (4 warps)
 
-// Shared memory: Q [nh][rsk], `stages` times K [nkv][DK][rsk] and V [nkv][DK][rsv], P [nh][PR] bytes, then floats: scores
-// [nh][DS], corr [nh], the mixture [nh][nh].  A tile's keys and values arrive together, stages - 1 tiles ahead.
-__global__ void __launch_bounds__(MT, 1) attn_mix_decode_mma_kernel(DecodeArgs a, int stages) {
-  extern __shared__ __align__(16) unsigned char smraw[];
+struct MixScratch {
+  float* scores;                        // [n_seqs][keys][nh]
+  bf16* weights;                        // [n_seqs][nh][keys]
+  float* chunks;                        // [n_seqs][nh][keys / CHUNK][2]: maximum (whole log2 units), sum
+  int keys;                             // most keys of a sequence, whole chunks
+};
+
+__device__ __forceinline__ int first_page_key(const DecodeArgs& a, int len) { return mask_first(len - 1, a.window, a.chunked) / LLG_PAGE * LLG_PAGE; }
+__device__ __forceinline__ int page_at(const DecodeArgs& a, int slot, int pos) {
+  return a.page_table[(long long)slot * a.table_width + (pos / LLG_PAGE) % a.ring_pages];
+}
+
+// HD32: the head's elements in steps of 32, at most (a remainder of 16 is one product more)
+template <int HD32>
+__global__ void __launch_bounds__(128) mix_scores_kernel(DecodeArgs a, MixScratch w) {
   pdl_launch_dependents();
+  const int nh = a.nh, nkv = a.nkv, hd = a.hd, G = nh / nkv;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int kv = blockIdx.y, b = blockIdx.z;
   pdl_wait();
-  const int nh = a.nh, nkv = a.nkv, hd = a.hd, vd = a.vd > 0 ? a.vd : a.hd, G = nh / nkv, RC = (G + 15) / 16;
-  const int rsk = hd * 2 + 16, rsv = vd * 2 + 16;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
-  const int split = blockIdx.x, b = blockIdx.y;
-  unsigned char* Qs = smraw;
-  unsigned char* Ks = Qs + (size_t)nh * rsk;
-  const int k_bytes = nkv * DK * rsk, stage_bytes = k_bytes + nkv * DK * rsv;
-  unsigned char* Ps = Ks + (size_t)stages * stage_bytes;
-  float* S = reinterpret_cast<float*>(Ps + (size_t)nh * PR);
-  float* corr = S + nh * DS;
-  float* T = corr + nh;
-  const int len = a.len_before[b] + 1, slot = a.slots[b];
-  const int lo = mask_first(len - 1, a.window, a.chunked);
-  const int t0 = lo / DK, t_end = (len + DK - 1) / DK;
-  const int per = (t_end - t0 + a.n_splits - 1) / a.n_splits;
-  const int my0 = min(t_end, t0 + split * per), my1 = min(t_end, my0 + per);
-  const bf16 *qg = (const bf16*)a.q + (long long)b * nh * hd, *kp = (const bf16*)a.k_pages, *vp = (const bf16*)a.v_pages;
-  const int k_cpr = hd / 8, v_cpr = vd / 8;
-  const int k_ch = tid % k_cpr, k_r0 = tid / k_cpr, k_step = MT / k_cpr, v_ch = tid % v_cpr, v_r0 = tid / v_cpr, v_step = MT / v_cpr;
-  const uint32_t k_to = smem_u32(Ks) + k_ch * 16, v_to = smem_u32(Ks) + k_bytes + v_ch * 16;
-  const bool k_copies = k_r0 < k_step, v_copies = v_r0 < v_step;
-  // the page of a tile is looked up one tile ahead of its copies
-  auto page_of = [&](int tile) {
-    return tile < my1 ? a.page_table[(long long)slot * a.table_width + (tile * DK / LLG_PAGE) % a.ring_pages] : 0;
-  };
-  int page = page_of(my0);
-  auto load = [&](int tile, int stage) {
-    if (tile < my1) {
-      const int pos0 = tile * DK;
-      const long long base = (long long)page * nkv * LLG_PAGE + pos0 % LLG_PAGE;
-      page = page_of(tile + 1);
-      if (k_copies) {
-        const bf16* src = kp + base * hd + k_ch * 8;
-        for (int r = k_r0; r < nkv * DK; r += k_step) {
-          const bool valid = pos0 + r % DK < len;
-          cp_async16(k_to + stage * stage_bytes + r * rsk, valid ? src + (long long)(r / DK * LLG_PAGE + r % DK) * hd : kp, valid);
-        }
-      }
-      if (v_copies) {
-        const bf16* src = vp + base * vd + v_ch * 8;
-        for (int r = v_r0; r < nkv * DK; r += v_step) {
-          const bool valid = pos0 + r % DK < len;
-          cp_async16(v_to + stage * stage_bytes + r * rsv, valid ? src + (long long)(r / DK * LLG_PAGE + r % DK) * vd : vp, valid);
-        }
-      }
-    }
-    cp_async_commit();
-  };
-  for (int idx = tid; idx < nh * (hd / 8); idx += MT) {
-    const int ch = idx % (hd / 8), h = idx / (hd / 8);
-    cp_async16(smem_u32(Qs + (size_t)h * rsk + ch * 16), qg + (long long)h * hd + ch * 8, true);
-  }
-  for (int st = 0; st < stages - 1; ++st) load(my0 + st, st);      // (the queries belong to the first group)
-  for (int idx = tid; idx < nh * nh; idx += MT) T[idx] = a.head_mix ? a.head_mix[idx] : (idx / nh == idx % nh ? 1.f : 0.f);
-  const int v16 = vd / 16, acc_items = nkv * RC * v16, qk_items = nkv * RC * (DK / 16);
-  float o[MAX_ACC][2][4];
-#pragma unroll
-  for (int i = 0; i < MAX_ACC; ++i)
-#pragma unroll
-    for (int e = 0; e < 4; ++e) o[i][0][e] = o[i][1][e] = 0.f;
-  float m[MAX_ROWS], l[MAX_ROWS];
-#pragma unroll
-  for (int i = 0; i < MAX_ROWS; ++i) {
-    m[i] = -INFINITY;
-    l[i] = 0.f;
-  }
+  const int len = a.len_before[b] + 1, base = first_page_key(a, len);
+  const int k0 = base + blockIdx.x * SCORE_KEYS;
+  if (k0 >= len) return;
+  const int slot = a.slots[b], steps = hd / 32, tail = hd % 32;
   const float two_over_cap = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
-  const int frag_row = (lane & 7) + ((lane >> 3) & 1) * 8;
-  // this warp's pieces of the outputs: shared-memory offsets of their weights' and values' rows, first head
-  int p_off[MAX_ACC], v_off[MAX_ACC], c_off[MAX_ACC];
+  const bf16* q = (const bf16*)a.q + ((long long)b * nh + kv * G) * hd;
 #pragma unroll
-  for (int i = 0; i < MAX_ACC; ++i) {
-    const int it = min(warp + i * MW, acc_items - 1), vc = it % v16, u = it / v16, row0 = u / RC * G + u % RC * 16;
-    p_off[i] = min(row0 + frag_row, nh - 1) * PR + (lane >> 4) * 16;
-    v_off[i] = (u / RC * DK + frag_row) * rsv + (lane >> 4) * 16 + vc * 32;
-    c_off[i] = min(row0 + g, nh - 1) | min(row0 + g + 8, nh - 1) << 16;
-  }
-  const uint32_t ps_at = smem_u32(Ps);
-  int stage = 0;
-  for (int tile = my0; tile < my1; ++tile) {
-    if (stages == 2) cp_async_wait<0>();
-    else if (stages == 3) cp_async_wait<1>();
-    else if (stages == 4) cp_async_wait<2>();
-    else if (stages == 5) cp_async_wait<3>();
-    else cp_async_wait<4>();
-    __syncthreads();                              // the tile is here; the tile before last is no longer read
-    load(tile + stages - 1, stage == 0 ? stages - 1 : stage - 1);
-    const uint32_t k_at = smem_u32(Ks) + stage * stage_bytes, v_at = k_at + k_bytes;
-    stage = stage + 1 == stages ? 0 : stage + 1;
-    for (int it = warp; it < qk_items; it += MW) {
-      const int kh = it % (DK / 16), u = it / (DK / 16), rc = RC == 1 ? 0 : u % RC, kv = RC == 1 ? u : u / RC;
-      const int row0 = kv * G + rc * 16;
-      const uint32_t q_addr = smem_u32(Qs + (size_t)min(row0 + frag_row, nh - 1) * rsk) + (lane >> 4) * 16;
-      const uint32_t k_addr = k_at + (kv * DK + kh * 16 + (lane & 7) + (lane >> 4) * 8) * rsk + ((lane >> 3) & 1) * 16;
-      float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll 4
-      for (int ks = 0; ks < hd / 16; ++ks) {
-        uint32_t qf[4], kb[4];
-        ldmatrix_x4(qf, q_addr + ks * 32);
-        ldmatrix_x4(kb, k_addr + ks * 32);
-        mma_16816(s[0], qf, kb[0], kb[1]);
-        mma_16816(s[1], qf, kb[2], kb[3]);
+  for (int it = 0; it < SCORE_KEYS / 64; ++it) {
+    const int kt = k0 + it * 64 + warp * 16;
+    if (kt >= len) break;
+    const bf16* row = (const bf16*)a.k_pages + (((long long)page_at(a, slot, kt) * nkv + kv) * LLG_PAGE + kt % LLG_PAGE + g) * hd;
+    uint4 k_lo[HD32], k_hi[HD32];
+    uint2 t_lo = make_uint2(0, 0), t_hi = make_uint2(0, 0);
+#pragma unroll
+    for (int c = 0; c < HD32; ++c)
+      if (c < steps) {
+        k_lo[c] = *reinterpret_cast<const uint4*>(row + c * 32 + t * 8);
+        k_hi[c] = *reinterpret_cast<const uint4*>(row + 8 * hd + c * 32 + t * 8);
       }
-#pragma unroll
-      for (int j = 0; j < 2; ++j)
-#pragma unroll
-        for (int r = 0; r < 2; ++r)
-          if (rc * 16 + g + r * 8 < G)
-            *reinterpret_cast<float2*>(S + (row0 + g + r * 8) * DS + kh * 16 + j * 8 + 2 * t) =
-                make_float2(capped(s[j][2 * r] * a.scale, a.softcap, two_over_cap), capped(s[j][2 * r + 1] * a.scale, a.softcap, two_over_cap));
+    if (tail) {
+      t_lo = *reinterpret_cast<const uint2*>(row + steps * 32 + t * 4);
+      t_hi = *reinterpret_cast<const uint2*>(row + 8 * hd + steps * 32 + t * 4);
     }
-    __syncthreads();
-    // mixture and softmax: half a warp per head, a lane per key
-    const int key = lane & 15, pos = tile * DK + key;
-    const bool valid = pos < len && pos >= lo;
+    float* dst = w.scores + ((long long)b * w.keys + kt - base + g) * nh + kv * G;
+    for (int g0 = 0; g0 < G; g0 += 8) {
+      const bf16* qr = q + (long long)min(g0 + g, G - 1) * hd;        // column g of the product: head g0 + g
+      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-    for (int i = 0; i < MAX_ROWS; ++i) {
-      const int h = 2 * warp + (lane >> 4) + i * 2 * MW;
-      if (2 * warp + i * 2 * MW >= nh) break;
-      const bool mine = h < nh;
-      const float* tr = T + (mine ? h : 0) * nh;
-      float s4[4] = {0.f, 0.f, 0.f, 0.f};
-      int gg = 0;
-      for (; gg + 4 <= nh; gg += 4) {
-#pragma unroll
-        for (int x = 0; x < 4; ++x) s4[x] = fmaf(tr[gg + x], S[(gg + x) * DS + key], s4[x]);
-      }
-      for (; gg < nh; ++gg) s4[0] = fmaf(tr[gg], S[gg * DS + key], s4[0]);
-      float s = (s4[0] + s4[1]) + (s4[2] + s4[3]);
-      if (!valid) s = -INFINITY;
-      float mx = s;
-#pragma unroll
-      for (int x = 8; x > 0; x >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, x));
-      const float m_new = fmaxf(m[i], ceilf(mx * LOG2E));
-      const float c = m_new == -INFINITY ? 1.f : pow2_whole(m[i] - m_new);
-      const float p = m_new == -INFINITY ? 0.f : fast_exp2(fmaf(s, LOG2E, -m_new));
-      m[i] = m_new;
-      l[i] = l[i] * c + p;                        // this lane's share of the sum
-      if (mine) {
-        *reinterpret_cast<bf16*>(Ps + (size_t)h * PR + key * 2) = __float2bfloat16_rn(p);
-        if (key == 0) corr[h] = c;
-      }
-    }
-    __syncthreads();
-#pragma unroll
-    for (int i = 0; i < MAX_ACC; ++i) {
-      const int it = warp + i * MW;
-      if (it >= acc_items) break;
-      const float c0 = corr[c_off[i] & 0xffff], c1 = corr[c_off[i] >> 16];
-      const uint32_t p_addr = ps_at + p_off[i], v_addr = v_at + v_off[i];
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        o[i][j][0] *= c0; o[i][j][1] *= c0; o[i][j][2] *= c1; o[i][j][3] *= c1;
+      for (int c = 0; c < HD32; ++c)
+        if (c < steps) {
+          const uint4 qf = *reinterpret_cast<const uint4*>(qr + c * 32 + t * 8);
+          const uint32_t a0[4] = {k_lo[c].x, k_hi[c].x, k_lo[c].y, k_hi[c].y}, a1[4] = {k_lo[c].z, k_hi[c].z, k_lo[c].w, k_hi[c].w};
+          mma_16816(s0, a0, qf.x, qf.y);
+          mma_16816(s1, a1, qf.z, qf.w);
+        }
+      if (tail) {
+        const uint2 qf = *reinterpret_cast<const uint2*>(qr + steps * 32 + t * 4);
+        const uint32_t a0[4] = {t_lo.x, t_hi.x, t_lo.y, t_hi.y};
+        mma_16816(s0, a0, qf.x, qf.y);
       }
 #pragma unroll
-      for (int kk = 0; kk < DK / 16; ++kk) {
-        uint32_t pa[4], vb[4];
-        ldmatrix_x4(pa, p_addr + kk * 32);
-        ldmatrix_x4_trans(vb, v_addr + kk * 16 * rsv);
-        mma_16816(o[i][0], pa, vb[0], vb[1]);
-        mma_16816(o[i][1], pa, vb[2], vb[3]);
+      for (int e = 0; e < 4; ++e) {                 // keys g (e < 2) and g + 8, heads g0 + 2t and g0 + 2t + 1
+        const int h = g0 + 2 * t + (e & 1);
+        if (h < G) dst[(long long)(e >> 1) * 8 * nh + h] = capped((s0[e] + s1[e]) * a.scale, a.softcap, two_over_cap);
       }
     }
   }
-  cp_async_wait<0>();
+}
+
+// rows of scores and of the mixture in shared memory, in floats: the heads filled up to a multiple of four, and four more
+// so that neighbouring rows start in different banks
+__host__ __device__ inline int heads_stride(int nh) { return (nh + 3) / 4 * 4 + 4; }
+
+// The mixture and a chunk's softmax: a warp takes four heads at a time, a lane two keys.
+__global__ void __launch_bounds__(256) mix_weights_kernel(DecodeArgs a, MixScratch w) {
+  extern __shared__ __align__(16) float msm[];
+  pdl_launch_dependents();
+  const int nh = a.nh, hs = heads_stride(nh), nh4 = (nh + 3) & ~3;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.y;
+  float* T = msm;                                 // [nh4][hs]
+  float* S = T + nh4 * hs;                        // [CHUNK][hs]
+  for (int idx = threadIdx.x; idx < nh4 * hs; idx += 256) {
+    const int h = idx / hs, gg = idx - h * hs;
+    T[idx] = h >= nh || gg >= nh ? 0.f : a.head_mix ? a.head_mix[h * nh + gg] : (h == gg ? 1.f : 0.f);
+  }
+  pdl_wait();
+  const int len = a.len_before[b] + 1, lo = mask_first(len - 1, a.window, a.chunked), base = lo / LLG_PAGE * LLG_PAGE;
+  const int r0 = blockIdx.x * CHUNK;
+  if (base + r0 >= len) return;
+  const float* src = w.scores + ((long long)b * w.keys + r0) * nh;
+  for (int idx = threadIdx.x; idx < CHUNK * nh; idx += 256) {
+    const int k = idx / nh, h = idx - k * nh;
+    S[k * hs + h] = base + r0 + k < len ? src[idx] : 0.f;
+  }
+  for (int idx = threadIdx.x; idx < CHUNK * (hs - nh); idx += 256) S[idx / (hs - nh) * hs + nh + idx % (hs - nh)] = 0.f;
+  __syncthreads();
+  for (int h0 = warp * 4; h0 < nh; h0 += 32) {
+    float acc[4][2] = {};
+    for (int gg = 0; gg < nh4; gg += 4) {
+      const float4 x = *reinterpret_cast<const float4*>(S + lane * hs + gg), y = *reinterpret_cast<const float4*>(S + (lane + 32) * hs + gg);
 #pragma unroll
-  for (int i = 0; i < MAX_ACC; ++i) {
-    const int it = warp + i * MW;
-    if (it >= acc_items) break;
-    const int vc = it % v16, u = it / v16, rc = u % RC, kv = u / RC;
+      for (int j = 0; j < 4; ++j) {
+        const float4 m = *reinterpret_cast<const float4*>(T + (h0 + j) * hs + gg);
+        acc[j][0] = fmaf(m.x, x.x, acc[j][0]); acc[j][1] = fmaf(m.x, y.x, acc[j][1]);
+        acc[j][0] = fmaf(m.y, x.y, acc[j][0]); acc[j][1] = fmaf(m.y, y.y, acc[j][1]);
+        acc[j][0] = fmaf(m.z, x.z, acc[j][0]); acc[j][1] = fmaf(m.z, y.z, acc[j][1]);
+        acc[j][0] = fmaf(m.w, x.w, acc[j][0]); acc[j][1] = fmaf(m.w, y.w, acc[j][1]);
+      }
+    }
+    const int p0 = base + r0 + lane, p1 = p0 + 32;
+    const bool v0 = p0 < len && p0 >= lo, v1 = p1 < len && p1 >= lo;
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      if (rc * 16 + g + r * 8 >= G) continue;
-      const int h = kv * G + rc * 16 + g + r * 8;
-      float* dst = a.part_o + (((long long)b * nh + h) * a.n_splits + split) * vd + vc * 16 + 2 * t;
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        dst[j * 8] = o[i][j][2 * r];
-        dst[j * 8 + 1] = o[i][j][2 * r + 1];
+    for (int j = 0; j < 4; ++j) {
+      const int h = h0 + j;
+      if (h >= nh) break;
+      const float top = warp_max(fmaxf(v0 ? acc[j][0] : -INFINITY, v1 ? acc[j][1] : -INFINITY));
+      const float m = ceilf(top * LOG2E);         // whole log2 units: rescaling between chunks is exact
+      const float e0 = v0 ? fast_exp2(fmaf(acc[j][0], LOG2E, -m)) : 0.f, e1 = v1 ? fast_exp2(fmaf(acc[j][1], LOG2E, -m)) : 0.f;
+      const float sum = warp_sum(e0 + e1);
+      bf16* dst = w.weights + ((long long)b * nh + h) * w.keys + r0 + lane;
+      dst[0] = __float2bfloat16_rn(e0);
+      dst[32] = __float2bfloat16_rn(e1);
+      if (lane == 0) {
+        float* c = w.chunks + (((long long)b * nh + h) * (w.keys / CHUNK) + blockIdx.x) * 2;
+        c[0] = m;
+        c[1] = sum;
       }
     }
   }
-#pragma unroll
-  for (int i = 0; i < MAX_ROWS; ++i) {
-    const int h = 2 * warp + (lane >> 4) + i * 2 * MW;
-    if (2 * warp + i * 2 * MW >= nh) break;
-    float sum = l[i];
-#pragma unroll
-    for (int x = 8; x > 0; x >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, x);
-    if ((lane & 15) == 0 && h < nh) {
-      float* ml = a.part_ml + (((long long)b * nh + h) * a.n_splits + split) * 2;
-      ml[0] = m[i] == -INFINITY ? -INFINITY : m[i] * 0.6931471805599453f;      // natural units
-      ml[1] = sum;
+}
+
+// The weighted values: block (split, key/value head and up to 16 of its query heads, sequence); the four warps take a chunk's
+// four runs of 16 keys.  All partial results are relative to the sequence's largest maximum.
+template <int VD64>
+__global__ void __launch_bounds__(128) mix_values_kernel(DecodeArgs a, MixScratch w) {
+  pdl_launch_dependents();
+  __shared__ float top_of[16], merge[4][16][VD64 * 64 + 4];
+  const int nh = a.nh, nkv = a.nkv, vd = a.vd > 0 ? a.vd : a.hd, G = nh / nkv, RC = (G + 15) / 16;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+  const int split = blockIdx.x, kv = blockIdx.y / RC, h0 = kv * G + blockIdx.y % RC * 16, b = blockIdx.z;
+  const int gn = min(16, kv * G + G - h0);        // heads of this block
+  pdl_wait();
+  const int len = a.len_before[b] + 1, base = first_page_key(a, len), slot = a.slots[b];
+  const int n_chunks = (len - base + CHUNK - 1) / CHUNK, all = w.keys / CHUNK;
+  const int per = (n_chunks + a.n_splits - 1) / a.n_splits;
+  const int c0 = min(n_chunks, split * per), c1 = min(n_chunks, c0 + per);
+  const float* ch = w.chunks + ((long long)b * nh + h0) * all * 2;
+  // the largest maximum of every head, and this split's share of the sum
+  for (int h = warp; h < gn; h += 4) {
+    float m = -INFINITY, l = 0.f;
+    for (int c = lane; c < n_chunks; c += 32) m = fmaxf(m, ch[((long long)h * all + c) * 2]);
+    m = warp_max(m);
+    for (int c = c0 + lane; c < c1; c += 32) l += pow2_whole(ch[((long long)h * all + c) * 2] - m) * ch[((long long)h * all + c) * 2 + 1];
+    l = warp_sum(l);
+    if (lane == 0) {
+      top_of[h] = m;
+      float* ml = a.part_ml + (((long long)b * nh + h0 + h) * a.n_splits + split) * 2;
+      ml[0] = c0 < c1 ? m * 0.6931471805599453f : -INFINITY;          // natural units
+      ml[1] = l;
     }
+  }
+  __syncthreads();
+  const float m0 = top_of[min(g, gn - 1)], m1 = top_of[min(g + 8, gn - 1)];
+  const bf16* p0 = w.weights + ((long long)b * nh + h0 + min(g, gn - 1)) * w.keys + warp * 16 + 2 * t;
+  const bf16* p1 = w.weights + ((long long)b * nh + h0 + min(g + 8, gn - 1)) * w.keys + warp * 16 + 2 * t;
+  float o[VD64][8][4];
+#pragma unroll
+  for (int c = 0; c < VD64; ++c)
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[c][j][e] = 0.f;
+  auto scaled = [](uint32_t p, float f) {         // two weights times a power of two
+    const __nv_bfloat162 v = __hmul2(*reinterpret_cast<const __nv_bfloat162*>(&p), __float2bfloat162_rn(f));
+    return *reinterpret_cast<const uint32_t*>(&v);
+  };
+  int page = c0 < c1 ? page_at(a, slot, base + c0 * CHUNK) : 0;
+  for (int c = c0; c < c1; ++c) {
+    const bf16* rows = (const bf16*)a.v_pages + (((long long)page * nkv + kv) * LLG_PAGE + warp * 16) * vd;
+    uint4 v[VD64][4];
+#pragma unroll
+    for (int x = 0; x < VD64; ++x) {
+      const int d = x * 64 + g * 8;
+#pragma unroll
+      for (int r = 0; r < 4; ++r)
+        v[x][r] = d < vd ? *reinterpret_cast<const uint4*>(rows + (long long)(2 * t + (r & 1) + (r >> 1) * 8) * vd + d) : make_uint4(0, 0, 0, 0);
+    }
+    if (c + 1 < c1) page = page_at(a, slot, base + (c + 1) * CHUNK);
+    const float f0 = pow2_whole(ch[((long long)min(g, gn - 1) * all + c) * 2] - m0);
+    const float f1 = pow2_whole(ch[((long long)min(g + 8, gn - 1) * all + c) * 2] - m1);
+    const uint32_t pa[4] = {scaled(*reinterpret_cast<const uint32_t*>(p0 + c * CHUNK), f0), scaled(*reinterpret_cast<const uint32_t*>(p1 + c * CHUNK), f1),
+                            scaled(*reinterpret_cast<const uint32_t*>(p0 + c * CHUNK + 8), f0), scaled(*reinterpret_cast<const uint32_t*>(p1 + c * CHUNK + 8), f1)};
+#pragma unroll
+    for (int x = 0; x < VD64; ++x) {
+      const uint32_t r0[4] = {v[x][0].x, v[x][0].y, v[x][0].z, v[x][0].w}, r1[4] = {v[x][1].x, v[x][1].y, v[x][1].z, v[x][1].w};
+      const uint32_t r2[4] = {v[x][2].x, v[x][2].y, v[x][2].z, v[x][2].w}, r3[4] = {v[x][3].x, v[x][3].y, v[x][3].z, v[x][3].w};
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {               // element j of the four rows: the low or the high half of word j / 2
+        const uint32_t sel = j & 1 ? 0x7632u : 0x5410u;
+        mma_16816(o[x][j], pa, __byte_perm(r0[j / 2], r1[j / 2], sel), __byte_perm(r2[j / 2], r3[j / 2], sel));
+      }
+    }
+  }
+  // column n of product j is element 64 x + 8 n + j; add the four warps up
+#pragma unroll
+  for (int x = 0; x < VD64; ++x)
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) merge[warp][g + (e >> 1) * 8][x * 64 + 8 * (2 * t + (e & 1)) + j] = o[x][j][e];
+  __syncthreads();
+  for (int idx = threadIdx.x; idx < gn * vd; idx += 128) {
+    const int h = idx / vd, d = idx - h * vd;
+    a.part_o[(((long long)b * nh + h0 + h) * a.n_splits + split) * vd + d] = (merge[0][h][d] + merge[1][h][d]) + (merge[2][h][d] + merge[3][h][d]);
   }
 }
 
@@ -572,13 +593,8 @@ bool plan_prefill(int nh, int nkv, int hd, int vd, MixCut* out) {
   return false;
 }
 
-size_t decode_smem(int nh, int nkv, int hd, int vd, int stages) {
-  const size_t rsk = 2 * hd + 16, rsv = 2 * vd + 16;
-  return (size_t)nh * rsk + (size_t)stages * nkv * DK * (rsk + rsv) + (size_t)nh * PR + ((size_t)nh * DS + nh + (size_t)nh * nh) * sizeof(float);
-}
-
 bool head_sizes_ok(int nh, int nkv, int hd, int vd) {
-  return nh > 0 && nkv > 0 && nh % nkv == 0 && nh <= 2 * MW * MAX_ROWS && hd >= 16 && hd <= 128 && hd % 16 == 0 && vd >= 16 && vd <= 128 && vd % 16 == 0;
+  return nh > 0 && nkv > 0 && nh % nkv == 0 && nh <= 128 && hd >= 16 && hd <= 128 && hd % 16 == 0 && vd >= 16 && vd <= 128 && vd % 16 == 0;
 }
 
 }  // namespace
@@ -588,11 +604,7 @@ LLG_API int llg_attn_mix_prefill_mma_supported(int nh, int nkv, int hd, int vd) 
   MixCut p;
   return head_sizes_ok(nh, nkv, hd, vd) && plan_prefill(nh, nkv, hd, vd, &p);
 }
-LLG_API int llg_attn_mix_decode_mma_supported(int nh, int nkv, int hd, int vd) {
-  if (!head_sizes_ok(nh, nkv, hd, vd)) return 0;
-  const int G = nh / nkv;
-  return nkv * ((G + 15) / 16) * (vd / 16) <= MW * MAX_ACC && decode_smem(nh, nkv, hd, vd, 2) <= SMEM_MAX;
-}
+LLG_API int llg_attn_mix_decode_mma_supported(int nh, int nkv, int hd, int vd) { return head_sizes_ok(nh, nkv, hd, vd); }
 
 // tile_queries: queries per entry of `tiles`, a multiple of 64.
 LLG_API int llg_attn_mix_prefill_mma(const PrefillArgs* args, int tile_queries, cudaStream_t stream) {
@@ -638,21 +650,32 @@ LLG_API int llg_attn_mix_prefill_mma(const PrefillArgs* args, int tile_queries, 
 #undef GO
 }
 
-LLG_API int llg_attn_mix_decode_mma(const DecodeArgs* args, void* out, cudaStream_t stream) {
+// scores [n_seqs][keys][nh] float32, weights [n_seqs][nh][keys] bfloat16 and chunks [n_seqs][nh][keys / 64][2] float32 are scratch;
+// keys: a multiple of 64, no less than any sequence's keys (the new one included).
+LLG_API int llg_attn_mix_decode_mma(const DecodeArgs* args, void* out, float* scores, void* weights, float* chunks, int keys,
+                                    cudaStream_t stream) {
   const DecodeArgs& a = *args;
   const int vd = a.vd > 0 ? a.vd : a.hd;
-  LLG_REQUIRE(llg_attn_mix_decode_mma_supported(a.nh, a.nkv, a.hd, vd), "attn_mix_decode_mma: %d heads (%d) of %d and %d elements", a.nh,
-              a.nkv, a.hd, vd);
+  LLG_REQUIRE(head_sizes_ok(a.nh, a.nkv, a.hd, vd), "attn_mix_decode_mma: %d heads (%d) of %d and %d elements", a.nh, a.nkv, a.hd, vd);
   LLG_REQUIRE(a.scale > 0.f && a.softcap >= 0.f, "attn_mix_decode_mma: scale %g, cap %g", a.scale, a.softcap);
   LLG_REQUIRE(a.n_splits >= 1 && a.n_splits <= 65535 && a.n_seqs <= 65535, "attn_mix_decode_mma: grid too large");
   LLG_REQUIRE(a.window >= 0 && a.ring_pages > 0 && a.table_width >= a.ring_pages, "attn_mix_decode_mma: bad cache geometry");
+  LLG_REQUIRE(keys > 0 && keys % CHUNK == 0 && scores && weights && chunks, "attn_mix_decode_mma: scratch for %d keys", keys);
   if (a.n_seqs <= 0) return 0;
-  int stages = 2;
-  while (stages < MAX_STAGES && decode_smem(a.nh, a.nkv, a.hd, vd, stages + 1) <= SMEM_MAX) ++stages;
-  const size_t smem = decode_smem(a.nh, a.nkv, a.hd, vd, stages);
-  cudaError_t e = cudaFuncSetAttribute(attn_mix_decode_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  if (e != cudaSuccess) return llg_fail("attn_mix_decode_mma: shared memory %zu: %s", smem, cudaGetErrorString(e));
-  llg_launch(attn_mix_decode_mma_kernel, dim3(a.n_splits, a.n_seqs), dim3(MT), smem, stream, a, stages);
+  const MixScratch w{scores, (bf16*)weights, chunks, keys};
+  const int rc = (a.nh / a.nkv + 15) / 16;
+  const dim3 sgrid((keys + SCORE_KEYS - 1) / SCORE_KEYS, a.nkv, a.n_seqs);
+  if (a.hd <= 64) llg_launch(mix_scores_kernel<2>, sgrid, dim3(128), 0, stream, a, w);
+  else llg_launch(mix_scores_kernel<4>, sgrid, dim3(128), 0, stream, a, w);
+  const size_t smem = (size_t)(((a.nh + 3) & ~3) + CHUNK) * heads_stride(a.nh) * sizeof(float);
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(mix_weights_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return llg_fail("attn_mix_decode_mma: shared memory %zu: %s", smem, cudaGetErrorString(e));
+  }
+  llg_launch(mix_weights_kernel, dim3(keys / CHUNK, a.n_seqs), dim3(256), smem, stream, a, w);
+  const dim3 vgrid(a.n_splits, a.nkv * rc, a.n_seqs);
+  if (vd <= 64) llg_launch(mix_values_kernel<1>, vgrid, dim3(128), 0, stream, a, w);
+  else llg_launch(mix_values_kernel<2>, vgrid, dim3(128), 0, stream, a, w);
   attn_decode_reduce_kernel<bf16><<<dim3(a.nh, a.n_seqs), 64, 0, stream>>>(a.part_o, a.part_ml, (bf16*)out, a.nh, vd, a.n_splits, a.has_sink,
                                                                         a.sink_score, a.gate, a.sinks);
   return llg_check_launch("attn_mix_decode_mma");

@@ -438,7 +438,7 @@ def _load_lib(name: str):
         lib.llg_attn_mix_prefill_mma_supported.argtypes = [c_int, c_int, c_int, c_int]
         lib.llg_attn_mix_decode_mma_supported.argtypes = [c_int, c_int, c_int, c_int]
         lib.llg_attn_mix_prefill_mma.argtypes = [POINTER(_PrefillArgs), c_int, c_void_p]
-        lib.llg_attn_mix_decode_mma.argtypes = [POINTER(_DecodeArgs), c_void_p, c_void_p]
+        lib.llg_attn_mix_decode_mma.argtypes = [POINTER(_DecodeArgs), c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
     elif name == "matrix_memory":
         lib.llg_matrix_memory_fits.argtypes = [c_int, c_int]
         lib.llg_matrix_memory.argtypes = [POINTER(_MatrixMemoryArgs), c_int, c_void_p]
@@ -1870,6 +1870,13 @@ def attn_decode_plan(dtype: torch.dtype, n_seqs: int, n_heads: int, n_kv_heads: 
     sequence by its length for small batches).  Everything else, and values of another head size than the keys: the
     CUDA-core kernel."""
     if form.mixes:
+        vd = form.vd(head_dim)
+        if _use_mix_mma("decode", dtype, n_heads, n_kv_heads, head_dim, vd):
+            # behind the splits' partial results: scores, weights and every chunk's maximum and sum (csrc/attention_mix_mma.cu)
+            keys = -(-max(max_len, 1) // PAGE) * PAGE
+            splits = _splits_for(n_seqs, n_kv_heads * -(-n_heads // n_kv_heads // 16), max_len, sm_count(), 4)
+            floats = attn_decode_scratch_floats(n_seqs, n_heads, vd, splits) + sum(_mix_scratch(n_seqs, n_heads, keys)) + 12
+            return DecodePlan("mix_mma", splits, False, max_len, floats, 0)
         # one block works on all heads of a sequence's share of the keys
         splits = _splits_for(n_seqs, 1, max_len, sm_count(), 1)
         return DecodePlan("mix", splits, False, max_len, attn_decode_scratch_floats(n_seqs, n_heads, form.vd(head_dim), splits), 0)
@@ -1889,6 +1896,11 @@ def attn_decode_plan(dtype: torch.dtype, n_seqs: int, n_heads: int, n_kv_heads: 
         splits = max(splits, min(64, tiles, 2 * n_sms // n_kv_heads - (n_seqs - 1)))
     return DecodePlan("mma" if mma else "simt", splits, balance, max_len,
                       attn_decode_scratch_floats(n_seqs, n_heads, form.vd(head_dim), splits), n_seqs * n_kv_heads if mma else 0)
+
+
+def _mix_scratch(n_seqs: int, n_heads: int, keys: int):
+    """Floats of the (scores, weights, chunks) that decode attention with mixed scores keeps on the way."""
+    return n_seqs * keys * n_heads, -(-n_seqs * n_heads * keys // 2), n_seqs * n_heads * (keys // PAGE) * 2
 
 
 def attn_decode_scratch_floats(n_seqs: int, n_heads: int, head_dim: int, n_splits: int) -> int:
@@ -1936,7 +1948,7 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         raise KernelError("attn_decode: the scratch must be float32")
     if form.gated != (gate is not None) or (gate is not None and tuple(gate.shape) != (b, nh)):
         raise KernelError("attn_decode: a gated form needs a gate [sequences, heads], and only a gated form takes one")
-    if not form.one_head_size(hd) and plan is not None and plan.kind not in ("simt", "mix"):
+    if not form.one_head_size(hd) and plan is not None and plan.kind not in ("simt", "mix", "mix_mma"):
         raise KernelError(f"attn_decode: the {plan.kind} kernel takes keys and values of one head size")
     assert out.shape == (b, nh * vd) and v_pages.shape[3] == vd
     if plan is not None and plan.kind == "tma":
@@ -1960,7 +1972,7 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
     if plan is not None:
         n_splits, balance = plan.n_splits, plan.balance
     mma = form.one_head_size(hd) and _use_mma(q.dtype, hd) and not form.mixes
-    mix_mma = form.mixes and _use_mix_mma("decode", q.dtype, nh, nkv, hd, vd)
+    mix_mma = form.mixes and plan is not None and plan.kind == "mix_mma"
     lib = _lib("attention_mix_mma" if mix_mma else "attention_mix" if form.mixes else "attention_mma" if mma else "attention_simt")
     need = b * nh * n_splits * (vd + 2)
     if n_splits < 1 or scratch.numel() < need:
@@ -1981,7 +1993,15 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         _check(lib, lib.llg_attn_decode_mma(byref(a), _ptr(out, q.dtype), _ptr(counters, torch.int32),
                                             int(bool(balance) and b * nkv <= attn_decode_balance_pairs() and b <= 32), _stream()))
     elif mix_mma:
-        _check(lib, lib.llg_attn_mix_decode_mma(byref(a), _ptr(out, q.dtype), _stream()), kernels=2)
+        if scratch.numel() < plan.scratch_floats:
+            raise KernelError(f"attn_decode: scratch of {scratch.numel()} floats, {plan.scratch_floats} needed")
+        keys = -(-max(plan.max_len, 1) // PAGE) * PAGE
+        n_scores, n_weights, _ = _mix_scratch(b, nh, keys)
+        at = -(-need // 4) * 4                               # every part starts on 16 bytes
+        at_w = at + -(-n_scores // 4) * 4
+        at_c = at_w + -(-n_weights // 4) * 4
+        _check(lib, lib.llg_attn_mix_decode_mma(byref(a), _ptr(out, q.dtype), base + 4 * at, base + 4 * at_w, base + 4 * at_c, keys, _stream()),
+               kernels=4)
     elif form.mixes:
         _check(lib, lib.llg_attn_mix_decode_simt(byref(a), _ptr(out, q.dtype), _dt(q), _stream()), kernels=2)
     else:
