@@ -345,7 +345,6 @@ __global__ void __launch_bounds__(MT, 1) attn_mix_prefill_mma_kernel(PrefillArgs
 // 64 c + 8 g .. + 7 of keys 2t, 2t + 1, 2t + 8, 2t + 9, and product j of eight uses element j of each.
 
 constexpr int CHUNK = LLG_PAGE;         // keys per chunk of the softmax (one page)
-constexpr int SCORE_KEYS = 128;         // keys per block of the scores' kernel (4 warps)
 
 struct MixScratch {
   float* scores;                        // [n_seqs][keys][nh]
@@ -361,36 +360,38 @@ __device__ __forceinline__ int page_at(const DecodeArgs& a, int slot, int pos) {
 
 // HD32: the head's elements in steps of 32, at most (a remainder of 16 is one product more)
 template <int HD32>
-__global__ void __launch_bounds__(128) mix_scores_kernel(DecodeArgs a, MixScratch w) {
+__global__ void __launch_bounds__(128, 4) mix_scores_kernel(DecodeArgs a, MixScratch w) {
   pdl_launch_dependents();
   const int nh = a.nh, nkv = a.nkv, hd = a.hd, G = nh / nkv;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int kv = blockIdx.y, b = blockIdx.z;
   pdl_wait();
   const int len = a.len_before[b] + 1, base = first_page_key(a, len);
-  const int k0 = base + blockIdx.x * SCORE_KEYS;
-  if (k0 >= len) return;
+  const int n_chunks = (len - base + CHUNK - 1) / CHUNK, per = (n_chunks + gridDim.x - 1) / gridDim.x;
+  const int c0 = blockIdx.x * per, c1 = min(n_chunks, c0 + per);
+  if (c0 >= c1) return;
   const int slot = a.slots[b], steps = hd / 32, tail = hd % 32;
   const float two_over_cap = a.softcap > 0.f ? 2.0f / a.softcap : 0.f;
   const bf16* q = (const bf16*)a.q + ((long long)b * nh + kv * G) * hd;
-#pragma unroll
-  for (int it = 0; it < SCORE_KEYS / 64; ++it) {
-    const int kt = k0 + it * 64 + warp * 16;
-    if (kt >= len) break;
-    const bf16* row = (const bf16*)a.k_pages + (((long long)page_at(a, slot, kt) * nkv + kv) * LLG_PAGE + kt % LLG_PAGE + g) * hd;
-    uint4 k_lo[HD32], k_hi[HD32];
-    uint2 t_lo = make_uint2(0, 0), t_hi = make_uint2(0, 0);
+  struct Keys {
+    uint4 lo[HD32], hi[HD32];
+    uint2 t_lo, t_hi;
+  };
+  auto fetch = [&](Keys& k, int page) {
+    const bf16* row = (const bf16*)a.k_pages + (((long long)page * nkv + kv) * LLG_PAGE + warp * 16 + g) * hd;
 #pragma unroll
     for (int c = 0; c < HD32; ++c)
       if (c < steps) {
-        k_lo[c] = *reinterpret_cast<const uint4*>(row + c * 32 + t * 8);
-        k_hi[c] = *reinterpret_cast<const uint4*>(row + 8 * hd + c * 32 + t * 8);
+        k.lo[c] = *reinterpret_cast<const uint4*>(row + c * 32 + t * 8);
+        k.hi[c] = *reinterpret_cast<const uint4*>(row + 8 * hd + c * 32 + t * 8);
       }
     if (tail) {
-      t_lo = *reinterpret_cast<const uint2*>(row + steps * 32 + t * 4);
-      t_hi = *reinterpret_cast<const uint2*>(row + 8 * hd + steps * 32 + t * 4);
+      k.t_lo = *reinterpret_cast<const uint2*>(row + steps * 32 + t * 4);
+      k.t_hi = *reinterpret_cast<const uint2*>(row + 8 * hd + steps * 32 + t * 4);
     }
-    float* dst = w.scores + ((long long)b * w.keys + kt - base + g) * nh + kv * G;
+  };
+  auto score = [&](const Keys& k, int chunk) {
+    float* dst = w.scores + ((long long)b * w.keys + chunk * CHUNK + warp * 16 + g) * nh + kv * G;
     for (int g0 = 0; g0 < G; g0 += 8) {
       const bf16* qr = q + (long long)min(g0 + g, G - 1) * hd;        // column g of the product: head g0 + g
       float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
@@ -398,13 +399,13 @@ __global__ void __launch_bounds__(128) mix_scores_kernel(DecodeArgs a, MixScratc
       for (int c = 0; c < HD32; ++c)
         if (c < steps) {
           const uint4 qf = *reinterpret_cast<const uint4*>(qr + c * 32 + t * 8);
-          const uint32_t a0[4] = {k_lo[c].x, k_hi[c].x, k_lo[c].y, k_hi[c].y}, a1[4] = {k_lo[c].z, k_hi[c].z, k_lo[c].w, k_hi[c].w};
+          const uint32_t a0[4] = {k.lo[c].x, k.hi[c].x, k.lo[c].y, k.hi[c].y}, a1[4] = {k.lo[c].z, k.hi[c].z, k.lo[c].w, k.hi[c].w};
           mma_16816(s0, a0, qf.x, qf.y);
           mma_16816(s1, a1, qf.z, qf.w);
         }
       if (tail) {
         const uint2 qf = *reinterpret_cast<const uint2*>(qr + steps * 32 + t * 4);
-        const uint32_t a0[4] = {t_lo.x, t_hi.x, t_lo.y, t_hi.y};
+        const uint32_t a0[4] = {k.t_lo.x, k.t_hi.x, k.t_lo.y, k.t_hi.y};
         mma_16816(s0, a0, qf.x, qf.y);
       }
 #pragma unroll
@@ -413,6 +414,20 @@ __global__ void __launch_bounds__(128) mix_scores_kernel(DecodeArgs a, MixScratc
         if (h < G) dst[(long long)(e >> 1) * 8 * nh + h] = capped((s0[e] + s1[e]) * a.scale, a.softcap, two_over_cap);
       }
     }
+  };
+  // the next keys are on their way while the products of these run
+  Keys ka, kb;
+  auto page_of = [&](int c) { return c < c1 ? page_at(a, slot, base + c * CHUNK) : 0; };
+  int next = page_of(c0 + 1);
+  fetch(ka, page_of(c0));
+  for (int c = c0; c < c1; c += 2) {
+    if (c + 1 < c1) fetch(kb, next);
+    next = page_of(c + 2);
+    score(ka, c);
+    if (c + 1 >= c1) break;
+    if (c + 2 < c1) fetch(ka, next);
+    next = page_of(c + 3);
+    score(kb, c + 1);
   }
 }
 
@@ -428,20 +443,34 @@ __global__ void __launch_bounds__(256) mix_weights_kernel(DecodeArgs a, MixScrat
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, b = blockIdx.y;
   float* T = msm;                                 // [nh4][hs]
   float* S = T + nh4 * hs;                        // [CHUNK][hs]
-  for (int idx = threadIdx.x; idx < nh4 * hs; idx += 256) {
-    const int h = idx / hs, gg = idx - h * hs;
-    T[idx] = h >= nh || gg >= nh ? 0.f : a.head_mix ? a.head_mix[h * nh + gg] : (h == gg ? 1.f : 0.f);
+  const bool vec = nh % 4 == 0;
+  if (vec && a.head_mix) {
+    const int q4 = nh / 4, step = 256 / q4, c = threadIdx.x % q4;
+    for (int h = threadIdx.x / q4; h < nh && threadIdx.x < step * q4; h += step)
+      *reinterpret_cast<float4*>(T + h * hs + c * 4) = *reinterpret_cast<const float4*>(a.head_mix + h * nh + c * 4);
+  } else {
+    for (int idx = threadIdx.x; idx < nh4 * hs; idx += 256) {
+      const int h = idx / hs, gg = idx - h * hs;
+      T[idx] = h >= nh || gg >= nh ? 0.f : a.head_mix ? a.head_mix[h * nh + gg] : (h == gg ? 1.f : 0.f);
+    }
   }
   pdl_wait();
   const int len = a.len_before[b] + 1, lo = mask_first(len - 1, a.window, a.chunked), base = lo / LLG_PAGE * LLG_PAGE;
   const int r0 = blockIdx.x * CHUNK;
   if (base + r0 >= len) return;
   const float* src = w.scores + ((long long)b * w.keys + r0) * nh;
-  for (int idx = threadIdx.x; idx < CHUNK * nh; idx += 256) {
-    const int k = idx / nh, h = idx - k * nh;
-    S[k * hs + h] = base + r0 + k < len ? src[idx] : 0.f;
+  if (vec) {
+    const int q4 = nh / 4, step = 256 / q4, c = threadIdx.x % q4;
+    for (int k = threadIdx.x / q4; k < CHUNK && threadIdx.x < step * q4; k += step)
+      *reinterpret_cast<float4*>(S + k * hs + c * 4) =
+          base + r0 + k < len ? *reinterpret_cast<const float4*>(src + k * nh + c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+  } else {
+    for (int idx = threadIdx.x; idx < CHUNK * nh; idx += 256) {
+      const int k = idx / nh, h = idx - k * nh;
+      S[k * hs + h] = base + r0 + k < len ? src[idx] : 0.f;
+    }
+    for (int idx = threadIdx.x; idx < CHUNK * (hs - nh); idx += 256) S[idx / (hs - nh) * hs + nh + idx % (hs - nh)] = 0.f;
   }
-  for (int idx = threadIdx.x; idx < CHUNK * (hs - nh); idx += 256) S[idx / (hs - nh) * hs + nh + idx % (hs - nh)] = 0.f;
   __syncthreads();
   for (int h0 = warp * 4; h0 < nh; h0 += 32) {
     float acc[4][2] = {};
@@ -478,15 +507,14 @@ __global__ void __launch_bounds__(256) mix_weights_kernel(DecodeArgs a, MixScrat
   }
 }
 
-// The weighted values: block (split, key/value head and up to 16 of its query heads, sequence); the four warps take a chunk's
-// four runs of 16 keys.  All partial results are relative to the sequence's largest maximum.
-template <int VD64>
-__global__ void __launch_bounds__(128) mix_values_kernel(DecodeArgs a, MixScratch w) {
+// The weighted values: block (split, key/value head, up to 16 of its query heads and 64 of its elements, sequence); the four
+// warps take a chunk's four runs of 16 keys, and the next chunk's values are on their way while a chunk's products run.  All partial results are relative to the sequence's largest maximum.
+__global__ void __launch_bounds__(128, 4) mix_values_kernel(DecodeArgs a, MixScratch w) {
   pdl_launch_dependents();
-  __shared__ float top_of[16], merge[4][16][VD64 * 64 + 4];
-  const int nh = a.nh, nkv = a.nkv, vd = a.vd > 0 ? a.vd : a.hd, G = nh / nkv, RC = (G + 15) / 16;
+  __shared__ float top_of[16], merge[4][16][64 + 4];
+  const int nh = a.nh, nkv = a.nkv, vd = a.vd > 0 ? a.vd : a.hd, G = nh / nkv, RC = (G + 15) / 16, NX = (vd + 63) / 64;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-  const int split = blockIdx.x, kv = blockIdx.y / RC, h0 = kv * G + blockIdx.y % RC * 16, b = blockIdx.z;
+  const int split = blockIdx.x, x = blockIdx.y % NX, u = blockIdx.y / NX, kv = u / RC, h0 = kv * G + u % RC * 16, b = blockIdx.z;
   const int gn = min(16, kv * G + G - h0);        // heads of this block
   pdl_wait();
   const int len = a.len_before[b] + 1, base = first_page_key(a, len), slot = a.slots[b];
@@ -501,8 +529,8 @@ __global__ void __launch_bounds__(128) mix_values_kernel(DecodeArgs a, MixScratc
     m = warp_max(m);
     for (int c = c0 + lane; c < c1; c += 32) l += pow2_whole(ch[((long long)h * all + c) * 2] - m) * ch[((long long)h * all + c) * 2 + 1];
     l = warp_sum(l);
-    if (lane == 0) {
-      top_of[h] = m;
+    if (lane == 0) top_of[h] = m;
+    if (lane == 0 && x == 0) {
       float* ml = a.part_ml + (((long long)b * nh + h0 + h) * a.n_splits + split) * 2;
       ml[0] = c0 < c1 ? m * 0.6931471805599453f : -INFINITY;          // natural units
       ml[1] = l;
@@ -512,55 +540,72 @@ __global__ void __launch_bounds__(128) mix_values_kernel(DecodeArgs a, MixScratc
   const float m0 = top_of[min(g, gn - 1)], m1 = top_of[min(g + 8, gn - 1)];
   const bf16* p0 = w.weights + ((long long)b * nh + h0 + min(g, gn - 1)) * w.keys + warp * 16 + 2 * t;
   const bf16* p1 = w.weights + ((long long)b * nh + h0 + min(g + 8, gn - 1)) * w.keys + warp * 16 + 2 * t;
-  float o[VD64][8][4];
+  float o[8][4];
 #pragma unroll
-  for (int c = 0; c < VD64; ++c)
+  for (int j = 0; j < 8; ++j)
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) o[c][j][e] = 0.f;
+    for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
   auto scaled = [](uint32_t p, float f) {         // two weights times a power of two
     const __nv_bfloat162 v = __hmul2(*reinterpret_cast<const __nv_bfloat162*>(&p), __float2bfloat162_rn(f));
     return *reinterpret_cast<const uint32_t*>(&v);
   };
-  int page = c0 < c1 ? page_at(a, slot, base + c0 * CHUNK) : 0;
-  for (int c = c0; c < c1; ++c) {
-    const bf16* rows = (const bf16*)a.v_pages + (((long long)page * nkv + kv) * LLG_PAGE + warp * 16) * vd;
-    uint4 v[VD64][4];
+  const int d = x * 64 + g * 8;
+  const bool there = d < vd;
+  struct Rows {
+    uint4 r[4];
+    uint32_t p[4];
+    float f0, f1;
+  };
+  auto fetch = [&](Rows& v, int c, int page) {
+    const bf16* rows = (const bf16*)a.v_pages + (((long long)page * nkv + kv) * LLG_PAGE + warp * 16 + 2 * t) * vd + d;
 #pragma unroll
-    for (int x = 0; x < VD64; ++x) {
-      const int d = x * 64 + g * 8;
+    for (int r = 0; r < 4; ++r)
+      v.r[r] = there ? *reinterpret_cast<const uint4*>(rows + (long long)((r & 1) + (r >> 1) * 8) * vd) : make_uint4(0, 0, 0, 0);
+    v.p[0] = *reinterpret_cast<const uint32_t*>(p0 + c * CHUNK);
+    v.p[1] = *reinterpret_cast<const uint32_t*>(p1 + c * CHUNK);
+    v.p[2] = *reinterpret_cast<const uint32_t*>(p0 + c * CHUNK + 8);
+    v.p[3] = *reinterpret_cast<const uint32_t*>(p1 + c * CHUNK + 8);
+    v.f0 = ch[((long long)min(g, gn - 1) * all + c) * 2];
+    v.f1 = ch[((long long)min(g + 8, gn - 1) * all + c) * 2];
+  };
+  auto add = [&](const Rows& v) {
+    const float f0 = pow2_whole(v.f0 - m0), f1 = pow2_whole(v.f1 - m1);
+    const uint32_t pa[4] = {scaled(v.p[0], f0), scaled(v.p[1], f1), scaled(v.p[2], f0), scaled(v.p[3], f1)};
+    const uint32_t w0[4] = {v.r[0].x, v.r[0].y, v.r[0].z, v.r[0].w}, w1[4] = {v.r[1].x, v.r[1].y, v.r[1].z, v.r[1].w};
+    const uint32_t w2[4] = {v.r[2].x, v.r[2].y, v.r[2].z, v.r[2].w}, w3[4] = {v.r[3].x, v.r[3].y, v.r[3].z, v.r[3].w};
 #pragma unroll
-      for (int r = 0; r < 4; ++r)
-        v[x][r] = d < vd ? *reinterpret_cast<const uint4*>(rows + (long long)(2 * t + (r & 1) + (r >> 1) * 8) * vd + d) : make_uint4(0, 0, 0, 0);
+    for (int j = 0; j < 8; ++j) {                 // element j of the four rows: the low or the high half of word j / 2
+      const uint32_t sel = j & 1 ? 0x7632u : 0x5410u;
+      mma_16816(o[j], pa, __byte_perm(w0[j / 2], w1[j / 2], sel), __byte_perm(w2[j / 2], w3[j / 2], sel));
     }
-    if (c + 1 < c1) page = page_at(a, slot, base + (c + 1) * CHUNK);
-    const float f0 = pow2_whole(ch[((long long)min(g, gn - 1) * all + c) * 2] - m0);
-    const float f1 = pow2_whole(ch[((long long)min(g + 8, gn - 1) * all + c) * 2] - m1);
-    const uint32_t pa[4] = {scaled(*reinterpret_cast<const uint32_t*>(p0 + c * CHUNK), f0), scaled(*reinterpret_cast<const uint32_t*>(p1 + c * CHUNK), f1),
-                            scaled(*reinterpret_cast<const uint32_t*>(p0 + c * CHUNK + 8), f0), scaled(*reinterpret_cast<const uint32_t*>(p1 + c * CHUNK + 8), f1)};
-#pragma unroll
-    for (int x = 0; x < VD64; ++x) {
-      const uint32_t r0[4] = {v[x][0].x, v[x][0].y, v[x][0].z, v[x][0].w}, r1[4] = {v[x][1].x, v[x][1].y, v[x][1].z, v[x][1].w};
-      const uint32_t r2[4] = {v[x][2].x, v[x][2].y, v[x][2].z, v[x][2].w}, r3[4] = {v[x][3].x, v[x][3].y, v[x][3].z, v[x][3].w};
-#pragma unroll
-      for (int j = 0; j < 8; ++j) {               // element j of the four rows: the low or the high half of word j / 2
-        const uint32_t sel = j & 1 ? 0x7632u : 0x5410u;
-        mma_16816(o[x][j], pa, __byte_perm(r0[j / 2], r1[j / 2], sel), __byte_perm(r2[j / 2], r3[j / 2], sel));
-      }
+  };
+  if (c0 < c1) {
+    Rows va, vb;
+    auto page_of = [&](int c) { return c < c1 ? page_at(a, slot, base + c * CHUNK) : 0; };
+    int next = page_of(c0 + 1);
+    fetch(va, c0, page_of(c0));
+    for (int c = c0; c < c1; c += 2) {
+      if (c + 1 < c1) fetch(vb, c + 1, next);
+      next = page_of(c + 2);
+      add(va);
+      if (c + 1 >= c1) break;
+      if (c + 2 < c1) fetch(va, c + 2, next);
+      next = page_of(c + 3);
+      add(vb);
     }
   }
   // column n of product j is element 64 x + 8 n + j; add the four warps up
 #pragma unroll
-  for (int x = 0; x < VD64; ++x)
+  for (int j = 0; j < 8; ++j)
 #pragma unroll
-    for (int j = 0; j < 8; ++j)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) merge[warp][g + (e >> 1) * 8][x * 64 + 8 * (2 * t + (e & 1)) + j] = o[x][j][e];
+    for (int e = 0; e < 4; ++e) merge[warp][g + (e >> 1) * 8][8 * (2 * t + (e & 1)) + j] = o[j][e];
   __syncthreads();
-  for (int idx = threadIdx.x; idx < gn * vd; idx += 128) {
-    const int h = idx / vd, d = idx - h * vd;
-    a.part_o[(((long long)b * nh + h0 + h) * a.n_splits + split) * vd + d] = (merge[0][h][d] + merge[1][h][d]) + (merge[2][h][d] + merge[3][h][d]);
+  const int dn = min(64, vd - x * 64);
+  for (int idx = threadIdx.x; idx < gn * 64; idx += 128) {
+    const int h = idx / 64, e = idx % 64;
+    if (e < dn)
+      a.part_o[(((long long)b * nh + h0 + h) * a.n_splits + split) * vd + x * 64 + e] =
+          (merge[0][h][e] + merge[1][h][e]) + (merge[2][h][e] + merge[3][h][e]);
   }
 }
 
@@ -664,7 +709,10 @@ LLG_API int llg_attn_mix_decode_mma(const DecodeArgs* args, void* out, float* sc
   if (a.n_seqs <= 0) return 0;
   const MixScratch w{scores, (bf16*)weights, chunks, keys};
   const int rc = (a.nh / a.nkv + 15) / 16;
-  const dim3 sgrid((keys + SCORE_KEYS - 1) / SCORE_KEYS, a.nkv, a.n_seqs);
+  // as many blocks as the GPU holds at once (four per multiprocessor), each with an equal share of its sequence's keys
+  int shares = 4 * llg_sm_count() / (a.nkv * a.n_seqs);
+  shares = shares < 1 ? 1 : shares > keys / CHUNK ? keys / CHUNK : shares;
+  const dim3 sgrid(shares, a.nkv, a.n_seqs);
   if (a.hd <= 64) llg_launch(mix_scores_kernel<2>, sgrid, dim3(128), 0, stream, a, w);
   else llg_launch(mix_scores_kernel<4>, sgrid, dim3(128), 0, stream, a, w);
   const size_t smem = (size_t)(((a.nh + 3) & ~3) + CHUNK) * heads_stride(a.nh) * sizeof(float);
@@ -673,9 +721,7 @@ LLG_API int llg_attn_mix_decode_mma(const DecodeArgs* args, void* out, float* sc
     if (e != cudaSuccess) return llg_fail("attn_mix_decode_mma: shared memory %zu: %s", smem, cudaGetErrorString(e));
   }
   llg_launch(mix_weights_kernel, dim3(keys / CHUNK, a.n_seqs), dim3(256), smem, stream, a, w);
-  const dim3 vgrid(a.n_splits, a.nkv * rc, a.n_seqs);
-  if (vd <= 64) llg_launch(mix_values_kernel<1>, vgrid, dim3(128), 0, stream, a, w);
-  else llg_launch(mix_values_kernel<2>, vgrid, dim3(128), 0, stream, a, w);
+  llg_launch(mix_values_kernel, dim3(a.n_splits, a.nkv * rc * ((vd + 63) / 64), a.n_seqs), dim3(128), 0, stream, a, w);
   attn_decode_reduce_kernel<bf16><<<dim3(a.nh, a.n_seqs), 64, 0, stream>>>(a.part_o, a.part_ml, (bf16*)out, a.nh, vd, a.n_splits, a.has_sink,
                                                                         a.sink_score, a.gate, a.sinks);
   return llg_check_launch("attn_mix_decode_mma");

@@ -1874,7 +1874,7 @@ def attn_decode_plan(dtype: torch.dtype, n_seqs: int, n_heads: int, n_kv_heads: 
         if _use_mix_mma("decode", dtype, n_heads, n_kv_heads, head_dim, vd):
             # behind the splits' partial results: scores, weights and every chunk's maximum and sum (csrc/attention_mix_mma.cu)
             keys = -(-max(max_len, 1) // PAGE) * PAGE
-            splits = _splits_for(n_seqs, n_kv_heads * -(-n_heads // n_kv_heads // 16), max_len, sm_count(), 4)
+            splits = _splits_for(n_seqs, n_kv_heads * -(-n_heads // n_kv_heads // 16) * -(-vd // 64), max_len, sm_count(), 4)
             floats = attn_decode_scratch_floats(n_seqs, n_heads, vd, splits) + sum(_mix_scratch(n_seqs, n_heads, keys)) + 12
             return DecodePlan("mix_mma", splits, False, max_len, floats, 0)
         # one block works on all heads of a sequence's share of the keys
