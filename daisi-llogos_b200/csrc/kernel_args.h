@@ -554,9 +554,8 @@ struct RetentionArgs {
 // state_s [slots][nh][dim][vdim], state_n [slots][nh][dim] and state_m [slots][nh] hold S, n and m before the step's first
 // token and receive them after its last.  A block owns `cols` columns of a head's S.  A head cut into several runs of
 // columns leaves its o in raw, and n and m in next, and a second kernel finishes (norm, gate, n and m into the state).
-// With carry, pieces of LLG_MEMORY_PIECE tokens run side by side from zero, are joined, and run again; a piece's entry in
+// With carry, pieces of `piece` tokens run side by side from zero, are joined, and run again; a piece's entry in
 // carry is S [dim][vdim], n [dim] and three numbers: the sum of its f, its own maximum, the maximum it starts from.
-#define LLG_MEMORY_PIECE 128
 #define LLG_MEMORY_CARRY_EXTRA 3
 struct MatrixMemoryArgs {
   const float* rows;          // [n_partials][n_tokens][row_width]
@@ -575,7 +574,7 @@ struct MatrixMemoryArgs {
   void* out;                  // [n_tokens][nh * vdim]
   int out_dtype;
   float* carry;               // [n_seqs][pieces][nh][dim * vdim + dim + LLG_MEMORY_CARRY_EXTRA] or null
-  int pieces;
+  int pieces, piece;
   float* raw;                 // [n_tokens][nh * vdim], where cols < vdim
   float* next;                // [n_seqs][nh][dim + 1], where cols < vdim and there is no carry
   int n_seqs, n_tokens, nh, dim, vdim, cols;

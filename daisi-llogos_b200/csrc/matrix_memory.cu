@@ -20,7 +20,6 @@ LLG_API const char* llg_last_error() { return g_llg_error; }
 
 namespace {
 
-constexpr int MEM_THREADS = 256;
 constexpr int MEM_BATCH = 16;
 constexpr int JOIN_BATCH = 8;
 
@@ -38,23 +37,23 @@ __device__ __forceinline__ void piece_range(const MatrixMemoryArgs& a, int b, in
   lo = t_begin;
   hi = t_end;
   if (pieces) {
-    lo = t_begin + piece * LLG_MEMORY_PIECE;
+    lo = t_begin + piece * a.piece;
     if (lo > t_end) lo = t_end;
-    hi = (piece == a.pieces - 1 || lo + LLG_MEMORY_PIECE > t_end) ? t_end : lo + LLG_MEMORY_PIECE;
+    hi = (piece == a.pieces - 1 || lo + a.piece > t_end) ? t_end : lo + a.piece;
   }
 }
 
 // MODE 0: a sequence from its state to its state; 1: a piece from zero, only its state is wanted; 2: a piece from the
 // state the join left.
-template <typename OT, int MODE, int R>
-__global__ void __launch_bounds__(MEM_THREADS, 2) matrix_memory_kernel(MatrixMemoryArgs a, int runs) {
+template <typename OT, int MODE, int R, int TH>
+__global__ void __launch_bounds__(TH, 512 / TH) matrix_memory_kernel(MatrixMemoryArgs a, int runs) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float smem[];
   __shared__ float s_i[MEM_BATCH], s_f[MEM_BATCH];
   const int h = blockIdx.x, piece = blockIdx.y / runs, run = blockIdx.y % runs, b = blockIdx.z;
   const int dim = a.dim, vdim = a.vdim, cols = a.cols;
-  const int slices = MEM_THREADS / cols;
+  const int slices = TH / cols;
   const int dp = slices * R;                  // padded length of a q, k or n row
   const int sl = threadIdx.x / cols, j = threadIdx.x - sl * cols;
   const int c0 = run * cols;                  // first column of this block
@@ -83,7 +82,7 @@ __global__ void __launch_bounds__(MEM_THREADS, 2) matrix_memory_kernel(MatrixMem
     const int i = sl * R + r;
     S[r] = (MODE != 1 && active && i < dim) ? src_s[(long long)i * vdim + c0 + j] : 0.f;
   }
-  for (int i = threadIdx.x; i < dp; i += MEM_THREADS) sn[i] = (MODE != 1 && i < dim) ? src_n[i] : 0.f;
+  for (int i = threadIdx.x; i < dp; i += TH) sn[i] = (MODE != 1 && i < dim) ? src_n[i] : 0.f;
   float m = MODE == 1 ? -INFINITY : MODE == 0 ? *gm : cr[(long long)dim * vdim + dim + 2];
   float f_total = 0.f;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -97,12 +96,12 @@ __global__ void __launch_bounds__(MEM_THREADS, 2) matrix_memory_kernel(MatrixMem
       for (int s = 1; s < a.n_partials; ++s) v += p[s * a.partial_stride];
       return v;
     };
-    for (int idx = threadIdx.x; idx < nb * dp; idx += MEM_THREADS) {
+    for (int idx = threadIdx.x; idx < nb * dp; idx += TH) {
       const int t = idx / dp, i = idx - t * dp;
       sk[idx] = i < dim ? summed(t, a.k_col + h * dim + i) : 0.f;
       if (MODE != 1) sq[idx] = i < dim ? summed(t, a.q_col + h * dim + i) * a.q_scale : 0.f;
     }
-    for (int idx = threadIdx.x; idx < nb * cols; idx += MEM_THREADS) {
+    for (int idx = threadIdx.x; idx < nb * cols; idx += TH) {
       const int t = idx / cols, c = idx - t * cols;
       sv[idx] = c < nc ? summed(t, a.v_col + h * vdim + c0 + c) : 0.f;
     }
@@ -158,7 +157,7 @@ __global__ void __launch_bounds__(MEM_THREADS, 2) matrix_memory_kernel(MatrixMem
         }
         if (MODE != 1) po[(t * slices + sl) * cols + j] = o;
       }
-      for (int i = threadIdx.x; i < dp; i += MEM_THREADS) {       // a row of n has one owner
+      for (int i = threadIdx.x; i < dp; i += TH) {       // a row of n has one owner
         const float v = fmaf(kp, sn[i], tk * sk[t * dp + i]);
         sn[i] = v;
         if (MODE != 1) pn[t * dp + i] = v * sq[t * dp + i];
@@ -167,7 +166,7 @@ __global__ void __launch_bounds__(MEM_THREADS, 2) matrix_memory_kernel(MatrixMem
     m = m_last;
     if (MODE != 1) {
       __syncthreads();
-      for (int t = warp; t < nb; t += MEM_THREADS / 32) {
+      for (int t = warp; t < nb; t += TH / 32) {
         float dot = 0.f;
         for (int i = lane; i < dp; i += 32) dot += pn[t * dp + i];
         dot = warp_sum(dot);
@@ -209,7 +208,7 @@ __global__ void __launch_bounds__(MEM_THREADS, 2) matrix_memory_kernel(MatrixMem
       const bool aside = MODE == 0 && !whole;
       float* nx = aside ? a.next + ((long long)b * a.nh + h) * (dim + 1) : nullptr;
       float* dn = MODE == 1 ? cr + (long long)dim * vdim : aside ? nx : gn;
-      for (int i = threadIdx.x; i < dim; i += MEM_THREADS) dn[i] = sn[i];
+      for (int i = threadIdx.x; i < dim; i += TH) dn[i] = sn[i];
       if (threadIdx.x == 0) {
         if (MODE == 1) {
           cr[(long long)dim * vdim + dim] = f_total;
@@ -295,13 +294,28 @@ __global__ void __launch_bounds__(128) matrix_memory_finish_kernel(MatrixMemoryA
   }
 }
 
-size_t memory_smem(int dim, int cols, int* r_out) {
-  const int slices = MEM_THREADS / cols;
+// Rows of a column per thread (4, 8, 16 or 32; 0: more than that) and shared memory of a block of `threads` threads.
+size_t memory_smem(int dim, int cols, int threads, int* r_out) {
+  const int slices = threads / cols;
+  if (slices == 0) {
+    *r_out = 0;
+    return 0;
+  }
   const int rows = (dim + slices - 1) / slices;
-  const int r = rows <= 4 ? 4 : rows <= 8 ? 8 : rows <= 16 ? 16 : 32;
-  if (r_out) *r_out = rows <= 32 ? r : 0;
+  const int r = threads == 512 ? 32 : rows <= 4 ? 4 : rows <= 8 ? 8 : rows <= 16 ? 16 : 32;      // (512 threads have one form)
+  *r_out = rows <= 32 ? r : 0;
   const size_t dp = (size_t)slices * r;
   return (3 * MEM_BATCH * dp + dp + (size_t)MEM_BATCH * cols + (size_t)MEM_BATCH * slices * cols) * sizeof(float);
+}
+
+// The threads of a block that can own `cols` columns of `dim` rows: 256, else 512, else 0.
+int memory_threads(int dim, int cols) {
+  for (int th = 256; th <= 512; th *= 2) {
+    int r = 0;
+    const size_t smem = memory_smem(dim, cols, th, &r);
+    if (r > 0 && smem <= 220 * 1024) return th;
+  }
+  return 0;
 }
 
 template <typename K>
@@ -313,18 +327,18 @@ int memory_attr(K kernel, size_t smem) {
   return 0;
 }
 
-template <typename OT, int R>
+template <typename OT, int R, int TH>
 int memory_run(const MatrixMemoryArgs& a, size_t smem, cudaStream_t stream) {
   const int runs = (a.vdim + a.cols - 1) / a.cols;
   if (!a.carry) {
-    if (memory_attr(matrix_memory_kernel<OT, 0, R>, smem)) return 1;
-    llg_launch(matrix_memory_kernel<OT, 0, R>, dim3(a.nh, runs, a.n_seqs), dim3(MEM_THREADS), smem, stream, a, runs);
+    if (memory_attr(matrix_memory_kernel<OT, 0, R, TH>, smem)) return 1;
+    llg_launch(matrix_memory_kernel<OT, 0, R, TH>, dim3(a.nh, runs, a.n_seqs), dim3(TH), smem, stream, a, runs);
   } else {
-    if (memory_attr(matrix_memory_kernel<OT, 1, R>, smem) || memory_attr(matrix_memory_kernel<OT, 2, R>, smem)) return 1;
+    if (memory_attr(matrix_memory_kernel<OT, 1, R, TH>, smem) || memory_attr(matrix_memory_kernel<OT, 2, R, TH>, smem)) return 1;
     const dim3 grid(a.nh, (unsigned)(a.pieces * runs), a.n_seqs);
-    llg_launch(matrix_memory_kernel<OT, 1, R>, grid, dim3(MEM_THREADS), smem, stream, a, runs);
+    llg_launch(matrix_memory_kernel<OT, 1, R, TH>, grid, dim3(TH), smem, stream, a, runs);
     llg_launch(matrix_memory_join_kernel, dim3((a.dim * a.vdim + a.dim + 255) / 256, a.nh, a.n_seqs), dim3(256), 0, stream, a);
-    llg_launch(matrix_memory_kernel<OT, 2, R>, grid, dim3(MEM_THREADS), smem, stream, a, runs);
+    llg_launch(matrix_memory_kernel<OT, 2, R, TH>, grid, dim3(TH), smem, stream, a, runs);
   }
   if (runs > 1) {
     const long long head_blocks = ((long long)a.n_tokens * a.nh + 3) / 4;
@@ -338,23 +352,22 @@ int memory_run(const MatrixMemoryArgs& a, size_t smem, cudaStream_t stream) {
 template <typename OT>
 int memory_launch(const MatrixMemoryArgs& a, cudaStream_t stream) {
   int r = 0;
-  const size_t smem = memory_smem(a.dim, a.cols, &r);
-  if (r == 4) return memory_run<OT, 4>(a, smem, stream);
-  if (r == 8) return memory_run<OT, 8>(a, smem, stream);
-  if (r == 16) return memory_run<OT, 16>(a, smem, stream);
-  return memory_run<OT, 32>(a, smem, stream);
+  const int th = memory_threads(a.dim, a.cols);
+  const size_t smem = memory_smem(a.dim, a.cols, th, &r);
+  if (th == 256) {
+    if (r == 4) return memory_run<OT, 4, 256>(a, smem, stream);
+    if (r == 8) return memory_run<OT, 8, 256>(a, smem, stream);
+    if (r == 16) return memory_run<OT, 16, 256>(a, smem, stream);
+    return memory_run<OT, 32, 256>(a, smem, stream);
+  }
+  return memory_run<OT, 32, 512>(a, smem, stream);
 }
 
 }  // namespace
 
-LLG_API int llg_matrix_memory_piece() { return LLG_MEMORY_PIECE; }
-
 // 1 when a block can own `cols` columns of a head with a state of `dim` rows.
 LLG_API int llg_matrix_memory_fits(int dim, int cols) {
-  if (dim <= 0 || cols <= 0 || cols > MEM_THREADS) return 0;
-  int r = 0;
-  const size_t smem = memory_smem(dim, cols, &r);
-  return r > 0 && smem <= 220 * 1024;
+  return dim > 0 && cols > 0 && memory_threads(dim, cols) > 0;
 }
 
 LLG_API int llg_matrix_memory(const MatrixMemoryArgs* args, int max_count, cudaStream_t stream) {
@@ -372,8 +385,8 @@ LLG_API int llg_matrix_memory(const MatrixMemoryArgs* args, int max_count, cudaS
   const int runs = (a.vdim + a.cols - 1) / a.cols;
   LLG_REQUIRE(runs == 1 || (a.raw && (a.carry || a.next)), "matrix_memory: a head in several runs of columns needs raw and next");
   if (a.carry)
-    LLG_REQUIRE(a.pieces >= 1 && (long long)a.pieces * runs <= 65535 && (long long)a.pieces * LLG_MEMORY_PIECE >= max_count,
-                "matrix_memory: %d pieces of %d tokens do not hold a sequence of %d", a.pieces, LLG_MEMORY_PIECE, max_count);
+    LLG_REQUIRE(a.pieces >= 1 && a.piece >= 1 && (long long)a.pieces * runs <= 65535 && (long long)a.pieces * a.piece >= max_count,
+                "matrix_memory: %d pieces of %d tokens do not hold a sequence of %d", a.pieces, a.piece, max_count);
   if (a.n_seqs == 0 || a.n_tokens == 0) return 0;
   if (a.out_dtype == LLG_F32) return memory_launch<float>(a, stream);
   if (a.out_dtype == LLG_BF16) return memory_launch<__nv_bfloat16>(a, stream);

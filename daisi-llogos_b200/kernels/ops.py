@@ -347,7 +347,7 @@ class _MatrixMemoryArgs(Structure):
         ("f_col", c_int), ("i_bias", c_void_p), ("f_bias", c_void_p),
         ("gate_cap", c_float), ("q_scale", c_float), ("denom_eps", c_float), ("eps", c_float), ("norm_w", c_void_p),
         ("state_s", c_void_p), ("state_n", c_void_p), ("state_m", c_void_p), ("slots", c_void_p), ("cu_tokens", c_void_p),
-        ("out", c_void_p), ("out_dtype", c_int), ("carry", c_void_p), ("pieces", c_int), ("raw", c_void_p), ("next", c_void_p),
+        ("out", c_void_p), ("out_dtype", c_int), ("carry", c_void_p), ("pieces", c_int), ("piece", c_int), ("raw", c_void_p), ("next", c_void_p),
         ("n_seqs", c_int), ("n_tokens", c_int), ("nh", c_int), ("dim", c_int), ("vdim", c_int), ("cols", c_int),
     ]
 
@@ -442,9 +442,6 @@ def _load_lib(name: str):
     elif name == "matrix_memory":
         lib.llg_matrix_memory_fits.argtypes = [c_int, c_int]
         lib.llg_matrix_memory.argtypes = [POINTER(_MatrixMemoryArgs), c_int, c_void_p]
-        if lib.llg_matrix_memory_piece() != MEMORY_PIECE:
-            raise KernelError(f"the matrix memory kernel works on pieces of {lib.llg_matrix_memory_piece()} tokens, Python "
-                              f"expects {MEMORY_PIECE}")
     elif name == "attention_mma":
         lib.llg_attn_mma_supported.argtypes = [c_int]
         lib.llg_attn_prefill_mma.argtypes = [POINTER(_PrefillArgs), c_void_p]
@@ -1238,39 +1235,39 @@ def retention(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, g_col: 
     _check(lib, lib.llg_retention(byref(a), max_count, _stream()), kernels=3 if carry is not None else 1)
 
 
-MEMORY_PIECE = 128          # tokens per piece of ``matrix_memory``; checked against the library at first use
 MEMORY_CARRY_EXTRA = 3
 _MEMORY_COLS = (256, 128, 64, 32, 16, 8)
+_MEMORY_PIECES = (128, 64)          # tokens per piece of a prompt
+_memory_plan_cache = {}
 
 
-def matrix_memory_pieces(max_count: int) -> int:
-    """Pieces per sequence that ``matrix_memory`` wants a carry for when the longest sequence of a step brings ``max_count``
-    tokens (1: no carry)."""
-    return max(1, -(-int(max_count) // MEMORY_PIECE))
-
-
-_memory_cols_cache = {}
-
-
-def matrix_memory_cols(dim: int, vdim: int, groups: int) -> int:
-    """Columns of a head's state per block, for a step of ``groups`` (sequence or piece, head) pairs: all of them where a
-    block can hold them and there are pairs enough for every multiprocessor, else a run of a power of two."""
-    key = (dim, vdim, groups)
-    cols = _memory_cols_cache.get(key)
-    if cols is not None:
-        return cols
+def matrix_memory_plan(dim: int, vdim: int, n_heads: int, n_seqs: int, max_count: int):
+    """``(piece, pieces, cols)`` for a step whose longest sequence brings ``max_count`` tokens: tokens per piece and pieces
+    per sequence (one piece: no carry), and the columns of a head's state that a block owns.  All of them where a block can
+    hold them; else, and where a prompt has too few (piece, head) pairs for the multiprocessors, shorter pieces and then
+    runs of a power of two."""
+    key = (dim, vdim, n_heads, n_seqs, max_count)
+    plan = _memory_plan_cache.get(key)
+    if plan is not None:
+        return plan
     lib = _lib("matrix_memory")
     fits = [c for c in (vdim,) + tuple(c for c in _MEMORY_COLS if c < vdim) if lib.llg_matrix_memory_fits(dim, c)]
     if not fits:
         raise KernelError(f"matrix_memory: a state of {dim} x {vdim} elements a head does not fit any block")
-    want = 2 * sm_count()
-    cols = fits[0]
-    for c in fits:
-        cols = c
-        if groups * -(-vdim // c) >= want:
-            break
-    _memory_cols_cache[key] = cols
-    return cols
+    plan = (max_count, 1, fits[0])
+    if max_count > _MEMORY_PIECES[-1]:
+        for piece in _MEMORY_PIECES:
+            pieces = -(-max_count // piece)
+            plan = (piece, pieces, fits[0])
+            if n_seqs * pieces * n_heads * -(-vdim // fits[0]) >= sm_count():
+                break
+        groups = n_seqs * plan[1] * n_heads
+        cols = next((c for c in fits if groups * -(-vdim // c) >= sm_count()), fits[-1])
+        plan = (plan[0], plan[1], cols)
+    if len(_memory_plan_cache) > 4096:
+        _memory_plan_cache.clear()
+    _memory_plan_cache[key] = plan
+    return plan
 
 
 def matrix_memory_supported(dim: int, vdim: int) -> bool:
@@ -1283,7 +1280,7 @@ def matrix_memory(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, g_c
                   dim: int, vdim: int, i_bias: Optional[torch.Tensor], f_bias: Optional[torch.Tensor], gate_cap: float,
                   q_scale: float, denom_eps: float, eps: float, norm_w: torch.Tensor, state_s: torch.Tensor,
                   state_n: torch.Tensor, state_m: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor,
-                  out: torch.Tensor, cols: int, carry: Optional[torch.Tensor] = None, raw: Optional[torch.Tensor] = None,
+                  out: torch.Tensor, cols: int, carry: Optional[torch.Tensor] = None, piece: int = 0, raw: Optional[torch.Tensor] = None,
                   next_nm: Optional[torch.Tensor] = None) -> None:
     """A matrix memory per head along every sequence of a step, from float32 partials ``rows`` ``[P, N, width]`` that hold q and k
     (``n_heads * dim`` columns each), v and the output gate's arguments (``n_heads * vdim`` each) and the two gates' arguments
@@ -1294,8 +1291,8 @@ def matrix_memory(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, g_c
         o = S'^T q / (max(|n' . q|, e^-m') + denom_eps),  out = o / sqrt(mean(o^2) + eps) * norm_w * sigmoid(g)
 
     ``state_s`` float32 ``[slots, n_heads, dim, vdim]``, ``state_n`` ``[slots, n_heads, dim]``, ``state_m`` ``[slots, n_heads]``; ``cols``
-    from ``matrix_memory_cols``.  ``carry`` float32 ``[B, pieces, n_heads, dim * vdim + dim + 3]`` lets a long prompt run in
-    pieces side by side (``pieces = matrix_memory_pieces(longest sequence)``).  With ``cols < vdim``: ``raw`` float32 ``[N, n_heads *
+    from ``matrix_memory_plan``.  ``carry`` float32 ``[B, pieces, n_heads, dim * vdim + dim + 3]`` lets a long prompt run in
+    pieces of ``piece`` tokens side by side.  With ``cols < vdim``: ``raw`` float32 ``[N, n_heads *
     vdim]`` and, without a carry, ``next_nm`` float32 ``[B, n_heads, dim + 1]``."""
     lib = _lib("matrix_memory")
     p_n, n, width = rows.shape
@@ -1317,8 +1314,8 @@ def matrix_memory(rows: torch.Tensor, *, q_col: int, k_col: int, v_col: int, g_c
     max_count = 0
     if carry is not None:
         assert carry.dim() == 4 and carry.shape[0] >= n_seqs and carry.shape[2:] == (n_heads, dim * vdim + dim + MEMORY_CARRY_EXTRA)
-        a.carry, a.pieces = _ptr(carry, torch.float32), carry.shape[1]
-        max_count = min(n, carry.shape[1] * MEMORY_PIECE)
+        a.carry, a.pieces, a.piece = _ptr(carry, torch.float32), carry.shape[1], piece
+        max_count = min(n, carry.shape[1] * piece)
     if cols < vdim:
         assert raw is not None and raw.shape == (n, n_heads * vdim)
         assert carry is not None or (next_nm is not None and next_nm.shape == (n_seqs, n_heads, dim + 1))

@@ -81,8 +81,7 @@ class MatrixMemory(Mixer):
         qk, v = self.nh * self.hd, self.nh * self.vd
         rows = linear(ctx, x, self.w_in, "memory.in", torch.float32)
         out = ctx.buffer("memory.out", (n, v))
-        pieces = ops.matrix_memory_pieces(ctx.max_count)
-        cols = ops.matrix_memory_cols(self.hd, self.vd, ctx.n_seqs * pieces * self.nh)
+        piece, pieces, cols = ops.matrix_memory_plan(self.hd, self.vd, self.nh, ctx.n_seqs, ctx.max_count)
         carry = raw = aside = None
         if pieces > 1:
             carry = ctx.buffer("memory.carry", (ctx.n_seqs, pieces, self.nh, self.hd * self.vd + self.hd + ops.MEMORY_CARRY_EXTRA),
@@ -95,7 +94,7 @@ class MatrixMemory(Mixer):
                           n_heads=self.nh, dim=self.hd, vdim=self.vd, i_bias=self.b_i, f_bias=self.b_f, gate_cap=self.cap,
                           q_scale=float(self.hd) ** -0.5, denom_eps=DENOMINATOR_EPS, eps=self.eps, norm_w=self.norm_w,
                           state_s=cache["memory"].state, state_n=cache["normaliser"].state, state_m=cache["maximum"].state,
-                          slots=ctx.slots, cu_tokens=ctx.cu_tokens, out=out, cols=cols, carry=carry, raw=raw, next_nm=aside)
+                          slots=ctx.slots, cu_tokens=ctx.cu_tokens, out=out, cols=cols, carry=carry, piece=piece, raw=raw, next_nm=aside)
         return Branch(linear(ctx, out, self.w_o, "memory.proj", torch.float32))
 
 

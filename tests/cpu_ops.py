@@ -346,16 +346,12 @@ MEMORY_PIECE = 4
 MEMORY_CARRY_EXTRA = 3
 
 
-def matrix_memory_pieces(max_count):
-    return -(-max_count // MEMORY_PIECE)
-
-
-def matrix_memory_cols(dim, vdim, groups):
-    return vdim if groups % 2 else max(1, vdim // 2)
+def matrix_memory_plan(dim, vdim, n_heads, n_seqs, max_count):
+    return MEMORY_PIECE, -(-max_count // MEMORY_PIECE), vdim if n_seqs % 2 else max(1, vdim // 2)
 
 
 def matrix_memory(rows, *, q_col, k_col, v_col, g_col, i_col, f_col, n_heads, dim, vdim, i_bias, f_bias, gate_cap, q_scale,
-                  denom_eps, eps, norm_w, state_s, state_n, state_m, slots, cu_tokens, out, cols, carry=None, raw=None,
+                  denom_eps, eps, norm_w, state_s, state_n, state_m, slots, cu_tokens, out, cols, carry=None, piece=0, raw=None,
                   next_nm=None):
     x = rows.float().sum(0)
     n, nh = x.shape[0], n_heads

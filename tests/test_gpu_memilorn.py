@@ -236,7 +236,7 @@ def test_routing_by_sigmoids_as_they_are(n_exp, top):
 
 
 MEMORY_SIZES = [(3, 16, 24, (5, 1, 9)), (2, 32, 40, (300, 1, 130)), (2, 64, 300, (5, 2, 1)), (5, 6, 6, (129, 128)), (1, 128, 128, (3, 140)),
-                (1, 200, 72, (17, 270)), (2, 10, 7, (1, 1, 1))]
+                (1, 200, 72, (17, 270)), (2, 10, 7, (1, 1, 1)), (2, 10, 300, (4, 70, 1))]
 
 
 @pytest.mark.parametrize("dtype", DTYPES, ids=IDS)
@@ -271,23 +271,24 @@ def test_matrix_memory_in_one_walk_and_in_pieces(dtype, nh, dim, vdim, counts):
         y = MP.unit_rms(y, 1e-5).reshape(c, vv) * nw.double() * torch.sigmoid(part(3, vv)[o:o + c])
         refs.append((y, last))
         o += c
-    lib_cols = sorted({vdim} | {c for c in (64, 32, 8) if c < vdim} | {ops.matrix_memory_cols(dim, vdim, nh * len(counts))})
+    lib_cols = sorted({vdim} | {c for c in (64, 32, 8) if c < vdim} | {ops.matrix_memory_plan(dim, vdim, nh, len(counts), max(counts))[2]})
     fits = ops._lib("matrix_memory").llg_matrix_memory_fits
     for cols in [c for c in lib_cols if fits(dim, c)]:
-        for pieces in (False, True):
+        for piece in (0, 128, 64, 20):
+            pieces = piece > 0
             S, N, M = s0.clone().cuda(), n0.clone().cuda(), m0.clone().cuda()
             out = torch.empty(n, vv, dtype=dtype, device="cuda")
-            carry = torch.empty(len(counts), ops.matrix_memory_pieces(max(counts)), nh, dim * vdim + dim + 3, device="cuda") if pieces else None
+            carry = torch.empty(len(counts), -(-max(counts) // piece), nh, dim * vdim + dim + 3, device="cuda") if pieces else None
             raw = torch.empty(n, vv, device="cuda") if cols < vdim else None
             nxt = torch.empty(len(counts), nh, dim + 1, device="cuda") if cols < vdim and not pieces else None
             ops.matrix_memory(rows.cuda(), q_col=cols_of[0], k_col=cols_of[1], v_col=cols_of[2], g_col=cols_of[3], i_col=cols_of[4],
                               f_col=cols_of[5], n_heads=nh, dim=dim, vdim=vdim, i_bias=ib.cuda(), f_bias=fb.cuda(), gate_cap=cap,
                               q_scale=dim ** -0.5, denom_eps=1e-6, eps=1e-5, norm_w=nw.cuda(), state_s=S, state_n=N, state_m=M,
-                              slots=sl, cu_tokens=cu, out=out, cols=cols, carry=carry, raw=raw, next_nm=nxt)
+                              slots=sl, cu_tokens=cu, out=out, cols=cols, carry=carry, piece=piece, raw=raw, next_nm=nxt)
             o = 0
             for b, c in enumerate(counts):
                 y, (s, nn, m) = refs[b]
-                what = (cols, pieces, b)
+                what = (cols, piece, b)
                 near(out[o:o + c], y, 2e-4 if dtype == torch.float32 else 2e-2, ("memory", *what))
                 near(S[slots[b]], s, 1e-4, ("S", *what))
                 near(N[slots[b]], nn, 1e-4, ("n", *what))
