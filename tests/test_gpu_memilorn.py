@@ -623,6 +623,52 @@ def test_configurations_drawn_at_random(llogos, tmp_path, seed):
     eng.cache.audit()
 
 
+def _random_tensor_config(seed):
+    """As ``_random_config``, of sizes that the tensor-core kernels take."""
+    g = torch.Generator().manual_seed(5000 + seed)
+    pick = lambda xs: xs[int(torch.randint(0, len(xs), (1,), generator=g))]
+    layers = []
+    for kind in torch.randperm(3, generator=g).tolist():
+        n_exp = pick([2, 4, 8])
+        mlp = MM.moe(n_exp, pick([1, 2]), pick([32, 72, 136]), pick([0.8, 3.0]), shared=pick([None, (64, 0.9)]))
+        if kind == 0:
+            mix = MM.mlstm(pick([2, 4, 6]), pick([32, 48, 96]), pick([32, 80, 128]), pick([6.0, 15.0]))
+        elif kind == 1:
+            mix = MM.latent(pick([2, 4, 6, 9]), pick([16, 32, 48]), pick([16, 32, 64]), pick([32, 64, 96, 128, 192]))
+        else:
+            kv, dim = pick([1, 2, 4, 5]), pick([16, 48, 80, 112, 128])
+            mix = MM.attention(kv * pick([1, 2, 3, 4, 5]), kv, dim, pick([16, 32, 96, 128]), pick([None, 8, dim]), base=pick([500.0, 1e6]),
+                               cap=pick([0.0, 15.0, 50.0]))
+        layers.append(MM.layer(mix, mlp))
+    return MM.config(layers, vocab=pick([160, 257]), width=pick([64, 128, 200]), loop=pick([None, (0, 2, 2), (1, 3, 2)]))
+
+
+@pytest.mark.parametrize("seed", range(8))
+def test_tensor_core_configurations_drawn_at_random(llogos, tmp_path, seed):
+    """bfloat16: a prompt whole, and a batch of two unequal prompts decoded together, against the plain model."""
+    cfg = _random_tensor_config(seed)
+    d = str(tmp_path / "m")
+    w = {k: v.float() for k, v in MM.write_model(llogos, d, cfg, seed=seed, steady_routing=True).items()}
+    model = llogos.weights.load_model(d, dtype=torch.bfloat16, device="cuda:0")
+    eng = llogos.engine.Engine(model, max_tokens=64 * 12)
+    key = {("random", torch.bfloat16): (d, cfg, w)}
+    for store in (_tokens, _refs, _pools):
+        for k in [k for k in store if k[0] == "random"]:
+            del store[k]
+    pairs = [sequence(key, "random", torch.bfloat16, n, n) for n in (230, 45)]
+    (a, ra), (b, rb) = pairs
+    slot = eng.open()
+    close(eng.step([(slot, a)], [list(range(len(a)))]), ra, torch.bfloat16, ("random", seed, "whole"))
+    eng.close(slot)
+    slots = [eng.open(), eng.open()]
+    cut = [len(a) - 14, len(b) - 14]
+    lg = eng.step([(slots[0], a[:cut[0]]), (slots[1], b[:cut[1]])])
+    close(lg[0], ra[cut[0] - 1], torch.bfloat16, ("random", seed, "prompt"))
+    got = [eng.step([(slots[0], [a[cut[0] + k]]), (slots[1], [b[cut[1] + k]])]).clone() for k in range(14)]
+    close(torch.stack([g[0] for g in got]), ra[cut[0]:], torch.bfloat16, ("random", seed, "decoded, long"))
+    close(torch.stack([g[1] for g in got]), rb[cut[1]:], torch.bfloat16, ("random", seed, "decoded, short"))
+
+
 # ---- faults that random weights would hide ---------------------------------------------------------
 
 A_TOK, B_TOK = 11, 12
