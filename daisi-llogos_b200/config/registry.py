@@ -151,3 +151,7 @@ register_architecture(_piratar.NAME, _piratar.PiratarConfig.from_dict, _piratar.
 from . import memilorn as _memilorn  # noqa: E402
 
 register_architecture(_memilorn.NAME, _memilorn.MemilornConfig.from_dict, _memilorn.memilorn_spec)
+
+from . import penasun as _penasun  # noqa: E402
+
+register_architecture(_penasun.NAME, _penasun.PenasunConfig.from_dict, _penasun.penasun_spec)

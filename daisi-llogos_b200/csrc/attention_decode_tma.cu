@@ -360,7 +360,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     if (a.has_sink) L += fast_exp2((a.sinks ? a.sinks[pend_row % a.nh] : a.sink_score) * LOG2E - M);       // the sink's weight beside the keys'; it carries no value
     float inv = L > 0.f ? 1.0f / L : 0.f;
     if (a.gate) inv *= a.gate[pend_row];
-    if (live) {
+    if (live && a.out_f32) {
+      *reinterpret_cast<float4*>((float*)a.out + pend_row * HD + 4 * lane) = make_float4(acc.x * inv, acc.y * inv, acc.z * inv, acc.w * inv);
+    } else if (live) {
       uint2 packed;
       packed.x = pack_bf16(acc.x * inv, acc.y * inv);
       packed.y = pack_bf16(acc.z * inv, acc.w * inv);
@@ -538,7 +540,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
           float inv = L > 0.f ? 1.0f / L : 0.f;
           if (a.gate) inv *= a.gate[head_row];
 #pragma unroll
-          for (int dd = 0; dd < HD / 32; ++dd) out[head_row * HD + lane + 32 * dd] = __float2bfloat16_rn(acc[dd] * inv);
+          for (int dd = 0; dd < HD / 32; ++dd) {
+            const long long at = head_row * HD + lane + 32 * dd;
+            if (a.out_f32) ((float*)a.out)[at] = acc[dd] * inv;
+            else out[at] = __float2bfloat16_rn(acc[dd] * inv);
+          }
         } else {
           if (pending) join_if_last();                  // a ticket of an earlier pair (or of this pair's head h0 - 4)
           float* mine = a.part + ((long long)(blockIdx.x + pair) * G + head) * (HD + PART_PAD);

@@ -302,8 +302,12 @@ __global__ void __launch_bounds__(128, 3) attn_prefill_mma_kernel(PrefillArgs a)
     bf16* dst = out + ((long long)(tok0 + q_off + row) * a.nh + h) * hd;
 #pragma unroll
     for (int j = 0; j < HDMAX / 8; ++j) {
-      if (j * 8 < hd)
-        *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * t) = pack_bf16(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+      if (j * 8 < hd) {
+        if (a.out_f32)
+          *reinterpret_cast<float2*>((float*)a.out + (dst - out) + j * 8 + 2 * t) = make_float2(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+        else
+          *reinterpret_cast<uint32_t*>(dst + j * 8 + 2 * t) = pack_bf16(o[j][2 * r] * inv, o[j][2 * r + 1] * inv);
+      }
     }
   }
 }
@@ -674,7 +678,11 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(DecodeArgs a, bf16
 #pragma unroll
     for (int dd = 0; dd < HDMAX / 32; ++dd) {
       const int d = lane + 32 * dd;
-      if (d < hd) out[((long long)b * a.nh + head) * hd + d] = __float2bfloat16_rn(oacc[dd] * inv);
+      const long long at = ((long long)b * a.nh + head) * hd + d;
+      if (d < hd) {
+        if (a.out_f32) reinterpret_cast<float*>(out)[at] = oacc[dd] * inv;
+        else out[at] = __float2bfloat16_rn(oacc[dd] * inv);
+      }
     }
   }
  }   // items

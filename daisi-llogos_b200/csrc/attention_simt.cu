@@ -159,7 +159,11 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(PrefillArgs a) {
 #pragma unroll
     for (int dd = 0; dd < MAXD; ++dd) {
       const int d = lane + 32 * dd;
-      if (d < vd) out[((long long)(tok0 + q_off + qi) * a.nh + h) * vd + d] = from_f32<T>(acc[i][dd] * inv);
+      const long long at = ((long long)(tok0 + q_off + qi) * a.nh + h) * vd + d;
+      if (d < vd) {
+        if (a.out_f32) reinterpret_cast<float*>(out)[at] = acc[i][dd] * inv;
+        else out[at] = from_f32<T>(acc[i][dd] * inv);
+      }
     }
   }
 }
@@ -364,8 +368,12 @@ LLG_API int llg_attn_decode_simt(const DecodeArgs* args, void* out, int dtype, c
     cudaError_t e = cudaFuncSetAttribute(attn_decode_kernel<T, D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     if (e != cudaSuccess) return llg_fail("attn_decode: shared memory %zu: %s", smem, cudaGetErrorString(e));           \
     attn_decode_kernel<T, D><<<grid, 128, smem, stream>>>(a);                                                           \
-    attn_decode_reduce_kernel<T><<<rgrid, 64, 0, stream>>>(a.part_o, a.part_ml, (T*)out, a.nh, vd, a.n_splits,          \
-                                                          a.has_sink, a.sink_score, a.gate, a.sinks);                  \
+    if (a.out_f32)                                                                                                      \
+      attn_decode_reduce_kernel<float><<<rgrid, 64, 0, stream>>>(a.part_o, a.part_ml, (float*)out, a.nh, vd, a.n_splits, \
+                                                            a.has_sink, a.sink_score, a.gate, a.sinks);                \
+    else                                                                                                                \
+      attn_decode_reduce_kernel<T><<<rgrid, 64, 0, stream>>>(a.part_o, a.part_ml, (T*)out, a.nh, vd, a.n_splits,        \
+                                                            a.has_sink, a.sink_score, a.gate, a.sinks);                \
   } while (0)
   if (dtype == LLG_F32) {
     if (large) DECODE(float, MAXD_LARGE);
@@ -440,5 +448,6 @@ int llg_attn_decode_noalloc(const void* q, const void* k_pages, const void* v_pa
   a.chunked = 0;
   a.softcap = 0.f;
   a.head_mix = nullptr;
+  a.out_f32 = 0;
   return llg_attn_decode_simt(&a, out, dtype, stream);
 }

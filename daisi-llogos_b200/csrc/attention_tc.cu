@@ -25,6 +25,11 @@
 // A row's accumulator is rescaled in place (tcgen05.ld / tcgen05.st) only when its maximum grows by
 // more than a factor of 2^8 in the weights, warp by warp and only when some row of the warp needs it.
 //
+// With MAPS (differential attention) the two halves of a query and of a key are two maps over the same values: the block's
+// two groups are the two maps of ONE tile of 128 queries, whose scores are products over their half of the head; keys,
+// values and queries arrive once for both.  At the end every thread reads a half of its row of both accumulators, takes
+// the difference, and the two threads of a row exchange their sums of squares for the head's unit norm.
+//
 // Every mbarrier wait is bounded; on expiry the thread records an error (llg_attn_tc_status) and
 // raises a flag that ends the other roles' waits; every role waits for its own copies in flight,
 // and the block frees its tensor memory and returns.
@@ -217,7 +222,7 @@ struct TileInfo {
   int nq[GROUPS], pos0[GROUPS], n_tiles[GROUPS], n_max;
 };
 
-template <int HD>
+template <int HD, bool MAPS>
 __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k_pages,
                                                                  const __grid_constant__ CUtensorMap map_v_pages,
                                                                  const __grid_constant__ CUtensorMap map_k_new,
@@ -230,13 +235,16 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_co
   constexpr int CPR = HD / 8;                 // 16-byte chunks per row of the head
   // The tiles need 1024-byte alignment (swizzle); the declaration asks for it and the kernel checks it.
   extern __shared__ __align__(1024) unsigned char smem[];
-  unsigned char* Qs = smem;                          // [GROUPS]
-  unsigned char* Ks = Qs + GROUPS * Q_BYTES;         // [KST]
+  constexpr int Q_TILES = MAPS ? 1 : GROUPS;
+  constexpr int G_STEP = MAPS ? 0 : BQ;              // queries from one group's tile to the next one's
+  unsigned char* Qs = smem;                          // [Q_TILES]
+  unsigned char* Ks = Qs + Q_TILES * Q_BYTES;        // [KST]
   unsigned char* Vs = Ks + KST * KV_BYTES;           // [VST]
   __shared__ uint64_t k_full[KST], k_free[KST], v_full[VST], v_free[VST];
   __shared__ uint64_t s_full[GROUPS][2], p_ready[GROUPS][2], o_done[GROUPS], q_ready;
   __shared__ uint32_t tmem_base_slot;
   __shared__ int abort_flag;
+  __shared__ float map_share[MAPS ? 2 * GROUPS : 1][MAPS ? BQ : 1];      // 1 / sum of each map's weights, sums of squares
 
   pdl_launch_dependents();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -293,8 +301,8 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_co
     ti.slot = a.slots[ti.b];
     ti.n_max = 0;
     for (int g = 0; g < GROUPS; ++g) {
-      ti.nq[g] = max(0, min(BQ, total - q_off - g * BQ));
-      ti.pos0[g] = ti.lb + q_off + g * BQ;
+      ti.nq[g] = max(0, min(BQ, total - q_off - g * G_STEP));
+      ti.pos0[g] = ti.lb + q_off + g * G_STEP;
     }
     // the first group's window starts earliest; the second masks the tiles that lie before its own
     int kb = mask_first(ti.pos0[0], a.window, a.chunked);
@@ -305,7 +313,7 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_co
     }
   }
   const int h = blockIdx.x, kvh = h / (a.nh / a.nkv);
-  const int k_end = ti.pos0[0] + (ti.nq[1] > 0 ? BQ + ti.nq[1] : ti.nq[0]);   // keys past it are never copied
+  const int k_end = ti.pos0[0] + (ti.nq[1] > 0 ? G_STEP + ti.nq[1] : ti.nq[0]);   // keys past it are never copied
   const int q_tok0 = ti.tok0 + ti.pos0[0] - ti.lb;                              // first token of the first query tile
 
   // queries: thread r of group g copies its part of tile g; the issuing lane waits for all of them,
@@ -313,10 +321,11 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_co
   if (tid < WORKERS) {
     const int g = tid / BQ, r = tid % BQ;
     const int ch = r % CPR;
-    for (int row = r / CPR; row < BQ; row += BQ / CPR) {
+    constexpr int ROWS = BQ / CPR;                   // rows a group copies side by side; with MAPS the groups share the tile's rows
+    for (int row = r / CPR + (MAPS ? g * ROWS : 0); row < BQ; row += MAPS ? GROUPS * ROWS : ROWS) {
       const bool valid = row < ti.nq[g];
-      const bf16* src = (const bf16*)a.q + ((long long)(q_tok0 + g * BQ + (valid ? row : 0)) * a.nh + h) * HD + ch * 8;
-      cp_async16(smem_u32(Qs + g * Q_BYTES) + (uint32_t)((ch >> 3) * (BQ * 128)) + swz(row, ch & 7), src, valid);
+      const bf16* src = (const bf16*)a.q + ((long long)(q_tok0 + g * G_STEP + (valid ? row : 0)) * a.nh + h) * HD + ch * 8;
+      cp_async16(smem_u32(Qs + (MAPS ? 0 : g * Q_BYTES)) + (uint32_t)((ch >> 3) * (BQ * 128)) + swz(row, ch & 7), src, valid);
     }
     cp_async_commit();
     cp_async_wait<0>();
@@ -404,10 +413,11 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_co
       constexpr uint32_t IDESC_O = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(HD >> 3) << 17) | ((uint32_t)(BQ >> 4) << 24);
       // scores of key tile t for group g into the group's score buffer t % 2
       auto issue_scores = [&](int g, int t) {
-        const uint32_t qa = smem_u32(Qs + g * Q_BYTES), ka = smem_u32(Ks + (t % KST) * KV_BYTES);
+        const uint32_t qa = smem_u32(Qs + (MAPS ? 0 : g * Q_BYTES)), ka = smem_u32(Ks + (t % KST) * KV_BYTES);
 #pragma unroll
-        for (int ks = 0; ks < HD / 16; ++ks) {
-          const uint32_t blk = ks >> 2, kk = ks & 3;      // 64-wide block, 16-wide step inside it (32 bytes)
+        for (int ks = 0; ks < (MAPS ? HD / 32 : HD / 16); ++ks) {
+          const int at = MAPS ? g * (HD / 32) + ks : ks;
+          const uint32_t blk = at >> 2, kk = at & 3;      // 64-wide block, 16-wide step inside it (32 bytes)
           umma_bf16(tmem + g * G_COLS + (uint32_t)(t & 1) * TK, desc_kmajor(qa + blk * (BQ * 128) + kk * 32),
                     desc_kmajor(ka + blk * (TK * 128) + kk * 32), IDESC_S, ks != 0);
         }
@@ -571,7 +581,47 @@ __global__ void __launch_bounds__(384, 1) attn_prefill_tc_kernel(const __grid_co
       ok = false;
     }
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-    if (ok && !*abortp) {
+    if (MAPS) {
+      // the two groups meet (both have the same queries, so all 256 threads come here, also after a wait that ran out)
+      map_share[g][r] = l_run > 0.f ? 1.0f / l_run : 0.f;
+      asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+      asm volatile("bar.sync 1, %0;" ::"n"(WORKERS) : "memory");
+      asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+      const bool whole = !*abortp;                       // uniform behind the barrier: no wait is left that could run out
+      float o[HD / 2], ss = 0.f;
+      if (whole) {
+        const float w1 = map_share[0][r], w2 = -a.map_lambda * map_share[GROUPS - 1][r];
+        const uint32_t row = tmem + O_COL + ((uint32_t)(gw * 32) << 16) + (uint32_t)(g * (HD / 2));
+#pragma unroll
+        for (int c0 = 0; c0 < HD / 2; c0 += 16) {
+          uint32_t r1[16], r2[16];
+          tmem_ld16(row + c0, r1);
+          tmem_ld16(row + G_COLS + c0, r2);
+          asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+          for (int c = 0; c < 16; ++c) {
+            const float v = fmaf(w2, __uint_as_float(r2[c]), w1 * __uint_as_float(r1[c]));
+            o[c0 + c] = v;
+            ss = fmaf(v, v, ss);
+          }
+        }
+      }
+      map_share[GROUPS + g][r] = ss;
+      asm volatile("bar.sync 1, %0;" ::"n"(WORKERS) : "memory");
+      if (whole && r < ti.nq[g]) {
+        const float f = a.map_scale / sqrtf((map_share[GROUPS][r] + map_share[2 * GROUPS - 1][r]) / (float)HD + a.map_eps);
+        bf16* dst = (bf16*)a.out + ((long long)(q_tok0 + r) * a.nh + h) * HD + g * (HD / 2);
+#pragma unroll
+        for (int c0 = 0; c0 < HD / 2; c0 += 8) {
+          uint4 v;
+          v.x = pack_bf16(o[c0] * f, o[c0 + 1] * f);
+          v.y = pack_bf16(o[c0 + 2] * f, o[c0 + 3] * f);
+          v.z = pack_bf16(o[c0 + 4] * f, o[c0 + 5] * f);
+          v.w = pack_bf16(o[c0 + 6] * f, o[c0 + 7] * f);
+          *reinterpret_cast<uint4*>(dst + c0) = v;
+        }
+      }
+    } else if (ok && !*abortp) {
       // a sink joins the sum with its own weight 2^(sink - M) and carries no value; a gate scales the head's output
       if (a.has_sink) l_run += fast_exp2((a.sinks ? a.sinks[h] : a.sink_score) * LOG2E - m_run);
       float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
@@ -666,13 +716,13 @@ bool kv_map(const void* base, long long rows, int nkv, int hd, CUtensorMap* resu
   return true;
 }
 
-template <int HD>
+template <int HD, bool MAPS>
 int launch(const PrefillArgs& a, cudaStream_t stream) {
   constexpr int KVB = (HD / 64) * TK * 128;
-  constexpr int smem = GROUPS * (HD / 64) * BQ * 128 + (KST + VST) * KVB;
+  constexpr int smem = (MAPS ? 1 : GROUPS) * (HD / 64) * BQ * 128 + (KST + VST) * KVB;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<HD, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
     if (e != cudaSuccess) return llg_fail("attn_prefill_tc: shared memory %d: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
@@ -681,7 +731,7 @@ int launch(const PrefillArgs& a, cudaStream_t stream) {
   if (!kv_map(a.k_pages, page_rows, 0, HD, &mkp) || !kv_map(a.v_pages, page_rows, 0, HD, &mvp) ||
       !kv_map(a.k_new, a.n_tokens, a.nkv, HD, &mkn) || !kv_map(a.v_new, a.n_tokens, a.nkv, HD, &mvn))
     return llg_fail("attn_prefill_tc: cuTensorMapEncodeTiled failed or is not available");
-  cudaError_t le = llg_launch(attn_prefill_tc_kernel<HD>, dim3(a.nh, a.n_tiles), dim3(THREADS), (size_t)smem, stream, mkp, mvp, mkn,
+  cudaError_t le = llg_launch(attn_prefill_tc_kernel<HD, MAPS>, dim3(a.nh, a.n_tiles), dim3(THREADS), (size_t)smem, stream, mkp, mvp, mkn,
                               mvn, a);
   if (le != cudaSuccess) return llg_fail("attn_prefill_tc: launch: %s", cudaGetErrorString(le));
   return llg_check_launch("attn_prefill_tc");
@@ -706,7 +756,12 @@ LLG_API int llg_attn_prefill_tc(const PrefillArgs* args, cudaStream_t stream) {
                   ((uintptr_t)a.v_pages % 16) == 0,
               "attn_prefill_tc: keys and values must be 16-byte aligned");
   if (a.n_tiles <= 0) return 0;
-  return a.hd == 64 ? launch<64>(a, stream) : launch<128>(a, stream);
+  LLG_REQUIRE(a.maps == 0 || a.maps == 2, "attn_prefill_tc: %d maps (0 or 2)", a.maps);
+  if (a.maps == 2) {
+    LLG_REQUIRE(!a.has_sink && !a.gate && a.map_eps > 0.f, "attn_prefill_tc: two maps go with neither a sink nor gates");
+    return a.hd == 64 ? launch<64, true>(a, stream) : launch<128, true>(a, stream);
+  }
+  return a.hd == 64 ? launch<64, false>(a, stream) : launch<128, false>(a, stream);
 }
 
 // Error code recorded when a wait ran out (0 = none); clears it.  Synchronises the device.

@@ -31,7 +31,7 @@ enum { F32 = 0, BF16 = 1 };
 // Entry points of the kernel libraries (filled in by the caller with the addresses of the loaded functions; an entry
 // may stay empty as long as no step needs it, so that a caller loads only the libraries its model uses).
 struct RunnerApi {
-  int (*add_rmsnorm)(float*, const float*, int, long long, const void*, int, float, void*, int, const int*, int, int, float*, cudaStream_t);
+  int (*add_rmsnorm)(float*, const float*, int, long long, const void*, int, float, void*, int, const int*, int, int, float*, const float*, cudaStream_t);
   int (*gemm_tc)(const void*, const void*, void*, int, int, int, int, int, int, int, const RowScale*, cudaStream_t);
   int (*gemm_simt)(const void*, int, const void*, int, void*, int, int, int, int, const RowScale*, cudaStream_t);
   int (*qk_prep)(const QkPrepArgs*, int, cudaStream_t);
@@ -162,7 +162,7 @@ int norm_after(const RunnerStep& s, const float* pending, int pending_parts, con
   const bool defer = s.dtype == BF16 && s.ss != nullptr;
   NEED(add_rmsnorm);
   if (g_api.add_rmsnorm(s.residual, pending, pending ? pending_parts : 0, (long long)n * s.hidden, norm_w, norm_w_dtype, eps, s.norm_out,
-                        s.dtype, nullptr, n, s.hidden, defer ? s.ss : nullptr, s.stream))
+                        s.dtype, nullptr, n, s.hidden, defer ? s.ss : nullptr, nullptr, s.stream))
     return fail("add_rmsnorm", g_api.err_elementwise);
   ++*launches;
   *scale = defer ? RowScale{s.ss, s.ss_parts, 1.0f / (float)s.hidden, eps} : RowScale{nullptr, 0, 0.f, 0.f};

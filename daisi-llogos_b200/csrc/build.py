@@ -44,6 +44,7 @@ SOURCES: Dict[str, List[str]] = {
     "recurrent": ["recurrent.cu", "common.cuh", "kernel_args.h"],
     "attention_mix_mma": ["attention_mix_mma.cu", "common.cuh", "kernel_args.h", "attention_reduce.cuh"],
     "matrix_memory": ["matrix_memory.cu", "common.cuh", "kernel_args.h"],
+    "state_space": ["state_space.cu", "common.cuh", "kernel_args.h"],
     "addnorm": ["addnorm.cu", "common.cuh", "kernel_args.h"],
     "moe": ["moe.cu", "common.cuh", "kernel_args.h"],
 }

@@ -79,7 +79,7 @@ __device__ __forceinline__ void vec_store4(__nv_bfloat16* p, const float (&v)[4]
 // ---- residual add + RMSNorm ---------------------------------------------------------
 
 // For output row j (token r = rows ? rows[j] : j):
-//   v = residual[r] + sum_s branch[s][r]   (written back to residual when there is a branch)
+//   v = residual[r] + branch_bias + sum_s branch[s][r]   (written back to residual when there is a branch)
 //   out[j] = v * rsqrt(mean(v^2) + eps) * weight         (eps inside the root, weight after)
 // With ss_out the division is left to the consumer of out (RowScale in kernel_args.h): out[j] = v * weight and
 // ss_out[j] = sum(v^2), whole or in parts.
@@ -87,7 +87,7 @@ template <typename OT, typename WT>
 __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const float* __restrict__ branch,
                                    int n_partials, long long partial_stride, const WT* __restrict__ weight,
                                    float eps, OT* __restrict__ out, const int* __restrict__ rows, int hidden,
-                                   float* __restrict__ ss_out) {
+                                   float* __restrict__ ss_out, const float* __restrict__ branch_bias) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[32];
@@ -99,6 +99,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const float* __
     float v = res[i];
     if (branch) {
       const float* b = branch + (long long)r * hidden + i;
+      if (branch_bias) v += branch_bias[i];
       for (int s = 0; s < n_partials; ++s) v += b[s * partial_stride];
       res[i] = v;
     }
@@ -121,7 +122,7 @@ template <typename OT, typename WT, int VPT>
 __global__ void add_rmsnorm_vec4_kernel(float* __restrict__ residual, const float* __restrict__ branch,
                                         int n_partials, long long partial_stride, const WT* __restrict__ weight,
                                         float eps, OT* __restrict__ out, const int* __restrict__ rows, int hidden,
-                                        float* __restrict__ ss_out) {
+                                        float* __restrict__ ss_out, const float* __restrict__ branch_bias) {
   __shared__ float red[32];
   pdl_launch_dependents();
   const int nv = hidden >> 2;
@@ -147,6 +148,10 @@ __global__ void add_rmsnorm_vec4_kernel(float* __restrict__ residual, const floa
     if (i < nv) {
       v = res[i];
       if (branch) {
+        if (branch_bias) {
+          const float4 bb = reinterpret_cast<const float4*>(branch_bias)[i];
+          v.x += bb.x; v.y += bb.y; v.z += bb.z; v.w += bb.w;
+        }
         const float4* b = reinterpret_cast<const float4*>(branch + (long long)r * hidden) + i;
         const long long ps = partial_stride >> 2;
         int s = 0;
@@ -207,12 +212,15 @@ __global__ void __launch_bounds__(PARTS_THREADS) add_rmsnorm_parts_kernel(float*
                                                                            int n_partials, long long partial_stride,
                                                                            const WT* __restrict__ weight, OT* __restrict__ out,
                                                                            const int* __restrict__ rows, int hidden,
-                                                                           float* __restrict__ ss_out) {
+                                                                           float* __restrict__ ss_out,
+                                                                           const float* __restrict__ branch_bias) {
   __shared__ float red[32];
   pdl_launch_dependents();
   const int i = blockIdx.x * PARTS_THREADS + threadIdx.x;          // float4 of the row (the host checks divisibility)
   float wv[4];
   vec_load4(weight + 4 * i, wv);                                   // no result of an earlier kernel
+  float4 bb = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (branch_bias) bb = reinterpret_cast<const float4*>(branch_bias)[i];
   const int j = blockIdx.y;
   if (threadIdx.x == 0) LLG_STAMP(3, 0, 0, blockIdx.x + gridDim.x * blockIdx.y);
   pdl_wait();
@@ -221,6 +229,7 @@ __global__ void __launch_bounds__(PARTS_THREADS) add_rmsnorm_parts_kernel(float*
   float4* res = reinterpret_cast<float4*>(residual + (long long)r * hidden);
   float4 v = res[i];
   if (branch) {
+    if (branch_bias) { v.x += bb.x; v.y += bb.y; v.z += bb.z; v.w += bb.w; }
     const float4* b = reinterpret_cast<const float4*>(branch + (long long)r * hidden) + i;
     const long long ps = partial_stride >> 2;
     constexpr int AT_ONCE = 12;                                    // all asked for before the first is added, added in order
@@ -251,13 +260,15 @@ LLG_API int llg_add_rmsnorm_parts(int n_out, int hidden) {
 
 LLG_API int llg_add_rmsnorm(float* residual, const float* branch, int n_partials, long long partial_stride,
                             const void* weight, int weight_dtype, float eps, void* out, int out_dtype,
-                            const int* rows, int n_out, int hidden, float* ss_out, cudaStream_t stream) {
+                            const int* rows, int n_out, int hidden, float* ss_out, const float* branch_bias, cudaStream_t stream) {
   LLG_REQUIRE(n_out >= 0 && hidden > 0, "add_rmsnorm: bad sizes n_out=%d hidden=%d", n_out, hidden);
   LLG_REQUIRE(eps > 0.f, "add_rmsnorm: eps must be positive");
   LLG_REQUIRE(!branch || n_partials >= 1, "add_rmsnorm: a branch needs n_partials >= 1");
+  LLG_REQUIRE(branch || !branch_bias, "add_rmsnorm: a bias without a branch");
   if (n_out == 0) return 0;
   const bool vec = hidden % 4 == 0 && partial_stride % 4 == 0 && ((uintptr_t)residual % 16) == 0 &&
-                   ((uintptr_t)branch % 16) == 0 && ((uintptr_t)weight % 16) == 0 && ((uintptr_t)out % 16) == 0;
+                   ((uintptr_t)branch % 16) == 0 && ((uintptr_t)weight % 16) == 0 && ((uintptr_t)out % 16) == 0 &&
+                   ((uintptr_t)branch_bias % 16) == 0;
   int threads = hidden >= 2048 ? 512 : (hidden >= 512 ? 256 : 128);
   // vector path: few rows (decode) want many threads per row, many rows want the row in registers
   int vpt = 1;
@@ -282,22 +293,22 @@ LLG_API int llg_add_rmsnorm(float* residual, const float* branch, int n_partials
   do {                                                                                                         \
     if (parts > 1)                                                                                             \
       llg_launch(add_rmsnorm_parts_kernel<OT, WT>, dim3(parts, n_out), PARTS_THREADS, 0, stream, residual, branch, \
-                 n_partials, partial_stride, (const WT*)weight, (OT*)out, rows, hidden, ss_out);               \
+                 n_partials, partial_stride, (const WT*)weight, (OT*)out, rows, hidden, ss_out, branch_bias);               \
     else if (vec_ok && vpt <= 1)                                                                                    \
       llg_launch(add_rmsnorm_vec4_kernel<OT, WT, 1>, n_out, threads, 0, stream, residual, branch, n_partials,    \
-                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out);                      \
+                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out, branch_bias);                      \
     else if (vec_ok && vpt <= 2)                                                                               \
       llg_launch(add_rmsnorm_vec4_kernel<OT, WT, 2>, n_out, threads, 0, stream, residual, branch, n_partials,    \
-                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out);                      \
+                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out, branch_bias);                      \
     else if (vec_ok && vpt <= 4)                                                                               \
       llg_launch(add_rmsnorm_vec4_kernel<OT, WT, 4>, n_out, threads, 0, stream, residual, branch, n_partials,    \
-                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out);                      \
+                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out, branch_bias);                      \
     else if (vec_ok)                                                                                           \
       llg_launch(add_rmsnorm_vec4_kernel<OT, WT, 8>, n_out, threads, 0, stream, residual, branch, n_partials,    \
-                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out);                      \
+                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out, branch_bias);                      \
     else                                                                                                       \
       llg_launch(add_rmsnorm_kernel<OT, WT>, n_out, threads, 0, stream, residual, branch, n_partials,            \
-                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out);                      \
+                 partial_stride, (const WT*)weight, eps, (OT*)out, rows, hidden, ss_out, branch_bias);                      \
   } while (0)
   if (out_dtype == LLG_F32 && weight_dtype == LLG_F32) LAUNCH(float, float);
   else if (out_dtype == LLG_F32 && weight_dtype == LLG_BF16) LAUNCH(float, __nv_bfloat16);
@@ -309,6 +320,11 @@ LLG_API int llg_add_rmsnorm(float* residual, const float* branch, int n_partials
 }
 
 // ---- query/key preparation ----------------------------------------------------------
+
+// What queries at a position are multiplied by (QkPrepArgs.q_scale; the host checks the table's reach).
+__device__ __forceinline__ float query_scale(const QkPrepArgs& a, int pos) {
+  return a.q_scale ? a.q_scale[pos < a.q_scale_positions ? pos : a.q_scale_positions - 1] : 1.0f;
+}
 
 template <typename IT, typename OT, typename WT>
 __global__ void qk_prep_kernel(QkPrepArgs a) {
@@ -390,8 +406,18 @@ __global__ void qk_prep_kernel(QkPrepArgs a) {
     __syncwarp();
   }
   if (kind == 0) {
+    const float qs = query_scale(a, pos);
+    if (a.q_maps == 2) {
+      OT* o = (OT*)a.q_out + ((long long)n * a.nh + h) * 2 * hd;
+      for (int d = lane; d < hd; d += 32) {
+        const float v = x[d] * qs;
+        o[d] = from_f32<OT>(2 * d < hd ? v : 0.f);
+        o[hd + d] = from_f32<OT>(2 * d < hd ? 0.f : v);
+      }
+      return;
+    }
     OT* o = (OT*)a.q_out + ((long long)n * a.nh + h) * hd;
-    for (int d = lane; d < hd; d += 32) o[d] = from_f32<OT>(x[d]);
+    for (int d = lane; d < hd; d += 32) o[d] = from_f32<OT>(x[d] * qs);
     return;
   }
   const int kvh = kind == 1 ? h - a.nh : h - a.nh - a.nkv;
@@ -442,6 +468,7 @@ __global__ void __launch_bounds__(256) qk_prep_vec_kernel(QkPrepArgs a) {
     vec_load4(bsrc + HALF, b1);
   }
   const int pos = a.positions[n];
+  const float qs = kind == 0 ? query_scale(a, pos) : 1.0f;
   const bool rotate = kind != 2 && a.cos_table;
   if (rotate) {
     const int p = pos < a.table_positions ? pos : a.table_positions - 1;
@@ -526,6 +553,22 @@ __global__ void __launch_bounds__(256) qk_prep_vec_kernel(QkPrepArgs a) {
     }
   }
   if (kind == 0) {
+    if (a.q_scale) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) {
+        x0[k] *= qs;
+        x1[k] *= qs;
+      }
+    }
+    if (a.q_maps == 2) {
+      const float none[4] = {0.f, 0.f, 0.f, 0.f};
+      OT* o = (OT*)a.q_out + ((long long)n * a.nh + h) * 2 * HD + 4 * l;
+      vec_store4(o, x0);
+      vec_store4(o + HALF, none);
+      vec_store4(o + HD, none);
+      vec_store4(o + HD + HALF, x1);
+      return;
+    }
     OT* o = (OT*)a.q_out + ((long long)n * a.nh + h) * HD + 4 * l;
     vec_store4(o, x0);
     vec_store4(o + HALF, x1);
@@ -552,6 +595,8 @@ LLG_API int llg_qk_prep(const QkPrepArgs* args, int out_dtype, cudaStream_t stre
   LLG_REQUIRE(!a.cos_table || (a.rotary_dim > 0 && a.rotary_dim % 2 == 0 && a.rotary_dim <= a.hd),
               "qk_prep: rotary_dim %d must be even and at most head_dim %d", a.rotary_dim, a.hd);
   LLG_REQUIRE(a.n_partials >= 1, "qk_prep: n_partials must be >= 1");
+  LLG_REQUIRE(a.q_maps == 0 || (a.q_maps == 2 && a.hd % 2 == 0), "qk_prep: %d maps of a query of %d elements (0 or 2)", a.q_maps, a.hd);
+  LLG_REQUIRE(!a.q_scale || a.q_scale_positions > 0, "qk_prep: an empty table of query factors");
   LLG_REQUIRE(!a.k_pages || (a.page_table && a.slots && a.seq_of_token && a.ring_pages > 0),
               "qk_prep: a cache write needs page_table, slots and seq_of_token");
   if (a.n_tokens == 0) return 0;
@@ -599,6 +644,70 @@ LLG_API int llg_qk_prep(const QkPrepArgs* args, int out_dtype, cudaStream_t stre
   }
 #undef LAUNCH
   return llg_check_launch("qk_prep");
+}
+
+// ---- the difference of two maps' outputs -------------------------------------------
+//
+// raw [n_tokens][nh][2][vd] float32: o = raw[.][0] - lambda raw[.][1], divided by sqrt(mean(o^2) + eps) over the vd elements of a
+// head and multiplied by scale.  A warp per (token, head).
+template <typename OT>
+__global__ void __launch_bounds__(128) map_difference_kernel(const float* __restrict__ raw, OT* __restrict__ out, long long items, int vd,
+                                                             float lambda, float eps, float scale) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const long long item = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (item >= items) return;
+  const float *r1 = raw + item * 2 * vd, *r2 = r1 + vd;
+  OT* o = out + item * vd;
+  float ss = 0.f;
+  if ((vd & 3) == 0 && vd <= 512) {
+    float v[4][4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int d = 4 * (lane + 32 * k);
+      if (d < vd) {
+        float a1[4], a2[4];
+        vec_load4(r1 + d, a1);
+        vec_load4(r2 + d, a2);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          v[k][e] = fmaf(-lambda, a2[e], a1[e]);
+          ss = fmaf(v[k][e], v[k][e], ss);
+        }
+      }
+    }
+    const float f = scale / sqrtf(warp_sum(ss) / (float)vd + eps);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int d = 4 * (lane + 32 * k);
+      if (d < vd) {
+        const float y[4] = {v[k][0] * f, v[k][1] * f, v[k][2] * f, v[k][3] * f};
+        vec_store4(o + d, y);
+      }
+    }
+    return;
+  }
+  for (int d = lane; d < vd; d += 32) {
+    const float v = fmaf(-lambda, r2[d], r1[d]);
+    ss = fmaf(v, v, ss);
+  }
+  const float f = scale / sqrtf(warp_sum(ss) / (float)vd + eps);
+  for (int d = lane; d < vd; d += 32) o[d] = from_f32<OT>(fmaf(-lambda, r2[d], r1[d]) * f);
+}
+
+LLG_API int llg_map_difference(const float* raw, void* out, int out_dtype, int n_tokens, int nh, int vd, float lambda, float eps,
+                               float scale, cudaStream_t stream) {
+  LLG_REQUIRE(n_tokens >= 0 && nh > 0 && vd > 0 && eps > 0.f, "map_difference: bad sizes");
+  LLG_REQUIRE(((uintptr_t)raw & 15u) == 0 && ((uintptr_t)out & 15u) == 0, "map_difference: operands must be 16-byte aligned");
+  if (n_tokens == 0) return 0;
+  const long long items = (long long)n_tokens * nh;
+  const unsigned grid = (unsigned)((items + 3) / 4);
+  if (out_dtype == LLG_F32) llg_launch(map_difference_kernel<float>, grid, 128, 0, stream, raw, (float*)out, items, vd, lambda, eps, scale);
+  else if (out_dtype == LLG_BF16)
+    llg_launch(map_difference_kernel<__nv_bfloat16>, grid, 128, 0, stream, raw, (__nv_bfloat16*)out, items, vd, lambda, eps, scale);
+  else return llg_fail("map_difference: unknown output type %d", out_dtype);
+  return llg_check_launch("map_difference");
 }
 
 // ---- cache write after a prompt step ------------------------------------------------

@@ -503,6 +503,11 @@ __global__ void __launch_bounds__(GEMM_THREADS) gemm_tc_kernel(const __grid_cons
                   }
                 }
               }
+              if (kind == 0 && a.q_scale) {
+                const float qs = a.q_scale[pos < a.q_scale_positions ? pos : a.q_scale_positions - 1];
+  #pragma unroll
+                for (int d = 0; d < HD; ++d) h[d] *= qs;
+              }
               if (live) {
                 auto store_head = [&](bf* dst) {
   #pragma unroll
@@ -981,6 +986,8 @@ LLG_API int llg_gemm_tc_qkv(const void* x, const void* w, int n, int k, const Qk
   LLG_REQUIRE(a.n_tokens == n && a.positions && a.q_out, "gemm_tc_qkv: the preparation's sizes do not fit the product");
   LLG_REQUIRE(!a.k_pages || (a.page_table && a.slots && a.seq_of_token && a.ring_pages > 0),
               "gemm_tc_qkv: a cache write needs page_table, slots and seq_of_token");
+  LLG_REQUIRE(a.q_maps == 0, "gemm_tc_qkv: queries split into maps are the preparation kernel's");
+  LLG_REQUIRE(!a.q_scale || a.q_scale_positions > 0, "gemm_tc_qkv: an empty table of query factors");
   if ((a.q_norm_w || a.k_norm_w) && a.bias)
     LLG_REQUIRE(a.norm_w_dtype == a.bias_dtype, "gemm_tc_qkv: norm weights and bias must share a dtype");
   auto aligned = [](const void* p) { return ((uintptr_t)p & 15u) == 0; };

@@ -92,6 +92,12 @@ struct QkPrepArgs {
   const float* v_first_in;    // [n_tokens][nkv][vd] float32 or null
   float* v_first_out;         // [n_tokens][nkv][vd] float32 or null: receives the values as projected (before any blend)
   float* gate_out;            // [n_tokens][nh] or null: a row of qkv then ends with nh more numbers z, and gate_out = sigmoid(z)
+  // All preparations read these two:
+  const float* q_scale;       // [q_scale_positions] or null: queries are multiplied by q_scale[position] before they are rounded
+  int q_scale_positions;
+  int q_maps;                 // 2: q_out is [n_tokens][2 * nh][hd]: a query head's two halves as two heads, each with zeros in
+                              // the other half's place, so that either meets its own half of the key (0: plain; the
+                              // product whose epilogue is the preparation writes plain queries only)
 };
 
 // Attention for a step with several tokens per sequence (attention_simt.cu, attention_mma.cu, attention_tc.cu).
@@ -125,6 +131,12 @@ struct PrefillArgs {
   // Only the kernels of attention_mix.cu read these:
   float softcap;            // > 0: a score s becomes softcap * tanh(s / softcap)
   const float* head_mix;    // [nh][nh] or null: then head h's score is sum_g head_mix[h][g] * (head g's score)
+  int out_f32;              // 1: out is float32 whatever the operands' type (not read by attention_tc.cu and attention_mix*.cu)
+  // Only attention_tc.cu reads these.  maps = 2: the two halves of a query and of a key are two maps, each with a softmax of
+  // its own over the same values; with their outputs a1, a2, o = a1 - map_lambda a2 is divided by sqrt(mean(o^2) + map_eps) over
+  // the head and multiplied by map_scale.
+  int maps;
+  float map_lambda, map_eps, map_scale;
 };
 
 // Attention of one new token per sequence, split kernels (attention_simt.cu, attention_mma.cu).
@@ -150,6 +162,7 @@ struct DecodeArgs {
   int chunked;
   float softcap;            // as in PrefillArgs (attention_mix.cu only)
   const float* head_mix;
+  int out_f32;              // as in PrefillArgs (the join's output)
 };
 
 // Attention of one new token per sequence, TMA kernel (attention_decode_tma.cu).
@@ -171,6 +184,7 @@ struct DecodeTmaArgs {
   const float* gate;          // [n_seqs][nh] or null
   const float* sinks;         // as in PrefillArgs
   int chunked;
+  int out_f32;                // 1: out is float32
 };
 
 // Residual kept as several streams (hyper-connections), elementwise.cu: hc_add_rmsnorm.  For output row j (token
@@ -311,11 +325,15 @@ struct MinGruArgs {
 //            the `top` eligible experts of largest s, weights = s / (sum of the chosen s + sum_eps) * scale.
 //   score 2: s = softmax over all experts' logits; the `top` experts of largest s, weights as for score 1.
 // raw = 1 (scores 1 and 2): weights = s * scale, not divided by the chosen scores' sum.
+// groups > 0 (scores 1 and 2): n_exp experts in `groups` equal groups of neighbours, a group judged by the sum of its
+// group_top largest choice scores; only experts of the keep_groups best groups can be chosen.
+// correction (scores 1 and 2): groups are judged and experts chosen by s + correction, weights are made of s alone.
 struct RouterRule {
   int score;
   int groups, keep_groups, group_top;
   float scale, sum_eps;
   int raw;
+  const float* correction;    // [n_exp] or null
 };
 
 // Preparation for latent attention (latent.cu: latent_prep).  A row of the input product holds, per token, up to three
@@ -485,10 +503,11 @@ struct ConvArgs {
   const int* cu_tokens;       // [n_seqs + 1]
   const int* seq_of_token;    // [n_tokens]
   const int* len_before;      // [n_seqs]
-  float* out;                 // [n_tokens][channels]
+  float* out;                 // [n_tokens][channels], or null where out2 is wanted alone
   void* out2;                 // or null: the same values once more in out2_dtype
   int out2_dtype;
   int n_seqs, n_tokens;
+  int act;                    // 0: none; else 1 + an activation kind of llg_act, applied to what is written
 };
 
 // The real-gated linear recurrent unit over a step's sequences (recurrent.cu).  Per channel c of block b = c / block_width:
@@ -578,4 +597,28 @@ struct MatrixMemoryArgs {
   float* raw;                 // [n_tokens][nh * vdim], where cols < vdim
   float* next;                // [n_seqs][nh][dim + 1], where cols < vdim and there is no carry
   int n_seqs, n_tokens, nh, dim, vdim, cols;
+};
+
+// A state-space recurrence with a scalar decay per head and step (state_space.cu).  A row of `mixed` is x [nh][vdim], then B
+// [groups][n_state], then C [groups][n_state] (head h reads group h / (nh / groups)); with d = softplus(dt + dt_bias[h]), dt
+// the sum of the partials' column dt_col + h:
+//   S <- exp(-exp(a_log[h]) d) S + d B x^T        (S is [n_state][vdim])
+//   out = (S^T C + d_skip[h] x) * silu(z)         (z the sums of the columns from z_col on; z_col < 0: no gate)
+// state [slots][nh][n_state][vdim] holds S before the step's first token of a sequence and receives it after its last.
+// A block owns `cols` columns of a head's S (a column's walk needs no other column).
+struct StateSpaceArgs {
+  const void* mixed;          // [n_tokens][nh * vdim + 2 * groups * n_state]
+  int mixed_dtype;
+  const float* rows;          // [n_partials][n_tokens][row_width]
+  int n_partials;
+  long long partial_stride;
+  int row_width, z_col, dt_col;
+  const float* dt_bias;       // [nh]
+  const float* a_log;         // [nh]
+  const float* d_skip;        // [nh]
+  float* state;
+  const int* slots;           // [n_seqs]
+  const int* cu_tokens;       // [n_seqs + 1]
+  float* out;                 // [n_tokens][nh * vdim]
+  int n_seqs, n_tokens, nh, groups, n_state, vdim, cols;
 };

@@ -3,7 +3,7 @@
 //
 //   moe_route   : z = W_r x + b in float32 (x may be bfloat16), the `top` largest per token (ties: the lower index), weights
 //                 softmax over the chosen z alone; or, by a RouterRule, sigmoid scores chosen within the best groups of
-//                 experts and divided by their sum.
+//                 experts and divided by their sum; experts may be chosen by corrected scores and weighed by plain ones.
 //   moe_plan    : one block counts the pairs of every expert, lays the experts' runs out one after another, each filled
 //                 up to whole tiles, and gives every pair its row.  Which row of its expert's run a pair gets depends on
 //                 the order in which the threads arrive; no result depends on it (a row's values come from its own token
@@ -12,6 +12,8 @@
 //                 16-byte boundaries on the tensor cores (mma.sync), everything else on the CUDA cores.
 //   moe_combine : out[n] = sum_k weight[n][k] y[row of (n, k)] + the shared expert's partial sums (a design whose weights
 //                 are on the experts' inputs has them in the first product's epilogue, and adds its rows as they are).
+//   Identity experts: the router may know more experts than there are matrices for; a pair whose choice lies beyond them
+//                 has no row (moe_plan says -1) and moe_combine adds its token's input times its weight instead.
 #include "common.cuh"
 #include "kernel_args.h"
 
@@ -24,7 +26,7 @@ namespace {
 
 // One warp turns a token's logits z[0 .. n_exp) (shared memory, overwritten) into its `top` experts and their weights by
 // `rule` (RouterRule in kernel_args.h).  Ties go to the lower index.  gsc: n_exp floats of scratch beside z (group
-// scores and the marks of the groups that stay).
+// scores and the marks of the groups that stay), and n_exp more with a correction (the scores without it).
 __device__ __forceinline__ void choose_and_weigh(float* z, float* gsc, float* chosen, int n_exp, int top, const RouterRule& rule,
                                                  int* __restrict__ choice, float* __restrict__ weight, int lane) {
   if (rule.score == 2) {
@@ -45,50 +47,60 @@ __device__ __forceinline__ void choose_and_weigh(float* z, float* gsc, float* ch
   if (rule.score == 1) {
     for (int e = lane; e < n_exp; e += 32) z[e] = 1.0f / (1.0f + expf(-z[e]));
     __syncwarp();
-    if (rule.groups > 0) {
-      const int per = n_exp / rule.groups;
-      // a group's score: the sum of its group_top largest scores (a lane per group, the largest taken one after another)
-      for (int g = lane; g < rule.groups; g += 32) {
-        const float* zg = z + g * per;
-        float total = 0.f, prev = INFINITY;
-        int prev_i = -1;
-        for (int t = 0; t < rule.group_top && t < per; ++t) {
-          float best = -INFINITY;
-          int arg = -1;
-          for (int i = 0; i < per; ++i) {
-            const float v = zg[i];
-            const bool after = v < prev || (v == prev && i > prev_i);     // not taken yet
-            if (after && v > best) { best = v; arg = i; }
-          }
-          if (arg < 0) break;
-          total += best;
-          prev = best;
-          prev_i = arg;
-        }
-        gsc[g] = total;
-      }
-      __syncwarp();
-      // the keep_groups best groups stay: their mark is 2 (no sum of scores reaches it), the others' scores fall to -1
-      for (int k = 0; k < rule.keep_groups; ++k) {
+  }
+  const float* plain = nullptr;           // the scores that make the weights, where they are not the ones that choose
+  if (rule.score != 0 && rule.correction) {
+    float* keep = gsc + n_exp;
+    for (int e = lane; e < n_exp; e += 32) {
+      keep[e] = z[e];
+      z[e] += rule.correction[e];
+    }
+    plain = keep;
+    __syncwarp();
+  }
+  if (rule.score != 0 && rule.groups > 0) {
+    const int per = n_exp / rule.groups;
+    // a group's score: the sum of its group_top largest scores (a lane per group, the largest taken one after another)
+    for (int g = lane; g < rule.groups; g += 32) {
+      const float* zg = z + g * per;
+      float total = 0.f, prev = INFINITY;
+      int prev_i = -1;
+      for (int t = 0; t < rule.group_top && t < per; ++t) {
         float best = -INFINITY;
-        int arg = 0x7fffffff;
-        for (int g = lane; g < rule.groups; g += 32) {
-          const float v = gsc[g];
-          if (v <= (float)per && v > best) { best = v; arg = g; }
+        int arg = -1;
+        for (int i = 0; i < per; ++i) {
+          const float v = zg[i];
+          const bool after = v < prev || (v == prev && i > prev_i);     // not taken yet
+          if (after && v > best) { best = v; arg = i; }
         }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-          const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
-          if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
-        }
-        if (lane == 0 && arg != 0x7fffffff) gsc[arg] = 2.0f * (float)per + 1.0f;
-        __syncwarp();
+        if (arg < 0) break;
+        total += best;
+        prev = best;
+        prev_i = arg;
       }
-      for (int e = lane; e < n_exp; e += 32)
-        if (gsc[e / per] <= (float)per) z[e] = -1.0f;
+      gsc[g] = total;
+    }
+    __syncwarp();
+    // the keep_groups best groups stay: their mark is infinity (no sum of scores reaches it), the others' scores fall away
+    for (int k = 0; k < rule.keep_groups; ++k) {
+      float best = -INFINITY;
+      int arg = 0x7fffffff;
+      for (int g = lane; g < rule.groups; g += 32) {
+        const float v = gsc[g];
+        if (v < INFINITY && v > best) { best = v; arg = g; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
+        if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
+      }
+      if (lane == 0 && arg != 0x7fffffff) gsc[arg] = INFINITY;
       __syncwarp();
     }
+    for (int e = lane; e < n_exp; e += 32)
+      if (gsc[e / per] != INFINITY) z[e] = -INFINITY;
+    __syncwarp();
   }
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -106,7 +118,7 @@ __device__ __forceinline__ void choose_and_weigh(float* z, float* gsc, float* ch
     if (arg == 0x7fffffff) arg = 0;                 // nothing but -inf or NaN left: still a valid index
     if (lane == 0) {
       choice[k] = arg;
-      chosen[k] = best;
+      chosen[k] = plain ? plain[arg] : best;
       z[arg] = -INFINITY;
     }
     __syncwarp();
@@ -140,7 +152,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const XT* __restrict__ x
   pdl_wait();
   extern __shared__ float sm[];
   float* xs = sm;                   // [hidden]
-  float* z = sm + hidden;           // [n_exp + 1], then [n_exp] of scratch
+  float* z = sm + hidden;           // [n_exp + 1], then [n_exp] of scratch, twice with a correction
   __shared__ float chosen[LLG_MOE_MAX_TOP];
   const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) xs[i] = to_f32(x[(long long)n * hidden + i]);
@@ -174,7 +186,7 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float* __restrict__
   const int n = blockIdx.x * 4 + warp;
   if (n >= n_tokens) return;
   const int width = n_exp + (extra ? 1 : 0);
-  float* z = sm + warp * (2 * n_exp + 1);
+  float* z = sm + warp * ((rule.correction ? 3 : 2) * n_exp + 1);
   for (int e = lane; e < width; e += 32) {
     float v = bias && e < n_exp ? bias[e] : 0.f;
     for (int s = 0; s < n_partials; ++s) v += logits[s * partial_stride + (long long)n * width + e];
@@ -220,7 +232,7 @@ __global__ void __launch_bounds__(1024) moe_plan_kernel(const int* __restrict__ 
   }
   for (int p = tid; p < n_pairs; p += nt) {
     const int e = choice[p];
-    int row = 0;
+    int row = -1;                                   // an identity expert's pair: no matrices, no row
     if (e >= 0 && e < n_exp) {
       row = starts[e] + atomicAdd(&cursor[e], 1);
       token_of_row[row] = p / top;
@@ -443,10 +455,18 @@ __global__ void moe_gather_rows_kernel(const uint4* __restrict__ x, const int* _
   out[i] = t >= 0 ? x[(long long)t * chunks + c] : make_uint4(0u, 0u, 0u, 0u);
 }
 
+__device__ __forceinline__ float4 load_four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load_four(const __nv_bfloat16* p) {
+  const uint2 t = *reinterpret_cast<const uint2*>(p);
+  const __nv_bfloat162 lo = *reinterpret_cast<const __nv_bfloat162*>(&t.x), hi = *reinterpret_cast<const __nv_bfloat162*>(&t.y);
+  return make_float4(__low2float(lo), __high2float(lo), __low2float(hi), __high2float(hi));
+}
+
+template <typename XT>
 __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair,
                                    const float* __restrict__ weight, const float* __restrict__ shared, int n_shared,
                                    long long shared_stride, const float* __restrict__ shared_scale, float* __restrict__ out,
-                                   int hidden, int top) {
+                                   int hidden, int top, const XT* __restrict__ x) {
   pdl_launch_dependents();
   pdl_wait();
   const int n = blockIdx.x;
@@ -454,7 +474,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
     float v = 0.f;
     for (int k = 0; k < top; ++k) {
       const int row = row_of_pair[(long long)n * top + k];
-      v = fmaf(weight ? weight[(long long)n * top + k] : 1.0f, y[(long long)row * hidden + d], v);
+      const float u = row >= 0 ? y[(long long)row * hidden + d] : x ? to_f32(x[(long long)n * hidden + d]) : 0.f;
+      v = fmaf(weight ? weight[(long long)n * top + k] : 1.0f, u, v);
     }
     float sh = 0.f;
     for (int s = 0; s < n_shared; ++s) sh += shared[s * shared_stride + (long long)n * hidden + d];
@@ -464,10 +485,11 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const int* __res
 
 // The same with four columns a thread (rows that start on 16-byte boundaries): every load of a thread is independent of
 // the others, so the few rows of a decode step are not a chain of waits.
+template <typename XT>
 __global__ void moe_combine_vec4_kernel(const float* __restrict__ y, const int* __restrict__ row_of_pair,
                                         const float* __restrict__ weight, const float* __restrict__ shared, int n_shared,
                                         long long shared_stride, const float* __restrict__ shared_scale,
-                                        float* __restrict__ out, int hidden, int top) {
+                                        float* __restrict__ out, int hidden, int top, const XT* __restrict__ x) {
   pdl_launch_dependents();
   pdl_wait();
   const int n = blockIdx.x;
@@ -477,7 +499,9 @@ __global__ void moe_combine_vec4_kernel(const float* __restrict__ y, const int* 
   for (int k = 0; k < top; ++k) {
     const int row = row_of_pair[(long long)n * top + k];
     const float wk = weight ? weight[(long long)n * top + k] : 1.0f;
-    const float4 u = *reinterpret_cast<const float4*>(y + (long long)row * hidden + d);
+    float4 u = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (row >= 0) u = *reinterpret_cast<const float4*>(y + (long long)row * hidden + d);
+    else if (x) u = load_four(x + (long long)n * hidden + d);
     v.x = fmaf(wk, u.x, v.x); v.y = fmaf(wk, u.y, v.y); v.z = fmaf(wk, u.z, v.z); v.w = fmaf(wk, u.w, v.w);
   }
   float4 sh = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -495,7 +519,8 @@ __global__ void moe_combine_vec4_kernel(const float* __restrict__ y, const int* 
 static int check_rule(const char* what, const RouterRule& r, int n_exp, int top) {
   LLG_REQUIRE(r.score >= 0 && r.score <= 2, "%s: score kind %d is not known", what, r.score);
   LLG_REQUIRE(!r.raw || r.score != 0, "%s: undivided scores go with sigmoid or softmax-over-all scores", what);
-  LLG_REQUIRE(r.groups >= 0 && (r.groups == 0 || r.score == 1), "%s: groups of experts go with sigmoid scores", what);
+  LLG_REQUIRE(r.groups >= 0 && (r.groups == 0 || r.score != 0), "%s: groups of experts go with sigmoid or softmax-over-all scores", what);
+  LLG_REQUIRE(!r.correction || r.score != 0, "%s: a correction goes with sigmoid or softmax-over-all scores", what);
   if (r.groups > 0) {
     LLG_REQUIRE(n_exp % r.groups == 0 && r.keep_groups > 0 && r.keep_groups <= r.groups && r.group_top > 0,
                 "%s: %d experts in %d groups of which %d stay, judged by %d scores", what, n_exp, r.groups, r.keep_groups, r.group_top);
@@ -512,10 +537,10 @@ LLG_API int llg_moe_route(const void* x, int x_dtype, const float* w, const floa
   LLG_REQUIRE(n_exp > 0 && n_exp <= LLG_MOE_MAX_EXPERTS, "moe_route: %d experts are outside [1, %d]", n_exp, LLG_MOE_MAX_EXPERTS);
   LLG_REQUIRE(top > 0 && top <= n_exp && top <= LLG_MOE_MAX_TOP, "moe_route: top %d of %d experts (at most %d)", top, n_exp,
               LLG_MOE_MAX_TOP);
-  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f, 0};
+  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f, 0, nullptr};
   if (check_rule("moe_route", r, n_exp, top)) return 1;
   if (n_tokens == 0) return 0;
-  const size_t smem = (size_t)(hidden + 2 * n_exp + 1) * sizeof(float);
+  const size_t smem = (size_t)(hidden + (r.correction ? 3 : 2) * n_exp + 1) * sizeof(float);
   LLG_REQUIRE(smem <= 200 * 1024, "moe_route: rows of %d elements do not fit shared memory", hidden);
   if (x_dtype == LLG_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_route_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -539,10 +564,12 @@ LLG_API int llg_moe_topk(const float* logits, int n_partials, long long partial_
   LLG_REQUIRE(n_exp > 0 && n_exp <= LLG_MOE_MAX_EXPERTS, "moe_topk: %d experts are outside [1, %d]", n_exp, LLG_MOE_MAX_EXPERTS);
   LLG_REQUIRE(top > 0 && top <= n_exp && top <= LLG_MOE_MAX_TOP, "moe_topk: top %d of %d experts (at most %d)", top, n_exp,
               LLG_MOE_MAX_TOP);
-  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f, 0};
+  const RouterRule r = rule ? *rule : RouterRule{0, 0, 0, 0, 1.0f, 0.0f, 0, nullptr};
   if (check_rule("moe_topk", r, n_exp, top)) return 1;
   if (n_tokens == 0) return 0;
-  llg_launch(moe_topk_kernel, dim3((n_tokens + 3) / 4), dim3(128), (size_t)4 * (2 * n_exp + 1) * sizeof(float), stream, logits,
+  const size_t smem = (size_t)4 * ((r.correction ? 3 : 2) * n_exp + 1) * sizeof(float);
+  if (smem > 48 * 1024) cudaFuncSetAttribute(moe_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  llg_launch(moe_topk_kernel, dim3((n_tokens + 3) / 4), dim3(128), smem, stream, logits,
              n_partials, partial_stride, bias, choice, weight, n_tokens, n_exp, top, r, extra);
   return llg_check_launch("moe_topk");
 }
@@ -659,24 +686,32 @@ LLG_API int llg_moe_gather_rows(const void* x, const int* token_of_row, void* ou
   return llg_check_launch("moe_gather_rows");
 }
 
-// weight: null = every pair counts once.  shared_scale: null, or [n_tokens]: the sum of the shared expert's partials is multiplied by it.
+// weight: null = every pair counts once.  shared_scale: null, or [n_tokens]: the sum of the shared expert's partials is
+// multiplied by it.  x: null, or [n_tokens][hidden]: what a pair without a row (row_of_pair -1, an identity expert) stands for.
 LLG_API int llg_moe_combine(const float* y, const int* row_of_pair, const float* weight, const float* shared, int n_shared,
                             long long shared_stride, const float* shared_scale, float* out, int n_tokens, int hidden, int top,
-                            cudaStream_t stream) {
+                            const void* x, int x_dtype, cudaStream_t stream) {
   LLG_REQUIRE(n_tokens >= 0 && hidden > 0 && top > 0, "moe_combine: bad sizes");
   LLG_REQUIRE(!shared || n_shared >= 1, "moe_combine: a shared expert's partials need at least one");
+  LLG_REQUIRE(!x || x_dtype == LLG_F32 || x_dtype == LLG_BF16, "moe_combine: unknown type %d of the identity experts' input", x_dtype);
   if (n_tokens == 0) return 0;
   const bool vec = hidden % 4 == 0 && shared_stride % 4 == 0 && ((uintptr_t)y % 16) == 0 && ((uintptr_t)shared % 16) == 0 &&
-                   ((uintptr_t)out % 16) == 0;
-  if (vec) {
-    const int threads = 128;
-    dim3 grid(n_tokens, (hidden / 4 + threads - 1) / threads);
-    llg_launch(moe_combine_vec4_kernel, grid, dim3(threads), 0, stream, y, row_of_pair, weight, shared, shared ? n_shared : 0,
-               shared_stride, shared ? shared_scale : nullptr, out, hidden, top);
-  } else {
-    const int threads = hidden >= 1024 ? 256 : 128;
-    llg_launch(moe_combine_kernel, dim3(n_tokens, 1), dim3(threads), 0, stream, y, row_of_pair, weight, shared,
-               shared ? n_shared : 0, shared_stride, shared ? shared_scale : nullptr, out, hidden, top);
-  }
+                   ((uintptr_t)out % 16) == 0 && ((uintptr_t)x % 16) == 0;
+#define COMBINE(XT)                                                                                                            \
+  do {                                                                                                                         \
+    if (vec) {                                                                                                                 \
+      const int threads = 128;                                                                                                 \
+      dim3 grid(n_tokens, (hidden / 4 + threads - 1) / threads);                                                               \
+      llg_launch(moe_combine_vec4_kernel<XT>, grid, dim3(threads), 0, stream, y, row_of_pair, weight, shared,                  \
+                 shared ? n_shared : 0, shared_stride, shared ? shared_scale : nullptr, out, hidden, top, (const XT*)x);       \
+    } else {                                                                                                                   \
+      const int threads = hidden >= 1024 ? 256 : 128;                                                                          \
+      llg_launch(moe_combine_kernel<XT>, dim3(n_tokens, 1), dim3(threads), 0, stream, y, row_of_pair, weight, shared,          \
+                 shared ? n_shared : 0, shared_stride, shared ? shared_scale : nullptr, out, hidden, top, (const XT*)x);       \
+    }                                                                                                                          \
+  } while (0)
+  if (x && x_dtype == LLG_BF16) COMBINE(__nv_bfloat16);
+  else COMBINE(float);
+#undef COMBINE
   return llg_check_launch("moe_combine");
 }

@@ -178,12 +178,16 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ConvArgs a) {
     return v + ib;
   };
   O2* out2 = (O2*)a.out2;
+  auto put = [&](int token, float v) {
+    if (a.act) v = llg_act(a.act - 1, v);
+    if (a.out) a.out[(long long)token * a.channels + c] = v;
+    if (out2) out2[(long long)token * a.channels + c] = from_f32<O2>(v);
+  };
   if (p >= K - 1) {
     float acc = 0.f;
     for (int j = 0; j < K; ++j) acc = fmaf(w[j], input(p - (K - 1) + j), acc);
     acc += ob;
-    a.out[(long long)n * a.channels + c] = acc;
-    if (out2) out2[(long long)n * a.channels + c] = from_f32<O2>(acc);
+    put(n, acc);
     return;
   }
   // p == 0 and K >= 2: vals[0 .. K-2] the inputs before the step, vals[K-1 + q] the step's first ones
@@ -197,8 +201,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ConvArgs a) {
     float acc = 0.f;
     for (int j = 0; j < K; ++j) acc = fmaf(w[j], vals[q + j], acc);
     acc += ob;
-    a.out[(long long)(t0 + q) * a.channels + c] = acc;
-    if (out2) out2[(long long)(t0 + q) * a.channels + c] = from_f32<O2>(acc);
+    put(t0 + q, acc);
   }
   float fresh[LLG_CONV_MAX_TAPS];
   for (int s = 0; s < K - 1; ++s) {
@@ -232,6 +235,11 @@ __global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a) {
     return v + ib;
   };
   O2* out2 = (O2*)a.out2;
+  auto put = [&](int token, float v) {
+    if (a.act) v = llg_act(a.act - 1, v);
+    if (a.out) a.out[(long long)token * a.channels + c] = v;
+    if (out2) out2[(long long)token * a.channels + c] = from_f32<O2>(v);
+  };
   float win[K - 1];                                // win[d - 1]: the input of the token d before the current one
   int have = 0;                                    // how many of them are held
   const int n_last = n_first + CONV_RUN < a.n_tokens ? n_first + CONV_RUN : a.n_tokens;
@@ -258,8 +266,7 @@ __global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a) {
 #pragma unroll
           for (int j = 0; j < K; ++j) acc = fmaf(w[j], vals[q + j], acc);
           acc += ob;
-          a.out[(long long)(t0 + q) * a.channels + c] = acc;
-          if (out2) out2[(long long)(t0 + q) * a.channels + c] = from_f32<O2>(acc);
+          put(t0 + q, acc);
         }
       }
       float fresh[K - 1];
@@ -289,8 +296,7 @@ __global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a) {
       acc = fmaf(w[j], v, acc);
     }
     acc = fmaf(w[K - 1], x, acc) + ob;
-    a.out[(long long)n * a.channels + c] = acc;
-    if (out2) out2[(long long)n * a.channels + c] = from_f32<O2>(acc);
+    put(n, acc);
 #pragma unroll
     for (int d = K - 2; d > 0; --d) win[d] = win[d - 1];
     win[0] = x;
@@ -758,6 +764,8 @@ LLG_API int llg_causal_conv(const ConvArgs* args, cudaStream_t stream) {
   LLG_REQUIRE(a.n_seqs >= 0 && a.n_tokens >= 0 && a.channels > 0 && a.n_partials >= 1, "causal_conv: bad sizes");
   LLG_REQUIRE(a.taps >= 1 && a.taps <= LLG_CONV_MAX_TAPS, "causal_conv: %d taps (1 to %d)", a.taps, LLG_CONV_MAX_TAPS);
   LLG_REQUIRE(a.col0 >= 0 && a.col0 + a.channels <= a.row_width, "causal_conv: %d channels at column %d of %d", a.channels, a.col0, a.row_width);
+  LLG_REQUIRE(a.out || a.out2, "causal_conv: no output");
+  LLG_REQUIRE(a.act >= 0 && a.act <= 4, "causal_conv: unknown activation %d", a.act);
   LLG_REQUIRE(a.taps == 1 || a.state, "causal_conv: more than one tap needs the sequences' state");
   if (a.n_tokens == 0) return 0;
   dim3 grid(a.n_tokens, (a.channels + 127) / 128);

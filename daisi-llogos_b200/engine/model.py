@@ -28,6 +28,7 @@ from ..parts import norm as _norm  # noqa: F401
 from ..parts import position as _position  # noqa: F401
 from ..parts import recurrent as _recurrent  # noqa: F401
 from ..parts import sandwich as _sandwich  # noqa: F401
+from ..parts import state_space as _state_space  # noqa: F401
 
 
 EMBEDDING_UNIT = "embedding"      # the cache unit of an embedding that keeps state (schedule entries are numbered)

@@ -144,6 +144,7 @@ class _QkPrepArgs(Structure):
         ("n_tokens", c_int), ("nh", c_int), ("nkv", c_int), ("hd", c_int),
         ("row_scale", _RowScale),
         ("vd", c_int), ("v_mix", c_void_p), ("v_first_in", c_void_p), ("v_first_out", c_void_p), ("gate_out", c_void_p),
+        ("q_scale", c_void_p), ("q_scale_positions", c_int), ("q_maps", c_int),
     ]
 
 
@@ -157,6 +158,7 @@ class _PrefillArgs(Structure):
         ("scale", c_float), ("window", c_int), ("n_tokens", c_int), ("n_pages", c_int),
         ("vd", c_int), ("has_sink", c_int), ("sink_score", c_float), ("gate", c_void_p),
         ("sinks", c_void_p), ("chunked", c_int), ("softcap", c_float), ("head_mix", c_void_p),
+        ("out_f32", c_int), ("maps", c_int), ("map_lambda", c_float), ("map_eps", c_float), ("map_scale", c_float),
     ]
 
 
@@ -169,6 +171,7 @@ class _DecodeArgs(Structure):
         ("scale", c_float), ("window", c_int),
         ("vd", c_int), ("has_sink", c_int), ("sink_score", c_float), ("gate", c_void_p),
         ("sinks", c_void_p), ("chunked", c_int), ("softcap", c_float), ("head_mix", c_void_p),
+        ("out_f32", c_int),
     ]
 
 
@@ -199,7 +202,7 @@ class _DecodeTmaArgs(Structure):
         ("slots", c_void_p), ("len_before", c_void_p), ("part", c_void_p), ("counters", c_void_p), ("out", c_void_p),
         ("n_seqs", c_int), ("nh", c_int), ("nkv", c_int), ("hd", c_int), ("scale", c_float), ("window", c_int),
         ("has_sink", c_int), ("sink_score", c_float), ("gate", c_void_p),
-        ("sinks", c_void_p), ("chunked", c_int),
+        ("sinks", c_void_p), ("chunked", c_int), ("out_f32", c_int),
     ]
 
 
@@ -277,6 +280,7 @@ class _ConvArgs(Structure):
         ("in_bias", c_void_p), ("weight", c_void_p), ("bias", c_void_p), ("state", c_void_p),
         ("slots", c_void_p), ("cu_tokens", c_void_p), ("seq_of_token", c_void_p), ("len_before", c_void_p),
         ("out", c_void_p), ("out2", c_void_p), ("out2_dtype", c_int), ("n_seqs", c_int), ("n_tokens", c_int),
+        ("act", c_int),
     ]
 
 
@@ -304,7 +308,16 @@ class _RetentionArgs(Structure):
 
 class _RouterRule(Structure):
     _fields_ = [("score", c_int), ("groups", c_int), ("keep_groups", c_int), ("group_top", c_int), ("scale", c_float),
-                ("sum_eps", c_float), ("raw", c_int)]
+                ("sum_eps", c_float), ("raw", c_int), ("correction", c_void_p)]
+
+
+class _StateSpaceArgs(Structure):
+    _fields_ = [
+        ("mixed", c_void_p), ("mixed_dtype", c_int), ("rows", c_void_p), ("n_partials", c_int), ("partial_stride", c_longlong),
+        ("row_width", c_int), ("z_col", c_int), ("dt_col", c_int), ("dt_bias", c_void_p), ("a_log", c_void_p), ("d_skip", c_void_p),
+        ("state", c_void_p), ("slots", c_void_p), ("cu_tokens", c_void_p), ("out", c_void_p),
+        ("n_seqs", c_int), ("n_tokens", c_int), ("nh", c_int), ("groups", c_int), ("n_state", c_int), ("vdim", c_int), ("cols", c_int),
+    ]
 
 
 class _LatentPrepArgs(Structure):
@@ -394,7 +407,8 @@ def _load_lib(name: str):
         lib.llg_embed_rows.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
         lib.llg_embed_rows_copies.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_longlong, c_void_p]
         lib.llg_add_rmsnorm.argtypes = [c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_int, c_float,
-                                        c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p]
+                                        c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p]
+        lib.llg_map_difference.argtypes = [c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_void_p]
         lib.llg_qk_prep.argtypes = [POINTER(_QkPrepArgs), c_int, c_void_p]
         lib.llg_kv_write.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
                                      c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
@@ -456,6 +470,12 @@ def _load_lib(name: str):
         lib.llg_attn_decode_tma_scratch_floats.restype = c_longlong
         lib.llg_attn_decode_tma.argtypes = [POINTER(_DecodeTmaArgs), c_void_p, c_void_p, c_int, c_int, c_void_p]
         lib.llg_attn_decode_tma_status.restype = c_int
+    elif name == "state_space":
+        lib.llg_state_space_fits.argtypes = [c_int, c_int]
+        lib.llg_state_space_mma_fits.argtypes = [c_int, c_int]
+        lib.llg_state_space_walk.argtypes = [POINTER(_StateSpaceArgs), c_void_p]
+        lib.llg_state_space_mma.argtypes = [POINTER(_StateSpaceArgs), c_void_p]
+        lib.llg_part_rmsnorm.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]
     elif name == "layernorm":
         lib.llg_add_layernorm.argtypes = [POINTER(_LayerNormArgs), c_void_p]
     elif name == "groupnorm":
@@ -496,7 +516,7 @@ def _load_lib(name: str):
         lib.llg_moe_gather_rows.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p]
         lib.llg_grouped_linear.argtypes = [POINTER(_GroupedLinearArgs), c_int, c_int, c_void_p]
         lib.llg_moe_combine.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_int,
-                                        c_int, c_int, c_void_p]
+                                        c_int, c_int, c_void_p, c_int, c_void_p]
     elif name == "init":
         lib.llg_fill_normal.argtypes = [c_void_p, c_int, c_longlong, c_ulonglong, ctypes.c_double, ctypes.c_double, c_void_p]
         lib.llg_fill.argtypes = [c_void_p, c_int, c_longlong, c_float, c_void_p]
@@ -548,8 +568,9 @@ def embed_rows(table: torch.Tensor, token_ids: torch.Tensor, out_residual: torch
 
 
 def add_rmsnorm(residual: torch.Tensor, branch: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
-                out: torch.Tensor, rows: Optional[torch.Tensor] = None, ss_out: Optional[torch.Tensor] = None) -> None:
-    """residual += sum of branch partials (if any); out[j] = RMSNorm(residual[rows[j] or j]) * weight.
+                out: torch.Tensor, rows: Optional[torch.Tensor] = None, ss_out: Optional[torch.Tensor] = None,
+                branch_bias: Optional[torch.Tensor] = None) -> None:
+    """residual += sum of branch partials (if any) + ``branch_bias`` (float32 ``[H]``, if any); out[j] = RMSNorm(residual[rows[j] or j]) * weight.
 
     ``residual`` is float32 ``[N, H]``; ``branch`` float32 ``[S, N, H]`` or None; ``out`` ``[M, H]``.
     With ``ss_out`` (float32 ``[M, norm_ss_parts(M, H)]``) the division is left to whoever consumes ``out``: ``out[j]``
@@ -559,7 +580,7 @@ def add_rmsnorm(residual: torch.Tensor, branch: Optional[torch.Tensor], weight: 
     lib = _lib("elementwise")
     n, hidden = residual.shape
     m = out.shape[0]
-    assert out.shape[1] == hidden and weight.shape == (hidden,)
+    assert out.shape[1] == hidden and weight.shape == (hidden,) and (branch_bias is None or branch_bias.shape == (hidden,))
     if rows is not None:
         assert rows.numel() == m
     else:
@@ -572,7 +593,8 @@ def add_rmsnorm(residual: torch.Tensor, branch: Optional[torch.Tensor], weight: 
         n_part, stride = branch.shape[0], n * hidden
     _check(lib, lib.llg_add_rmsnorm(_ptr(residual, torch.float32), _ptr(branch, torch.float32), n_part, stride,
                                     _ptr(weight), _dt(weight), float(eps), _ptr(out), _dt(out),
-                                    _ptr(rows, torch.int32), m, hidden, _ptr(ss_out, torch.float32), _stream()))
+                                    _ptr(rows, torch.int32), m, hidden, _ptr(ss_out, torch.float32),
+                                    _ptr(branch_bias, torch.float32), _stream()))
 
 
 _ss_parts = {}
@@ -692,7 +714,7 @@ def qk_prep(qkv: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim: int,
             seq_of_token: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
             row_scale: Optional[RowScale] = None, value_dim: int = 0, v_mix: Optional[torch.Tensor] = None,
             v_first_in: Optional[torch.Tensor] = None, v_first_out: Optional[torch.Tensor] = None,
-            gate_out: Optional[torch.Tensor] = None) -> None:
+            gate_out: Optional[torch.Tensor] = None, q_scale: Optional[torch.Tensor] = None, q_maps: int = 0) -> None:
     """Per-head norm (optional), bias (optional), rotation, and the writes of q, k, v.
 
     ``qkv`` is ``[S, N, (nh + nkv) * hd + nkv * vd]`` (partials are summed; ``vd = value_dim or hd``).  Queries go to
@@ -701,7 +723,9 @@ def qk_prep(qkv: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim: int,
     partials are multiplied by it before anything else.  Values blended across layers: ``v_first_out`` (float32
     ``[N, nkv, vd]``) receives the values as projected; with ``v_first_in`` and ``v_mix`` (one float32 number lam on the
     device) the values written are ``(1 - lam) v + lam v_first_in``.  ``gate_out`` (float32 ``[N, nh]``): the rows of ``qkv`` end
-    with one more number z per query head, and ``gate_out`` receives ``sigmoid(z)``.
+    with one more number z per query head, and ``gate_out`` receives ``sigmoid(z)``.  ``q_scale`` (float32, a number per
+    position): queries are multiplied by their position's.  ``q_maps`` 2: ``q_out`` is ``[N, 2 nh, hd]``, a query head's two
+    halves as two heads with zeros in the other half's place.
     """
     lib = _lib("elementwise")
     s, n, width = qkv.shape
@@ -720,8 +744,16 @@ def qk_prep(qkv: torch.Tensor, *, n_heads: int, n_kv_heads: int, head_dim: int,
     a.v_mix, a.v_first_in = _ptr(v_mix, torch.float32), _ptr(v_first_in, torch.float32)
     a.v_first_out = _ptr(v_first_out, torch.float32)
     a.gate_out = _ptr(gate_out, torch.float32)
+    assert q_out.shape == (n, n_heads * (q_maps or 1), head_dim), q_out.shape
+    a.q_maps = q_maps
+    _set_q_scale(a, q_scale)
     _set_scale(a, row_scale, n)
     _check(lib, lib.llg_qk_prep(byref(a), _dt(q_out), _stream()))
+
+
+def _set_q_scale(a: "_QkPrepArgs", q_scale: Optional[torch.Tensor]) -> None:
+    if q_scale is not None:
+        a.q_scale, a.q_scale_positions = _ptr(q_scale, torch.float32), q_scale.numel()
 
 
 def _set_scale(a: "_QkPrepArgs", row_scale: Optional[RowScale], n: int) -> None:
@@ -782,7 +814,7 @@ def gemm_tc_qkv(x: torch.Tensor, w: torch.Tensor, *, n_heads: int, n_kv_heads: i
                 k_pages: Optional[torch.Tensor] = None, v_pages: Optional[torch.Tensor] = None,
                 page_table: Optional[torch.Tensor] = None, ring_pages: int = 0,
                 seq_of_token: Optional[torch.Tensor] = None, slots: Optional[torch.Tensor] = None,
-                row_scale: Optional[RowScale] = None) -> None:
+                row_scale: Optional[RowScale] = None, q_scale: Optional[torch.Tensor] = None) -> None:
     """The q/k/v projection ``x w^T`` on the tensor cores with ``qk_prep`` as its epilogue (one kernel; the float32
     q/k/v array is never written).  Same arguments and results as ``gemm_tc`` followed by ``qk_prep``."""
     lib = _lib("gemm_tc")
@@ -790,6 +822,7 @@ def gemm_tc_qkv(x: torch.Tensor, w: torch.Tensor, *, n_heads: int, n_kv_heads: i
     assert w.shape == ((n_heads + 2 * n_kv_heads) * head_dim, k) and q_out.dtype == torch.bfloat16
     a = _prep_args(n, n_heads, n_kv_heads, head_dim, q_norm_w, k_norm_w, norm_eps, bias, cos, sin, rotary_dim, pairing,
                    positions, q_out, k_new, v_new, k_pages, v_pages, page_table, ring_pages, seq_of_token, slots)
+    _set_q_scale(a, q_scale)
     _set_scale(a, row_scale, n)
     _check(lib, lib.llg_gemm_tc_qkv(_ptr(x, torch.bfloat16), _ptr(w, torch.bfloat16), n, k, byref(a), _stream()))
 
@@ -1136,18 +1169,18 @@ def retention_supported(dim: int, vdim: int) -> bool:
 
 
 def causal_conv(rows: torch.Tensor, col0: int, weight: torch.Tensor, state: Optional[torch.Tensor], slots: torch.Tensor,
-                cu_tokens: torch.Tensor, seq_of_token: torch.Tensor, len_before: torch.Tensor, out: torch.Tensor,
+                cu_tokens: torch.Tensor, seq_of_token: torch.Tensor, len_before: torch.Tensor, out: Optional[torch.Tensor],
                 in_bias: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
-                out2: Optional[torch.Tensor] = None) -> None:
+                out2: Optional[torch.Tensor] = None, act: Optional[str] = None) -> None:
     """A causal convolution per channel along every sequence of a step.  The inputs are the ``C`` columns from ``col0`` of
     float32 partials ``rows`` ``[P, N, width]``, plus ``in_bias``; ``out[n, c] = sum_j weight[c, j] * input(position - K + 1 + j)
     + bias[c]`` (``weight`` float32 ``[C, K]``; zeros before a sequence's start).  ``state`` float32 ``[slots, K - 1, C]`` holds a
-    sequence's last ``K - 1`` inputs before the step and receives those after it.  ``out`` float32 ``[N, C]``; ``out2``: the
-    same once more in another type."""
+    sequence's last ``K - 1`` inputs before the step and receives those after it.  ``out`` float32 ``[N, C]`` (None: only ``out2`` is
+    wanted); ``out2``: the same once more in another type.  ``act``: an activation of ``ACTIVATIONS`` on what is written."""
     lib = _lib("recurrent")
     p_n, n, width = rows.shape
     c, k = weight.shape
-    assert out.shape == (n, c) and (out2 is None or out2.shape == (n, c))
+    assert (out is not None or out2 is not None) and all(t is None or t.shape == (n, c) for t in (out, out2))
     assert k == 1 or (state is not None and state.shape[1:] == (k - 1, c)), "the state holds taps - 1 rows of inputs"
     a = _ConvArgs()
     a.rows, a.n_partials, a.partial_stride = _ptr(rows, torch.float32), p_n, n * width
@@ -1159,6 +1192,7 @@ def causal_conv(rows: torch.Tensor, col0: int, weight: torch.Tensor, state: Opti
     a.out, a.out2 = _ptr(out, torch.float32), _ptr(out2)
     a.out2_dtype = _dt(out2) if out2 is not None else F32
     a.n_seqs, a.n_tokens = slots.numel(), n
+    a.act = 1 + ACTIVATIONS[act] if act is not None else 0
     _check(lib, lib.llg_causal_conv(byref(a), _stream()))
 
 
@@ -1395,14 +1429,23 @@ class RouterRule:
     the sigmoid scores are.  "sigmoid": scores ``s = sigmoid(logit)``; with ``groups`` the experts form that many equal groups of
     neighbours, a group is judged by the sum of its ``group_score_top`` largest scores and only the ``keep_groups`` best
     groups' experts can be chosen; the ``top`` largest eligible scores, ``weight = s / (sum of the chosen + weight_sum_eps) *
-    weight_scale``.  ``normalize`` False: ``weight = s * weight_scale`` instead."""
+    weight_scale``.  ``normalize`` False: ``weight = s * weight_scale`` instead.  Groups may also
+    go with "softmax_all".  ``correction`` (float32 ``[experts]`` on the device): groups are judged and experts chosen by ``s +
+    correction``, the weights are made of ``s``."""
 
     def __init__(self, score: str = "softmax", groups: int = 0, keep_groups: int = 0, group_score_top: int = 2,
-                 weight_scale: float = 1.0, weight_sum_eps: float = 0.0, normalize: bool = True):
+                 weight_scale: float = 1.0, weight_sum_eps: float = 0.0, normalize: bool = True,
+                 correction: Optional[torch.Tensor] = None):
         if score not in ROUTER_SCORES:
             raise KernelError(f"router rule: score '{score}' is not known ({', '.join(ROUTER_SCORES)})")
         self.c = _RouterRule(ROUTER_SCORES[score], int(groups), int(keep_groups), int(group_score_top),
-                             float(weight_scale), float(weight_sum_eps), int(not normalize))
+                             float(weight_scale), float(weight_sum_eps), int(not normalize), _ptr(correction, torch.float32))
+        self.correction = correction              # keeps the tensor alive
+
+
+def _check_rule(rule: Optional["RouterRule"], n_exp: int) -> None:
+    if rule is not None and rule.correction is not None and rule.correction.numel() != n_exp:
+        raise KernelError(f"router rule: a correction of {rule.correction.numel()} numbers for {n_exp} experts")
 
 
 def _rule_ref(rule: Optional["RouterRule"]):
@@ -1421,6 +1464,7 @@ def moe_route(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional[torch.
     n_exp = w_router.shape[0] - (1 if extra_out is not None else 0)
     assert w_router.shape[1] == hidden and choice.shape == (n, top) and weight.shape == (n, top)
     assert b_router is None or b_router.shape == (n_exp,)
+    _check_rule(rule, n_exp)
     assert extra_out is None or extra_out.shape == (n,)
     _check(lib, lib.llg_moe_route(_ptr(x), _dt(x), _ptr(w_router, torch.float32), _ptr(b_router, torch.float32),
                                   _ptr(choice, torch.int32), _ptr(weight, torch.float32), n, hidden, n_exp, top,
@@ -1436,6 +1480,7 @@ def moe_topk(logits: torch.Tensor, b_router: Optional[torch.Tensor], choice: tor
     n_exp = width - (1 if extra_out is not None else 0)
     top = choice.shape[1]
     assert choice.shape == (n, top) and weight.shape == (n, top) and (b_router is None or b_router.shape == (n_exp,))
+    _check_rule(rule, n_exp)
     assert extra_out is None or extra_out.shape == (n,)
     _check(lib, lib.llg_moe_topk(_ptr(logits, torch.float32), s, n * width, _ptr(b_router, torch.float32),
                                  _ptr(choice, torch.int32), _ptr(weight, torch.float32), n, n_exp, top,
@@ -1449,7 +1494,8 @@ def moe_plan(choice: torch.Tensor, n_experts: int, row_of_pair: torch.Tensor, to
     filled up to whole tiles of ``MOE_TILE_ROWS``: ``row_of_pair[n * top + k]`` the pair's row, ``token_of_row[r]`` the
     row's token (-1: a filling row), ``tile_expert[t]`` the expert of tile t (-1: unused).  ``token_of_row`` has
     ``moe_row_capacity(N * top, n_experts, tile)`` entries and ``tile_expert`` one per tile: their sizes say which tile
-    size is meant.  With ``weight`` ``[N, top]``, ``weight_of_row`` receives every row's pair's weight (0 for filling rows)."""
+    size is meant.  With ``weight`` ``[N, top]``, ``weight_of_row`` receives every row's pair's weight (0 for filling rows).
+    A choice that is not below ``n_experts`` (an identity expert) gets no row: its ``row_of_pair`` is -1."""
     lib = _moe_lib()
     n, top = choice.shape
     cap = token_of_row.numel()
@@ -1539,9 +1585,10 @@ def moe_down(act: torch.Tensor, tile_expert: torch.Tensor, w_down: torch.Tensor,
 
 
 def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, weight: Optional[torch.Tensor], shared: Optional[torch.Tensor],
-                out: torch.Tensor, shared_scale: Optional[torch.Tensor] = None) -> None:
+                out: torch.Tensor, shared_scale: Optional[torch.Tensor] = None, identity: Optional[torch.Tensor] = None) -> None:
     """out[n] = sum_k weight[n, k] y[row_of_pair[n * top + k]] (``weight`` None: every row counts once) + the sum of ``shared``'s partials ``[S, N, H]`` (if any),
-    that sum times ``shared_scale[n]`` where given (float32 ``[N]``)."""
+    that sum times ``shared_scale[n]`` where given (float32 ``[N]``).  A pair without a row (``row_of_pair`` -1) stands for
+    ``identity[n]`` (``[N, H]``, the mixture's own input), or for nothing without it."""
     lib = _moe_lib()
     n, hidden = out.shape
     top = row_of_pair.numel() // max(n, 1)
@@ -1551,9 +1598,11 @@ def moe_combine(y: torch.Tensor, row_of_pair: torch.Tensor, weight: Optional[tor
         assert shared.dim() == 3 and shared.shape[1:] == (n, hidden)
         n_shared = shared.shape[0]
     assert shared_scale is None or (shared is not None and shared_scale.shape == (n,))
+    assert identity is None or identity.shape == (n, hidden)
     _check(lib, lib.llg_moe_combine(_ptr(y, torch.float32), _ptr(row_of_pair, torch.int32), _ptr(weight, torch.float32),
                                     _ptr(shared, torch.float32), n_shared, n * hidden, _ptr(shared_scale, torch.float32),
-                                    _ptr(out, torch.float32), n, hidden, top, _stream()))
+                                    _ptr(out, torch.float32), n, hidden, top, _ptr(identity),
+                                    _dt(identity) if identity is not None else F32, _stream()))
 
 
 ACTIVATIONS = {"relu2": 0, "gelu_tanh": 1, "silu": 2, "relu": 3}
@@ -1689,11 +1738,12 @@ class AttentionForm:
     c)``), ``head_mix`` (a float32 tensor ``[nh, nh]`` on the device: behind the cap, head h's scores become ``sum_g
     head_mix[h, g] s_g``).  The last two run on kernels of their own (csrc/attention_mix_mma.cu on the tensor cores,
     csrc/attention_mix.cu on the CUDA cores): a block then works on all
-    query heads of its queries."""
+    query heads of its queries.  ``maps`` (a ``MapDifference``): a query head and a key head hold two maps, half of their elements
+    each, that attend to the same values; see ``maps_in_kernel`` for who takes the difference of the two outputs."""
 
     def __init__(self, value_dim: int = 0, sink: Optional[float] = None, gated: bool = False,
                  sinks: Optional[torch.Tensor] = None, chunked: bool = False, softcap: float = 0.0,
-                 head_mix: Optional[torch.Tensor] = None):
+                 head_mix: Optional[torch.Tensor] = None, maps: Optional["MapDifference"] = None):
         self.value_dim, self.sink, self.gated = int(value_dim), (None if sink is None else float(sink)), bool(gated)
         if sinks is not None and (sinks.dtype != torch.float32 or sinks.dim() != 1):
             raise KernelError("AttentionForm: per-head sinks are a float32 vector [query heads]")
@@ -1704,6 +1754,9 @@ class AttentionForm:
         if head_mix is not None and (head_mix.dtype != torch.float32 or head_mix.dim() != 2 or head_mix.shape[0] != head_mix.shape[1]):
             raise KernelError("AttentionForm: the mix of the heads' scores is a float32 matrix [query heads, query heads]")
         self.head_mix = head_mix
+        self.maps = maps
+        if maps is not None and (self.mixes or self.gated or sink is not None or sinks is not None):
+            raise KernelError("AttentionForm: two maps go with neither capped or mixed scores nor sinks nor gates")
 
     @property
     def mixes(self) -> bool:
@@ -1712,7 +1765,7 @@ class AttentionForm:
 
     def plain(self, head_dim: int) -> bool:
         return (self.value_dim in (0, head_dim) and self.sink is None and self.sinks is None and not self.gated
-                and not self.chunked and not self.mixes)
+                and not self.chunked and not self.mixes and self.maps is None)
 
     def one_head_size(self, head_dim: int) -> bool:
         """Keys and values of one head size: what the tensor-core kernels take (sink and gate they all apply)."""
@@ -1723,6 +1776,31 @@ class AttentionForm:
 
 
 PLAIN_ATTENTION = AttentionForm()
+
+
+class MapDifference:
+    """What becomes of the outputs ``a1``, ``a2`` of an attention's two maps: ``o = a1 - lam a2``, divided by ``sqrt(mean(o^2) + eps)``
+    over a head's values and multiplied by ``scale``."""
+
+    def __init__(self, lam: float, eps: float, scale: float):
+        self.lam, self.eps, self.scale = float(lam), float(eps), float(scale)
+        if not self.eps > 0:
+            raise KernelError("MapDifference: eps must be positive")
+
+
+def maps_in_kernel(dtype: torch.dtype, head_dim: int, form: AttentionForm) -> bool:
+    """Whether the prompt attention kernel itself takes two maps (``form.maps``): queries ``[N, nh, head_dim]`` as they are, finished
+    output ``[N, nh * vd]``.  Otherwise, and in decode steps, the caller gives the maps as heads of their own (``qk_prep(...,
+    q_maps=2)``), gets float32 ``[N, 2 nh * vd]`` and calls ``map_difference``."""
+    return _prefill_kernel(dtype, head_dim, form) == "tc"
+
+
+def map_difference(raw: torch.Tensor, out: torch.Tensor, maps: MapDifference) -> None:
+    """out[n, h] = the ``MapDifference`` of ``raw[n, h, 0]`` and ``raw[n, h, 1]``; ``raw`` float32 ``[N, nh, 2, vd]``, ``out`` ``[N, nh * vd]``."""
+    lib = _lib("elementwise")
+    n, nh, two, vd = raw.shape
+    assert two == 2 and out.shape == (n, nh * vd)
+    _check(lib, lib.llg_map_difference(_ptr(raw, torch.float32), _ptr(out), _dt(out), n, nh, vd, maps.lam, maps.eps, maps.scale, _stream()))
 
 
 def _prefill_kernel(dtype: torch.dtype, head_dim: int, form: AttentionForm) -> str:
@@ -1741,6 +1819,8 @@ USE_MIX_MMA = True           # tests switch it off to reach the CUDA-core kernel
 
 def prefill_tile_queries(dtype: torch.dtype, head_dim: int, form: AttentionForm = PLAIN_ATTENTION) -> int:
     """Queries per block of the prompt attention kernel that ``attn_prefill`` will run."""
+    if form.maps is not None and _prefill_kernel(dtype, head_dim, form) == "tc":
+        return 128                   # the kernel's two tiles of 128 queries are the two maps of one
     return {"tc": 256, "mma": 64, "simt": 16, "mix": MIX_TILE_QUERIES}[_prefill_kernel(dtype, head_dim, form)]
 
 
@@ -1748,6 +1828,7 @@ def _set_form(a, form: AttentionForm, head_dim: int, gate: Optional[torch.Tensor
     """The fields of a prompt or decode argument block that say which form of attention is wanted."""
     a.vd = 0 if form.value_dim in (0, head_dim) else form.value_dim
     a.softcap = form.softcap
+    a.out_f32 = int(form.maps is not None)
     if form.head_mix is not None:
         if form.head_mix.shape[0] != a.nh:
             raise KernelError(f"attention: a mix of {form.head_mix.shape[0]} heads' scores for {a.nh} query heads")
@@ -1780,7 +1861,7 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
     the tensor cores: head sizes 64 and 128 with tcgen05 (csrc/attention_tc.cu), other multiples of 16 up
     to 128 with mma.sync (csrc/attention_mma.cu); everything else on the CUDA cores
     (csrc/attention_simt.cu).  ``form`` (an ``AttentionForm``) and ``gate`` ask for values of another head size, a
-    sink and gated heads; ``out`` is then ``[N, nh * value_dim]``.
+    sink and gated heads; ``out`` is then ``[N, nh * value_dim]``.  With ``form.maps``: ``maps_in_kernel``.
     """
     n, nh, hd = q.shape
     nkv = k_new.shape[1]
@@ -1803,11 +1884,14 @@ def attn_prefill(q, k_new, v_new, k_pages, v_pages, page_table, ring_pages, tile
     a.page_table, a.table_width, a.ring_pages = _ptr(page_table, torch.int32), page_table.shape[1], ring_pages
     a.tiles, a.cu_tokens = _ptr(tiles, torch.int32), _ptr(cu_tokens, torch.int32)
     a.len_before, a.slots = _ptr(len_before, torch.int32), _ptr(slots, torch.int32)
-    a.out = _ptr(out, q.dtype)
+    own_maps = form.maps is not None and _prefill_kernel(q.dtype, hd, form) == "tc"
+    a.out = _ptr(out, torch.float32 if form.maps is not None and not own_maps else q.dtype)
     a.n_tiles, a.nh, a.nkv, a.hd = tiles.shape[0], nh, nkv, hd
     a.scale, a.window = float(scale), int(window)
     a.n_tokens, a.n_pages = k_new.shape[0], k_pages.shape[0]
     _set_form(a, form, hd, gate)
+    if own_maps:
+        a.out_f32, a.maps, a.map_lambda, a.map_eps, a.map_scale = 0, 2, form.maps.lam, form.maps.eps, form.maps.scale
     if mix_mma:
         _check(lib, lib.llg_attn_mix_prefill_mma(byref(a), tile_queries, _stream()))
     elif kernel == "mix":
@@ -1829,6 +1913,49 @@ def _use_tma_decode(dtype: torch.dtype, head_dim: int, n_heads: int, n_kv_heads:
     """bfloat16 decode attention with a geometry the TMA kernel takes (csrc/attention_decode_tma.cu)."""
     return (USE_TMA_DECODE_ATTENTION and dtype == torch.bfloat16 and head_dim in (64, 128) and n_kv_heads > 0
             and n_heads % n_kv_heads == 0 and n_heads // n_kv_heads <= 8 and n_seqs <= 1024)
+
+
+STATE_SPACE_MMA_TOKENS = 16      # steps whose longest sequence brings fewer tokens take the walk also in bfloat16
+USE_STATE_SPACE_MMA = True       # tests switch it off to reach the walk with many tokens
+
+
+def state_space_supported(n_state: int, vdim: int) -> bool:
+    """Whether a head's state of ``n_state`` x ``vdim`` numbers fits the blocks of the state-space walk."""
+    return bool(_lib("state_space").llg_state_space_fits(n_state, vdim))
+
+
+def state_space(mixed: torch.Tensor, rows: torch.Tensor, *, z_col: int, dt_col: int, dt_bias: torch.Tensor, a_log: torch.Tensor,
+                d_skip: torch.Tensor, n_heads: int, groups: int, n_state: int, vdim: int, state: torch.Tensor, slots: torch.Tensor,
+                cu_tokens: torch.Tensor, out: torch.Tensor, max_count: int) -> None:
+    """``S <- exp(-exp(a_log) d) S + d B x^T`` and ``out = (S^T C + d_skip x) silu(z)`` per head along every sequence of a step, with ``d =
+    softplus(dt + dt_bias)``.  ``mixed`` ``[N, nh * vdim + 2 * groups * n_state]`` holds x, B and C (head h reads group ``h // (nh /
+    groups)``); ``rows`` (float32 partials ``[P, N, width]``) the columns of z from ``z_col`` (negative: no gate) and of dt from
+    ``dt_col``; ``state`` float32 ``[slots, nh, n_state, vdim]``; ``out`` float32 ``[N, nh * vdim]``.  Steps of several tokens in bfloat16
+    run in chunks on the tensor cores, everything else walks token by token."""
+    lib = _lib("state_space")
+    p_n, n, width = rows.shape
+    assert mixed.shape == (n, n_heads * vdim + 2 * groups * n_state) and out.shape == (n, n_heads * vdim)
+    assert state.shape[1:] == (n_heads, n_state, vdim) and all(t.shape == (n_heads,) for t in (dt_bias, a_log, d_skip))
+    a = _StateSpaceArgs()
+    a.mixed, a.mixed_dtype = _ptr(mixed), _dt(mixed)
+    a.rows, a.n_partials, a.partial_stride = _ptr(rows, torch.float32), p_n, n * width
+    a.row_width, a.z_col, a.dt_col = width, int(z_col), int(dt_col)
+    a.dt_bias, a.a_log, a.d_skip = _ptr(dt_bias, torch.float32), _ptr(a_log, torch.float32), _ptr(d_skip, torch.float32)
+    a.state, a.slots, a.cu_tokens = _ptr(state, torch.float32), _ptr(slots, torch.int32), _ptr(cu_tokens, torch.int32)
+    a.out = _ptr(out, torch.float32)
+    a.n_seqs, a.n_tokens, a.nh, a.groups, a.n_state, a.vdim = slots.numel(), n, n_heads, groups, n_state, vdim
+    mma = (USE_STATE_SPACE_MMA and mixed.dtype == torch.bfloat16 and max_count >= STATE_SPACE_MMA_TOKENS
+           and lib.llg_state_space_mma_fits(n_state, vdim))
+    _check(lib, (lib.llg_state_space_mma if mma else lib.llg_state_space_walk)(byref(a), _stream()))
+
+
+def part_rmsnorm(x: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, out: torch.Tensor) -> None:
+    """out[n] = x[n] with each of ``parts`` equal parts divided by its own root mean square, times ``weight`` (float32)."""
+    lib = _lib("state_space")
+    n, width = x.shape
+    assert out.shape == (n, width) and weight.shape == (width,)
+    _check(lib, lib.llg_part_rmsnorm(_ptr(x, torch.float32), _ptr(weight, torch.float32), _ptr(out), _dt(out), n, width, int(parts), float(eps),
+                                     _stream()))
 
 
 class DecodePlan:
@@ -1948,6 +2075,7 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
     if not form.one_head_size(hd) and plan is not None and plan.kind not in ("simt", "mix", "mix_mma"):
         raise KernelError(f"attn_decode: the {plan.kind} kernel takes keys and values of one head size")
     assert out.shape == (b, nh * vd) and v_pages.shape[3] == vd
+    out_dtype = torch.float32 if form.maps is not None else q.dtype        # two maps: the caller takes their difference
     if plan is not None and plan.kind == "tma":
         lib = _lib("attention_decode_tma")
         if scratch.numel() < plan.scratch_floats:
@@ -1958,7 +2086,8 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         a.q = _ptr(q, torch.bfloat16)
         a.page_table, a.table_width, a.ring_pages = _ptr(page_table, torch.int32), page_table.shape[1], ring_pages
         a.slots, a.len_before = _ptr(slots, torch.int32), _ptr(len_before, torch.int32)
-        a.part, a.counters, a.out = _ptr(scratch), _ptr(counters, torch.int32), _ptr(out, torch.bfloat16)
+        a.part, a.counters = _ptr(scratch), _ptr(counters, torch.int32)
+        a.out, a.out_f32 = _ptr(out, out_dtype), int(form.maps is not None)
         a.n_seqs, a.nh, a.nkv, a.hd = b, nh, nkv, hd
         a.scale, a.window = float(scale), int(window)
         _set_sink(a, form)
@@ -1987,7 +2116,7 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
     if mma:
         if counters is None or counters.numel() < b * nkv:
             raise KernelError(f"attn_decode: needs {b * nkv} zeroed int32 counters")
-        _check(lib, lib.llg_attn_decode_mma(byref(a), _ptr(out, q.dtype), _ptr(counters, torch.int32),
+        _check(lib, lib.llg_attn_decode_mma(byref(a), _ptr(out, out_dtype), _ptr(counters, torch.int32),
                                             int(bool(balance) and b * nkv <= attn_decode_balance_pairs() and b <= 32), _stream()))
     elif mix_mma:
         if scratch.numel() < plan.scratch_floats:
@@ -1997,12 +2126,12 @@ def attn_decode(q, k_pages, v_pages, page_table, ring_pages, slots, len_before, 
         at = -(-need // 4) * 4                               # every part starts on 16 bytes
         at_w = at + -(-n_scores // 4) * 4
         at_c = at_w + -(-n_weights // 4) * 4
-        _check(lib, lib.llg_attn_mix_decode_mma(byref(a), _ptr(out, q.dtype), base + 4 * at, base + 4 * at_w, base + 4 * at_c, keys, _stream()),
+        _check(lib, lib.llg_attn_mix_decode_mma(byref(a), _ptr(out, out_dtype), base + 4 * at, base + 4 * at_w, base + 4 * at_c, keys, _stream()),
                kernels=4)
     elif form.mixes:
-        _check(lib, lib.llg_attn_mix_decode_simt(byref(a), _ptr(out, q.dtype), _dt(q), _stream()), kernels=2)
+        _check(lib, lib.llg_attn_mix_decode_simt(byref(a), _ptr(out, out_dtype), _dt(q), _stream()), kernels=2)
     else:
-        _check(lib, lib.llg_attn_decode_simt(byref(a), _ptr(out, q.dtype), _dt(q), _stream()), kernels=2)
+        _check(lib, lib.llg_attn_decode_simt(byref(a), _ptr(out, out_dtype), _dt(q), _stream()), kernels=2)
 
 
 def fill_normal(out: torch.Tensor, key: int, mean: float, std: float) -> None:

@@ -102,7 +102,9 @@ def model_costs(model) -> ModelCosts:
             kv.append((need.num_kv_heads * (need.head_dim + values) * elem, need.window))
         for part in block.parts.values():
             nh, hd = getattr(part, "nh", None), getattr(part, "hd", None) or getattr(part, "kd", None)
-            if nh and hd and getattr(part, "SCORES_PAIRS", True):
+            if hasattr(part, "flops_per_pair"):
+                attn += part.flops_per_pair()
+            elif nh and hd and getattr(part, "SCORES_PAIRS", True):
                 attn += 2 * nh * (hd + (getattr(part, "vd", None) or hd))
     return ModelCosts(matrix, head, elem, tuple(kv), attn, active)
 

@@ -15,6 +15,15 @@ value, not scaled); and values blended across layers: the first layer of a group
 (float32, per step) to the others, which cache ``(1 - lam) v + lam v_first`` with a learned number ``lam`` each.  Ahead of
 the softmax the scaled scores may pass a cap ``c tanh(s / c)`` and then be mixed over the heads, ``s'_h = sum_g T[h, g] s_g``;
 every head's output may be multiplied by one number ``sigmoid(w_h . x)`` from the mixer's own input.
+
+Differential attention (``maps`` 2): a query head and a key head hold two maps of ``head_dim`` elements, one behind the other,
+each with a softmax of its own over the same values.  With their outputs a1, a2 and one number for the layer, ``lam = exp(lq1 .
+lk1) - exp(lq2 . lk2) + diff``, a head's output is ``o = a1 - lam a2`` divided by its root mean square over the values (no weight),
+times ``1 - diff``.  The cache keeps a key head's two maps as one row of ``2 head_dim`` elements and its values once.  A prompt
+step on the tcgen05 kernel runs both maps in one block, which also takes the difference; the other kernels get the maps as two
+query heads with zeros in the other map's half, leave float32 outputs, and ``ops.map_difference`` follows: a decode step then
+reads keys and values once for both maps.  Queries may be multiplied by a number per position (``q_scale``), and the output projection may have
+a bias, which enters the residual with the projection's partial sums (``Branch.bias``).
 """
 from __future__ import annotations
 
@@ -39,7 +48,10 @@ class Attention(Mixer):
     keys and values), out_gate (False, or True: the concatenated heads are multiplied by ``sigmoid(g_proj x)`` before
     the output projection; a tensor ``g_proj.weight`` [num_heads * value_dim, hidden]), head_gate (bool: one gate per query
     head instead, a tensor ``gate_proj.weight`` [num_heads, hidden]; its rows ride in the projections' product and the
-    attention kernel applies it), softcap (0: none), head_mix (bool: a tensor ``head_mix.weight`` [num_heads, num_heads])."""
+    attention kernel applies it), softcap (0: none), head_mix (bool: a tensor ``head_mix.weight`` [num_heads, num_heads]),
+    out_bias (bool: a tensor ``o_proj.bias`` [hidden]), q_scale (None, or the name of a position encoding that gives queries a factor
+    per position), maps (0, or 2 with ``diff`` and ``diff_eps``: q_proj and k_proj then have two maps of head_dim rows per head, and there
+    are tensors ``lq1``, ``lk1``, ``lq2``, ``lk2`` [head_dim])."""
 
     TAKES_ROW_SCALE = True
 
@@ -49,13 +61,18 @@ class Attention(Mixer):
         self.hidden = int(p["hidden_size"])
         self.nh = int(p["num_heads"])
         self.nkv = int(p["num_kv_heads"])
-        self.hd = int(p["head_dim"])
+        self.maps = int(p.get("maps", 0) or 0)
+        if self.maps not in (0, 2):
+            raise ValueError(f"attention: {self.maps} maps (none or 2)")
+        self.map_dim = int(p["head_dim"])
+        self.hd = self.map_dim * (self.maps or 1)            # elements of a query or key head, all its maps
         if self.nh % self.nkv:
             raise ValueError(f"{self.nh} heads are not a multiple of {self.nkv} key/value heads")
         # said when the model is built, not at its first step
         limit = getattr(env.ops, "ATTN_MAX_HEAD_DIM", None)
         if limit is not None and not 0 < self.hd <= limit:
-            raise ValueError(f"head_dim {self.hd}: the attention kernels take head sizes from 1 to {limit}")
+            raise ValueError(f"head_dim {self.hd}: the attention kernels take head sizes from 1 to {limit}"
+                             + (f" (two maps of {self.map_dim} elements)" if self.maps else ""))
         self.qkv_bias = bool(p.get("qkv_bias", False))
         self.qk_norm = bool(p.get("qk_norm", False))
         self.qk_norm_eps = float(p.get("qk_norm_eps", 1e-6))
@@ -96,7 +113,16 @@ class Attention(Mixer):
                              f"kernels for capped and mixed scores take")
         self.own_form = (self.vd != self.hd or self.mask != "window" or self.sink_kind is not None or self.head_gate
                          or self.softcap > 0 or self.head_mix)
-        self.special = self.own_form or bool(self.conv_taps) or self.out_gate
+        self.out_bias = bool(p.get("out_bias", False))
+        self.q_scale = env.encodings[p["q_scale"]] if p.get("q_scale") is not None else None
+        self.diff = self.diff_eps = 0.0
+        if self.maps:
+            if self.softcap or self.head_mix or self.head_gate or self.sink_kind is not None or self.conv_taps or not self.own_kv:
+                raise ValueError("attention: two maps go with plain scores, without sinks, gates per head, convolutions or a borrowed cache")
+            self.diff, self.diff_eps = float(p["diff"]), float(p["diff_eps"])
+        self.own_form = self.own_form or bool(self.maps)
+        self.special = self.own_form or bool(self.conv_taps) or self.out_gate or self.out_bias or self.q_scale is not None
+        self.b_o = None
         self.w_gate = self.w_conv = None
         if self.conv_taps:
             self.TAKES_ROW_SCALE = False      # the convolution mixes rows: every row arrives finished
@@ -138,6 +164,10 @@ class Attention(Mixer):
             t["gate_proj.weight"] = TensorDecl((self.nh, self.hidden))
         if self.head_mix:
             t["head_mix.weight"] = TensorDecl((self.nh, self.nh), "stream_mix")
+        if self.out_bias:
+            t["o_proj.bias"] = TensorDecl((self.hidden,), "bias")
+        if self.maps:
+            t.update({name: TensorDecl((self.map_dim,), "bias") for name in ("lq1", "lk1", "lq2", "lk2")})
         return t
 
     def bind(self, tensors):
@@ -175,8 +205,13 @@ class Attention(Mixer):
             mix = {}
             if self.softcap > 0 or self.head_mix:
                 mix = dict(softcap=self.softcap, head_mix=as_f32(tensors["head_mix.weight"], self.env) if self.head_mix else None)
+            if self.maps:
+                dots = [float(torch.dot(*(tensors[n].to("cpu", torch.float64) for n in pair))) for pair in (("lq1", "lk1"), ("lq2", "lk2"))]
+                mix["maps"] = self.env.ops.MapDifference(math.exp(dots[0]) - math.exp(dots[1]) + self.diff, self.diff_eps, 1.0 - self.diff)
             self.form = self.env.ops.AttentionForm(value_dim=self.vd, sinks=self.sinks, chunked=self.mask == "chunk",
                                                    gated=self.head_gate, **mix)
+        if self.out_bias:
+            self.b_o = as_f32(tensors["o_proj.bias"], self.env)
 
     def cache_need(self):
         if not self.own_kv:
@@ -189,6 +224,10 @@ class Attention(Mixer):
     def qkv_width_of(self) -> int:
         """Columns of the q | k | v rows of a layer that projects its own keys and values."""
         return (self.nh + self.nkv) * self.hd + self.nkv * self.vd
+
+    def flops_per_pair(self) -> int:
+        """Flops of one (query, key) pair, all heads."""
+        return 2 * self.nh * (self.hd + self.vd * (self.maps or 1))
 
     def check_borrowed(self, need) -> None:
         if self.own_kv:
@@ -217,6 +256,13 @@ class Attention(Mixer):
         scale_kw = {"row_scale": row_scale} if row_scale is not None else {}
         form_kw = {"form": self.form} if self.form is not None else {}
         extra = {}                    # what only the general preparation kernel does
+        maps = self.form.maps if self.maps else None
+        # two maps: the prompt kernel of some sizes takes a head's both maps at once; everywhere else each is a head of its own
+        split_maps = maps is not None and (ctx.decode or not ops.maps_in_kernel(ctx.dtype, self.hd, self.form))
+        if split_maps:
+            extra["q_maps"] = self.maps
+        if self.q_scale is not None:
+            scale_kw["q_scale"] = self.q_scale.query_scale()
         if self.vd != self.hd:
             extra["value_dim"] = self.vd
         if self.blend_group is not None:
@@ -256,8 +302,10 @@ class Attention(Mixer):
             ops.causal_conv(qkv, 0, self.w_conv, conv_state, ctx.slots, ctx.cu_tokens, ctx.seq_of_token, ctx.len_before,
                             mixed[0])
             qkv = mixed
-        q = ctx.buffer("attn.q", (n, self.nh, self.hd))
-        out = ctx.buffer("attn.out", (n, self.nh * self.vd))
+        nh = self.nh * (self.maps if split_maps else 1)              # query heads of the attention kernel
+        q = ctx.buffer("attn.q", (n, nh, self.hd))
+        result = ctx.buffer("attn.out", (n, self.nh * self.vd))
+        out = ctx.buffer("attn.maps", (n, nh * self.vd), torch.float32) if split_maps else result
         common = dict(n_heads=self.nh, n_kv_heads=nkv_in, head_dim=self.hd,
                       q_norm_w=self.q_norm_w, k_norm_w=self.k_norm_w, norm_eps=self.qk_norm_eps,
                       bias=self.b_qkv, cos=rot.cos if rot else None, sin=rot.sin if rot else None,
@@ -272,7 +320,7 @@ class Attention(Mixer):
                 prep(qkv, **common)
             # which kernel runs and how it splits the keys is the kernels' business: the plan says what scratch it wants
             plan_kw = {"form": self.form} if self.form is not None else {}
-            plan = ops.attn_decode_plan(q.dtype, ctx.n_seqs, self.nh, self.nkv, self.hd, ctx.max_len_after, **plan_kw)
+            plan = ops.attn_decode_plan(q.dtype, ctx.n_seqs, nh, self.nkv, self.hd, ctx.max_len_after, **plan_kw)
             scratch = ctx.buffer("attn.scratch", (max(1, plan.scratch_floats),), torch.float32)
             counters = None
             if plan.n_counters:
@@ -313,9 +361,11 @@ class Attention(Mixer):
                     cache.shared.setdefault("after_last_reader", []).append(write_ring)
                 else:
                     write_ring()
+        if split_maps:
+            ops.map_difference(out.view(n, self.nh, self.maps, self.vd), result, maps)
         if gate is not None:
-            ops.sigmoid_gate(out, gate, gate_col)
-        return Branch(linear(ctx, out, self.w_o, "attn.proj", torch.float32))
+            ops.sigmoid_gate(result, gate, gate_col)
+        return Branch(linear(ctx, result, self.w_o, "attn.proj", torch.float32), bias=self.b_o)
 
 
 register_part("mixer", "attention", Attention)

@@ -63,7 +63,8 @@ class Branch:
     partials ``[s_i, n_tokens, hidden]`` that enter the residual together with ``data`` (sublayers that read the
     same norm's output side by side); ``scale``: the factor on the whole sum as it is added.  ``terms``: instead of all
     that, the summands one by one (``Term``), each with a norm and a factor of its own; ``data`` is then the first term's.
-    Only norms that say so take ``more``, a scale other than 1 or terms (``Norm.check_plain`` is for the others).
+    ``bias`` (float32 ``[H]``): added to every token together with ``data`` (the bias of the sublayer's last projection).
+    Only norms that say so take ``more``, a scale other than 1, terms or a bias (``Norm.check_plain`` is for the others).
     """
 
     data: torch.Tensor
@@ -71,6 +72,7 @@ class Branch:
     more: Tuple[torch.Tensor, ...] = ()
     scale: float = 1.0
     terms: Tuple[Term, ...] = ()
+    bias: Optional[torch.Tensor] = None
 
     @property
     def n_partials(self) -> int:
@@ -93,6 +95,8 @@ class Branch:
         """The branch as a list of summands, whichever way it was built (``write`` has no such reading)."""
         if self.write is not None:
             raise ValueError("a branch that enters the residual through a part of its own has no plain terms")
+        if self.bias is not None:
+            raise ValueError("a branch with a bias has no plain terms: only a norm that takes the bias can add it")
         if self.terms:
             return self.terms
         return tuple(Term(d, scale=self.scale) for d in (self.data,) + tuple(self.more))
@@ -175,8 +179,10 @@ class Norm(Part):
         raise NotImplementedError
 
     @staticmethod
-    def check_plain(branch: Optional[Branch], who: str) -> None:
+    def check_plain(branch: Optional[Branch], who: str, takes_bias: bool = False) -> None:
         """For norms that add one set of partials, unscaled: refuses a branch that asks for more."""
+        if branch is not None and branch.bias is not None and not takes_bias:
+            raise ValueError(f"{who}: the pending branch carries a bias; this norm adds outputs as they are")
         if branch is not None and (branch.more or branch.scale != 1.0 or branch.terms):
             raise ValueError(f"{who}: the pending branch carries several sublayers' outputs or a scale; "
                              f"this norm adds one output as it is")
@@ -217,6 +223,10 @@ class PositionEncoding(Part):
 
     def rotation(self):
         """``None`` or a ``Rotation`` that a mixer applies to its queries and keys."""
+        return None
+
+    def query_scale(self):
+        """``None`` or a float32 tensor with a number per position that a mixer multiplies its queries by."""
         return None
 
     def on_embeddings(self, residual, ctx) -> None:

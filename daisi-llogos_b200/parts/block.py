@@ -69,7 +69,7 @@ class ParallelBlock(Block):
         # neither consumer gets a row scale: both read the same finished rows
         h = p["norm1"].forward(residual, pending, ctx)
         a = p["mixer"].forward(h, ctx, cache)
-        if a.more or a.scale != 1.0 or a.write is not None:
+        if a.more or a.scale != 1.0 or a.write is not None or a.bias is not None:
             raise ValueError("parallel block: the mixer's branch must be plain partials")
         if "ffn" not in p:
             return Branch(a.data, scale=self.scale)

@@ -11,7 +11,11 @@ runs) where the layer has one; with ``shared_gate`` the shared expert's output i
 number per token, whose row ``w_sg`` rides in the router's product.  Further forms, by parameter: weights that are the chosen
 scores themselves (``normalize`` False); weights on the experts' INPUT, ``sum_e expert_e(w_e h)``, which the first product's
 epilogue applies (it is linear in its rows) and the sum at the end does not; experts gated in a clamped form (``activation``
-"clamped", parts/feedforward.py), the shared expert with constants of its own.
+"clamped", parts/feedforward.py), the shared expert with constants of its own; groups also with "softmax_all"; scores that are
+corrected by a learned number per expert where groups are judged and experts chosen, but not where they become weights
+(``correction``); and IDENTITY experts (``identity`` of them, behind the others in the router's rows and in the groups), which
+return their input and have no matrices: their pairs get no row in the layout below, and the weighted sum adds the token's
+input instead.
 
 On the device the step's (token, choice) pairs are put in the order of their experts, every expert's run of rows
 filled up to a whole tile (``ops.moe_plan``), so that two grouped products (gate/up with the gating as its epilogue,
@@ -36,8 +40,9 @@ class MoeFeedForward(FeedForward):
     keep_groups (0: every expert is eligible), group_score_top (default 2), weight_scale (default 1), weight_sum_eps
     (default 0), normalize (default True: scores other than "softmax" are divided by the chosen ones' sum), weight_on ("output",
     the default, or "input"), activation ("silu", or "clamped" with gate_alpha, up_offset, limit), shared_params (further params
-    of the shared expert), shared_gate (bool: a tensor ``shared_gate.weight`` [1, hidden]).  Tensors: ``router.weight`` [experts, hidden],
-    ``router.bias`` [experts], and per expert i ``experts.<i>.{gate_proj,up_proj,down_proj}.weight``."""
+    of the shared expert), shared_gate (bool: a tensor ``shared_gate.weight`` [1, hidden]), identity (how many identity experts the
+    router has besides), correction (bool: a tensor ``correction`` [routed]).  Tensors: ``router.weight`` [routed, hidden] with ``routed`` =
+    experts + identity experts, ``router.bias`` [routed], and per expert i ``experts.<i>.{gate_proj,up_proj,down_proj}.weight``."""
 
     def __init__(self, params, prefix, env):
         super().__init__(params, prefix, env)
@@ -46,11 +51,15 @@ class MoeFeedForward(FeedForward):
         self.n_exp = int(p["num_experts"])
         self.top = int(p["top"])
         self.inter = int(p["expert_size"])
-        if not 0 < self.top <= self.n_exp:
-            raise ValueError(f"moe: top {self.top} of {self.n_exp} experts")
+        self.identity = int(p.get("identity", 0) or 0)
+        if self.identity < 0 or self.n_exp <= 0:
+            raise ValueError(f"moe: {self.n_exp} experts and {self.identity} identity experts")
+        self.n_routed = self.n_exp + self.identity               # what the router chooses from
+        if not 0 < self.top <= self.n_routed:
+            raise ValueError(f"moe: top {self.top} of {self.n_routed} experts")
         limit = getattr(env.ops, "MOE_MAX_EXPERTS", None)
-        if limit is not None and self.n_exp > limit:
-            raise ValueError(f"moe: {self.n_exp} experts; the routing kernels take up to {limit}")
+        if limit is not None and self.n_routed > limit:
+            raise ValueError(f"moe: {self.n_routed} experts; the routing kernels take up to {limit}")
         top_limit = getattr(env.ops, "MOE_MAX_TOP", None)
         if top_limit is not None and self.top > top_limit:
             raise ValueError(f"moe: top {self.top}; the routing kernels take up to {top_limit}")
@@ -60,11 +69,11 @@ class MoeFeedForward(FeedForward):
             raise ValueError(f"moe: score '{self.score}' is not known (softmax, sigmoid, softmax_all)")
         self.groups, self.keep_groups = int(p.get("groups") or 0), int(p.get("keep_groups") or 0)
         if self.groups:
-            if self.score != "sigmoid":
-                raise ValueError("moe: groups of experts go with sigmoid scores")
-            if self.n_exp % self.groups or not 0 < self.keep_groups <= self.groups:
-                raise ValueError(f"moe: {self.n_exp} experts in {self.groups} groups of which {self.keep_groups} are kept")
-            if self.top > self.keep_groups * (self.n_exp // self.groups):
+            if self.score == "softmax":
+                raise ValueError("moe: groups of experts go with sigmoid or softmax_all scores")
+            if self.n_routed % self.groups or not 0 < self.keep_groups <= self.groups:
+                raise ValueError(f"moe: {self.n_routed} experts in {self.groups} groups of which {self.keep_groups} are kept")
+            if self.top > self.keep_groups * (self.n_routed // self.groups):
                 raise ValueError(f"moe: top {self.top} exceeds the experts of {self.keep_groups} groups")
         self.group_score_top = int(p.get("group_score_top", 2))
         self.weight_scale = float(p.get("weight_scale", 1.0))
@@ -75,6 +84,12 @@ class MoeFeedForward(FeedForward):
         self.weight_on = str(p.get("weight_on", "output"))
         if self.weight_on not in ("output", "input"):
             raise ValueError(f"moe: weight_on '{self.weight_on}' is not known (output, input)")
+        if self.identity and self.weight_on != "output":
+            raise ValueError("moe: identity experts go with weights on the experts' outputs")
+        self.corrected = bool(p.get("correction", False))
+        if self.corrected and self.score == "softmax":
+            raise ValueError("moe: a correction goes with sigmoid or softmax_all scores")
+        self.correction = None
         activation = str(p.get("activation", "silu"))
         if activation not in ("silu", "clamped"):
             raise ValueError(f"moe: the experts' activation '{activation}' is not known (silu, clamped)")
@@ -109,9 +124,11 @@ class MoeFeedForward(FeedForward):
         return self.prefix + rel
 
     def tensors(self):
-        t = {"router.weight": TensorDecl((self.n_exp, self.hidden))}
+        t = {"router.weight": TensorDecl((self.n_routed, self.hidden))}
         if self.router_bias:
-            t["router.bias"] = TensorDecl((self.n_exp,), "bias")
+            t["router.bias"] = TensorDecl((self.n_routed,), "bias")
+        if self.corrected:
+            t["correction"] = TensorDecl((self.n_routed,), "bias")
         if self.shared_gate:
             t["shared_gate.weight"] = TensorDecl((1, self.hidden))
         for i in range(self.n_exp):
@@ -135,6 +152,7 @@ class MoeFeedForward(FeedForward):
         self.w_router_same = w_r if w_r.dtype == self.env.dtype else None
         self.w_router = as_f32(w_r, self.env) if self.w_router_same is None else None
         self.b_router = as_f32(tensors["router.bias"], self.env) if self.router_bias else None
+        self.correction = as_f32(tensors["correction"], self.env) if self.corrected else None
         per = {what: [tensors[self._expert(i, what)] for i in range(self.n_exp)] for what in ("gate", "up", "down")}
         if len({w.dtype for ws in per.values() for w in ws}) != 1:
             raise ValueError(f"{self.prefix}: the experts' matrices are stored with different types")
@@ -148,7 +166,7 @@ class MoeFeedForward(FeedForward):
     def active_matrix_params(self) -> int:
         """Elements of the matrices one token passes through: the router, ``top`` experts, the shared expert."""
         shared = 3 * self.hidden * self.shared.inter if self.shared is not None else 0
-        return self.n_exp * self.hidden + self.top * 3 * self.hidden * self.inter + shared
+        return self.n_routed * self.hidden + self.top * 3 * self.hidden * self.inter + shared
 
     def forward(self, x, ctx) -> Branch:
         ops = ctx.ops
@@ -160,7 +178,9 @@ class MoeFeedForward(FeedForward):
         shared_scale = ctx.buffer("moe.shared_scale", (n,), torch.float32) if self.shared_gate else None
         rule = {} if plain else dict(rule=ops.RouterRule(self.score, self.groups, self.keep_groups, self.group_score_top,
                                                         self.weight_scale, self.weight_sum_eps,
-                                                        **({} if self.normalize else {"normalize": False})), extra_out=shared_scale)
+                                                        **({} if self.normalize else {"normalize": False}),
+                                                        **({"correction": self.correction} if self.corrected else {})),
+                                     extra_out=shared_scale)
         if self.w_router_same is not None and x.dtype == self.w_router_same.dtype and hasattr(ops, "moe_topk"):
             ops.moe_topk(linear(ctx, x, self.w_router_same, "moe.logits", torch.float32), self.b_router, choice, weight, **rule)
         else:
@@ -191,10 +211,10 @@ class MoeFeedForward(FeedForward):
         ops.moe_down(act, tile_expert, self.w_down, y)
         shared = self.shared.forward(x, ctx).data if self.shared is not None else None
         out = ctx.buffer("moe.out", (1, n, self.hidden), torch.float32)
-        if shared_scale is not None:
-            ops.moe_combine(y, row_of_pair, weight, shared, out[0], shared_scale=shared_scale)
-        else:
-            ops.moe_combine(y, row_of_pair, weight, shared, out[0])
+        combine_kw = {} if shared_scale is None else {"shared_scale": shared_scale}
+        if self.identity:
+            combine_kw["identity"] = x
+        ops.moe_combine(y, row_of_pair, weight, shared, out[0], **combine_kw)
         return Branch(out)
 
 

@@ -19,6 +19,10 @@ import torch
 from .base import Branch, Norm, TensorDecl, as_f32, register_part
 
 
+def _bias(branch: Optional[Branch]) -> dict:
+    return {} if branch is None or branch.bias is None else {"branch_bias": branch.bias}
+
+
 class RmsNorm(Norm):
     """params: size, eps, weight_offset (default 0; 1 for a weight that holds its difference from one: the row is multiplied by
     ``1 + weight``), out_name (the workspace buffer of the output, default "norm.out": two norms whose outputs are alive
@@ -68,10 +72,10 @@ class RmsNorm(Norm):
     def forward(self, residual, branch: Optional[Branch], ctx, rows=None):
         if self.weight_offset or (branch is not None and branch.terms):
             return self.forward_many(residual, branch, ctx, (), rows)[0]
-        self.check_plain(branch, "rmsnorm")
+        self.check_plain(branch, "rmsnorm", takes_bias=True)
         m = residual.shape[0] if rows is None else rows.numel()
         out = ctx.buffer("norm.out", (m, self.size))
-        ctx.ops.add_rmsnorm(residual, branch.data if branch is not None else None, self.weight, self.eps, out, rows)
+        ctx.ops.add_rmsnorm(residual, branch.data if branch is not None else None, self.weight, self.eps, out, rows, **_bias(branch))
         return out
 
     def forward_unscaled(self, residual, branch: Optional[Branch], ctx, rows=None):
@@ -79,11 +83,12 @@ class RmsNorm(Norm):
         make_scale = getattr(ops, "RowScale", None)
         if make_scale is None or ctx.dtype != torch.bfloat16 or self.weight_offset or (branch is not None and branch.terms):
             return self.forward(residual, branch, ctx, rows), None
-        self.check_plain(branch, "rmsnorm")
+        self.check_plain(branch, "rmsnorm", takes_bias=True)
         m = residual.shape[0] if rows is None else rows.numel()
         out = ctx.buffer("norm.out", (m, self.size))
         ss = ctx.buffer("norm.ss", (m, ops.norm_ss_parts(m, self.size)), torch.float32)
-        ops.add_rmsnorm(residual, branch.data if branch is not None else None, self.weight, self.eps, out, rows, ss_out=ss)
+        ops.add_rmsnorm(residual, branch.data if branch is not None else None, self.weight, self.eps, out, rows, ss_out=ss,
+                        **_bias(branch))
         return out, make_scale(ss, self.size, self.eps)
 
 
@@ -116,6 +121,8 @@ class LayerNorm(Norm):
             raise ValueError(f"{self.prefix}: a layer norm's weight and bias are stored with different types")
 
     def forward(self, residual, branch: Optional[Branch], ctx, rows=None):
+        if branch is not None and branch.bias is not None:
+            raise ValueError("layernorm: the pending branch carries a bias; this norm adds outputs as they are")
         if residual.dim() != 2:
             raise ValueError("layernorm: the residual must be one stream [tokens, hidden]")
         m = residual.shape[0] if rows is None else rows.numel()

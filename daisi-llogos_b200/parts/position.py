@@ -114,9 +114,40 @@ class RotaryEncoding(PositionEncoding):
         return self._rotation
 
 
+class QueryTemperature(PositionEncoding):
+    """Queries grow with their position: a query at position p is multiplied by ``1 + coef ln(floor((p + 1) / every) + 1)``.
+    The factors are worked out in float64 and kept as float32, one per position.  params: coef, every."""
+
+    def __init__(self, params, prefix, env):
+        super().__init__(params, prefix, env)
+        self.coef, self.every = float(params["coef"]), float(params["every"])
+        if not self.every > 0:
+            raise ValueError(f"query temperature: 'every' must be positive, got {self.every}")
+        self._table: Optional[torch.Tensor] = None
+        self._retired = []        # as in RotaryEncoding
+
+    def limit(self) -> Optional[int]:
+        return None if self._table is None else int(self._table.shape[0])
+
+    def prepare(self, max_positions: int) -> None:
+        if self._table is not None:
+            if self._table.shape[0] >= max_positions:
+                return
+            self._retired.append(self._table)
+        pos = torch.arange(max_positions, dtype=torch.float64)
+        factor = 1.0 + self.coef * torch.log(torch.floor((pos + 1.0) / self.every) + 1.0)
+        self._table = factor.to(torch.float32).to(self.env.device).contiguous()
+
+    def query_scale(self) -> torch.Tensor:
+        if self._table is None:
+            raise RuntimeError("QueryTemperature.prepare() has not run")
+        return self._table
+
+
 class NoEncoding(PositionEncoding):
     """No position information (mixers then skip the rotation)."""
 
 
 register_part("position", "rotary", RotaryEncoding)
+register_part("position", "query_temperature", QueryTemperature)
 register_part("position", "none", NoEncoding)

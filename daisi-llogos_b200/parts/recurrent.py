@@ -263,7 +263,7 @@ class SideBySide(Mixer):
         for side, part in self.sides.items():
             view = cache[side] if part.cache_need() is not None else None
             b = part.forward(x, ctx, view)
-            if b.more or b.terms or b.scale != 1.0 or b.write is not None:
+            if b.more or b.terms or b.scale != 1.0 or b.write is not None or b.bias is not None:
                 raise ValueError("side by side: a side's branch must be plain partials")
             terms.append(Term(b.data, self.out_w[side], self.eps, self.scale))
         return Branch.of_terms(terms)

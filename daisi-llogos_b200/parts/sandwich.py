@@ -129,7 +129,7 @@ class SandwichBlock(Block):
 
     @staticmethod
     def _through(post: GatedPostNorm, branch: Branch, h, ctx) -> Branch:
-        if branch.more or branch.scale != 1.0 or branch.write is not None:
+        if branch.more or branch.scale != 1.0 or branch.write is not None or branch.bias is not None:
             raise ValueError("sandwich: a sublayer's branch must be plain partials")
         gate = post.gate_arguments(h, ctx)
         return Branch(branch.data, write=post, more=() if gate is None else (gate,))

@@ -24,12 +24,13 @@ def embed_rows(table, token_ids, out_residual):
     out_residual.copy_(rows if out_residual.dim() == 2 else rows.expand_as(out_residual))
 
 
-def add_rmsnorm(residual, branch, weight, eps, out, rows=None):
+def add_rmsnorm(residual, branch, weight, eps, out, rows=None, branch_bias=None):
     if branch is not None:
+        total = branch.sum(0) if branch_bias is None else branch.sum(0) + branch_bias
         if rows is None:
-            residual += branch.sum(0)
+            residual += total
         else:
-            residual[rows.long()] += branch.sum(0)[rows.long()]
+            residual[rows.long()] += total[rows.long()]
     x = residual if rows is None else residual[rows.long()]
     y = x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight.float()
     out.copy_(y.to(out.dtype))
@@ -47,7 +48,7 @@ def _rows_of(page_table, ring_pages, slot, pos, kvh, nkv):
 def qk_prep(qkv, *, n_heads, n_kv_heads, head_dim, q_norm_w, k_norm_w, norm_eps, bias, cos, sin, rotary_dim,
             pairing, positions, q_out, k_new=None, v_new=None, k_pages=None, v_pages=None, page_table=None,
             ring_pages=0, seq_of_token=None, slots=None, value_dim=0, v_mix=None, v_first_in=None, v_first_out=None,
-            gate_out=None):
+            gate_out=None, q_scale=None, q_maps=0):
     x = qkv.float().sum(0)
     if gate_out is not None:
         gate_out.copy_(torch.sigmoid(x[:, x.shape[1] - n_heads:]))
@@ -89,7 +90,16 @@ def qk_prep(qkv, *, n_heads, n_kv_heads, head_dim, q_norm_w, k_norm_w, norm_eps,
             a, b = r[..., 0:2 * half:2].clone(), r[..., 1:2 * half:2].clone()
             r[..., 0:2 * half:2] = a * c - b * s
             r[..., 1:2 * half:2] = a * s + b * c
-    q_out.copy_(x[:, :nh].to(q_out.dtype))
+    q = x[:, :nh]
+    if q_scale is not None:
+        q = q * q_scale[positions.long()][:, None, None]
+    if q_maps:
+        part = hd // q_maps
+        split = torch.zeros(n, nh, q_maps, hd)
+        for m in range(q_maps):
+            split[:, :, m, m * part:(m + 1) * part] = q[:, :, m * part:(m + 1) * part]
+        q = split.view(n, nh * q_maps, hd)
+    q_out.copy_(q.to(q_out.dtype))
     if nkv == 0:
         return
     k = x[:, nh:nh + nkv].to(q_out.dtype)
@@ -275,8 +285,10 @@ CONV_MAX_TAPS = 16
 RETENTION_PIECE = 4
 
 
-def causal_conv(rows, col0, weight, state, slots, cu_tokens, seq_of_token, len_before, out, in_bias=None, bias=None, out2=None):
+def causal_conv(rows, col0, weight, state, slots, cu_tokens, seq_of_token, len_before, out, in_bias=None, bias=None, out2=None, act=None):
     c, k = weight.shape
+    if out is None:
+        out = torch.empty(out2.shape)
     x = rows.float().sum(0)[:, col0:col0 + c]
     if in_bias is not None:
         x = x + in_bias.float()
@@ -286,11 +298,38 @@ def causal_conv(rows, col0, weight, state, slots, cu_tokens, seq_of_token, len_b
         seq = torch.cat([past, x[t0:t1]])               # the state holds zeros where the sequence had not begun
         for t in range(t1 - t0):
             y = (seq[t:t + k] * weight.float().t()).sum(0)
-            out[t0 + t] = y if bias is None else y + bias.float()
+            y = y if bias is None else y + bias.float()
+            out[t0 + t] = y if act is None else _act(y, act)
         if k > 1:
             state[int(slots[b])] = seq[seq.shape[0] - (k - 1):]
     if out2 is not None:
         out2.copy_(out.to(out2.dtype))
+
+
+def state_space(mixed, rows, *, z_col, dt_col, dt_bias, a_log, d_skip, n_heads, groups, n_state, vdim, state, slots, cu_tokens, out,
+                max_count):
+    inner, gn = n_heads * vdim, groups * n_state
+    r = rows.float().sum(0)
+    dt = torch.nn.functional.softplus(r[:, dt_col:dt_col + n_heads] + dt_bias)
+    of = torch.arange(n_heads) // (n_heads // groups)
+    x = mixed[:, :inner].float().view(-1, n_heads, vdim)
+    b_all = mixed[:, inner:inner + gn].float().view(-1, groups, n_state)[:, of]
+    c_all = mixed[:, inner + gn:].float().view(-1, groups, n_state)[:, of]
+    for b in range(slots.numel()):
+        s = state[int(slots[b])].clone()
+        for t in range(int(cu_tokens[b]), int(cu_tokens[b + 1])):
+            s = torch.exp(-torch.exp(a_log) * dt[t])[:, None, None] * s + (dt[t][:, None] * b_all[t])[:, :, None] * x[t][:, None, :]
+            y = (s * c_all[t][:, :, None]).sum(1) + d_skip[:, None] * x[t]
+            if z_col >= 0:
+                y = y.reshape(-1) * torch.nn.functional.silu(r[t, z_col:z_col + inner])
+            out[t] = y.reshape(-1)
+        state[int(slots[b])] = s
+
+
+def part_rmsnorm(x, weight, parts, eps, out):
+    v = x.float().view(x.shape[0], parts, -1)
+    v = v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps)
+    out.copy_((v.reshape(x.shape) * weight).to(out.dtype))
 
 
 def rglru_scan(rows, y_col, y_bias, u, gates, gate_bias, lam, decay_scale, state, slots, cu_tokens, out, carry=None):
@@ -403,8 +442,8 @@ def moe_row_capacity(pairs, n_experts, tile=MOE_TILE_ROWS):
 
 class RouterRule:
     def __init__(self, score="softmax", groups=0, keep_groups=0, group_score_top=2, weight_scale=1.0, weight_sum_eps=0.0,
-                 normalize=True):
-        self.normalize = normalize
+                 normalize=True, correction=None):
+        self.normalize, self.correction = normalize, correction
         self.score, self.groups, self.keep_groups, self.group_score_top = score, groups, keep_groups, group_score_top
         self.weight_scale, self.weight_sum_eps = weight_scale, weight_sum_eps
 
@@ -424,14 +463,15 @@ def moe_route(x, w_router, b_router, choice, weight, rule=None, extra_out=None):
         return
     s = torch.softmax(z, dim=-1) if rule.score == "softmax_all" else torch.sigmoid(z)
     n, n_exp = s.shape
-    masked = s
+    masked = s if rule.correction is None else s + rule.correction
     if rule.groups:
         per = n_exp // rule.groups
-        gs = torch.topk(s.view(n, rule.groups, per), min(rule.group_score_top, per), dim=-1).values.sum(-1)
+        gs = torch.topk(masked.view(n, rule.groups, per), min(rule.group_score_top, per), dim=-1).values.sum(-1)
         best = torch.topk(gs, rule.keep_groups, dim=-1).indices
         ok = torch.zeros_like(gs, dtype=torch.bool).scatter_(1, best, True)
-        masked = s.masked_fill(~ok[:, :, None].expand(-1, -1, per).reshape(n, n_exp), -1.0)
-    val, idx = torch.topk(masked, top, dim=-1)
+        masked = masked.masked_fill(~ok[:, :, None].expand(-1, -1, per).reshape(n, n_exp), float("-inf"))
+    idx = torch.topk(masked, top, dim=-1).indices
+    val = s.gather(1, idx)
     choice.copy_(idx.to(torch.int32))
     if not rule.normalize:
         weight.copy_(val * rule.weight_scale)
@@ -444,6 +484,7 @@ def moe_plan(choice, n_experts, row_of_pair, token_of_row, tile_expert, weight=N
         weight_of_row.zero_()
     top = choice.shape[1]
     flat = choice.reshape(-1).tolist()
+    row_of_pair.fill_(-1)
     token_of_row.fill_(-1)
     tile_expert.fill_(-1)
     row = 0
@@ -497,10 +538,13 @@ def moe_down(act, tile_expert, w_down, y):
             y[r] = w_down[e].float() @ act[r].float()
 
 
-def moe_combine(y, row_of_pair, weight, shared, out, shared_scale=None):
+def moe_combine(y, row_of_pair, weight, shared, out, shared_scale=None, identity=None):
     n = out.shape[0]
     rows = row_of_pair.view(n, -1).long()
-    out.copy_((y[rows] if weight is None else weight[:, :, None] * y[rows]).sum(1))
+    got = y[rows.clamp(min=0)]
+    if identity is not None:
+        got = torch.where((rows < 0)[:, :, None], identity.float()[:, None, :], got)
+    out.copy_((got if weight is None else weight[:, :, None] * got).sum(1))
     if shared is not None:
         out += shared.sum(0) if shared_scale is None else shared.sum(0) * shared_scale[:, None]
 
@@ -618,8 +662,8 @@ def zero_rows(base, rows):
 
 
 class AttentionForm:
-    def __init__(self, value_dim=0, sink=None, gated=False, sinks=None, chunked=False, softcap=0.0, head_mix=None):
-        self.softcap, self.head_mix = softcap, head_mix
+    def __init__(self, value_dim=0, sink=None, gated=False, sinks=None, chunked=False, softcap=0.0, head_mix=None, maps=None):
+        self.softcap, self.head_mix, self.maps = softcap, head_mix, maps
         self.value_dim, self.sink, self.gated = int(value_dim), sink, bool(gated)
         self.sinks, self.chunked = sinks, bool(chunked)
 
@@ -631,6 +675,21 @@ class AttentionForm:
 
 
 PLAIN_ATTENTION = AttentionForm()
+
+
+class MapDifference:
+    def __init__(self, lam, eps, scale):
+        self.lam, self.eps, self.scale = lam, eps, scale
+
+
+def maps_in_kernel(dtype, head_dim, form):
+    return False                                 # every map is a head of its own here
+
+
+def map_difference(raw, out, maps):
+    o = raw[:, :, 0] - maps.lam * raw[:, :, 1]
+    o = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + maps.eps) * maps.scale
+    out.copy_(o.reshape(out.shape).to(out.dtype))
 
 
 def _lowest(form, window, pos):
