@@ -30,7 +30,9 @@ closest model the library has, at equal latent, expert and feed-forward sizes; `
 input) beside Rukedra at equal widths, experts and feed-forward sizes; ``--design memilorn`` puts the Memilorn design (a
 matrix memory with exponential gates, attention with capped scores mixed over the heads, latent attention, a mixture weighed
 on its input) beside the two closest models the library has, Piratar (retention, attention over every key) and Rukedra
-(latent attention over every key), at equal widths, heads, states and experts.
+(latent attention over every key), at equal widths, heads, states and experts; ``--design penasun`` puts the Penasun design (a
+state-space recurrence with a scalar decay per head, differential attention, a mixture with identity experts) beside Memilorn
+(a matrix-valued state, the same experts) and Piratar (retention, attention over every key, short convolutions).
 """
 import argparse
 import json
@@ -459,6 +461,23 @@ def memilorn_config(size):
     return {"architecture": "Memilorn", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-6}, "layers": layers}
 
 
+def penasun_config(size):
+    """Penasun at a size, four layers: a state-space recurrence and differential attention in turn, each with a mixture.  The
+    recurrence is twice as wide as the model in heads of 64, 128 state rows and eight groups, with four taps; a head of attention
+    holds both maps in one head size of the stock model (half of it each; values of the whole of it), so the cached rows are the
+    stock model's; the experts (sixteen, four per token) are Memilorn's, beside four identity experts, in four groups of which two
+    stay; there is no shared expert."""
+    width, heads, kv, hd, ff, window, _ = DESIGN_SIZES[size]
+    ssm = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 8, "conv": 4, "norm_groups": 8}
+    att = {"heads": heads, "kv_heads": kv, "dim": hd // 2, "vdim": hd, "scale": (hd // 2) ** -0.5, "diff": 0.5,
+           "q_temp": {"coef": 0.1, "every": 4096}}
+    moe = {"kind": "moe", "router": {"experts": FIPAVIK_EXPERTS, "top": FIPAVIK_TOP, "identity": 4, "scale": 2.5,
+                                     "groups": {"count": 4, "keep": 2}}, "expert": {"ff": ff // 8, "limit": 7.0}}
+    layers = [{"type": t, "mixer": dict(m), "mlp": dict(moe)} for t, m in (("mamba2", ssm), ("attention", att)) * 2]
+    assert len(layers) == DESIGN_LAYERS
+    return {"architecture": "Penasun", "vocab": DESIGN_VOCAB, "width": width, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 def design_configs(size, design="karitar"):
     """The configuration of ``design`` (Karitar or Fipavik) at a size and the closest stock model's (Qwen3: grouped-query
     attention with normed queries and keys and the same window, pre-norm blocks) with the same width, heads, head size
@@ -483,6 +502,8 @@ def design_configs(size, design="karitar"):
         return {"piratar": piratar_config(size), "rukedra": rukedra_config(size)}
     if design == "memilorn":
         return {"memilorn": memilorn_config(size), "piratar": piratar_config(size), "rukedra": rukedra_config(size)}
+    if design == "penasun":
+        return {"penasun": penasun_config(size), "memilorn": memilorn_config(size), "piratar": piratar_config(size)}
     return {"karitar": karitar, "qwen3": qwen3}
 
 
@@ -490,7 +511,8 @@ _TIMED_OPS = ("embed_rows", "add_rmsnorm", "hc_add_rmsnorm", "qk_prep", "qkv_row
               "act_rows", "silu_mul", "attn_prefill", "attn_decode", "kv_write", "add_layernorm", "latent_prep", "head_linear",
               "moe_route", "moe_topk", "moe_plan", "moe_gather_rows", "moe_gated", "moe_down", "moe_combine",
               "gated_add_group_rmsnorm", "mingru_scan", "sigmoid_gate", "tanh_cap", "multi_add_rmsnorm", "hash_embed",
-              "table_gate", "causal_conv", "rglru_scan", "retention", "matrix_memory")
+              "table_gate", "causal_conv", "rglru_scan", "retention", "matrix_memory", "state_space", "part_rmsnorm",
+              "map_difference")
 
 # What the float32 multiply-adds of a B200's CUDA cores can do at most (148 multiprocessors x 128 lanes x 2 flops at
 # 1.9 GHz): the arithmetic bound of kernels whose products must stay float32 (retention's state).
@@ -512,6 +534,7 @@ def _kernel_label(name, args, kw):
     return name
 
 
+_MATRIX_SHARE = [1.0]        # set by probe_designs: of the experts a router chooses from, the share that has matrices
 _TENSOR_PER_FP32 = [1.0]     # set by probe_designs: the measured matrix peak over FP32_TFLOPS
 
 
@@ -533,6 +556,12 @@ def _kernel_cost(name, args, kw, keys_read):
         if getattr(kw.get("form"), "head_mix", None) is not None:
             # the mixture of the heads' scores: float32 products, counted against the CUDA cores' peak as retention's are
             mixed = 2.0 * nh * nh * pairs * _TENSOR_PER_FP32[0]
+        if getattr(kw.get("form"), "maps", None) is not None:
+            # two maps: scores over half of a key each, both over the same values; a kernel that does not take a head's both maps
+            # at once gets them as heads of their own and leaves float32
+            out = args[11 if name == "attn_prefill" else 7]
+            n_maps = 2 * nh if out.dtype == q.dtype else nh
+            return rows * nkv * (hd + vd) * q.element_size() + q.nbytes + out.nbytes, 2.0 * n_maps * (hd / 2 + vd) * pairs
         return rows * nkv * (hd + vd) * q.element_size() + 2 * q.nbytes, 2.0 * nh * (hd + vd) * pairs + mixed
     if name in ("add_rmsnorm", "hc_add_rmsnorm"):
         # the residual (one array or several streams) is read and, with a branch, written back; only the rows that
@@ -566,9 +595,8 @@ def _kernel_cost(name, args, kw, keys_read):
         rows, table, out = args[0], args[1], args[4]
         return rows.nbytes + out.nbytes + out.numel() * table.element_size(), 0.0
     if name == "causal_conv":
-        rows, weight, out = args[0], args[2], args[8]
-        out2 = kw.get("out2")
-        return rows.shape[0] * out.numel() * 4 + out.nbytes + (out2.nbytes if out2 is not None else 0), 0.0
+        rows, outs = args[0], [t for t in (args[8], kw.get("out2")) if t is not None]
+        return rows.shape[0] * outs[0].numel() * 4 + sum(t.nbytes for t in outs), 0.0
     if name == "rglru_scan":
         # y's partial sums, u, the gates' arguments and the outputs; with the scan in pieces u and the gates are read twice
         rows, u, gates, out = args[0], args[3], args[4], args[11]
@@ -593,6 +621,15 @@ def _kernel_cost(name, args, kw, keys_read):
         moved = rows.nbytes * (2 if carry is not None else 1) + out.nbytes + 2 * kw["slots"].numel() * state[0].numel() * 4
         flops = 4.0 * n * nh * dim * vdim * (2 if carry is not None else 1)
         return moved, flops * _TENSOR_PER_FP32[0]
+    if name == "state_space":
+        # x, B and C, the sums of z and of the step sizes, the outputs, and every sequence's state in and out.  Update and read-out:
+        # float32 products against the CUDA cores' peak where tokens are walked one by one (a decode step), tensor-core products in
+        # chunks (a prompt step)
+        mixed, rows, out, state = args[0], args[1], kw["out"], kw["state"]
+        n, nh = out.shape[0], kw["n_heads"]
+        moved = mixed.nbytes + rows.shape[0] * n * (out.shape[1] + nh) * 4 + out.nbytes + 2 * kw["slots"].numel() * state[0].numel() * 4
+        flops = 4.0 * n * nh * kw["n_state"] * kw["vdim"]
+        return moved, flops * (1.0 if kw["max_count"] > 1 else _TENSOR_PER_FP32[0])
     if name == "sigmoid_gate":
         x, gate = args[0], args[1]
         return 2 * x.nbytes + gate.shape[0] * x.numel() * 4, 0.0
@@ -608,7 +645,7 @@ def _kernel_cost(name, args, kw, keys_read):
         rows_out = args[4] if name == "moe_gated" else args[3]
         tiles = args[2] if name == "moe_gated" else args[1]
         n_exp, n_in, n_out = w.shape[0], w.shape[2], rows_out.shape[1]
-        pairs = max(1, rows_out.shape[0] - n_exp * (rows_out.shape[0] // tiles.numel() - 1))
+        pairs = max(1, int((rows_out.shape[0] - n_exp * (rows_out.shape[0] // tiles.numel() - 1)) * _MATRIX_SHARE[0]))
         mats = 2 if name == "moe_gated" else 1
         moved = min(n_exp, pairs) * mats * n_out * n_in * w.element_size() + pairs * (n_in * args[0].element_size() + n_out * rows_out.element_size())
         return moved, 2.0 * mats * pairs * n_out * n_in
@@ -636,6 +673,8 @@ def probe_designs(torch, L, ops, pk, sizes, batch, which="karitar"):
         context = DESIGN_SIZES[size][6]
         for design, cfg in design_configs(size, which).items():
             model = L.weights.random_model(cfg, seed=0, dtype=torch.bfloat16, device=dev, std=0.02)
+            router = cfg.get("layers", [{}])[0].get("mlp", {}).get("router", {})
+            _MATRIX_SHARE[0] = router.get("experts", 1) / (router.get("experts", 1) + router.get("identity", 0))
             out = {}
             for graphs in (True, False):
                 eng = L.engine.Engine(model, max_tokens=(batch + 1) * pages_of(context), max_seq_len=context, n_slots=batch + 1,
@@ -751,7 +790,7 @@ def main():
     ap.add_argument("--tokens", type=int, default=0,
                     help="with --probe timeline: the time line of a prompt step of so many tokens instead of a decode step")
     ap.add_argument("--sizes", default=",".join(DESIGN_SIZES), help="with --probe designs: which of " + ", ".join(DESIGN_SIZES))
-    ap.add_argument("--design", choices=["karitar", "fipavik", "rukedra", "piratar", "memilorn"], default="karitar",
+    ap.add_argument("--design", choices=["karitar", "fipavik", "rukedra", "piratar", "memilorn", "penasun"], default="karitar",
                     help="with --probe designs: the design that stands beside the closest stock model")
     ap.add_argument("--probe", choices=["decode-attention", "leave-one-out", "timeline", "designs"],
                     help="instead of the bench line, print a table: decode attention alone over batch shapes; what "

@@ -605,7 +605,7 @@ struct MatrixMemoryArgs {
 //   S <- exp(-exp(a_log[h]) d) S + d B x^T        (S is [n_state][vdim])
 //   out = (S^T C + d_skip[h] x) * silu(z)         (z the sums of the columns from z_col on; z_col < 0: no gate)
 // state [slots][nh][n_state][vdim] holds S before the step's first token of a sequence and receives it after its last.
-// A block owns `cols` columns of a head's S (a column's walk needs no other column).
+// A block owns `cols` columns of a head's S (a column's walk needs no other column); 0: the library chooses.
 struct StateSpaceArgs {
   const void* mixed;          // [n_tokens][nh * vdim + 2 * groups * n_state]
   int mixed_dtype;

@@ -156,6 +156,10 @@ LLG_API int llg_mingru_scan(const MinGruArgs* args, int max_count, cudaStream_t 
 
 namespace {
 
+__device__ __noinline__ float other_act(int kind, float v) { return llg_act(kind, v); }
+// silu in line, every other kind as a call: the switch over all kinds would be repeated for each token of a run
+__device__ __forceinline__ float conv_act(int kind, float v) { return kind == 2 ? __fdividef(v, 1.0f + __expf(-v)) : other_act(kind, v); }
+
 template <typename O2>
 __global__ void __launch_bounds__(128) causal_conv_kernel(ConvArgs a) {
   pdl_launch_dependents();
@@ -179,7 +183,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ConvArgs a) {
   };
   O2* out2 = (O2*)a.out2;
   auto put = [&](int token, float v) {
-    if (a.act) v = llg_act(a.act - 1, v);
+    if (a.act) v = conv_act(a.act - 1, v);
     if (a.out) a.out[(long long)token * a.channels + c] = v;
     if (out2) out2[(long long)token * a.channels + c] = from_f32<O2>(v);
   };
@@ -217,13 +221,9 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(ConvArgs a) {
 // step) are still all done by the thread that meets the sequence's first token, state first, new state last.
 constexpr int CONV_RUN = 8;
 
+// Run `run` of one channel, whatever of it lies in which sequence.
 template <typename O2, int K>
-__global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int n_first = blockIdx.x * CONV_RUN;
-  const int c = blockIdx.y * blockDim.x + threadIdx.x;
-  if (c >= a.channels) return;
+__device__ __noinline__ void conv_run_of_channel(const ConvArgs& a, int n_first, int c) {
   const float ib = a.in_bias ? a.in_bias[c] : 0.f, ob = a.bias ? a.bias[c] : 0.f;
   float w[K];
 #pragma unroll
@@ -236,13 +236,13 @@ __global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a) {
   };
   O2* out2 = (O2*)a.out2;
   auto put = [&](int token, float v) {
-    if (a.act) v = llg_act(a.act - 1, v);
+    if (a.act) v = conv_act(a.act - 1, v);
     if (a.out) a.out[(long long)token * a.channels + c] = v;
     if (out2) out2[(long long)token * a.channels + c] = from_f32<O2>(v);
   };
+  const int n_last = n_first + CONV_RUN < a.n_tokens ? n_first + CONV_RUN : a.n_tokens;
   float win[K - 1];                                // win[d - 1]: the input of the token d before the current one
   int have = 0;                                    // how many of them are held
-  const int n_last = n_first + CONV_RUN < a.n_tokens ? n_first + CONV_RUN : a.n_tokens;
   for (int n = n_first; n < n_last; ++n) {
     const int b = a.seq_of_token[n];
     const int t0 = a.cu_tokens[b];
@@ -301,6 +301,76 @@ __global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a) {
     for (int d = K - 2; d > 0; --d) win[d] = win[d - 1];
     win[0] = x;
     if (have < K - 1) ++have;
+  }
+}
+
+__device__ __forceinline__ void load_run(const float* p, float (&v)[1]) { v[0] = *p; }
+__device__ __forceinline__ void load_run(const float* p, float (&v)[2]) {
+  const float2 t = *reinterpret_cast<const float2*>(p);
+  v[0] = t.x;
+  v[1] = t.y;
+}
+template <typename T> __device__ __forceinline__ void store_run(T* p, const float (&v)[1]) { *p = from_f32<T>(v[0]); }
+__device__ __forceinline__ void store_run(float* p, const float (&v)[2]) { *reinterpret_cast<float2*>(p) = make_float2(v[0], v[1]); }
+__device__ __forceinline__ void store_run(__nv_bfloat16* p, const float (&v)[2]) {
+  *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(v[0], v[1]);
+}
+
+// A thread owns VEC neighbouring channels of a run; neighbouring blocks own neighbouring channels of the same run, so the rows
+// are read through.  Where the run lies inside one sequence and all taps inside the step, every input is asked for before the
+// first is used; the others go channel by channel.
+template <typename O2, int K, int VEC>
+__global__ void __launch_bounds__(128) causal_conv_run_kernel(ConvArgs a, int channel_blocks) {
+  pdl_launch_dependents();
+  const int run = blockIdx.x / channel_blocks;
+  const int n_first = run * CONV_RUN;
+  const int c = ((blockIdx.x - run * channel_blocks) * blockDim.x + threadIdx.x) * VEC;
+  if (c >= a.channels) return;
+  const int n_last = n_first + CONV_RUN < a.n_tokens ? n_first + CONV_RUN : a.n_tokens;
+  const int b = a.seq_of_token[n_first];
+  const bool inside = n_last - n_first == CONV_RUN && a.seq_of_token[n_last - 1] == b && n_first - a.cu_tokens[b] >= K - 1;
+  float w[VEC][K], ib[VEC], ob[VEC];
+#pragma unroll
+  for (int e = 0; e < VEC; ++e) {
+    ib[e] = a.in_bias ? a.in_bias[c + e] : 0.f;
+    ob[e] = a.bias ? a.bias[c + e] : 0.f;
+#pragma unroll
+    for (int j = 0; j < K; ++j) w[e][j] = a.weight[(long long)(c + e) * K + j];
+  }
+  pdl_wait();
+  if (!inside) {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) conv_run_of_channel<O2, K>(a, n_first, c + e);
+    return;
+  }
+  float v[CONV_RUN + K - 1][VEC];
+  const float* r = a.rows + (long long)(n_first - (K - 1)) * a.row_width + a.col0 + c;
+#pragma unroll
+  for (int i = 0; i < CONV_RUN + K - 1; ++i) load_run(r + (long long)i * a.row_width, v[i]);
+  for (int s = 1; s < a.n_partials; ++s) {
+    r += a.partial_stride;
+#pragma unroll
+    for (int i = 0; i < CONV_RUN + K - 1; ++i) {
+      float u[VEC];
+      load_run(r + (long long)i * a.row_width, u);
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) v[i][e] += u[e];
+    }
+  }
+  long long at = (long long)n_first * a.channels + c;
+#pragma unroll
+  for (int k = 0; k < CONV_RUN; ++k, at += a.channels) {
+    float o[VEC];
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) {
+      float acc = 0.f;
+#pragma unroll
+      for (int j = 0; j < K; ++j) acc = fmaf(w[e][j], v[k + j][e] + ib[e], acc);
+      o[e] = acc + ob[e];
+      if (a.act) o[e] = conv_act(a.act - 1, o[e]);
+    }
+    if (a.out) store_run(a.out + at, o);
+    if (a.out2) store_run((O2*)a.out2 + at, o);
   }
 }
 
@@ -774,11 +844,19 @@ LLG_API int llg_causal_conv(const ConvArgs* args, cudaStream_t stream) {
   const bool bf = a.out2 && a.out2_dtype == LLG_BF16;
   // steps of many tokens and 2 to 4 taps: runs of tokens a thread
   if (a.taps >= 2 && a.taps <= 4 && a.n_tokens >= 4 * CONV_RUN) {
-    dim3 runs((a.n_tokens + CONV_RUN - 1) / CONV_RUN, grid.y);
-#define CONV_RUN_LAUNCH(K)                                                                               \
-  do {                                                                                                   \
-    if (bf) llg_launch(causal_conv_run_kernel<__nv_bfloat16, K>, runs, dim3(128), 0, stream, a);         \
-    else llg_launch(causal_conv_run_kernel<float, K>, runs, dim3(128), 0, stream, a);                    \
+    // two channels a thread where every row and every output starts on the boundary that takes
+    const bool two = a.channels % 2 == 0 && a.col0 % 2 == 0 && a.row_width % 2 == 0 && a.partial_stride % 2 == 0 &&
+                     ((uintptr_t)a.rows & 7u) == 0 && ((uintptr_t)a.out & 7u) == 0 && ((uintptr_t)a.out2 & 7u) == 0;
+    const int cb = (a.channels + (two ? 255 : 127)) / (two ? 256 : 128);
+    const long long blocks = (long long)((a.n_tokens + CONV_RUN - 1) / CONV_RUN) * cb;
+    LLG_REQUIRE(blocks < 2147483647LL, "causal_conv: too many tokens and channels");
+    const dim3 runs((unsigned)blocks);
+#define CONV_RUN_LAUNCH(K)                                                                                       \
+  do {                                                                                                           \
+    if (bf && two) llg_launch(causal_conv_run_kernel<__nv_bfloat16, K, 2>, runs, dim3(128), 0, stream, a, cb);   \
+    else if (bf) llg_launch(causal_conv_run_kernel<__nv_bfloat16, K, 1>, runs, dim3(128), 0, stream, a, cb);     \
+    else if (two) llg_launch(causal_conv_run_kernel<float, K, 2>, runs, dim3(128), 0, stream, a, cb);            \
+    else llg_launch(causal_conv_run_kernel<float, K, 1>, runs, dim3(128), 0, stream, a, cb);                     \
   } while (0)
     if (a.taps == 2) CONV_RUN_LAUNCH(2);
     else if (a.taps == 3) CONV_RUN_LAUNCH(3);

@@ -133,7 +133,7 @@ __global__ void __launch_bounds__(SS_THREADS) state_space_walk_kernel(StateSpace
 // ---- the chunked form on the tensor cores --------------------------------------------------------------------------
 
 constexpr int CH = 64;                   // tokens of a chunk
-constexpr int MM_THREADS = 128;          // four warps: warp w owns tokens 16 w .. of a chunk and every fourth 16 rows of the state
+constexpr int MM_THREADS = 256;
 constexpr float LEAST_LOG2 = -160.f;     // a decay below 2^-160 forgets everything; bounding it keeps the running sums short
 
 __device__ __forceinline__ uint32_t smem_at(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -169,21 +169,40 @@ __device__ __forceinline__ void split2(float v0, float v1, uint32_t& hi, uint32_
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
 
+// Two groups of four warps share a chunk; warp w of either group owns tokens 16 w .. of it.
+//   inside : C B^T, the factors, their product with x, and the output (with what the other group hands over, D x and the gate)
+//   across : C S0 for the chunk's tokens, handed over in shared memory as the registers hold it, then the state's update;
+//            warp w owns every fourth 16 rows of the state
+// One barrier of the block a chunk; the groups meet once more where the read-out is handed over.  The next chunk's rows are
+// requested at a chunk's start, its step sizes and their running sums are worked out beside the chunk.
+//
 // MT: 16-row tiles of the state per warp (n_state <= 64 MT); NV: 8-column tiles (8 NV columns of vdim a block).
 // Shared memory (bfloat16): two stages of B [CH][n_state + 8], C the same, x [CH][8 NV + 8]; the state as two parts
-// [2][n_state][8 NV + 8]; the weighed x as two parts [2][CH][8 NV + 8].
+// [2][n_state][8 NV + 8], or the read-out of S0 in float32 [4][NV][32][4]; the weighed x as two parts [2][CH][8 NV + 8].
+// bfloat16 places of the state's parts, in whose place the read-out is handed over once they have been read
+__host__ __device__ constexpr int state_halves(int n_state, int cols) {
+  return 2 * n_state * (cols + 8) > 2 * CH * cols ? 2 * n_state * (cols + 8) : 2 * CH * cols;
+}
+
+__device__ __forceinline__ void group_sync(int id) { asm volatile("bar.sync %0, 128;" ::"r"(id) : "memory"); }
+
 template <int MT, int NV>
-__global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceArgs a) {
+__global__ void __launch_bounds__(MM_THREADS, MT <= 2 && NV <= 4 ? 2 : 1) state_space_mma_kernel(StateSpaceArgs a) {
   pdl_launch_dependents();
   extern __shared__ __align__(16) unsigned char raw_smem[];
-  __shared__ float s_step[CH], s_log[CH];
+  // per token of a chunk: the step size d, the running sum of log2 decays a, d 2^{a_end - a} (what its x weighs in the state behind
+  // the chunk), and d 2^{E - a} with E the sum at the end of its sixteen tokens (its part of a factor for later tokens)
+  __shared__ float s_step[2][CH], s_log[2][CH], s_last[2][CH], s_part[2][CH];
   constexpr int VS = 8 * NV, LDV = VS + 8;
   const int N = a.n_state, LDN = N + 8, NT = N / 16;
   bf16* stage0 = reinterpret_cast<bf16*>(raw_smem);
   const int stage_halves = 2 * CH * LDN + CH * LDV;
   bf16* state_sm = stage0 + 2 * stage_halves;
-  bf16* wx = state_sm + 2 * N * LDV;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  bf16* wx = state_sm + state_halves(N, VS);
+  float4* handed = reinterpret_cast<float4*>(state_sm);
+  const int tid = threadIdx.x, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const bool across = tid >= 128;
+  const int warp = (tid >> 5) & 3;                       // inside its group
   const int runs = a.vdim / VS;
   const int h = blockIdx.x / runs, c0 = (blockIdx.x - h * runs) * VS, b = blockIdx.y;
   const int lo = a.cu_tokens[b], hi = a.cu_tokens[b + 1];
@@ -197,7 +216,7 @@ __global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceA
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
       const int row = (warp + 4 * mt) * 16 + g;
-      const bool in = warp + 4 * mt < NT;
+      const bool in = across && warp + 4 * mt < NT;
       const float* p = gstate + (long long)row * a.vdim + v * 8 + 2 * t4;
       const float2 u = in ? *reinterpret_cast<const float2*>(p) : make_float2(0.f, 0.f);
       const float2 w = in ? *reinterpret_cast<const float2*>(p + 8LL * a.vdim) : make_float2(0.f, 0.f);
@@ -207,16 +226,34 @@ __global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceA
   pdl_wait();
 
   const bf16* mixed = (const bf16*)a.mixed;
+  const int per = N / 8;                                 // 16-byte pieces of a row of B or C
+  const int t_first = tid / per, c_first = tid - t_first * per, t_step = MM_THREADS / per, c_step = MM_THREADS - t_step * per;
   auto load_chunk = [&](int n0, int stage) {
     bf16* base = stage0 + stage * stage_halves;
-    const int per = N / 8;
-    for (int idx = tid; idx < CH * per; idx += MM_THREADS) {
-      const int t = idx / per, c = idx - t * per;
-      const bool valid = n0 + t < hi;
-      const bf16* row = mixed + (long long)(valid ? n0 + t : lo) * mixed_w + c * 8;
-      copy16(smem_at(base + t * LDN + c * 8), row + b_col, valid);
-      copy16(smem_at(base + (CH + t) * LDN + c * 8), row + c_col, valid);
+    if (n0 + CH <= hi && c_step == 0) {
+      // a whole chunk whose pieces divide among the threads: the same piece of every t_step-th row
+      const bf16* src = mixed + (long long)(n0 + t_first) * mixed_w + c_first * 8;
+      const long long src_step = (long long)t_step * mixed_w;
+      uint32_t dst = smem_at(base + t_first * LDN + c_first * 8);
+      const uint32_t dst_step = (uint32_t)(t_step * LDN * 2), to_c = (uint32_t)(CH * LDN * 2);
+      for (int t = t_first; t < CH; t += t_step) {
+        copy16(dst, src + b_col, true);
+        copy16(dst + to_c, src + c_col, true);
+        src += src_step;
+        dst += dst_step;
+      }
+    } else {
+      for (int t = t_first, c = c_first; t < CH;) {
+        const bool valid = n0 + t < hi;
+        const bf16* row = mixed + (long long)(valid ? n0 + t : lo) * mixed_w + c * 8;
+        copy16(smem_at(base + t * LDN + c * 8), row + b_col, valid);
+        copy16(smem_at(base + (CH + t) * LDN + c * 8), row + c_col, valid);
+        t += t_step;
+        c += c_step;
+        if (c >= per) { c -= per; ++t; }
+      }
     }
+#pragma unroll
     for (int idx = tid; idx < CH * NV; idx += MM_THREADS) {
       const int t = idx / NV, c = idx - t * NV;
       const bool valid = n0 + t < hi;
@@ -224,76 +261,149 @@ __global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceA
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  // warp 0: the step sizes' arguments of tokens n0 + 2 lane and n0 + 2 lane + 1
+  // the first warp: the step sizes' arguments of tokens n0 + 2 lane and n0 + 2 lane + 1, and what becomes of them
   float arg0 = 0.f, arg1 = 0.f;
   auto fetch_steps = [&](int n0) {
     const int n = n0 + 2 * lane;
     const float* p = a.rows + a.dt_col + h;
-    arg0 = arg1 = dt_bias;
-    for (int s = 0; s < a.n_partials; ++s) {
+    // nothing is added to the first loads' results here: they would be waited for
+    arg0 = n < hi ? p[(long long)n * a.row_width] : 0.f;
+    arg1 = n + 1 < hi ? p[(long long)(n + 1) * a.row_width] : 0.f;
+    for (int s = 1; s < a.n_partials; ++s) {
       if (n < hi) arg0 += p[s * a.partial_stride + (long long)n * a.row_width];
       if (n + 1 < hi) arg1 += p[s * a.partial_stride + (long long)(n + 1) * a.row_width];
     }
   };
+  auto put_steps = [&](int n0, int buf) {
+    // tokens past the end: no step and no decay, so they change nothing
+    const int n = n0 + 2 * lane;
+    const float d0 = n < hi ? softplus_f(arg0 + dt_bias) : 0.f, d1 = n + 1 < hi ? softplus_f(arg1 + dt_bias) : 0.f;
+    const float l0 = fmaxf(rate2 * d0, LEAST_LOG2), l1 = fmaxf(rate2 * d1, LEAST_LOG2);
+    float incl = l0 + l1;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, incl, o);
+      if (lane >= o) incl += up;
+    }
+    const float up1 = __shfl_up_sync(0xffffffffu, incl, 1), log0 = (lane ? up1 : 0.f) + l0;
+    const float end = __shfl_sync(0xffffffffu, incl, 31), block_end = __shfl_sync(0xffffffffu, incl, lane | 7);
+    *reinterpret_cast<float2*>(&s_step[buf][2 * lane]) = make_float2(d0, d1);
+    *reinterpret_cast<float2*>(&s_log[buf][2 * lane]) = make_float2(log0, incl);
+    *reinterpret_cast<float2*>(&s_last[buf][2 * lane]) = make_float2(d0 * exp2_fast(end - log0), d1 * exp2_fast(end - incl));
+    *reinterpret_cast<float2*>(&s_part[buf][2 * lane]) = make_float2(d0 * exp2_fast(block_end - log0), d1 * exp2_fast(block_end - incl));
+  };
   load_chunk(lo, 0);
-  if (warp == 0) fetch_steps(lo);
+  if (tid < 32) {
+    fetch_steps(lo);
+    put_steps(lo, 0);
+  }
   int stage = 0;
   for (int n0 = lo; n0 < hi; n0 += CH, stage ^= 1) {
-    if (warp == 0) {
-      // tokens past the end: no step and no decay, so they change nothing
-      const int n = n0 + 2 * lane;
-      const float d0 = n < hi ? softplus_f(arg0) : 0.f, d1 = n + 1 < hi ? softplus_f(arg1) : 0.f;
-      const float l0 = fmaxf(rate2 * d0, LEAST_LOG2), l1 = fmaxf(rate2 * d1, LEAST_LOG2);
-      float incl = l0 + l1;
+    const bool more = n0 + CH < hi;
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();                       // the chunk and its sums of logs are there; the other stage may be written again
+    if (more) load_chunk(n0 + CH, stage ^ 1);
+    const bf16* Bs = stage0 + stage * stage_halves;
+    const bf16* Cs = Bs + CH * LDN;
+    const bf16* Xs = Cs + CH * LDN;
+    const float *slog = s_log[stage], *sstep = s_step[stage];
+    const int r0 = warp * 16 + g, r1 = r0 + 8;
+    const float a0 = slog[r0], a1 = slog[r1];
+    if (across) {
+      // the state before the chunk, in two parts, for the group's products with C
 #pragma unroll
-      for (int o = 1; o < 32; o <<= 1) {
-        const float up = __shfl_up_sync(0xffffffffu, incl, o);
-        if (lane >= o) incl += up;
-      }
-      const float before = __shfl_up_sync(0xffffffffu, incl, 1);
-      s_step[2 * lane] = d0;
-      s_step[2 * lane + 1] = d1;
-      s_log[2 * lane] = (lane ? before : 0.f) + l0;
-      s_log[2 * lane + 1] = incl;
-    }
-    // the state before the chunk, in two parts, for everybody's products with C
+      for (int mt = 0; mt < MT; ++mt) {
+        if (warp + 4 * mt < NT) {
 #pragma unroll
-    for (int mt = 0; mt < MT; ++mt) {
-      if (warp + 4 * mt < NT) {
-#pragma unroll
-        for (int v = 0; v < NV; ++v) {
-          bf16* p = state_sm + ((warp + 4 * mt) * 16 + g) * LDV + v * 8 + 2 * t4;
-          uint32_t h0, l0, h1, l1;
-          split2(S[mt][v][0], S[mt][v][1], h0, l0);
-          split2(S[mt][v][2], S[mt][v][3], h1, l1);
-          *reinterpret_cast<uint32_t*>(p) = h0;
-          *reinterpret_cast<uint32_t*>(p + 8 * LDV) = h1;
-          *reinterpret_cast<uint32_t*>(p + N * LDV) = l0;
-          *reinterpret_cast<uint32_t*>(p + N * LDV + 8 * LDV) = l1;
+          for (int v = 0; v < NV; ++v) {
+            bf16* p = state_sm + ((warp + 4 * mt) * 16 + g) * LDV + v * 8 + 2 * t4;
+            uint32_t h0, l0, h1, l1;
+            split2(S[mt][v][0], S[mt][v][1], h0, l0);
+            split2(S[mt][v][2], S[mt][v][3], h1, l1);
+            *reinterpret_cast<uint32_t*>(p) = h0;
+            *reinterpret_cast<uint32_t*>(p + 8 * LDV) = h1;
+            *reinterpret_cast<uint32_t*>(p + N * LDV) = l0;
+            *reinterpret_cast<uint32_t*>(p + N * LDV + 8 * LDV) = l1;
+          }
         }
       }
-    }
-    const bool more = n0 + CH < hi;
-    if (more) {
-      load_chunk(n0 + CH, stage ^ 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();                       // the chunk, its sums of logs and the state are in shared memory
-    bf16* Bs = stage0 + stage * stage_halves;
-    bf16* Cs = Bs + CH * LDN;
-    bf16* Xs = Cs + CH * LDN;
-    const int r0 = warp * 16 + g, r1 = r0 + 8;
-    // asked for now, used at the end: the gates' arguments and (warp 0) the next chunk's step sizes
-    float z[NV][4];
-    if (a.z_col >= 0) {
+      group_sync(1);
+      float y[NV][4];
 #pragma unroll
       for (int v = 0; v < NV; ++v)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) z[v][e] = 0.f;
-      for (int s = 0; s < a.n_partials; ++s) {
-        const float* zp = a.rows + s * a.partial_stride + (long long)(n0 + r0) * a.row_width + a.z_col + x_col + 2 * t4;
+        for (int e = 0; e < 4; ++e) y[v][e] = 0.f;
+#pragma unroll 4
+      for (int kk = 0; kk < NT; ++kk) {
+        uint32_t ca[4];
+        ldm4(ca, smem_at(Cs + (warp * 16 + (lane & 15)) * LDN + kk * 16 + (lane >> 4) * 8));
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          uint32_t sb[4];                  // both parts of 16 rows and 8 columns of the state
+          ldm4_trans(sb, smem_at(state_sm + ((lane >> 4) * N + kk * 16 + (lane & 15)) * LDV + v * 8));
+          mma16816(y[v], ca, sb[0], sb[1]);
+          mma16816(y[v], ca, sb[2], sb[3]);
+        }
+      }
+      const float e0 = exp2_fast(a0), e1 = exp2_fast(a1);
+      group_sync(1);                       // nobody reads the state's parts any more: the read-out takes their place
+#pragma unroll
+      for (int v = 0; v < NV; ++v) handed[(warp * NV + v) * 32 + lane] = make_float4(y[v][0] * e0, y[v][1] * e0, y[v][2] * e1, y[v][3] * e1);
+      asm volatile("bar.arrive 2, 256;" ::: "memory");
+      // x times e^{a_end - a_s} d_s in two parts, then S = e^{a_end} S0 + B^T (weighed x)
+      const float log_end = slog[CH - 1];
+      for (int idx = tid - 128; idx < CH * NV * 4; idx += 128) {
+        const int s = idx / (NV * 4), c = (idx - s * (NV * 4)) * 2;
+        const float w = s_last[stage][s];
+        const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(Xs + s * LDV + c);
+        uint32_t hi2, lo2;
+        split2(w * __low2float(x), w * __high2float(x), hi2, lo2);
+        *reinterpret_cast<uint32_t*>(wx + s * LDV + c) = hi2;
+        *reinterpret_cast<uint32_t*>(wx + (CH + s) * LDV + c) = lo2;
+      }
+      const float e_end = exp2_fast(log_end);
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int v = 0; v < NV; ++v)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) S[mt][v][e] *= e_end;
+      group_sync(1);
+#pragma unroll
+      for (int kk = 0; kk < CH / 16; ++kk) {
+        uint32_t ba[MT][4];                // B^T
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+          if (warp + 4 * mt < NT)
+            ldm4_trans(ba[mt], smem_at(Bs + (kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * LDN + (warp + 4 * mt) * 16 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+          uint32_t wb[4];                  // both parts of the weighed x of 16 tokens
+          ldm4_trans(wb, smem_at(wx + ((lane >> 4) * CH + kk * 16 + (lane & 15)) * LDV + v * 8));
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            if (warp + 4 * mt < NT) {
+              mma16816(S[mt][v], ba[mt], wb[0], wb[1]);
+              mma16816(S[mt][v], ba[mt], wb[2], wb[3]);
+            }
+          }
+        }
+      }
+      continue;
+    }
+    // asked for now, used at the end: the gates' arguments and (first warp) the next chunk's step sizes
+    float z[NV][4];
+    if (a.z_col >= 0) {
+      const float* zp = a.rows + (long long)(n0 + r0) * a.row_width + a.z_col + x_col + 2 * t4;
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        z[v][0] = n0 + r0 < hi ? zp[v * 8] : 0.f;
+        z[v][1] = n0 + r0 < hi ? zp[v * 8 + 1] : 0.f;
+        z[v][2] = n0 + r1 < hi ? zp[8LL * a.row_width + v * 8] : 0.f;
+        z[v][3] = n0 + r1 < hi ? zp[8LL * a.row_width + v * 8 + 1] : 0.f;
+      }
+      for (int s = 1; s < a.n_partials; ++s) {
+        zp += a.partial_stride;
 #pragma unroll
         for (int v = 0; v < NV; ++v) {
           if (n0 + r0 < hi) { z[v][0] += zp[v * 8]; z[v][1] += zp[v * 8 + 1]; }
@@ -302,18 +412,7 @@ __global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceA
       }
     }
     if (more && warp == 0) fetch_steps(n0 + CH);
-    const float log_end = s_log[CH - 1];
-    // x times e^{a_end - a_s} d_s in two parts, for the state's update
-    for (int idx = tid; idx < CH * NV * 4; idx += MM_THREADS) {
-      const int s = idx / (NV * 4), c = (idx - s * (NV * 4)) * 2;
-      const float w = exp2_fast(log_end - s_log[s]) * s_step[s];
-      const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(Xs + s * LDV + c);
-      uint32_t hi2, lo2;
-      split2(w * __low2float(x), w * __high2float(x), hi2, lo2);
-      *reinterpret_cast<uint32_t*>(wx + s * LDV + c) = hi2;
-      *reinterpret_cast<uint32_t*>(wx + (CH + s) * LDV + c) = lo2;
-    }
-    // C B^T for this warp's tokens (columns up to its own last token), and C S0
+    // C B^T for this warp's tokens (columns up to its own last token)
     float G[8][4], y[NV][4];
 #pragma unroll
     for (int i = 0; i < 8; ++i)
@@ -323,6 +422,7 @@ __global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceA
     for (int v = 0; v < NV; ++v)
 #pragma unroll
       for (int e = 0; e < 4; ++e) y[v][e] = 0.f;
+#pragma unroll 4
     for (int kk = 0; kk < NT; ++kk) {
       uint32_t ca[4];
       ldm4(ca, smem_at(Cs + (warp * 16 + (lane & 15)) * LDN + kk * 16 + (lane >> 4) * 8));
@@ -335,95 +435,67 @@ __global__ void __launch_bounds__(MM_THREADS) state_space_mma_kernel(StateSpaceA
           mma16816(G[2 * sp + 1], ca, bb[2], bb[3]);
         }
       }
-#pragma unroll
-      for (int v = 0; v < NV; ++v) {
-        uint32_t sb[4];                    // both parts of 16 rows and 8 columns of the state
-        ldm4_trans(sb, smem_at(state_sm + ((lane >> 4) * N + kk * 16 + (lane & 15)) * LDV + v * 8));
-        mma16816(y[v], ca, sb[0], sb[1]);
-        mma16816(y[v], ca, sb[2], sb[3]);
-      }
-    }
-    const float a0 = s_log[r0], a1 = s_log[r1];
-    {
-      const float e0 = exp2_fast(a0), e1 = exp2_fast(a1);
-#pragma unroll
-      for (int v = 0; v < NV; ++v) { y[v][0] *= e0; y[v][1] *= e0; y[v][2] *= e1; y[v][3] *= e1; }
     }
 #pragma unroll
-    for (int kp = 0; kp < 2; ++kp) {
-      if (2 * kp > warp) continue;
-      uint32_t xb[NV][4];                  // x of 32 tokens: the operands of two products
-#pragma unroll
-      for (int v = 0; v < NV; ++v) ldm4_trans(xb[v], smem_at(Xs + (kp * 32 + lane) * LDV + v * 8));
-#pragma unroll
-      for (int k2 = 0; k2 < 2; ++k2) {
-        const int kk = 2 * kp + k2;
-        if (kk > warp) continue;
-        uint32_t ah[4], al[4];
+    for (int kk = 0; kk < 4; ++kk) {
+      if (kk > warp) continue;
+      uint32_t ah[4], al[4];
+      if (kk < warp) {
+        // sixteen earlier tokens: 2^{a_t - a_s} d_s as 2^{a_t - E} times the token's part up to E, neither above d_s
+        const float block_end = slog[kk * 16 + 15], e0 = exp2_fast(a0 - block_end), e1 = exp2_fast(a1 - block_end);
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
-          const int s = kk * 16 + half * 8 + 2 * t4;
-          const float2 la = *reinterpret_cast<const float2*>(s_log + s), d = *reinterpret_cast<const float2*>(s_step + s);
+          const float2 q = *reinterpret_cast<const float2*>(&s_part[stage][kk * 16 + half * 8 + 2 * t4]);
           const float(&gv)[4] = G[2 * kk + half];
-          const float m00 = s <= r0 ? gv[0] * (exp2_fast(a0 - la.x) * d.x) : 0.f;
-          const float m01 = s + 1 <= r0 ? gv[1] * (exp2_fast(a0 - la.y) * d.y) : 0.f;
-          const float m10 = s <= r1 ? gv[2] * (exp2_fast(a1 - la.x) * d.x) : 0.f;
-          const float m11 = s + 1 <= r1 ? gv[3] * (exp2_fast(a1 - la.y) * d.y) : 0.f;
-          split2(m00, m01, ah[2 * half], al[2 * half]);
-          split2(m10, m11, ah[2 * half + 1], al[2 * half + 1]);
+          split2(gv[0] * (e0 * q.x), gv[1] * (e0 * q.y), ah[2 * half], al[2 * half]);
+          split2(gv[2] * (e1 * q.x), gv[3] * (e1 * q.y), ah[2 * half + 1], al[2 * half + 1]);
         }
+      } else
 #pragma unroll
-        for (int v = 0; v < NV; ++v) {
-          mma16816(y[v], ah, xb[v][2 * k2], xb[v][2 * k2 + 1]);
-          mma16816(y[v], al, xb[v][2 * k2], xb[v][2 * k2 + 1]);
+      for (int half = 0; half < 2; ++half) {
+        const int s = kk * 16 + half * 8 + 2 * t4;
+        const float2 la = *reinterpret_cast<const float2*>(slog + s), d = *reinterpret_cast<const float2*>(sstep + s);
+        const float(&gv)[4] = G[2 * kk + half];
+        const float m00 = s <= r0 ? gv[0] * (exp2_fast(a0 - la.x) * d.x) : 0.f;
+        const float m01 = s + 1 <= r0 ? gv[1] * (exp2_fast(a0 - la.y) * d.y) : 0.f;
+        const float m10 = s <= r1 ? gv[2] * (exp2_fast(a1 - la.x) * d.x) : 0.f;
+        const float m11 = s + 1 <= r1 ? gv[3] * (exp2_fast(a1 - la.y) * d.y) : 0.f;
+        split2(m00, m01, ah[2 * half], al[2 * half]);
+        split2(m10, m11, ah[2 * half + 1], al[2 * half + 1]);
+      }
+#pragma unroll
+      for (int v = 0; v < NV; v += 2) {    // x of 16 tokens and up to 16 columns
+        uint32_t xb[4];
+        ldm4_trans(xb, smem_at(Xs + (kk * 16 + (lane & 15)) * LDV + (v + (NV > 1 ? lane >> 4 : 0)) * 8));
+        mma16816(y[v], ah, xb[0], xb[1]);
+        mma16816(y[v], al, xb[0], xb[1]);
+        if (NV > 1) {
+          mma16816(y[(v + 1) % NV], ah, xb[2], xb[3]);
+          mma16816(y[(v + 1) % NV], al, xb[2], xb[3]);
         }
       }
     }
+    if (more && warp == 0) put_steps(n0 + CH, stage ^ 1);
+    asm volatile("bar.sync 2, 256;" ::: "memory");       // what the state before the chunk gives is there
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
       const __nv_bfloat162 x0 = *reinterpret_cast<const __nv_bfloat162*>(Xs + r0 * LDV + v * 8 + 2 * t4);
       const __nv_bfloat162 x1 = *reinterpret_cast<const __nv_bfloat162*>(Xs + r1 * LDV + v * 8 + 2 * t4);
-      float o[4] = {fmaf(skip, __low2float(x0), y[v][0]), fmaf(skip, __high2float(x0), y[v][1]),
-                    fmaf(skip, __low2float(x1), y[v][2]), fmaf(skip, __high2float(x1), y[v][3])};
+      const float4 q = handed[(warp * NV + v) * 32 + lane];
+      float o[4] = {fmaf(skip, __low2float(x0), y[v][0] + q.x), fmaf(skip, __high2float(x0), y[v][1] + q.y),
+                    fmaf(skip, __low2float(x1), y[v][2] + q.z), fmaf(skip, __high2float(x1), y[v][3] + q.w)};
       if (a.z_col >= 0) {
 #pragma unroll
-        for (int e = 0; e < 4; ++e) o[e] *= z[v][e] / (1.0f + expf(-z[v][e]));
+        for (int e = 0; e < 4; ++e) o[e] *= __fdividef(z[v][e], 1.0f + __expf(-z[v][e]));
       }
       float* dst = a.out + (long long)(n0 + r0) * inner + x_col + v * 8 + 2 * t4;
       if (n0 + r0 < hi) *reinterpret_cast<float2*>(dst) = make_float2(o[0], o[1]);
       if (n0 + r1 < hi) *reinterpret_cast<float2*>(dst + 8LL * inner) = make_float2(o[2], o[3]);
     }
-    __syncthreads();                       // the weighed x is in shared memory; nobody reads the old state any more
-    const float e_end = exp2_fast(log_end);
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int v = 0; v < NV; ++v)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) S[mt][v][e] *= e_end;
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      uint32_t wb[NV][4];                  // both parts of the weighed x of 16 tokens
-#pragma unroll
-      for (int v = 0; v < NV; ++v) ldm4_trans(wb[v], smem_at(wx + ((lane >> 4) * CH + kk * 16 + (lane & 15)) * LDV + v * 8));
-#pragma unroll
-      for (int mt = 0; mt < MT; ++mt) {
-        if (warp + 4 * mt < NT) {
-          uint32_t ba[4];                  // B^T
-          ldm4_trans(ba, smem_at(Bs + (kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * LDN + (warp + 4 * mt) * 16 + ((lane >> 3) & 1) * 8));
-#pragma unroll
-          for (int v = 0; v < NV; ++v) {
-            mma16816(S[mt][v], ba, wb[v][0], wb[v][1]);
-            mma16816(S[mt][v], ba, wb[v][2], wb[v][3]);
-          }
-        }
-      }
-    }
-    __syncthreads();                       // the stage, the weighed x and the state's parts may be written again
   }
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt) {
-    if (warp + 4 * mt < NT) {
+    if (across && warp + 4 * mt < NT) {
 #pragma unroll
       for (int v = 0; v < NV; ++v) {
         float* p = gstate + (long long)((warp + 4 * mt) * 16 + g) * a.vdim + v * 8 + 2 * t4;
@@ -487,7 +559,7 @@ __global__ void part_rmsnorm_kernel(const float* __restrict__ x, const float* __
 
 template <typename K>
 int allow_smem(K kernel, size_t smem) {
-  if (smem > 48 * 1024) {
+  if (smem > 40 * 1024) {                   // the kernels' static shared memory counts toward the 48 KB that need no asking
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return llg_fail("state_space: shared memory %zu: %s", smem, cudaGetErrorString(e));
   }
@@ -512,9 +584,19 @@ WalkShape walk_shape(int n_state, int vdim) {
 }
 
 size_t mma_smem(int n_state, int cols) {
-  return (size_t)(2 * (2 * CH * (n_state + 8) + CH * (cols + 8)) + 2 * n_state * (cols + 8) + 2 * CH * (cols + 8)) * sizeof(bf16);
+  return (size_t)(2 * (2 * CH * (n_state + 8) + CH * (cols + 8)) + state_halves(n_state, cols) + 2 * CH * (cols + 8)) * sizeof(bf16);
 }
-int mma_cols(int vdim) { return vdim % 32 == 0 ? 32 : vdim % 16 == 0 ? 16 : vdim % 8 == 0 ? 8 : 0; }
+// Columns a block owns: as many as fit (fewer columns repeat C B^T more often), fewer where that would leave too many
+// multiprocessors without a block.  0: none fit.
+int mma_cols(int n_state, int vdim, long long heads) {
+  int last = 0;
+  for (int cols = 64; cols >= 8; cols /= 2) {
+    if (vdim % cols || mma_smem(n_state, cols) > 220 * 1024) continue;
+    last = cols;
+    if (heads * (vdim / cols) * 4 >= 3LL * llg_sm_count()) return cols;
+  }
+  return last;
+}
 
 int check_args(const StateSpaceArgs& a, const char* what) {
   LLG_REQUIRE(a.n_seqs >= 0 && a.n_tokens >= 0 && a.nh > 0 && a.groups > 0 && a.n_state > 0 && a.vdim > 0 && a.n_partials >= 1,
@@ -533,7 +615,7 @@ LLG_API int llg_state_space_fits(int n_state, int vdim) { return n_state > 0 && 
 
 // 1 when the tensor-core form takes it (bfloat16, prompt steps).
 LLG_API int llg_state_space_mma_fits(int n_state, int vdim) {
-  return n_state > 0 && n_state % 16 == 0 && n_state <= 256 && mma_cols(vdim) > 0 && mma_smem(n_state, mma_cols(vdim)) <= 220 * 1024;
+  return n_state > 0 && n_state % 16 == 0 && n_state <= 256 && mma_cols(n_state, vdim, 1) > 0;
 }
 
 LLG_API int llg_state_space_walk(const StateSpaceArgs* args, cudaStream_t stream) {
@@ -572,7 +654,9 @@ LLG_API int llg_state_space_mma(const StateSpaceArgs* args, cudaStream_t stream)
   LLG_REQUIRE(((uintptr_t)a.mixed & 15u) == 0 && ((uintptr_t)a.state & 15u) == 0 && ((uintptr_t)a.out & 15u) == 0,
               "state_space_mma: operands must be 16-byte aligned");
   if (a.n_seqs == 0 || a.n_tokens == 0) return 0;
-  a.cols = mma_cols(a.vdim);
+  if (a.cols == 0) a.cols = mma_cols(a.n_state, a.vdim, (long long)a.nh * a.n_seqs);
+  LLG_REQUIRE((a.cols == 8 || a.cols == 16 || a.cols == 32 || a.cols == 64) && a.vdim % a.cols == 0 && mma_smem(a.n_state, a.cols) <= 220 * 1024,
+              "state_space_mma: %d columns a block of a state of %d x %d", a.cols, a.n_state, a.vdim);
   const size_t smem = mma_smem(a.n_state, a.cols);
   const dim3 grid(a.nh * (a.vdim / a.cols), a.n_seqs);
 #define GO(MT, NV)                                                                   \
@@ -586,7 +670,8 @@ LLG_API int llg_state_space_mma(const StateSpaceArgs* args, cudaStream_t stream)
     else if (a.n_state <= 128) GO(2, NV); \
     else GO(4, NV);                    \
   } while (0)
-  if (a.cols == 32) GO_M(4);
+  if (a.cols == 64) GO_M(8);
+  else if (a.cols == 32) GO_M(4);
   else if (a.cols == 16) GO_M(2);
   else GO_M(1);
 #undef GO_M
