@@ -230,6 +230,8 @@ def penasun_spec(cfg: PenasunConfig) -> ModelSpec:
         schedule=tuple(ScheduleEntry(i) for i in range(len(layers))),
         final_norm=norm("final.norm"),
         head=PartSpec("linear_head", {"vocab_size": cfg.vocab, "hidden_size": cfg.width, "tied_to": "embed"}, ""),
+        # a layer without a feed-forward has no use for the norm ahead of it
+        ignorable_tensors=tuple(rf"l{i}\.norm2" for i, layer in enumerate(cfg.layers) if layer.mlp is None),
     )
     spec.validate()
     return spec

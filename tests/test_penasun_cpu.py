@@ -224,6 +224,15 @@ def test_cost_model_counts_both_maps_the_chosen_experts_and_no_pairs_for_a_state
     assert [u for u in costs.kv_units] == [(2 * (24 + 20) * 2, 0), (3 * (16 + 16) * 2, 0)]
 
 
+def test_a_norm_ahead_of_no_feed_forward_is_skipped_with_a_warning(llogos, tmp_path):
+    cfg = PM.CONFIGS["odd"]
+    w = PM.random_weights(cfg, 3)
+    w["l3.norm2"] = torch.ones(cfg["width"], dtype=torch.bfloat16)
+    PM.write_model(llogos, str(tmp_path), cfg, 0, weights=w)
+    model = llogos.weights.load_model(str(tmp_path), dtype=torch.float32, device="cpu", ops=cpu_ops)
+    assert any("l3.norm2" in x for x in model.load_warnings)
+
+
 def test_fixed_size_state_refuses_a_rollback(llogos, tmp_path):
     cfg = PM.CONFIGS["odd"]
     PM.write_model(llogos, str(tmp_path), cfg, seed=1)
